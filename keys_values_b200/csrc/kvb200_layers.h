@@ -1,0 +1,84 @@
+// C API of libkvb200_layers: kernels of models whose layers are described one by one (latent attention over a
+// ring of latents, routed experts, token shift, averages over the depth). Conventions as in kvb200.h: launches on
+// the given stream, returns KVB_OK or a negative code, dtype 0 = fp32, 1 = bf16; nothing synchronises the device.
+//
+// A pass works on B rows of T tokens (right padded). Row b belongs to the sequence in slot slots[b]; its first
+// token has position start[b], and count[b] <= T of its tokens are real. Padding is computed like tokens but never
+// reaches a cache or a state.
+#pragma once
+#include <stdint.h>
+
+#include "kvb200.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+// ---- layer_edge.cu
+// First tokens of a layer stack: x = embed[token] (+ bigram row), fp32, written to hist (entry 0 of the depth
+// history); then norm and token shift of the first layer as in kvb_layer_edge. bigram may be NULL; gain NULL: no norm.
+int kvb_embed_edge(const long long* idx, const int* prev_token, const void* embed, const void* bigram, long long buckets,
+                   long long mul_prev, long long mul_cur, float* hist, const float* gain, const float* shift, float* state, void* h,
+                   void* hs, const int* slots, const int* start, const int* count, int B, int T, int width, long long vocab, float eps,
+                   int dtype, int* status, void* stream);
+// Between two layers: X_new = x_in + mix (+ sum_k w[n,k] · expert_out[row[n,k]]); with a depth history (coef not NULL)
+// hist[n_hist] = X_new and x_out = sum_{j <= n_hist} coef[j] · X_j, else x_out = X_new. Then, unless gain is NULL,
+// h = x_out / rms(x_out) · gain and hs = h + (h_prev − h) · shift (shift NULL: hs not written). state (slots, width):
+// h of the last token of every sequence.
+int kvb_layer_edge(const float* x_in, const void* mix, const void* expert_out, const int* expert_row, const float* expert_w, int top,
+                   long long expert_ld, float* hist, int n_hist, long long hist_stride, const float* coef, float* x_out,
+                   const float* gain, const float* shift, float* state, void* h, void* hs, const int* slots, const int* start,
+                   const int* count, int B, int T, int width, float eps, int dtype, void* stream);
+// rows of x (fp32, rows[i] or i when rows is NULL) divided by their root mean square, times one number
+int kvb_scalar_rmsnorm(const float* x, const long long* rows, const float* gain, void* y, long long n, int width, float eps,
+                       int dtype, void* stream);
+// pos[slot] += count, prev_token[slot] = last token of the row; rows without tokens stay as they are
+int kvb_sequence_advance(const long long* idx, int* pos, int* prev_token, const int* slots, const int* count, int B, int T,
+                         void* stream);
+
+// ---- latent_attn.cu
+// One row of the latent storage: [c (kv_rank, padded to kvp) | rotated key part (rot, padded to rp)], kvp and rp
+// multiples of 8, padding zero. Queries: [unrotated (dim padded to dimp) | rotated (rot padded to rp)] per head.
+int kvb_latent_prep(const void* qkv, long long ld, const float* norm_w, const float* freq, void* q, void* latent, void* ring,
+                    const int* slots, const int* start, const int* count, int B, int T, int P, int ring_len, int heads, int dim,
+                    int dimp, int rot, int rot_dims, int rp, int kv_rank, int kvp, float eps, int dtype, void* stream);
+// latent[b, j] (j < P) = ring row of position start[b] − P + j, zero where there is none
+int kvb_ring_gather(const void* ring, void* latent, const int* slots, const int* start, int B, int T, int P, int ring_len, int lw,
+                    int dtype, void* stream);
+// the last min(count, ring_len) new rows of every sequence into its ring
+int kvb_ring_append(const void* latent, void* ring, const int* slots, const int* start, const int* count, int B, int T, int P,
+                    int ring_len, int lw, int dtype, void* stream);
+// Attention of T new tokens over P + T expanded keys: kv (B, P+T, heads, dimp + vdp) = [unrotated key | value],
+// latent (B, P+T, lw) holds the rotated key part at column kvp. out (B, T, heads, vdp).
+int kvb_latent_attend(const void* q, const void* kv, const void* latent, void* out, const int* start, int B, int T, int P, int heads,
+                      int dimp, int rp, int kvp, int vdp, int window, float scale, int dtype, void* stream);
+// One new token per sequence over its ring, in latent space: q_abs (heads, B, kvp) = W_uk^T q, q (B, heads, dimp + rp) for
+// the rotated part, out (heads, B, kvp) = weighted latents.
+long long kvb_latent_decode_scratch_bytes(int B, int heads, int kvp, int ring_len);
+int kvb_latent_decode(const void* q_abs, const void* q, const void* ring, void* out, void* scratch, const int* slots,
+                      const int* start, int B, int heads, int dimp, int rp, int kvp, int ring_len, float scale, int dtype,
+                      int simple, void* stream);
+
+// ---- latent_sm100.cu: kvb_latent_attend for bf16 on tcgen05
+int kvb_latent_attend_tc_supported(int dimp, int rp, int vdp);
+int kvb_latent_attend_tc(const void* q, const void* kv, const void* latent, void* out, const int* start, int B, int T, int P,
+                         int heads, int dimp, int rp, int kvp, int vdp, int window, float scale, int* status, void* stream);
+
+// ---- moe.cu
+// Router: softmax over n_expert fp32 logits, the `top` largest (ties: lower index first). weight (n, top) fp32, divided by
+// their sum if renormalize. Every choice gets a row of the buffer sorted by expert: the rows of an expert start at a multiple
+// of `tile`; row (n, top), tile_expert / tile_row (one entry per tile in use), plan[0] = number of tiles. counters: n_expert
+// ints of scratch.
+int kvb_moe_route(const float* logits, int* expert, float* weight, int* row, int* counters, int* plan, int* tile_expert,
+                  int* tile_row, long long n, int n_expert, int top, int tile, int max_tiles, int renormalize, void* stream);
+// sorted[row[n, k]] = h[n] (columns beyond width zero up to ld)
+int kvb_moe_gather(const void* h, const int* row, void* sorted, long long n, int top, int width, long long ld, int dtype, void* stream);
+// out[r] = act(w[expert of r's tile] · in[r]) for all rows of the tiles in use; in (rows, ldk), w (n_expert, n_out, ldk),
+// out (rows, ldo) with columns n_out .. ldo zero. act 0: none, 1: square of relu.
+int kvb_moe_gemm(const void* in, const void* w, void* out, const int* plan, const int* tile_expert, const int* tile_row, int tile,
+                 int max_tiles, int n_expert, int n_out, int k, long long ldk, long long ldo, int act, int dtype, int simple,
+                 int* status, void* stream);
+
+#ifdef __cplusplus
+}
+#endif

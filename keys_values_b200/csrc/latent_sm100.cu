@@ -1,0 +1,438 @@
+// Attention of several new tokens over keys and values expanded from latents, on tcgen05.
+//
+//   S = Q_u K_u^T + Q_r K_r^T (the rotated key part K_r is shared by the heads), P = exp2(S·c − m), O += P V
+//
+// The head sizes of keys (unrotated + rotated) and values differ and are run-time values: operands are staged as chunks of
+// 64 features ([128 rows x 128 B], 128B swizzle, TMA fills what lies beyond a tensor's last feature with zero), S sums over
+// the chunks of both parts, and the PV product has N = 64 · (value chunks). One CTA has NQT query tiles of 128 tokens of
+// one head, one softmax warpgroup each: with two tiles, one warpgroup works on its scores while the tensor core runs
+// PV and the next QK of the other. TMEM: NQT score tiles of 128 columns, NQT outputs of 64 · (value chunks) columns; P
+// aliases its S and is the A operand of the PV product.
+//
+// Masks are arithmetic: key row j of sequence b has position start[b] − P + j, query t sees
+// max(P + t − window + 1, P − start[b], 0) <= j <= P + t. Tiles outside the range of a query tile are skipped, tiles inside
+// the range of all its rows need no mask.
+#include <cuda.h>
+#include <limits.h>
+
+#include "common.cuh"
+#include "kvb200_layers.h"
+#include "tmap.cuh"
+
+namespace kvb {
+
+constexpr int LF_T = 128;
+constexpr int LF_CHUNK = LF_T * 128;  // bytes of [128 rows x 64 features]
+constexpr int LF_SMEM_LIMIT = 232448;
+constexpr int LF_SMEM_MIN = 120 * 1024;  // one CTA per SM: a CTA owns all 512 TMEM columns
+constexpr float LF_RESCALE_STEP = 8.f;   // log2 units
+constexpr int LF_MAX_STAGES = 4;
+
+struct LfParams {
+  __nv_bfloat16* out;
+  const int* start;
+  int B, heads, T, P, nQ, n_pair;
+  int nu, nr, nv;        // feature chunks of the unrotated / rotated key part and of the values
+  int ksu_last, ksr;     // 16-feature steps of the last unrotated chunk and of the rotated chunk(s) in total
+  int kst, vst;          // stages of K and V
+  int vdp, window;
+  float scale_log2;
+  int* status;
+};
+
+__device__ __forceinline__ float lf_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int NQT>
+__global__ void __launch_bounds__(64 + 128 * NQT, 1)
+latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant__ CUtensorMap tmQr,
+                    const __grid_constant__ CUtensorMap tmKu, const __grid_constant__ CUtensorMap tmKr,
+                    const __grid_constant__ CUtensorMap tmV, const LfParams p) {
+  extern __shared__ __align__(1024) uint8_t smem[];
+  if (smem_u32(smem) & 1023u) {
+    if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, STATUS_TIMEOUT_MISC);
+    return;
+  }
+  const int nk = p.nu + p.nr;
+  uint8_t* sQ = smem;
+  uint8_t* sK = sQ + NQT * nk * LF_CHUNK;
+  uint8_t* sV = sK + p.kst * nk * LF_CHUNK;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + p.vst * p.nv * LF_CHUNK);
+  uint64_t* q_full = bars;
+  uint64_t* o_full = bars + 1;
+  uint64_t* s_full = bars + 2;                 // [NQT]
+  uint64_t* p_full = bars + 4;                 // [NQT]
+  uint64_t* k_full = bars + 6;                 // [kst]
+  uint64_t* k_empty = k_full + LF_MAX_STAGES;
+  uint64_t* v_full = k_empty + LF_MAX_STAGES;  // [vst]
+  uint64_t* v_empty = v_full + LF_MAX_STAGES;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(v_empty + LF_MAX_STAGES);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pair = blockIdx.x % p.n_pair;
+  const int h = (blockIdx.x / p.n_pair) % p.heads;
+  const int b = blockIdx.x / (p.n_pair * p.heads);
+  const int lo_seq = max(0, p.P - p.start[b]);  // first key row that holds a token
+  // key tiles [ta, tb] of query tile u (empty if the tile has no query)
+  auto range = [&](int u, int& ta, int& tb) {
+    const int t0 = (pair * NQT + u) * LF_T;
+    if (t0 >= p.T) {
+      ta = INT_MAX;
+      tb = -1;
+      return;
+    }
+    const int t1 = min(t0 + LF_T, p.T) - 1;
+    const int lo = max(lo_seq, p.window > 0 ? p.P + t0 - p.window + 1 : 0);
+    ta = lo / LF_T;
+    tb = (p.P + t1) / LF_T;
+  };
+  int ra[NQT], rb[NQT];
+  int first = INT_MAX, last = -1;
+#pragma unroll
+  for (int u = 0; u < NQT; ++u) {
+    range(u, ra[u], rb[u]);
+    first = min(first, ra[u]);
+    last = max(last, rb[u]);
+  }
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    mbar_init(o_full, 1);
+    for (int u = 0; u < NQT; ++u) {
+      mbar_init(&s_full[u], 1);
+      mbar_init(&p_full[u], 4);
+    }
+    for (int i = 0; i < LF_MAX_STAGES; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_empty[i], 1);
+      mbar_init(&v_full[i], 1);
+      mbar_init(&v_empty[i], 1);
+    }
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  const int o_cols = 64 * p.nv;
+
+  if (warp == 0) {
+    // ------------------------------------------------------------ TMA producer
+    if (lane == 0) {
+      tma_prefetch_desc(&tmQu);
+      tma_prefetch_desc(&tmQr);
+      tma_prefetch_desc(&tmKu);
+      tma_prefetch_desc(&tmKr);
+      tma_prefetch_desc(&tmV);
+      mbar_expect_tx(q_full, (uint32_t)(NQT * nk * LF_CHUNK));
+      for (int u = 0; u < NQT; ++u) {
+        const int t0 = (pair * NQT + u) * LF_T;  // beyond T: zero rows
+        for (int c = 0; c < p.nu; ++c) tma_load_4d(sQ + (u * nk + c) * LF_CHUNK, &tmQu, q_full, 64 * c, h, t0, b);
+        for (int c = 0; c < p.nr; ++c) tma_load_4d(sQ + (u * nk + p.nu + c) * LF_CHUNK, &tmQr, q_full, 64 * c, h, t0, b);
+      }
+      bool ok = true;
+      int ks = 0, vs = 0;
+      uint32_t kph = 0, vph = 0;
+      for (int t = first; t <= last; ++t) {
+        if (!(ok = mbar_wait_bounded(&k_empty[ks], kph ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
+        mbar_expect_tx(&k_full[ks], (uint32_t)(nk * LF_CHUNK));
+        uint8_t* kd = sK + ks * nk * LF_CHUNK;
+        for (int c = 0; c < p.nu; ++c) tma_load_4d(kd + c * LF_CHUNK, &tmKu, &k_full[ks], 64 * c, h, t * LF_T, b);
+        for (int c = 0; c < p.nr; ++c) tma_load_4d(kd + (p.nu + c) * LF_CHUNK, &tmKr, &k_full[ks], 64 * c, 0, t * LF_T, b);
+        if (++ks == p.kst) {
+          ks = 0;
+          kph ^= 1;
+        }
+        if (!(ok = mbar_wait_bounded(&v_empty[vs], vph ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
+        mbar_expect_tx(&v_full[vs], (uint32_t)(p.nv * LF_CHUNK));
+        for (int c = 0; c < p.nv; ++c) tma_load_4d(sV + (vs * p.nv + c) * LF_CHUNK, &tmV, &v_full[vs], 64 * c, h, t * LF_T, b);
+        if (++vs == p.vst) {
+          vs = 0;
+          vph ^= 1;
+        }
+      }
+      if (!ok) {  // copies in flight get a bounded time to land before the shared memory is released
+        const long long c0 = clock64();
+        while (clock64() - c0 < 2000000LL) {
+        }
+      }
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------- MMA issuer
+    if (lane == 0) {
+      constexpr uint32_t idesc_qk = make_idesc_bf16(LF_T, LF_T, 0, 0);
+      const uint32_t idesc_pv = make_idesc_bf16(LF_T, o_cols, 0, 1);
+      const uint32_t q_addr = smem_u32(sQ), k_addr = smem_u32(sK), v_addr = smem_u32(sV);
+      const int su = (p.nu - 1) * 4 + p.ksu_last;  // 16-feature steps of the unrotated part
+      const int steps = su + p.ksr;
+      bool ok = mbar_wait_bounded(q_full, 0, abort_flag, p.status, STATUS_TIMEOUT_FULL);
+      int ks = 0, vs = 0;
+      uint32_t kph = 0, vph = 0;
+      uint32_t pph[NQT];
+#pragma unroll
+      for (int u = 0; u < NQT; ++u) pph[u] = 0;
+      for (int t = first; t <= last + 1 && ok; ++t) {
+        const bool have_k = t <= last, have_v = t > first;
+        bool k_ready = false, v_ready = false;
+#pragma unroll
+        for (int u = 0; u < NQT; ++u) {
+          if (have_v && t - 1 >= ra[u] && t - 1 <= rb[u]) {
+            if (!v_ready) {
+              if (!(ok = mbar_wait_bounded(&v_full[vs], vph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
+              v_ready = true;
+            }
+            if (!(ok = mbar_wait_bounded(&p_full[u], pph[u], abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
+            pph[u] ^= 1;
+            tc_fence_after();
+#pragma unroll
+            for (int kk = 0; kk < 8; ++kk)
+              umma_f16_ts(tmem_base + (uint32_t)(NQT * LF_T + u * o_cols), tmem_base + (uint32_t)(u * LF_T + 8 * kk),
+                          make_smem_desc_sw128(v_addr + (uint32_t)(vs * p.nv * LF_CHUNK + kk * 16 * 128), LF_CHUNK, 1024), idesc_pv,
+                          (t - 1 == ra[u] && kk == 0) ? 0u : 1u);
+          }
+          if (have_k && t >= ra[u] && t <= rb[u]) {
+            if (!k_ready) {
+              if (!(ok = mbar_wait_bounded(&k_full[ks], kph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
+              k_ready = true;
+            }
+            tc_fence_after();
+            for (int s = 0; s < steps; ++s) {
+              const int c = s < su ? (s >> 2) : p.nu + ((s - su) >> 2);
+              const int kk = s < su ? (s & 3) : ((s - su) & 3);
+              const uint32_t off = (uint32_t)(c * LF_CHUNK + kk * 32);
+              umma_f16_ss(tmem_base + (uint32_t)(u * LF_T), make_smem_desc_sw128(q_addr + (uint32_t)(u * nk * LF_CHUNK) + off, 16, 1024),
+                          make_smem_desc_sw128(k_addr + (uint32_t)(ks * nk * LF_CHUNK) + off, 16, 1024), idesc_qk, s != 0 ? 1u : 0u);
+            }
+            umma_commit(&s_full[u]);
+          }
+        }
+        if (!ok) break;
+        if (have_v) {
+          // a stage that no query tile of this CTA reads cannot occur between first and last: the ranges overlap or touch
+          umma_commit(&v_empty[vs]);
+          if (!v_ready && !(ok = mbar_wait_bounded(&v_full[vs], vph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
+          if (++vs == p.vst) {
+            vs = 0;
+            vph ^= 1;
+          }
+        }
+        if (have_k) {
+          umma_commit(&k_empty[ks]);
+          if (!k_ready && !(ok = mbar_wait_bounded(&k_full[ks], kph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
+          if (++ks == p.kst) {
+            ks = 0;
+            kph ^= 1;
+          }
+        }
+      }
+      if (ok) umma_commit(o_full);
+    }
+  } else {
+    // ------------------------------------------------- softmax + epilogue, one warpgroup per query tile
+    const int u = NQT == 1 ? 0 : (warp - 2) >> 2;
+    const int quarter = warp & 3;
+    const int row = quarter * 32 + lane;
+    const int t0 = (pair * NQT + u) * LF_T;
+    const int tq = t0 + row;
+    const int my_ra = u == 0 ? ra[0] : ra[NQT - 1], my_rb = u == 0 ? rb[0] : rb[NQT - 1];
+    const int hi = p.P + tq;
+    const int lo = max(lo_seq, p.window > 0 ? hi - p.window + 1 : 0);
+    // rows of the tile: all see keys in [lo of the last row, hi of the first row]
+    const int lo_max = max(lo_seq, p.window > 0 ? p.P + t0 + LF_T - 1 - p.window + 1 : 0), hi_min = p.P + t0;
+    const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
+    const uint32_t tmem_S = tmem_base + (uint32_t)(u * LF_T) + lane_base;
+    const uint32_t tmem_O = tmem_base + (uint32_t)(NQT * LF_T + u * o_cols) + lane_base;
+    const float c = p.scale_log2;
+    const float2 c2 = make_float2(c, c);
+    float m_used = -1e30f, l = 0.f;
+    bool ok = true;
+    uint32_t ph = 0;
+    for (int t = my_ra; t <= my_rb; ++t) {
+      if (!(ok = mbar_wait_bounded(&s_full[u], ph, abort_flag, p.status, STATUS_TIMEOUT_TMEM_FULL))) break;
+      ph ^= 1;
+      tc_fence_after();
+      uint32_t x[LF_T];
+#pragma unroll
+      for (int w = 0; w < 4; ++w) tmem_ld_32x32b_x32(tmem_S + (uint32_t)(32 * w), x + 32 * w);
+      tmem_ld_wait();
+      const int j0 = t * LF_T;
+      if (j0 < lo_max || j0 + LF_T - 1 > hi_min) {
+        const uint32_t span = (uint32_t)(hi - lo);
+        const uint32_t off = (uint32_t)(j0 - lo);
+#pragma unroll
+        for (int e = 0; e < LF_T; ++e)
+          if (off + (uint32_t)e > span) x[e] = 0xff800000u;
+      }
+      float a8[8];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) a8[i] = fmaxf(__uint_as_float(x[i]), __uint_as_float(x[8 + i]));
+#pragma unroll
+      for (int e = 16; e < LF_T; e += 16)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) a8[i] = fmax3(a8[i], __uint_as_float(x[e + 2 * i]), __uint_as_float(x[e + 2 * i + 1]));
+      const float m_tile = fmax3(fmax3(a8[0], a8[1], a8[2]), fmax3(a8[3], a8[4], a8[5]), fmaxf(a8[6], a8[7])) * c;
+      const bool raise = m_tile > m_used + LF_RESCALE_STEP;
+      const float m_new = raise ? m_tile : m_used;
+      // the PV product of the previous tile was issued before this tile's scores: it is complete, O is quiet
+      if (t > my_ra && __any_sync(0xffffffffu, raise)) {
+        const float f = raise ? lf_exp2(m_used - m_new) : 1.f;
+        l *= f;
+#pragma unroll 1
+        for (int c0 = 0; c0 < o_cols; c0 += 16) {
+          uint32_t o[16];
+          tmem_ld_32x32b_x16(tmem_O + (uint32_t)c0, o);
+          tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * f);
+          tmem_st_32x32b_x16(tmem_O + (uint32_t)c0, o);
+        }
+      }
+      m_used = m_new;
+      const float2 neg_m2 = make_float2(-m_used, -m_used);
+      float2 s0 = make_float2(0.f, 0.f), s1 = s0;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int e = 0; e < 32; e += 4) {
+          const uint32_t* xe = x + 32 * w + e;
+          const float2 x0 = ffma2(make_float2(__uint_as_float(xe[0]), __uint_as_float(xe[1])), c2, neg_m2);
+          const float2 x1 = ffma2(make_float2(__uint_as_float(xe[2]), __uint_as_float(xe[3])), c2, neg_m2);
+          const float2 y0 = make_float2(lf_exp2(x0.x), lf_exp2(x0.y));
+          const float2 y1 = make_float2(lf_exp2(x1.x), lf_exp2(x1.y));
+          s0 = fadd2(s0, y0);
+          s1 = fadd2(s1, y1);
+          pk[e >> 1] = pack_bf16x2(y0.x, y0.y);
+          pk[(e >> 1) + 1] = pack_bf16x2(y1.x, y1.y);
+        }
+        tmem_st_32x32b_x16(tmem_S + (uint32_t)(16 * w), pk);
+      }
+      s0 = fadd2(s0, s1);
+      l += s0.x + s0.y;
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&p_full[u]);
+    }
+    if (ok) ok = mbar_wait_bounded(o_full, 0, abort_flag, p.status, STATUS_TIMEOUT_TMEM_FULL);
+    if (ok && my_rb >= my_ra) {
+      tc_fence_after();
+      const float inv_l = l > 0.f ? 1.f / l : 0.f;
+      __nv_bfloat16* dst = p.out + (((long long)b * p.T + (tq < p.T ? tq : 0)) * p.heads + h) * p.vdp;
+#pragma unroll 1
+      for (int c0 = 0; c0 < p.vdp; c0 += 16) {
+        uint32_t o[16];
+        tmem_ld_32x32b_x16(tmem_O + (uint32_t)c0, o);
+        tmem_ld_wait();
+        if (tq < p.T) {
+#pragma unroll
+          for (int i = 0; i < 2; ++i) {
+            if (c0 + 8 * i >= p.vdp) break;
+            uint4 v;
+            v.x = pack_bf16x2(__uint_as_float(o[8 * i + 0]) * inv_l, __uint_as_float(o[8 * i + 1]) * inv_l);
+            v.y = pack_bf16x2(__uint_as_float(o[8 * i + 2]) * inv_l, __uint_as_float(o[8 * i + 3]) * inv_l);
+            v.z = pack_bf16x2(__uint_as_float(o[8 * i + 4]) * inv_l, __uint_as_float(o[8 * i + 5]) * inv_l);
+            v.w = pack_bf16x2(__uint_as_float(o[8 * i + 6]) * inv_l, __uint_as_float(o[8 * i + 7]) * inv_l);
+            *reinterpret_cast<uint4*>(dst + c0 + 8 * i) = v;
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+struct LfPlan {
+  int nqt, nu, nr, nv, kst, vst;
+  int smem;
+};
+
+// query tiles per CTA and stages that fit into shared and tensor memory; nqt = 0: not supported
+static LfPlan lf_plan(int dimp, int rp, int vdp) {
+  LfPlan pl;
+  pl.nqt = 0;
+  pl.nu = (dimp + 63) / 64;
+  pl.nr = (rp + 63) / 64;
+  pl.nv = (vdp + 63) / 64;
+  const int nk = pl.nu + pl.nr;
+  if (dimp <= 0 || rp <= 0 || vdp <= 0 || pl.nv > 4) return pl;
+  const int limit = LF_SMEM_LIMIT - 512;
+  for (int nqt = 2; nqt >= 1; --nqt) {
+    if (nqt * (LF_T + 64 * pl.nv) > 512) continue;
+    static const int stages[][2] = {{3, 3}, {2, 2}, {2, 1}, {1, 1}};
+    for (auto& st : stages) {
+      const int bytes = (nqt * nk + st[0] * nk + st[1] * pl.nv) * LF_CHUNK;
+      if (bytes > limit || (nqt == 2 && st[0] == 1)) continue;
+      pl.nqt = nqt;
+      pl.kst = st[0];
+      pl.vst = st[1];
+      pl.smem = bytes + 512 < LF_SMEM_MIN ? LF_SMEM_MIN : bytes + 512;
+      return pl;
+    }
+  }
+  return pl;
+}
+
+template <int NQT>
+static int lf_launch(const CUtensorMap* tm, LfParams& p, int smem, cudaStream_t s) {
+  static PerDeviceOnce once;
+  if (once.first()) cudaFuncSetAttribute(latent_flash_kernel<NQT>, cudaFuncAttributeMaxDynamicSharedMemorySize, LF_SMEM_LIMIT);
+  p.n_pair = (p.nQ + NQT - 1) / NQT;
+  latent_flash_kernel<NQT><<<p.B * p.heads * p.n_pair, 64 + 128 * NQT, smem, s>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+}  // namespace kvb
+
+extern "C" int kvb_latent_attend_tc_supported(int dimp, int rp, int vdp) {
+  return (dimp % 8 == 0 && rp % 8 == 0 && vdp % 8 == 0 && kvb::lf_plan(dimp, rp, vdp).nqt > 0) ? 1 : 0;
+}
+
+extern "C" int kvb_latent_attend_tc(const void* q, const void* kv, const void* latent, void* out, const int* start, int B, int T, int P,
+                                    int heads, int dimp, int rp, int kvp, int vdp, int window, float scale, int* status, void* stream) {
+  using namespace kvb;
+  if (B <= 0 || T <= 0 || P < 0 || heads <= 0 || window < 0 || !(scale > 0.f)) return KVB_ERR_ARG;
+  if ((dimp | rp | vdp | kvp) % 8) return KVB_ERR_ALIGN;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(latent) |
+       reinterpret_cast<uintptr_t>(out)) & 15)
+    return KVB_ERR_ALIGN;
+  const LfPlan pl = lf_plan(dimp, rp, vdp);
+  if (!pl.nqt) return KVB_ERR_UNSUPPORTED;
+  const uint64_t dq = dimp + rp, row = dimp + vdp, lw = kvp + rp, n = (uint64_t)P + T;
+  const uint32_t box[4] = {64, 1, LF_T, 1};
+  CUtensorMap tm[5];
+  int rc;
+  const __nv_bfloat16 *qb = (const __nv_bfloat16*)q, *kb = (const __nv_bfloat16*)kv, *lb = (const __nv_bfloat16*)latent;
+  const uint64_t sq[3] = {dq, heads * dq, (uint64_t)T * heads * dq};
+  const uint64_t sk[3] = {row, heads * row, n * heads * row};
+  const uint64_t sl[3] = {lw, lw, n * lw};
+  const uint64_t dqu[4] = {(uint64_t)dimp, (uint64_t)heads, (uint64_t)T, (uint64_t)B}, dqr[4] = {(uint64_t)rp, (uint64_t)heads, (uint64_t)T, (uint64_t)B};
+  const uint64_t dku[4] = {(uint64_t)dimp, (uint64_t)heads, n, (uint64_t)B}, dkr[4] = {(uint64_t)rp, 1, n, (uint64_t)B};
+  const uint64_t dv[4] = {(uint64_t)vdp, (uint64_t)heads, n, (uint64_t)B};
+  if ((rc = tmap_bf16(&tm[0], qb, 4, dqu, sq, box))) return rc;
+  if ((rc = tmap_bf16(&tm[1], qb + dimp, 4, dqr, sq, box))) return rc;
+  if ((rc = tmap_bf16(&tm[2], kb, 4, dku, sk, box))) return rc;
+  if ((rc = tmap_bf16(&tm[3], lb + kvp, 4, dkr, sl, box))) return rc;
+  if ((rc = tmap_bf16(&tm[4], kb + dimp, 4, dv, sk, box))) return rc;
+  LfParams p;
+  p.out = (__nv_bfloat16*)out; p.start = start;
+  p.B = B; p.heads = heads; p.T = T; p.P = P; p.nQ = (T + LF_T - 1) / LF_T;
+  p.nu = pl.nu; p.nr = pl.nr; p.nv = pl.nv; p.kst = pl.kst; p.vst = pl.vst;
+  p.ksu_last = (dimp - 64 * (pl.nu - 1) + 15) / 16;
+  p.ksr = (rp + 15) / 16;
+  p.vdp = vdp; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
+  return pl.nqt == 2 ? lf_launch<2>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1>(tm, p, pl.smem, (cudaStream_t)stream);
+}

@@ -1,0 +1,260 @@
+// Routed experts: softmax router with top-k choice, rows sorted by expert, grouped products.
+//
+//   route  one warp per token: softmax over the fp32 router logits, the k largest, a rank within every chosen expert;
+//   plan   one CTA: rows of an expert start at a multiple of the row tile; table of tiles for the grouped products;
+//   gather rows of the chosen tokens into the sorted buffer;
+//   gemm   out = act(W_e · in) per tile of rows of one expert. bf16: tcgen05 with the expert's weight rows as the
+//          M = 128 operand and the tokens as N (16 .. 256 columns), so that a decode step with a handful of tokens per
+//          expert streams the weights without padding the token side to 128; fp32: CUDA cores.
+// The weighted sum over a token's experts is part of the kernel that closes the layer (layer_edge.cu).
+#include <cuda.h>
+
+#include "common.cuh"
+#include "kvb200_layers.h"
+
+namespace kvb {
+
+constexpr int ROUTE_WARPS = 4;
+constexpr int ROUTE_MAX_EXPERTS = 2048;
+
+__global__ void __launch_bounds__(ROUTE_WARPS * 32)
+moe_route_kernel(const float* __restrict__ logits, int* __restrict__ expert, float* __restrict__ weight, int* __restrict__ row,
+                 int* __restrict__ counters, long long n, int E, int top, int renormalize) {
+  extern __shared__ float sc_all[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* sc = sc_all + warp * E;
+  const long long tok = (long long)blockIdx.x * ROUTE_WARPS + warp;
+  if (tok >= n) return;
+  const float* z = logits + tok * E;
+  float m = -INFINITY;
+  for (int e = lane; e < E; e += 32) {
+    const float v = z[e];
+    sc[e] = v;
+    m = fmaxf(m, v);
+  }
+  m = warp_max(m);
+  float l = 0.f;
+  for (int e = lane; e < E; e += 32) {
+    const float v = expf(sc[e] - m);
+    sc[e] = v;
+    l += v;
+  }
+  l = warp_sum(l);
+  __syncwarp();
+  float chosen = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -2.f;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const float v = sc[e];
+      if (v > best) {
+        best = v;
+        bi = e;
+      }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > best || (ov == best && oi < bi)) {
+        best = ov;
+        bi = oi;
+      }
+    }
+    if (bi >= E) bi = 0;  // scores that are not numbers: any expert
+    const float w = best / l;
+    chosen += w;
+    if (lane == 0) {
+      expert[tok * top + k] = bi;
+      weight[tok * top + k] = w;
+      row[tok * top + k] = atomicAdd(&counters[bi], 1);
+      sc[bi] = -1.f;
+    }
+    __syncwarp();
+  }
+  if (renormalize && lane < top)
+    for (int k = lane; k < top; k += 32) weight[tok * top + k] = weight[tok * top + k] / chosen;
+}
+
+// Exclusive prefix over the experts' tile counts, tile table. One CTA of 1024 threads.
+__global__ void __launch_bounds__(1024)
+moe_plan_kernel(int* __restrict__ counters, int* __restrict__ plan, int* __restrict__ tile_expert, int* __restrict__ tile_row, int E,
+                int tile, int max_tiles) {
+  __shared__ int sums[32];
+  __shared__ int carry;
+  if (threadIdx.x == 0) carry = 0;
+  __syncthreads();
+  for (int e0 = 0; e0 < E; e0 += 1024) {
+    const int e = e0 + threadIdx.x;
+    const int nt = e < E ? (counters[e] + tile - 1) / tile : 0;
+    int v = nt;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int t = __shfl_up_sync(0xffffffffu, v, o);
+      if (lane >= o) v += t;
+    }
+    if (lane == 31) sums[warp] = v;
+    __syncthreads();
+    if (warp == 0) {
+      int s = sums[lane];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int t = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += t;
+      }
+      sums[lane] = s;
+    }
+    __syncthreads();
+    const int base = carry + (warp > 0 ? sums[warp - 1] : 0) + v - nt;
+    if (e < E) {
+      counters[e] = base * tile;  // first row of the expert
+      for (int i = 0; i < nt && base + i < max_tiles; ++i) {
+        tile_expert[base + i] = e;
+        tile_row[base + i] = (base + i) * tile;
+      }
+    }
+    __syncthreads();
+    if (threadIdx.x == 1023) carry += sums[31];
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) plan[0] = min(carry, max_tiles);
+}
+
+__global__ void moe_rows_kernel(const int* __restrict__ expert, const int* __restrict__ counters, int* __restrict__ row, long long n) {
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) row[i] += counters[expert[i]];
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+moe_gather_kernel(const T* __restrict__ h, const int* __restrict__ row, T* __restrict__ sorted, int top, int width, long long ld) {
+  struct alignas(sizeof(T) * V) Vec { T v[V]; };
+  const long long n = blockIdx.x;
+  for (int c = threadIdx.x * V; c < ld; c += 128 * V) {
+    Vec x;
+    if (c < width) {
+      x = *reinterpret_cast<const Vec*>(h + n * width + c);
+    } else {
+#pragma unroll
+      for (int i = 0; i < V; ++i) x.v[i] = from_f32<T>(0.f);
+    }
+    for (int k = 0; k < top; ++k) *reinterpret_cast<Vec*>(sorted + (long long)row[n * top + k] * ld + c) = x;
+  }
+}
+
+__device__ __forceinline__ float moe_act(float v, int act) {
+  if (act == 1) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  return v;
+}
+
+// ---- CUDA-core product: 32 rows x 64 features per CTA
+constexpr int MS_R = 32, MS_F = 64, MS_K = 32;
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __restrict__ out, const int* __restrict__ plan,
+                       const int* __restrict__ tile_expert, const int* __restrict__ tile_row, int tile, int n_out, int k, long long ldk,
+                       long long ldo, int act) {
+  __shared__ float sa[MS_K][MS_R + 1];
+  __shared__ float sw[MS_K][MS_F + 1];
+  const int sub = tile / MS_R;
+  const int ti = blockIdx.x / sub;
+  if (ti >= plan[0]) return;
+  const long long r0 = (long long)tile_row[ti] + (blockIdx.x % sub) * MS_R;
+  const long long e = tile_expert[ti];
+  const int f0 = blockIdx.y * MS_F;
+  const T* we = w + e * n_out * ldk;
+  const int tr = threadIdx.x / 32, tf = threadIdx.x % 32;  // rows tr + 8 i, features tf and tf + 32
+  float acc[4][2] = {};
+  for (int k0 = 0; k0 < k; k0 += MS_K) {
+    for (int i = threadIdx.x; i < MS_R * MS_K; i += 256) {
+      const int r = i / MS_K, kk = i % MS_K;
+      sa[kk][r] = k0 + kk < k ? to_f32(in[(r0 + r) * ldk + k0 + kk]) : 0.f;
+    }
+    for (int i = threadIdx.x; i < MS_F * MS_K; i += 256) {
+      const int f = i / MS_K, kk = i % MS_K;
+      sw[kk][f] = (f0 + f < n_out && k0 + kk < k) ? to_f32(we[(long long)(f0 + f) * ldk + k0 + kk]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int kk = 0; kk < MS_K; ++kk) {
+      const float w0 = sw[kk][tf], w1 = sw[kk][tf + 32];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float a = sa[kk][tr + 8 * i];
+        acc[i][0] = fmaf(a, w0, acc[i][0]);
+        acc[i][1] = fmaf(a, w1, acc[i][1]);
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 2; ++j) {
+      const int f = f0 + tf + 32 * j;
+      if (f < ldo) out[(r0 + tr + 8 * i) * ldo + f] = from_f32<T>(f < n_out ? moe_act(acc[i][j], act) : 0.f);
+    }
+}
+
+int moe_gemm_tc(const void* in, const void* w, void* out, const int* plan, const int* tile_expert, const int* tile_row, int tile,
+                int max_tiles, int n_expert, int n_out, int k, long long ldk, long long ldo, int act, int* status, cudaStream_t s);
+
+}  // namespace kvb
+
+extern "C" int kvb_moe_route(const float* logits, int* expert, float* weight, int* row, int* counters, int* plan, int* tile_expert,
+                             int* tile_row, long long n, int n_expert, int top, int tile, int max_tiles, int renormalize, void* stream) {
+  using namespace kvb;
+  if (n <= 0 || n_expert <= 0 || top <= 0 || top > n_expert || tile <= 0) return KVB_ERR_ARG;
+  if (n_expert > ROUTE_MAX_EXPERTS) return KVB_ERR_TOO_LARGE;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (cudaMemsetAsync(counters, 0, sizeof(int) * n_expert, s) != cudaSuccess) return KVB_ERR_CUDA;
+  moe_route_kernel<<<(unsigned)((n + ROUTE_WARPS - 1) / ROUTE_WARPS), ROUTE_WARPS * 32, ROUTE_WARPS * n_expert * sizeof(float), s>>>(
+      logits, expert, weight, row, counters, n, n_expert, top, renormalize);
+  moe_plan_kernel<<<1, 1024, 0, s>>>(counters, plan, tile_expert, tile_row, n_expert, tile, max_tiles);
+  const long long m = n * top;
+  moe_rows_kernel<<<(unsigned)((m + 255) / 256), 256, 0, s>>>(expert, counters, row, m);
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+extern "C" int kvb_moe_gather(const void* h, const int* row, void* sorted, long long n, int top, int width, long long ld, int dtype,
+                              void* stream) {
+  using namespace kvb;
+  if (n <= 0 || top <= 0 || ld < width) return KVB_ERR_ARG;
+  cudaStream_t s = (cudaStream_t)stream;
+  const unsigned g = (unsigned)n;
+  const bool vec = width % 8 == 0 && ld % 8 == 0;
+  if (dtype == 0) {
+    if (vec) moe_gather_kernel<float, 4><<<g, 128, 0, s>>>((const float*)h, row, (float*)sorted, top, width, ld);
+    else moe_gather_kernel<float, 1><<<g, 128, 0, s>>>((const float*)h, row, (float*)sorted, top, width, ld);
+  } else if (dtype == 1) {
+    if (vec) moe_gather_kernel<__nv_bfloat16, 8><<<g, 128, 0, s>>>((const __nv_bfloat16*)h, row, (__nv_bfloat16*)sorted, top, width, ld);
+    else moe_gather_kernel<__nv_bfloat16, 1><<<g, 128, 0, s>>>((const __nv_bfloat16*)h, row, (__nv_bfloat16*)sorted, top, width, ld);
+  } else {
+    return KVB_ERR_ARG;
+  }
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+extern "C" int kvb_moe_gemm(const void* in, const void* w, void* out, const int* plan, const int* tile_expert, const int* tile_row,
+                            int tile, int max_tiles, int n_expert, int n_out, int k, long long ldk, long long ldo, int act, int dtype,
+                            int simple, int* status, void* stream) {
+  using namespace kvb;
+  if (max_tiles <= 0 || n_out <= 0 || k <= 0 || ldk < k || ldo < n_out || tile <= 0) return KVB_ERR_ARG;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (dtype == 1 && !simple)
+    return moe_gemm_tc(in, w, out, plan, tile_expert, tile_row, tile, max_tiles, n_expert, n_out, k, ldk, ldo, act, status, s);
+  if (tile % MS_R) return KVB_ERR_ARG;
+  const dim3 grid(max_tiles * (tile / MS_R), (unsigned)((ldo + MS_F - 1) / MS_F));
+  if (dtype == 0)
+    moe_gemm_simple_kernel<float><<<grid, 256, 0, s>>>((const float*)in, (const float*)w, (float*)out, plan, tile_expert, tile_row, tile,
+                                                       n_out, k, ldk, ldo, act);
+  else if (dtype == 1)
+    moe_gemm_simple_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>((const __nv_bfloat16*)in, (const __nv_bfloat16*)w, (__nv_bfloat16*)out,
+                                                               plan, tile_expert, tile_row, tile, n_out, k, ldk, ldo, act);
+  else return KVB_ERR_ARG;
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}

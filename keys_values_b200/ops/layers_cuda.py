@@ -1,0 +1,186 @@
+"""ctypes bindings to ``libkvb200_layers.so``: kernels of models that are described layer by layer.
+
+Same conventions as :mod:`keys_values_b200.ops.cuda` (outputs allocated with torch, raw pointers plus the
+current stream, status code checked); launches are counted and device-side errors reported through
+the same status word.
+"""
+from __future__ import annotations
+
+import ctypes
+from typing import Optional
+
+import torch
+
+from keys_values_b200.ops import cuda as _base
+from keys_values_b200.ops.cuda import NativeError, _check, _count, _ll, _p, _stream, status_word
+
+_LIB = None
+LIB_PATH = _base._ROOT / "libkvb200_layers.so"
+_CODE = {torch.float32: 0, torch.bfloat16: 1}
+# True: the CUDA-core kernels serve bf16 too (comparisons in tests and benchmarks)
+FORCE_SIMPLE = False
+
+
+def lib():
+    global _LIB
+    if _LIB is None:
+        if not LIB_PATH.exists():
+            raise NativeError(f"{LIB_PATH} is missing: run `python -m keys_values_b200.build_ext`")
+        _LIB = ctypes.CDLL(str(LIB_PATH))
+        _LIB.kvb_latent_decode_scratch_bytes.restype = ctypes.c_longlong
+    return _LIB
+
+
+def code(dtype: torch.dtype) -> int:
+    try:
+        return _CODE[dtype]
+    except KeyError:
+        raise NativeError(f"dtype {dtype}: these kernels exist for bfloat16 and float32")
+
+
+def _f(x: float) -> ctypes.c_float:
+    return ctypes.c_float(float(x))
+
+
+def _contiguous(*tensors) -> None:
+    for t in tensors:
+        if t is not None and not t.is_contiguous():
+            raise NativeError("layer kernels take contiguous tensors")
+
+
+# ---------------------------------------------------------------------------------------------- layer edges
+def embed_edge(idx, prev_token, embed, bigram, buckets, mul_prev, mul_cur, hist, gain, shift, state, h, hs, seq, eps) -> None:
+    B, T = idx.shape
+    _contiguous(idx, embed, bigram, hist, gain, shift, state, h, hs)
+    _check(lib().kvb_embed_edge(_p(idx), _p(prev_token), _p(embed), _p(bigram), _ll(buckets), _ll(mul_prev), _ll(mul_cur), _p(hist),
+                                _p(gain), _p(shift), _p(state), _p(h), _p(hs), _p(seq.slots), _p(seq.start), _p(seq.count), B, T,
+                                embed.shape[1], _ll(embed.shape[0]), _f(eps), code(embed.dtype), _p(status_word(idx.device)),
+                                _stream(idx)), "embed_edge")
+    _count()
+
+
+def layer_edge(x_in, mix, expert_out, expert_row, expert_w, hist, n_hist, coef, x_out, gain, shift, state, h, hs, seq, eps) -> None:
+    B, T, width = x_in.shape
+    _contiguous(x_in, mix, expert_out, expert_row, expert_w, coef, x_out, gain, shift, state, h, hs)
+    top = 0 if expert_w is None else expert_w.shape[1]
+    ld = 0 if expert_out is None else expert_out.shape[1]
+    _check(lib().kvb_layer_edge(_p(x_in), _p(mix), _p(expert_out), _p(expert_row), _p(expert_w), top, _ll(ld), _p(hist), n_hist,
+                                _ll(0 if hist is None else hist.stride(0)), _p(coef), _p(x_out), _p(gain), _p(shift), _p(state), _p(h),
+                                _p(hs), _p(seq.slots), _p(seq.start), _p(seq.count), B, T, width, _f(eps), code(mix.dtype),
+                                _stream(x_in)), "layer_edge")
+    _count()
+
+
+def scalar_rmsnorm(x, rows, gain, eps, dtype) -> torch.Tensor:
+    n = x.shape[0] if rows is None else rows.numel()
+    y = torch.empty((n, x.shape[1]), dtype=dtype, device=x.device)
+    _contiguous(x, rows, gain)
+    _check(lib().kvb_scalar_rmsnorm(_p(x), _p(rows), _p(gain), _p(y), _ll(n), x.shape[1], _f(eps), code(dtype), _stream(x)), "scalar_rmsnorm")
+    _count()
+    return y
+
+
+def sequence_advance(idx, pos, prev_token, seq) -> None:
+    B, T = idx.shape
+    _contiguous(idx)
+    _check(lib().kvb_sequence_advance(_p(idx), _p(pos), _p(prev_token), _p(seq.slots), _p(seq.count), B, T, _stream(idx)), "sequence_advance")
+    _count()
+
+
+# ------------------------------------------------------------------------------------------- latent attention
+def latent_prep(qkv, norm_w, freq, latent, ring, seq, P, shape, eps) -> torch.Tensor:
+    """``qkv (B, T, ·)`` → padded queries ``(B, T, heads, dimp + rp)``; latent rows go to ``latent`` or straight into ``ring``."""
+    B, T, ld = qkv.shape
+    s = shape
+    q = torch.empty((B, T, s.heads, s.dimp + s.rp), dtype=qkv.dtype, device=qkv.device)
+    _contiguous(qkv, norm_w, freq, latent, ring)
+    _check(lib().kvb_latent_prep(_p(qkv), _ll(ld), _p(norm_w), _p(freq), _p(q), _p(latent), _p(ring), _p(seq.slots), _p(seq.start),
+                                 _p(seq.count), B, T, P, 0 if ring is None else ring.shape[1], s.heads, s.dim, s.dimp, s.rot, s.rot_dims,
+                                 s.rp, s.kv_rank, s.kvp, _f(eps), code(qkv.dtype), _stream(qkv)), "latent_prep")
+    _count()
+    return q
+
+
+def ring_gather(ring, latent, seq, P) -> None:
+    B, n, lw = latent.shape
+    _check(lib().kvb_ring_gather(_p(ring), _p(latent), _p(seq.slots), _p(seq.start), B, n - P, P, ring.shape[1], lw, code(ring.dtype),
+                                 _stream(ring)), "ring_gather")
+    _count()
+
+
+def ring_append(latent, ring, seq, P) -> None:
+    B, n, lw = latent.shape
+    _check(lib().kvb_ring_append(_p(latent), _p(ring), _p(seq.slots), _p(seq.start), _p(seq.count), B, n - P, P, ring.shape[1], lw,
+                                 code(ring.dtype), _stream(ring)), "ring_append")
+    _count()
+
+
+def latent_attend(q, kv, latent, seq, P, shape, window, scale) -> torch.Tensor:
+    B, T = q.shape[:2]
+    s = shape
+    out = torch.empty((B, T, s.heads * s.vdp), dtype=q.dtype, device=q.device)
+    _contiguous(q, kv, latent)
+    args = (B, T, P, s.heads, s.dimp, s.rp, s.kvp, s.vdp, int(window), _f(scale))
+    if q.dtype == torch.bfloat16 and not FORCE_SIMPLE and lib().kvb_latent_attend_tc_supported(s.dimp, s.rp, s.vdp):
+        _check(lib().kvb_latent_attend_tc(_p(q), _p(kv), _p(latent), _p(out), _p(seq.start), *args, _p(status_word(q.device)), _stream(q)),
+               "latent_attend_tc")
+    else:
+        _check(lib().kvb_latent_attend(_p(q), _p(kv), _p(latent), _p(out), _p(seq.start), *args, code(q.dtype), _stream(q)), "latent_attend")
+    _count()
+    return out
+
+
+def latent_decode(q_abs, q, ring, seq, shape, scale) -> torch.Tensor:
+    """``q_abs (heads, B, kvp)``, ``q (B, 1, heads, dimp + rp)`` → weighted latents ``(heads, B, kvp)``."""
+    s = shape
+    H, B, kvp = q_abs.shape
+    C = ring.shape[1]
+    out = torch.empty_like(q_abs)
+    _contiguous(q_abs, q, ring)
+    nbytes = int(lib().kvb_latent_decode_scratch_bytes(B, H, kvp, C))
+    scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
+    _check(lib().kvb_latent_decode(_p(q_abs), _p(q), _p(ring), _p(out), _p(scratch), _p(seq.slots), _p(seq.start), B, H, s.dimp, s.rp, kvp,
+                                   C, _f(scale), code(q.dtype), int(FORCE_SIMPLE), _stream(q)), "latent_decode")
+    _count()
+    return out
+
+
+# ---------------------------------------------------------------------------------------------- routed experts
+def moe_tile(n_choices: int, n_expert: int, dtype: torch.dtype) -> int:
+    """Rows per tile of the grouped products: the expected number of tokens per expert, 16 … 256."""
+    if dtype != torch.bfloat16 or FORCE_SIMPLE:
+        return 32
+    per = n_choices / n_expert
+    tile = 16
+    while tile < 256 and tile < per:
+        tile *= 2
+    return tile
+
+
+def moe_forward(h, logits, up, down, top: int, act: int, renormalize: bool, n_up: int, n_down: int):
+    """``h (n, width)``, fp32 router ``logits (n, E)``, ``up (E, ff, ldw)``, ``down (E, width, ldf)`` (rows padded to
+    multiples of 8). Returns ``(expert_out, row (n, top), weight (n, top))``: row of every choice in ``expert_out``."""
+    n, width = h.shape
+    E = logits.shape[1]
+    dev, dt = h.device, h.dtype
+    _contiguous(h, logits, up, down)
+    tile = moe_tile(n * top, E, dt)
+    max_tiles = n * top // tile + min(E, n * top)
+    ints = torch.empty(E + 2 * n * top + 1 + 2 * max_tiles, dtype=torch.int32, device=dev)
+    counters, expert, row, plan, tile_expert, tile_row = torch.split(ints, [E, n * top, n * top, 1, max_tiles, max_tiles])
+    weight = torch.empty((n, top), dtype=torch.float32, device=dev)
+    _check(lib().kvb_moe_route(_p(logits), _p(expert), _p(weight), _p(row), _p(counters), _p(plan), _p(tile_expert), _p(tile_row), _ll(n), E,
+                               top, tile, max_tiles, int(renormalize), _stream(h)), "moe_route")
+    ldw, ldf = up.shape[2], down.shape[2]
+    ldo = (n_down + 7) // 8 * 8
+    sorted_h = torch.empty((max_tiles * tile, ldw), dtype=dt, device=dev)
+    _check(lib().kvb_moe_gather(_p(h), _p(row), _p(sorted_h), _ll(n), top, width, _ll(ldw), code(dt), _stream(h)), "moe_gather")
+    hidden = torch.empty((max_tiles * tile, ldf), dtype=dt, device=dev)
+    st = _p(status_word(dev))
+    _check(lib().kvb_moe_gemm(_p(sorted_h), _p(up), _p(hidden), _p(plan), _p(tile_expert), _p(tile_row), tile, max_tiles, E, n_up, width,
+                              _ll(ldw), _ll(ldf), act, code(dt), int(FORCE_SIMPLE), st, _stream(h)), "moe_gemm (up)")
+    out = torch.empty((max_tiles * tile, ldo), dtype=dt, device=dev)
+    _check(lib().kvb_moe_gemm(_p(hidden), _p(down), _p(out), _p(plan), _p(tile_expert), _p(tile_row), tile, max_tiles, E, n_down, n_up,
+                              _ll(ldf), _ll(ldo), 0, code(dt), int(FORCE_SIMPLE), st, _stream(h)), "moe_gemm (down)")
+    _count(6)
+    return out, row.view(n, top), weight

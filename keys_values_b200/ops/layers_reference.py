@@ -1,0 +1,147 @@
+"""PyTorch restatement of :mod:`keys_values_b200.ops.layers` for CPU tensors (same layouts, same padding)."""
+from __future__ import annotations
+
+import torch
+
+
+def _norm_and_shift(x, gain, shift, state, h, hs, seq, eps) -> None:
+    if gain is None:
+        return
+    hf = x * (gain / torch.sqrt(x.square().mean(-1, keepdim=True) + eps))
+    h.copy_(hf)
+    if shift is None:
+        return
+    slots = seq.slots.long()
+    first = torch.where(seq.start[:, None] > 0, state[slots], torch.zeros_like(state[slots]))
+    before = torch.cat((first[:, None], hf[:, :-1]), dim=1)
+    hs.copy_(hf + (before - hf) * shift)
+    for b, n in enumerate(seq.count.tolist()):
+        if n > 0:
+            state[slots[b]] = hf[b, n - 1]
+
+
+def embed_edge(idx, prev_token, embed, bigram, buckets, mul_prev, mul_cur, hist, gain, shift, state, h, hs, seq, eps) -> None:
+    if int(idx.min()) < 0 or int(idx.max()) >= embed.shape[0]:
+        raise IndexError("token id outside of the vocabulary")
+    x = embed[idx].float()
+    if bigram is not None:
+        prev = torch.cat((prev_token[seq.slots.long()].long()[:, None], idx[:, :-1]), dim=1)
+        row = (prev * mul_prev + idx * mul_cur) % buckets
+        row[:, 0] = torch.where(seq.start > 0, row[:, 0], torch.full_like(row[:, 0], buckets))
+        x = x + bigram[row].float()
+    hist.copy_(x)
+    _norm_and_shift(x, gain, shift, state, h, hs, seq, eps)
+
+
+def layer_edge(x_in, mix, expert_out, expert_row, expert_w, hist, n_hist, coef, x_out, gain, shift, state, h, hs, seq, eps) -> None:
+    sub = mix.float()
+    if expert_out is not None:
+        width = sub.shape[-1]
+        sub = sub + (expert_w[:, :, None] * expert_out[expert_row.long()][:, :, :width].float()).sum(1).view_as(sub)
+    new = x_in + sub
+    if coef is None:
+        x_out.copy_(new)
+    else:
+        hist[n_hist] = new
+        x_out.copy_((coef.view(-1, 1, 1, 1) * hist[: n_hist + 1]).sum(0))
+    _norm_and_shift(x_out, gain, shift, state, h, hs, seq, eps)
+
+
+def scalar_rmsnorm(x, rows, gain, eps, dtype):
+    x = x if rows is None else x[rows]
+    return (x * (gain / torch.sqrt(x.square().mean(-1, keepdim=True) + eps))).to(dtype)
+
+
+def sequence_advance(idx, pos, prev_token, seq) -> None:
+    for b, (slot, n) in enumerate(zip(seq.slots.tolist(), seq.count.tolist())):
+        if n > 0:
+            pos[slot] += n
+            prev_token[slot] = int(idx[b, n - 1])
+
+
+def _rotate(x, cos, sin, dims):
+    half = dims // 2
+    u, v, rest = x[..., :half], x[..., half:dims], x[..., dims:]
+    return torch.cat((u * cos - v * sin, v * cos + u * sin, rest), dim=-1)
+
+
+def latent_prep(qkv, norm_w, freq, latent, ring, seq, P, s, eps):
+    B, T, _ = qkv.shape
+    nq = s.heads * (s.dim + s.rot)
+    qf = qkv[..., :nq].float().view(B, T, s.heads, s.dim + s.rot)
+    c, kr = qkv[..., nq : nq + s.kv_rank].float(), qkv[..., nq + s.kv_rank :].float()
+    pos = seq.start[:, None] + torch.arange(T)
+    angle = pos.float()[..., None] * freq
+    cos, sin = angle.cos(), angle.sin()
+    q = torch.zeros(B, T, s.heads, s.dimp + s.rp, dtype=qkv.dtype)
+    q[..., : s.dim] = qf[..., : s.dim]
+    q[..., s.dimp : s.dimp + s.rot] = _rotate(qf[..., s.dim :], cos[:, :, None], sin[:, :, None], s.rot_dims)
+    row = torch.zeros(B, T, s.row, dtype=qkv.dtype)
+    row[..., : s.kv_rank] = c / torch.sqrt(c.square().mean(-1, keepdim=True) + eps) * norm_w
+    row[..., s.kvp : s.kvp + s.rot] = _rotate(kr, cos, sin, s.rot_dims)
+    if ring is not None:
+        for b, (slot, n) in enumerate(zip(seq.slots.tolist(), seq.count.tolist())):
+            if n > 0:
+                ring[slot, int(pos[b, 0]) % ring.shape[1]] = row[b, 0]
+    else:
+        latent[:, P:] = row
+    return q
+
+
+def ring_gather(ring, latent, seq, P) -> None:
+    C = ring.shape[1]
+    latent[:, :P] = 0
+    for b, (slot, start) in enumerate(zip(seq.slots.tolist(), seq.start.tolist())):
+        for j in range(P):
+            p = start - P + j
+            if p >= max(0, start - C):
+                latent[b, j] = ring[slot, p % C]
+
+
+def ring_append(latent, ring, seq, P) -> None:
+    C = ring.shape[1]
+    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
+        for t in range(max(0, n - C), n):
+            ring[slot, (start + t) % C] = latent[b, P + t]
+
+
+def latent_attend(q, kv, latent, seq, P, s, window, scale):
+    B, T = q.shape[:2]
+    N = P + T
+    kv = kv.view(B, N, s.heads, s.dimp + s.vdp).float()
+    qf = q.float()
+    score = torch.einsum("bthd,bjhd->bhtj", qf[..., : s.dimp], kv[..., : s.dimp])
+    score = (score + torch.einsum("bthr,bjr->bhtj", qf[..., s.dimp :], latent[..., s.kvp :].float())) * scale
+    j = torch.arange(N)
+    back = P + torch.arange(T)[:, None] - j
+    seen = (back >= 0) & ((back < window) if window > 0 else torch.ones_like(back, dtype=torch.bool))
+    seen = seen[None] & (j[None, None] >= P - seq.start[:, None, None])
+    w = score.masked_fill(~seen[:, None], float("-inf")).softmax(-1)
+    return torch.einsum("bhtj,bjhv->bthv", w, kv[..., s.dimp :]).reshape(B, T, s.heads * s.vdp).to(q.dtype)
+
+
+def latent_decode(q_abs, q, ring, seq, s, scale):
+    out = torch.empty_like(q_abs)
+    for b, (slot, start) in enumerate(zip(seq.slots.tolist(), seq.start.tolist())):
+        rows = ring[slot, : min(start + 1, ring.shape[1])].float()
+        qc = torch.cat((q_abs[:, b].float(), q[b, 0, :, s.dimp :].float()), dim=-1)
+        w = (qc @ rows.t() * scale).softmax(-1)
+        out[:, b] = (w @ rows[:, : s.kvp]).to(out.dtype)
+    return out
+
+
+def moe_forward(h, logits, up, down, top, act, renormalize, n_up, n_down):
+    n, width = h.shape
+    scores = logits.softmax(-1)
+    weight, expert = scores.topk(top, dim=-1)
+    if renormalize:
+        weight = weight / weight.sum(-1, keepdim=True)
+    out = torch.zeros(n * top, (n_down + 7) // 8 * 8, dtype=h.dtype)
+    for e in range(logits.shape[1]):
+        t, k = torch.where(expert == e)
+        if t.numel():
+            z = h[t].float() @ up[e, :n_up, :width].float().t()
+            if act == 1:
+                z = z.relu().square()
+            out[t * top + k, :n_down] = (z.to(h.dtype).float() @ down[e, :n_down, :n_up].float().t()).to(h.dtype)
+    return out, torch.arange(n * top, dtype=torch.int32).view(n, top), weight
