@@ -2,7 +2,7 @@
 
 Commands (``keys_values/__main__.py:38-47``): ``finetune_long_full``, ``finetune_long_lora``,
 ``finetune_offload_full``, ``finetune_offload_lora``, ``eval_long``, ``eval_long_ext``,
-``recomp_val_losses``, plus ``generate``. Every command maps to a ``setup(...)`` function;
+``recomp_val_losses``, plus ``generate``, ``convert_hf_checkpoint`` and ``trace_run``. Every command maps to a ``setup(...)`` function;
 dataclass parameters are filled from dotted flags, ``--config file.yaml`` supplies defaults.
 Output is teed to ``$KEYSVALS_LOG_DIR/gpu{LOCAL_RANK}.log`` when that variable is set."""
 from __future__ import annotations
@@ -22,7 +22,7 @@ def _commands() -> Dict[str, Callable]:
     from keys_values_b200.evaluation import longcontext_eval, longcontext_eval_ext
     from keys_values_b200.finetune import longcon_offload_full, longcon_offload_lora, longcontext_full, longcontext_lora
     from keys_values_b200.generate import base as generate_base
-    from keys_values_b200.tools import convert_hf_checkpoint, recompute_val_losses
+    from keys_values_b200.tools import convert_hf_checkpoint, recompute_val_losses, trace_run
 
     return {
         "finetune_long_full": longcontext_full.setup,
@@ -34,11 +34,12 @@ def _commands() -> Dict[str, Callable]:
         "recomp_val_losses": recompute_val_losses.setup,
         "generate": generate_base.main,
         "convert_hf_checkpoint": convert_hf_checkpoint.setup,
+        "trace_run": trace_run.setup,
     }
 
 
 PARSER_DATA = ("finetune_long_full", "finetune_long_lora", "finetune_offload_full", "finetune_offload_lora", "eval_long", "eval_long_ext",
-               "recomp_val_losses", "generate", "convert_hf_checkpoint")
+               "recomp_val_losses", "generate", "convert_hf_checkpoint", "trace_run")
 
 
 class TeeOutput:
@@ -121,6 +122,7 @@ def build_kwargs(fn: Callable, argv: List[str]) -> Dict[str, Any]:
             else:
                 val = argv[i + 1]
                 i += 2
+            key = key.replace("-", "_")
             if "." in key:
                 g, f = key.split(".", 1)
                 nested.setdefault(g, {})[f] = val

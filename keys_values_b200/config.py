@@ -81,6 +81,14 @@ class Config:
     scale_embeddings: bool = False
     lm_head_bias: bool = False
     final_logit_softcapping: Optional[float] = None
+    # Models described layer by layer (models/layered.py). Each entry: {"mixer": {"kind": "latent_attention", "n_head",
+    # "dim", "rot_dim", "v_dim", "kv_rank", "scale", "rope_base", "window" or None}, "mlp": None or {"kind": "routed",
+    # "n_expert", "top", "ff"}}; mixer and feed-forward are parallel under one norm.
+    layers: Optional[List[dict]] = None
+    bigram: Optional[dict] = None  # {"buckets", "mul_prev", "mul_cur"}: hashed embedding of (previous token, token)
+    token_shift: bool = False  # the mixer reads a learned blend of this and the previous token's normed input
+    depth_average: bool = False  # learned average over the embedding output and all layers' results
+    architecture: str = ""  # entry of models/registry.py the config was read by
     # Added by keys_values (config.py:26-30): use the in-repo RMSNorm
     own_rms_norm_implementation: bool = True
 
@@ -130,10 +138,15 @@ class Config:
 
     @classmethod
     def from_checkpoint(cls, path: Union[str, Path], **kwargs: Any) -> "Config":
-        """``path`` is a checkpoint directory holding ``model_config.yaml``."""
+        """``path`` is a checkpoint directory holding ``model_config.yaml``, or the ``config.json`` of a registered
+        architecture (``models/registry.py``)."""
         path = Path(path)
         if (config_path := path / "model_config.yaml").is_file():
             return cls.from_file(config_path, **kwargs)
+        from keys_values_b200.models.registry import config_from_directory
+
+        if (config := config_from_directory(path, **kwargs)) is not None:
+            return config
         if (model_name := path.name) in name_to_config:
             return cls.from_name(model_name, **kwargs)
         raise FileNotFoundError(f"For {str(path)!r} neither 'model_config.yaml' nor matching config exists.")
@@ -166,6 +179,10 @@ class Config:
 
         from keys_values_b200.models.model import RMSNorm
 
+        if self.norm_class_name == "ScalarRMSNorm":
+            from keys_values_b200.models.layered import ScalarRMSNorm
+
+            return ScalarRMSNorm
         if self.norm_class_name == "RMSNorm":
             return partial(RMSNorm, add_unit_offset="Gemma" in self.name)
         if self.norm_class_name == "LayerNorm" and "OLMo" in self.name:
@@ -177,6 +194,18 @@ class Config:
 # Registry of named architectures. Only architecture hyper-parameters live here:
 # weights come from a ``lit_model.pth`` or from random initialisation.
 # --------------------------------------------------------------------------
+def _layered(n_layer: int, mixer: dict, mlp: Optional[dict]) -> dict:
+    """Fields of a model of ``n_layer`` equal latent-attention layers with routed experts."""
+    mixer = dict(kind="latent_attention", **mixer)
+    mixer.setdefault("scale", (mixer["dim"] + mixer["rot_dim"]) ** -0.5)
+    mlp = None if mlp is None else dict(kind="routed", **mlp)
+    return dict(
+        n_layer=n_layer, n_head=mixer["n_head"], head_size=mixer["dim"] + mixer["rot_dim"], layers=[dict(mixer=mixer, mlp=mlp)] * n_layer,
+        norm_class_name="ScalarRMSNorm", shared_attention_norm=True, bias=False, architecture="Mezilix",
+        token_shift=True, depth_average=True,
+    )
+
+
 _llama_like = dict(
     rotary_percentage=1.0,
     parallel_residual=False,
@@ -226,6 +255,24 @@ configs: List[dict] = [
     dict(
         name="pythia-14m",
         block_size=512, n_layer=6, n_embd=128, n_head=4, padding_multiple=128,
+    ),
+    # Mezilix: latent attention over a window, routed experts, token shift, depth average, bigram embedding
+    dict(
+        name="tiny-mezilix", block_size=1 << 20, vocab_size=320, padded_vocab_size=320, n_embd=192, norm_eps=1e-5,
+        bigram=dict(buckets=211, mul_prev=37, mul_cur=5),
+        **_layered(3, dict(n_head=6, dim=24, rot_dim=8, v_dim=40, kv_rank=72, window=48, rope_base=10000.0), dict(n_expert=10, top=3, ff=56)),
+    ),
+    dict(
+        name="Mezilix-2k", block_size=1 << 20, vocab_size=32000, padded_vocab_size=32000, n_embd=2048, norm_eps=1e-5,
+        bigram=dict(buckets=65521, mul_prev=8191, mul_cur=31),
+        **_layered(16, dict(n_head=16, dim=128, rot_dim=64, v_dim=128, kv_rank=512, window=4096, rope_base=10000.0),
+                   dict(n_expert=64, top=6, ff=1408)),
+    ),
+    dict(
+        name="Mezilix-4k", block_size=1 << 20, vocab_size=32000, padded_vocab_size=32000, n_embd=4096, norm_eps=1e-5,
+        bigram=dict(buckets=65521, mul_prev=8191, mul_cur=31),
+        **_layered(16, dict(n_head=32, dim=128, rot_dim=64, v_dim=128, kv_rank=512, window=4096, rope_base=10000.0),
+                   dict(n_expert=16, top=2, ff=6144)),
     ),
     # Qwen 2.5
     dict(

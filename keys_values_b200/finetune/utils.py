@@ -93,6 +93,11 @@ def load_model_checkpoint(gpt_model, checkpoint_dir: Path, resume_dir: Optional[
             return shard_state_dict(_load_sd(path), gpt_model.full_config, comm.world, comm.rank)
     else:
         load = _load_sd
+    if resume_dir is None and gpt_model.config.architecture:
+        from keys_values_b200.models.registry import load_architecture_weights
+
+        if load_architecture_weights(gpt_model, checkpoint_dir):
+            return
     has_lora = any("lora_" in n for n, _ in gpt_model.named_parameters())
     base = checkpoint_dir / LIT_MODEL_FNAME
     if resume_dir is not None and not has_lora:

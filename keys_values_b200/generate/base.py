@@ -7,7 +7,7 @@ from the (quantized) cache storage. Parity: ``keys_values/generate/base.py:50-61
 """
 from __future__ import annotations
 
-from typing import Any, Iterator, List, Optional, Tuple, Union
+from typing import Any, Iterator, List, Optional, Sequence, Tuple, Union
 
 import torch
 
@@ -70,17 +70,29 @@ def batched_next_token(model: GPT, x: torch.Tensor, kwargs: Union[dict, List[dic
     return batched_sample(model(x)[:, -1:], kwargs).to(torch.int64)
 
 
-def _prefill(model: GPT, prompts: torch.Tensor, chunk_size: int, max_seq_length: int) -> torch.Tensor:
-    """Chunked prompt processing; returns the logits of the final prompt position ``(B,1,V)``."""
+def _prefill(model: GPT, prompts: torch.Tensor, chunk_size: int, max_seq_length: int, lengths: Optional[List[int]] = None) -> torch.Tensor:
+    """Chunked prompt processing; returns the logits of the final prompt position ``(B,1,V)`` (of every row's own final
+    position with ``lengths``)."""
     lcm = LongContextInferenceModel(model, CrossEntropyOnLogits(model.config), chunk_size=chunk_size)
     lcm.fixed_max_seq_length = max_seq_length
-    return lcm(prompts, None)
+    return lcm(prompts, None, lengths=lengths)
+
+
+def pad_prompts(prompts: Sequence[torch.Tensor]) -> Tuple[torch.Tensor, List[int]]:
+    """Right-padded ``(B, T)`` batch of 1-d prompts and their lengths."""
+    lengths = [int(p.numel()) for p in prompts]
+    if not lengths or min(lengths) == 0:
+        raise ValueError("every prompt must have at least one token")
+    out = torch.zeros((len(lengths), max(lengths)), dtype=torch.int64, device=prompts[0].device)
+    for row, p in zip(out, prompts):
+        row[: p.numel()] = p
+    return out, lengths
 
 
 @torch.inference_mode()
 def batched_generate_fn(
     model: GPT,
-    prompts: torch.Tensor,
+    prompts: Union[torch.Tensor, Sequence[torch.Tensor]],
     max_returned_tokens: int,
     prompt_chunksize: int = 1024,
     sample_args: Union[dict, List[dict], None] = None,
@@ -90,9 +102,14 @@ def batched_generate_fn(
     use_graph: bool = True,
 ) -> Iterator[List[Optional[torch.Tensor]]]:
     """Yields, step by step, one token (or ``None`` once a row has stopped) per batch row.
-    ``prompts (B, T)`` must have equal lengths (left-padded batches). On a GPU the single-token
+    ``prompts (B, T)`` must have equal lengths (left-padded batches); models that keep a position per row
+    (:class:`keys_values_b200.models.layered.LayeredGPT`) also take a list of 1-d prompts of different lengths, all of which
+    get ``max_returned_tokens`` minus the longest length new tokens. On a GPU the single-token
     steps are replayed from one CUDA graph as soon as all caches are full
     (:class:`keys_values_b200.generate.decode_graph.Decoder`); ``use_graph=False`` keeps them eager."""
+    lengths: Optional[List[int]] = None
+    if not torch.is_tensor(prompts):
+        prompts, lengths = pad_prompts(prompts)
     if prompts.ndim == 1:
         prompts = prompts.unsqueeze(0)
     B, T = prompts.shape
@@ -101,8 +118,8 @@ def batched_generate_fn(
     sample_args = sample_args if sample_args is not None else dict(temperature=0.0)
     if include_prompt:
         for t in range(T):
-            yield [prompts[b, t : t + 1] for b in range(B)]
-    logits = _prefill(model, prompts, prompt_chunksize, max_returned_tokens)
+            yield [prompts[b, t : t + 1] if lengths is None or t < lengths[b] else None for b in range(B)]
+    logits = _prefill(model, prompts, prompt_chunksize, max_returned_tokens, lengths)
     tokens = batched_sample(logits, sample_args).view(B, 1).to(torch.int64)
     from keys_values_b200.generate.decode_graph import Decoder
 
@@ -151,27 +168,31 @@ def generate(model: GPT, prompt: torch.Tensor, max_returned_tokens: int, prompt_
     return torch.cat(toks) if toks else torch.empty(0, dtype=torch.int64, device=prompt.device)
 
 
-def main(checkpoint_dir: str, prompt: str = "What food do llamas eat?", *, max_new_tokens: int = 50, cache_name: str = "h2o-default",
+def main(checkpoint_dir: str, prompt: str = "What food do llamas eat?", *, max_new_tokens: int = 50, cache_name: Optional[str] = None,
          cache_length: int = 4096, chunk_size: int = 1024, temperature: float = 0.8, top_k: Optional[int] = 50, top_p: float = 1.0,
-         precision: Optional[str] = None, device: Optional[str] = None, tp: int = 1, seed: int = 1337) -> Optional[str]:
+         precision: Optional[str] = None, device: Optional[str] = None, tp: int = 1, seed: int = 1337,
+         prompt_tokens: Optional[str] = None) -> Optional[str]:
     """CLI body of ``keys_values_b200 generate``: load a checkpoint directory, generate a reply. ``tp > 1``: the
-    model is sharded over ``tp`` ranks of this node (one process per GPU; gloo ranks on a machine without GPUs)."""
+    model is sharded over ``tp`` ranks of this node (one process per GPU; gloo ranks on a machine without GPUs).
+    ``cache_name``: default ``h2o-default``, for models with described layers ``latent-default``. ``prompt_tokens``: comma
+    separated token ids instead of a text, for checkpoints without a tokenizer; prints the generated ids."""
     from keys_values_b200.parallel.launch import launch
 
     result: List[str] = []
     launch(_generate_rank, tp, checkpoint_dir=checkpoint_dir, prompt=prompt, max_new_tokens=max_new_tokens, cache_name=cache_name,
            cache_length=cache_length, chunk_size=chunk_size, temperature=temperature, top_k=top_k, top_p=top_p, precision=precision,
-           device=device, seed=seed, result=result)
+           device=device, seed=seed, prompt_tokens=prompt_tokens, result=result)
     return result[0] if result else None  # spawned ranks print the text; it comes back only from an in-process run
 
 
 def _generate_rank(rank: int, local_rank: int, world: int, *, checkpoint_dir, prompt, max_new_tokens, cache_name, cache_length, chunk_size,
-                   temperature, top_k, top_p, precision, device, seed, result) -> None:
+                   temperature, top_k, top_p, precision, device, seed, prompt_tokens, result) -> None:
     from pathlib import Path
 
     from keys_values_b200.config import Config
     from keys_values_b200.finetune.utils import load_model_checkpoint
     from keys_values_b200.kvcache.factory import KVCacheFactory
+    from keys_values_b200.models.registry import create_model, default_cache_name
     from keys_values_b200.prompts import has_prompt_style, load_prompt_style, Default
     from keys_values_b200.tokenizer import Tokenizer
     from keys_values_b200.utils import get_default_supported_precision, str_to_torch_dtype
@@ -183,10 +204,13 @@ def _generate_rank(rank: int, local_rank: int, world: int, *, checkpoint_dir, pr
         dev = torch.device("cuda", local_rank) if torch.cuda.is_available() else torch.device("cpu")
     dtype = str_to_torch_dtype(precision or get_default_supported_precision(False))
     config = Config.from_checkpoint(ckpt)
-    tokenizer = Tokenizer(ckpt)
+    cache_name = default_cache_name(config, cache_name)
+    tokenizer = Tokenizer(ckpt) if prompt_tokens is None else None
     style = load_prompt_style(ckpt) if has_prompt_style(ckpt) else Default()
     comm = None
     if world > 1:
+        if config.layers is not None:
+            raise NotImplementedError("tensor parallelism of models with described layers")
         from keys_values_b200.parallel.tp import TPComm, TPGPT, load_sharded_checkpoint
 
         comm = TPComm(world, rank, dev, dtype=dtype)
@@ -196,18 +220,24 @@ def _generate_rank(rank: int, local_rank: int, world: int, *, checkpoint_dir, pr
         load_sharded_checkpoint(model, ckpt)
     else:
         with torch.device(dev):
-            model = GPT(config)
+            model = create_model(config)
         model = model.to(dtype)
         load_model_checkpoint(model, ckpt)
     model.eval()
     torch.manual_seed(seed)  # every rank draws the same samples
-    ids = tokenizer.encode(style.apply(prompt), device=dev).to(torch.int64)
+    if tokenizer is None:
+        ids = torch.tensor([int(t) for t in str(prompt_tokens).split(",")], dtype=torch.int64, device=dev)
+        if int(ids.min()) < 0 or int(ids.max()) >= config.padded_vocab_size:
+            raise ValueError(f"prompt_tokens must lie in [0, {config.padded_vocab_size})")
+    else:
+        ids = tokenizer.encode(style.apply(prompt), device=dev).to(torch.int64)
     total = ids.numel() + max_new_tokens
     model.max_seq_length = total
-    model.assign_kv_caches(KVCacheFactory.create(model, cache_name, 1, min(cache_length, total) if cache_name.startswith("dense") else cache_length,
+    model.assign_kv_caches(KVCacheFactory.create(model, cache_name, 1, min(cache_length, total) if cache_name.startswith("dense") else (total if cache_name.startswith("latent") else cache_length),
                                                  device=dev, dtype=dtype))
-    out = generate(model, ids, total, chunk_size, temperature, top_k, top_p, eos_id=tokenizer.eos_id, include_prompt=False)
-    text = tokenizer.decode(out)
+    out = generate(model, ids, total, chunk_size, temperature, top_k, top_p, eos_id=None if tokenizer is None else tokenizer.eos_id,
+                   include_prompt=False)
+    text = ",".join(str(t) for t in out.view(-1).tolist()) if tokenizer is None else tokenizer.decode(out)
     if rank == 0:
         print(text)
     result.append(text)

@@ -46,6 +46,7 @@ class DecodeGraph:
         """``None`` if the next single-token step of ``model`` can be captured, else the reason."""
         from keys_values_b200.kvcache.basics import LastRecentlyInsertedKVCache
         from keys_values_b200.kvcache.h2o import H2OKVCache
+        from keys_values_b200.kvcache.latent import LatentKVCache
 
         if not torch.cuda.is_available() or model.lm_head.weight.device.type != "cuda":
             return "model is not on a GPU"
@@ -53,6 +54,8 @@ class DecodeGraph:
             return "a start-of-layer hook is set"
         if torch.is_grad_enabled():
             return "gradients are enabled"
+        if all(isinstance(cache, LatentKVCache) for cache in model.get_kv_caches()):
+            return None  # rings of fixed size, positions in device memory: any step is like the next
         for cache in model.get_kv_caches():
             if type(cache) is LastRecentlyInsertedKVCache:
                 # ring of the most recent tokens: the slot is a function of the position
@@ -78,8 +81,7 @@ class DecodeGraph:
 
     # --------------------------------------------------------------------- capture
     def _advance_host(self) -> None:
-        for cache in self.model.get_kv_caches():
-            cache.advance_host_counters()
+        self.model.advance_host_counters()
 
     def _capture(self, tokens: torch.Tensor) -> None:
         from keys_values_b200.ops import cuda as cu

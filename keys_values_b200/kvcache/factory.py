@@ -2,7 +2,8 @@
 
 Names are ``<policy>-<buffers>`` with policy in ``dense, lastrec, smart-lastrec,
 h2o, h2o-vlen, qh2o, qh2o-vlen, h2o-orig`` and buffers in ``default,
-torch-quantized4, torch-quantized8, bnb-quantized4, bnb-quantized8``.
+torch-quantized4, torch-quantized8, bnb-quantized4, bnb-quantized8``; ``latent-default`` is the cache of
+latent-attention layers (``models/layered.py``).
 """
 from __future__ import annotations
 
@@ -14,6 +15,7 @@ from keys_values_b200.kvcache.base import KVCache, KVCacheParams
 from keys_values_b200.kvcache.basics import DenseKVCache, LastRecentlyInsertedKVCache
 from keys_values_b200.kvcache.buffers import DefaultKVCacheBuffers
 from keys_values_b200.kvcache.consts import SUPPORTED_QUANTIZERS, split_name
+from keys_values_b200.kvcache.latent import LatentKVCache
 from keys_values_b200.kvcache.h2o import H2OKVCache, H2OOriginalKVCache, VLengthH2OKVCache
 from keys_values_b200.kvcache.qh2o import QuantizedH2OKVCache, QuantizedVLengthH2OKVCache
 from keys_values_b200.kvcache.quant_buffers import (
@@ -41,6 +43,7 @@ SUPPORTED_CACHES: Dict[str, type] = {
     for q in SUPPORTED_QUANTIZERS
     if not (p.startswith("qh2o") and q == "default")
 }
+SUPPORTED_CACHES["latent-default"] = LatentKVCache
 
 
 class KVCacheFactory:
@@ -110,6 +113,8 @@ class KVCacheFactory:
     def _create(gpt_model, name, max_batch_size, cache_lengths, start, end, device, dtype, cache_kwargs) -> List[KVCache]:
         config = gpt_model.config
         cache_type = KVCacheFactory._cache_type(name)
+        if (cache_type is LatentKVCache) != (config.layers is not None):
+            raise ValueError(f"cache {name!r} does not fit model {config.name!r}")
         cache_kwargs = dict(cache_kwargs or {})
         max_num_ranges = cache_kwargs.pop("max_num_ranges", None)
         allocate_buffers = cache_kwargs.pop("allocate_buffers", False)

@@ -32,6 +32,8 @@ def create_chunk_sizes(gpt_model: GPT, seq_length: int, chunk_size: int, randomi
     With ``randomize_chunk_sizes`` later chunks draw from 5 values sampled in
     ``[cs − cs//2, cs + cs//2]``."""
     caches = gpt_model.get_kv_caches()
+    if all(c.max_prefill_length is None for c in caches):  # caches that take passes of any length
+        return [min(chunk_size, seq_length - s) for s in range(0, seq_length, chunk_size)]
     mpl = min(c.max_prefill_length for c in caches)
     points = sorted({c.cache_length for c in caches if c.cache_length <= seq_length})
     if not points:
@@ -229,18 +231,28 @@ class LongContextInferenceModel(GPTAndHeadModel):
                 self.cells.append(ChunksForCell(1, tuple(sizes[1:]), sizes[0]))
         else:
             # a tensor-parallel shard keeps the cell schedule of the whole model (its layer inputs are not sharded)
-            cell_len = max(default_cell_length(getattr(gpt, "full_config", gpt.config), max_c, self.chunks_per_cell_multiplier), 1)
+            if hasattr(gpt, "max_pass_tokens"):
+                cell_len = gpt.max_pass_tokens(input_ids.shape[0])
+            else:
+                cell_len = max(default_cell_length(getattr(gpt, "full_config", gpt.config), max_c, self.chunks_per_cell_multiplier), 1)
             self.cells = get_chunks_for_cells(sizes, cell_len)
 
     # --------------------------------------------------------------- forward
-    def forward(self, input_ids: torch.Tensor, targets: Optional[torch.Tensor] = None, scale_factor: float = 1.0):
+    def forward(self, input_ids: torch.Tensor, targets: Optional[torch.Tensor] = None, scale_factor: float = 1.0,
+                lengths: Optional[List[int]] = None):
         """With ``targets``: loss per batch row ``(B,)`` (normalised by the number of
-        target entries). Without: logits of the final position ``(B, 1, vocab)``. The result
+        target entries). Without: logits of the final position ``(B, 1, vocab)``; ``lengths`` gives the
+        lengths of right-padded rows for models that keep a position per row. The result
         stays on the device; callers that read it on the host follow the read with
         :func:`keys_values_b200.ops.check_status` (see :meth:`loss_value`)."""
+        if lengths is not None:
+            if targets is not None or len(lengths) != input_ids.shape[0] or not all(1 <= n <= input_ids.shape[1] for n in lengths):
+                raise ValueError("lengths: one per row, within the row, and only without targets")
+            if all(n == input_ids.shape[1] for n in lengths):
+                lengths = None
         self._init_members_from_tokens(input_ids, targets)
         with torch.no_grad():
-            return self._forward_internal(input_ids, targets, scale_factor)
+            return self._forward_internal(input_ids, targets, scale_factor, lengths)
 
     def loss_value(self, input_ids: torch.Tensor, targets: torch.Tensor, scale_factor: float = 1.0) -> torch.Tensor:
         """:meth:`forward` followed by a host read of the loss and of the device status word: raises if a
@@ -251,7 +263,7 @@ class LongContextInferenceModel(GPTAndHeadModel):
         _ops.check_status(input_ids.device)
         return loss
 
-    def _forward_internal(self, input_ids, targets, scale_factor: float = 1.0):
+    def _forward_internal(self, input_ids, targets, scale_factor: float = 1.0, lengths: Optional[List[int]] = None):
         def _dense(t):  # blocks of a tensor-parallel shard may hand on token rows sharded over the ranks
             return t.full() if hasattr(t, "full") else t
 
@@ -263,20 +275,24 @@ class LongContextInferenceModel(GPTAndHeadModel):
         last_x = None
         for cell_idx, cell in enumerate(self.cells):
             ids = input_ids[:, cell.start : cell.end]
-            x = gpt.embed(ids)
-            for layer_idx, block in enumerate(gpt.transformer.h):
+            counts = None if lengths is None else [min(max(n - cell.start, 0), cell.num_tokens) for n in lengths]
+            x = gpt.begin_pass(ids, counts)
+            for layer_idx in range(n_layer):
                 if self.layer_input_hook is not None:
-                    x = _dense(x)
-                    self.layer_input_hook(x, layer_idx, cell.start, cell.end)
+                    dense = _dense(x)
+                    self.layer_input_hook(dense, layer_idx, cell.start, cell.end)
+                    if not getattr(x, "carries_state", False):
+                        x = dense
                 ws = self.weight_streamer
                 if ws is not None:  # host-resident blocks: this one on the device, the next one on its way
                     ws.acquire(layer_idx)
                     ws.prefetch(layer_idx + 1)
-                x = block(x, ids, gpt.mha, chunk_sizes=cell.chunk_sizes)
+                x = gpt.run_layer(layer_idx, x, ids, chunk_sizes=cell.chunk_sizes)
                 if ws is not None:
                     ws.release(layer_idx)
                 if self.cell_boundary_hook is not None:
                     self.cell_boundary_hook(layer_idx, cell_idx, cell.end)
+            x = gpt.end_pass(x, ids)
             if self.layer_input_hook is not None:
                 x = _dense(x)
                 self.layer_input_hook(x, n_layer, cell.start, cell.end)
@@ -290,7 +306,16 @@ class LongContextInferenceModel(GPTAndHeadModel):
                         if torch.is_tensor(part):
                             loss_sum = part if loss_sum is None else loss_sum + part
                     pos += c
-            last_x = x
+            if lengths is not None:  # rows whose last token lies in this cell
+                rows = [b for b, n in enumerate(lengths) if cell.start < n <= cell.end]
+                if rows:
+                    at = torch.tensor([lengths[b] - 1 - cell.start for b in rows], device=x.device)
+                    rows = torch.tensor(rows, device=x.device)
+                    if last_x is None:
+                        last_x = x.new_zeros((x.shape[0], 1, x.shape[2]))
+                    last_x[rows, 0] = x[rows, at]
+            else:
+                last_x = x
         if targets is None:
             return gpt.head(last_x[:, -1:, :])
         num = head.num_target_entries(targets)

@@ -1,0 +1,385 @@
+"""Decoder models whose layers are described one by one (``config.layers``).
+
+Each entry of ``config.layers`` names its mixer and its feed-forward with their own sizes, so the layers of a model may
+differ. The mechanisms are modules of their own, picked by the description:
+
+* :class:`LatentAttention`: low-rank keys and values (one latent per token plus one rotated key part that the heads
+  share), optional sliding window, ring cache of latents (:class:`keys_values_b200.kvcache.latent.LatentKVCache`);
+* :class:`RoutedMLP`: softmax router, top-k experts without gates;
+* :class:`ScalarRMSNorm`: RMS norm with one gain for all coordinates;
+* token shift (``config.token_shift``): the mixer reads a learned blend of the token's normed input and the previous token's;
+* depth average (``config.depth_average``): what goes on to the next layer is a learned average of the embedding output
+  and all layers' results so far;
+* bigram embedding (``config.bigram``): a hashed row for the pair (previous token, token) is added to the embedding.
+
+Mixer and feed-forward of a layer are parallel: both read the output of the layer's one norm. The residual stream and the
+depth history are fp32. What lies between the sublayers of two layers (residual sum, weighted expert outputs, depth
+average, next norm, token shift) is one kernel, :func:`keys_values_b200.ops.layers.layer_edge`; therefore the stream that
+:meth:`LayeredGPT.run_layer` hands on is a :class:`LayerStream`, which carries the next layer's normed inputs along.
+"""
+from __future__ import annotations
+
+from typing import Any, Dict, Optional, Sequence
+
+import torch
+import torch.nn as nn
+import torch.nn.functional as F
+
+from keys_values_b200.config import Config
+from keys_values_b200.kvcache.sequences import SequencePass, SequenceTable
+from keys_values_b200.models.model import GPT
+from keys_values_b200.ops import layers as L
+
+# fp32 bytes of residual streams (depth history included) that one pass of a chunked prefill may hold
+MAX_STREAM_BYTES = 4 * 2**30
+MAX_PASS_TOKENS = 16384
+
+
+def latent_shape(spec: Dict[str, Any]) -> L.LatentShape:
+    return L.LatentShape(heads=spec["n_head"], dim=spec["dim"], rot=spec["rot_dim"], vdim=spec["v_dim"], kv_rank=spec["kv_rank"],
+                         rot_dims=spec.get("rope_dims", spec["rot_dim"]))
+
+
+class ScalarRMSNorm(nn.Module):
+    """``x / rms(x) · weight`` with a single number as weight."""
+
+    def __init__(self, size: int, eps: float = 1e-5) -> None:
+        super().__init__()
+        self.weight = nn.Parameter(torch.ones(()))
+        self.size = size
+        self.eps = eps
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        y = L.scalar_rmsnorm(x.reshape(-1, self.size).float(), self.weight.float(), self.eps, self.weight.dtype)
+        return y.view(x.shape)
+
+    def reset_parameters(self) -> None:
+        nn.init.ones_(self.weight)
+
+
+class _Packed(nn.Module):
+    """Module that keeps copies of its weights in the layout of the kernels, made on first use."""
+
+    def __init__(self) -> None:
+        super().__init__()
+        self._pack: Optional[Dict[str, torch.Tensor]] = None
+
+    def packed(self) -> Dict[str, torch.Tensor]:
+        if self._pack is None:
+            with torch.no_grad(), torch.inference_mode(False):
+                self._pack = self._make_pack()
+        return self._pack
+
+    def _make_pack(self) -> Dict[str, torch.Tensor]:
+        raise NotImplementedError
+
+    def drop_pack(self) -> None:
+        self._pack = None
+
+    def _apply(self, fn, *args, **kwargs):
+        self._pack = None
+        return super()._apply(fn, *args, **kwargs)
+
+    def _load_from_state_dict(self, *args: Any, **kwargs: Any) -> None:
+        self._pack = None
+        super()._load_from_state_dict(*args, **kwargs)
+
+
+def _pad_last(w: torch.Tensor, n: int) -> torch.Tensor:
+    return w.contiguous() if w.shape[-1] == n else F.pad(w, (0, n - w.shape[-1])).contiguous()
+
+
+class LatentAttention(_Packed):
+    def __init__(self, config: Config, block_idx: int, kv_cache=None) -> None:
+        super().__init__()
+        spec = config.layers[block_idx]["mixer"]
+        s = self.shape = latent_shape(spec)
+        if not spec["scale"] > 0:
+            raise ValueError(f"layer {block_idx}: attention scale must be positive")
+        self.scale = float(spec["scale"])
+        self.window = int(spec.get("window") or 0)
+        self.rope_base = float(spec["rope_base"])
+        self.eps = config.norm_eps
+        # rows: queries head by head [unrotated | rotated], latent, shared rotated key part
+        self.qkv = nn.Linear(config.n_embd, s.heads * (s.dim + s.rot) + s.kv_rank + s.rot, bias=False)
+        self.norm_kv = nn.Parameter(torch.ones(s.kv_rank))
+        self.key = nn.Linear(s.kv_rank, s.heads * s.dim, bias=False)
+        self.value = nn.Linear(s.kv_rank, s.heads * s.vdim, bias=False)
+        self.proj = nn.Linear(s.heads * s.vdim, config.n_embd, bias=False)
+        self.kv_cache = kv_cache
+        self.config = config
+        self.block_idx = block_idx
+
+    def _make_pack(self) -> Dict[str, torch.Tensor]:
+        s = self.shape
+        w = self.qkv.weight
+        key = F.pad(self.key.weight.view(s.heads, s.dim, s.kv_rank), (0, s.kvp - s.kv_rank, 0, s.dimp - s.dim)).contiguous()
+        value = F.pad(self.value.weight.view(s.heads, s.vdim, s.kv_rank), (0, s.kvp - s.kv_rank, 0, s.vdp - s.vdim))
+        exps = torch.arange(s.rot_dims // 2, dtype=torch.float64) * (-2.0 / s.rot_dims)
+        return {
+            "norm": self.norm_kv.float().contiguous(),
+            "freq": (self.rope_base**exps).to(device=w.device, dtype=torch.float32),
+            "key": key,  # (heads, dimp, kvp)
+            "value_t": value.transpose(1, 2).contiguous(),  # (heads, kvp, vdp)
+            "key_value": torch.cat((key, value), dim=1).view(-1, s.kvp).contiguous(),  # rows of a head: [key | value]
+            "proj": _pad_last(self.proj.weight.view(-1, s.heads, s.vdim), s.vdp).view(-1, s.heads * s.vdp),
+        }
+
+    def forward(self, x: torch.Tensor, seq: SequencePass) -> torch.Tensor:
+        """``x (B, T, width)`` → ``(B, T, width)``; the cache takes the rows of the pass."""
+        B, T, _ = x.shape
+        s, w = self.shape, self.packed()
+        qkv = F.linear(x, self.qkv.weight)
+        ring = self.kv_cache.allocate(x.device, x.dtype)
+        if T == 1:
+            q = L.latent_prep(qkv, w["norm"], w["freq"], None, ring, seq, 0, s, self.eps)
+            q_abs = torch.bmm(q[:, 0, :, : s.dimp].transpose(0, 1), w["key"])  # W_uk folded into the query
+            lat = L.latent_decode(q_abs, q, ring, seq, s, self.scale)
+            y = torch.empty((B, s.heads, s.vdp), dtype=x.dtype, device=x.device)
+            torch.bmm(lat, w["value_t"], out=y.transpose(0, 1))
+            return F.linear(y.view(B, 1, -1), w["proj"])
+        # rows before the pass that its first tokens still see
+        P = seq.max_start if self.window == 0 else min(seq.max_start, self.window - 1)
+        latent = torch.empty((B, P + T, s.row), dtype=x.dtype, device=x.device)
+        L.ring_gather(ring, latent, seq, P)
+        q = L.latent_prep(qkv, w["norm"], w["freq"], latent, None, seq, P, s, self.eps)
+        L.ring_append(latent, ring, seq, P)
+        kv = torch.mm(latent.view(-1, s.row)[:, : s.kvp], w["key_value"].t())
+        y = L.latent_attend(q, kv, latent, seq, P, s, self.window, self.scale)
+        return F.linear(y, w["proj"])
+
+    def create_default_kv_cache(self, batch_size: int, dtype=None, max_sequence_length: Optional[int] = None, device=None) -> None:
+        from keys_values_b200.kvcache.latent import LatentKVCache
+
+        length = self.config.block_size if max_sequence_length is None else max_sequence_length
+        self.kv_cache = LatentKVCache(self.config, batch_size, length, self.block_idx, dtype=dtype, device=device)
+
+
+class RoutedMLP(_Packed):
+    """``Σ over the chosen experts of score_e · down_e(act(up_e(x)))``. Returns the experts' outputs unsummed (the sum is
+    part of the kernel that closes the layer)."""
+
+    def __init__(self, config: Config, spec: Dict[str, Any]) -> None:
+        super().__init__()
+        E, ff, width = spec["n_expert"], spec["ff"], config.n_embd
+        if not 0 < spec["top"] <= E:
+            raise ValueError(f"top = {spec['top']} of {E} experts")
+        if spec.get("activation", "relu_squared") not in L.ACTIVATIONS:
+            raise ValueError(f"activation {spec['activation']!r}")
+        self.spec = spec
+        self.gate = nn.Linear(width, E, bias=False)
+        self.up = nn.Parameter(torch.empty(E, ff, width))
+        self.down = nn.Parameter(torch.empty(E, width, ff))
+        for p in (self.up, self.down):
+            nn.init.normal_(p, mean=0.0, std=0.02)
+
+    def _make_pack(self) -> Dict[str, torch.Tensor]:
+        E, ff, width = self.up.shape
+        return {"up": _pad_last(self.up.detach(), L.round8(width)), "down": _pad_last(self.down.detach(), L.round8(ff))}
+
+    def forward(self, x: torch.Tensor):
+        _, ff, width = self.up.shape
+        w = self.packed()
+        x = x.reshape(-1, width)
+        logits = L.linear_fp32(x, self.gate.weight)
+        return L.routed_experts(x, logits, w["up"], w["down"], self.spec["top"], self.spec.get("activation", "relu_squared"),
+                                bool(self.spec.get("renormalize", False)), ff, width)
+
+
+MIXERS = {"latent_attention": LatentAttention}
+FEED_FORWARDS = {"routed": RoutedMLP}
+
+
+class LayeredBlock(_Packed):
+    """Sublayers and layer-edge parameters of one layer."""
+
+    def __init__(self, config: Config, block_idx: int, kv_cache=None) -> None:
+        super().__init__()
+        spec = config.layers[block_idx]
+        self.norm_1 = config.norm_class(config.n_embd, eps=config.norm_eps)
+        self.attn = MIXERS[spec["mixer"]["kind"]](config, block_idx, kv_cache)
+        self.mlp = None if spec.get("mlp") is None else FEED_FORWARDS[spec["mlp"]["kind"]](config, spec["mlp"])
+        self.shift = nn.Parameter(torch.zeros(config.n_embd)) if config.token_shift else None
+        self.depth = None
+        if config.depth_average:  # the identity: all weight on the layer's own result
+            self.depth = nn.Parameter(F.one_hot(torch.tensor(block_idx + 1), block_idx + 2).float())
+        self.config = config
+        self.block_idx = block_idx
+
+    def _make_pack(self) -> Dict[str, Optional[torch.Tensor]]:
+        return {
+            "gain": self.norm_1.weight.float().contiguous(),
+            "shift": None if self.shift is None else self.shift.float().contiguous(),
+            "depth": None if self.depth is None else self.depth.float().contiguous(),
+        }
+
+
+class LayerStream:
+    """What one layer hands to the next: the fp32 residual stream, the depth history and the next layer's inputs."""
+
+    carries_state = True  # not replaceable by its dense tensor
+
+    def __init__(self, seq: SequencePass, x: torch.Tensor, history: Optional[torch.Tensor], h: torch.Tensor, shifted: Optional[torch.Tensor]):
+        self.seq = seq
+        self.x = x  # (B, T, width) fp32
+        self.history = history  # (n_layer + 1, B, T, width) fp32: embedding output, then every layer's result
+        self.h = h  # normed input of the next layer
+        self.shifted = shifted  # what the next layer's mixer reads
+        self.spare: Optional[torch.Tensor] = None  # retired stream buffer
+
+    def full(self) -> torch.Tensor:
+        return self.x
+
+
+class LayeredGPT(GPT):
+    """:class:`GPT` for configs with ``layers``. Rows of a batch may have different lengths: ``counts`` of
+    :meth:`forward` says how many tokens of each (right-padded) row are real."""
+
+    def __init__(self, config: Config, **mha_kwargs) -> None:
+        if config.layers is None or len(config.layers) != config.n_layer:
+            raise ValueError("config.layers must describe every layer")
+        super().__init__(config, **mha_kwargs)
+        self.bigram = None
+        if config.bigram is not None:  # the last row is for tokens without a predecessor
+            self.bigram = nn.Embedding(config.bigram["buckets"] + 1, config.n_embd)
+        self.sequences: Optional[SequenceTable] = None
+
+    def _make_block(self, config: Config, block_idx: int) -> LayeredBlock:
+        return LayeredBlock(config, block_idx)
+
+    def _make_mha(self, config: Config, **mha_kwargs) -> None:
+        return None  # positions, windows and scales belong to the layers
+
+    def _init_weights(self, module: nn.Module) -> None:
+        super()._init_weights(module)
+        if isinstance(module, RoutedMLP):
+            nn.init.normal_(module.up, mean=0.0, std=0.02)
+            nn.init.normal_(module.down, mean=0.0, std=0.02)
+        if isinstance(module, _Packed):
+            module.drop_pack()
+
+    @property
+    def max_seq_length(self) -> int:
+        return self._max_seq_length
+
+    @max_seq_length.setter
+    def max_seq_length(self, value: int) -> None:
+        if value <= 0:
+            raise ValueError(f"value = {value}, must be positive")
+        self._max_seq_length = value  # angles are computed per position: nothing is sized by the context
+
+    # ---------------------------------------------------------------- caches
+    def _check_kv_cache(self, cache) -> None:
+        from keys_values_b200.kvcache.latent import LatentKVCache
+
+        if cache is None:
+            return
+        if not isinstance(cache, LatentKVCache):
+            raise ValueError(f"{type(cache).__name__} does not fit a latent-attention layer (use cache name 'latent-default')")
+        if cache.shape != self.transformer.h[cache.block_idx].attn.shape:
+            raise ValueError(f"cache of layer {cache.block_idx} has sizes {cache.shape}, the layer has {self.transformer.h[cache.block_idx].attn.shape}")
+
+    def assign_kv_caches(self, kv_caches: Sequence[Any]) -> None:
+        super().assign_kv_caches(kv_caches)
+        self._make_sequences()
+
+    def set_kv_caches(self, batch_size: int, dtype=None, max_seq_length: Optional[int] = None, device=None) -> None:
+        super().set_kv_caches(batch_size, dtype, max_seq_length, device)
+        self._make_sequences()
+
+    def _make_sequences(self) -> None:
+        caches = self.get_kv_caches()
+        self.sequences = None
+        if any(c is None for c in caches):
+            return
+        c = self.config
+        self.sequences = SequenceTable(min(x.max_batch_size for x in caches), self.lm_head.weight.device,
+                                       c.n_layer if c.token_shift else 0, c.n_embd)
+        for x in caches:
+            x.sequences = self.sequences
+
+    def clear_kv_caches(self) -> None:
+        super().clear_kv_caches()
+        self.sequences = None
+
+    def reset(self) -> None:
+        super().reset()
+        if self.sequences is not None:
+            self.sequences.reset()
+
+    def advance_host_counters(self) -> None:
+        self.sequences.advance_host()
+
+    def max_pass_tokens(self, batch_size: int) -> int:
+        """Tokens per row that one pass of a chunked prefill may take."""
+        c = self.config
+        per_token = 4 * c.n_embd * ((c.n_layer + 1 if c.depth_average else 0) + 2)
+        return max(1, min(MAX_STREAM_BYTES // per_token, MAX_PASS_TOKENS) // batch_size)
+
+    # --------------------------------------------------------------- forward
+    def embed(self, idx: torch.Tensor) -> torch.Tensor:
+        raise NotImplementedError("the embedding is part of begin_pass")
+
+    def begin_pass(self, idx: torch.Tensor, counts: Optional[Sequence[int]] = None) -> LayerStream:
+        if self.sequences is None:
+            raise ValueError("KV caches must be assigned to the model (see KVCacheFactory.create)")
+        if torch.is_grad_enabled():
+            raise NotImplementedError("models with described layers run in inference only (use torch.inference_mode())")
+        c = self.config
+        B, T = idx.shape
+        seq = self.sequences.begin(B, T, counts)
+        for cache in self.get_kv_caches():
+            cache.check_capacity(seq.max_end)
+        wte = self.transformer.wte.weight
+        dev, dt = wte.device, wte.dtype
+        idx = idx.contiguous()
+        history = torch.empty((c.n_layer + 1, B, T, c.n_embd), dtype=torch.float32, device=dev) if c.depth_average else None
+        x = history[0] if history is not None else torch.empty((B, T, c.n_embd), dtype=torch.float32, device=dev)
+        h = torch.empty((B, T, c.n_embd), dtype=dt, device=dev)
+        shifted = torch.empty_like(h) if c.token_shift else None
+        first = self.transformer.h[0].packed()
+        bg = c.bigram or dict(buckets=0, mul_prev=0, mul_cur=0)
+        L.embed_edge(idx, self.sequences.prev_token, wte, None if self.bigram is None else self.bigram.weight, bg["buckets"], bg["mul_prev"],
+                     bg["mul_cur"], x, first["gain"], first["shift"], self._shift_state(0), h, shifted, seq, c.norm_eps)
+        return LayerStream(seq, x, history, h, shifted)
+
+    def _shift_state(self, block_idx: int) -> Optional[torch.Tensor]:
+        return None if self.sequences.shift is None else self.sequences.shift[block_idx]
+
+    def run_layer(self, block_idx: int, x: LayerStream, idx: torch.Tensor, chunk_sizes: Optional[Sequence[int]] = None) -> LayerStream:
+        c = self.config
+        block = self.transformer.h[block_idx]
+        mixed = block.attn(x.h if x.shifted is None else x.shifted, x.seq)
+        experts = None if block.mlp is None else block.mlp(x.h)
+        nxt = self.transformer.h[block_idx + 1].packed() if block_idx + 1 < c.n_layer else {"gain": None, "shift": None}
+        state = self._shift_state(block_idx + 1) if nxt["shift"] is not None else None
+        out = x.spare if x.spare is not None else torch.empty_like(x.x)
+        L.layer_edge(x.x, mixed, experts, x.history, block_idx + 1, block.packed()["depth"], out, nxt["gain"], nxt["shift"], state,
+                     x.h, x.shifted, x.seq, c.norm_eps)
+        x.spare = None if x.history is not None and block_idx == 0 else x.x  # the embedding output stays in the history
+        x.x = out
+        return x
+
+    def end_pass(self, x: LayerStream, idx: torch.Tensor) -> torch.Tensor:
+        self.sequences.finish(x.seq, idx.contiguous())
+        return x.x
+
+    def head(self, x: torch.Tensor) -> torch.Tensor:
+        """Logits in fp32."""
+        rows = x.reshape(-1, self.config.n_embd).contiguous()
+        h = L.scalar_rmsnorm(rows, self._final_gain(), self.config.norm_eps, self.lm_head.weight.dtype)
+        return L.linear_fp32(h, self.lm_head.weight).view(*x.shape[:-1], -1)
+
+    def _final_gain(self) -> torch.Tensor:
+        return self.transformer.ln_f.weight.float()
+
+    def clone(self, device: Optional[torch.device] = None) -> "LayeredGPT":
+        sequences, self.sequences = self.sequences, None
+        try:
+            other = super().clone(device)
+        finally:
+            self.sequences = sequences
+            for cache in self.get_kv_caches():
+                if cache is not None:
+                    cache.sequences = sequences
+        return other

@@ -275,13 +275,16 @@ class GPT(nn.Module):
                 ln_f=config.norm_class(config.n_embd, eps=config.norm_eps),
             )
         )
-        self.mha = MultiHeadSelfAttention(config, **mha_kwargs)
+        self.mha = self._make_mha(config, **mha_kwargs)
         self._max_seq_length = config.block_size
         self._start_of_layer_hook: Optional[StartOfLayerHook] = None
         self._default_kv_cache = False
 
     def _make_block(self, config: Config, block_idx: int) -> Block:
         return Block(config, block_idx)
+
+    def _make_mha(self, config: Config, **mha_kwargs):
+        return MultiHeadSelfAttention(config, **mha_kwargs)
 
     # ------------------------------------------------------------ properties
     @property
@@ -366,6 +369,11 @@ class GPT(nn.Module):
             if cache is not None:
                 cache.reset()
 
+    def advance_host_counters(self) -> None:
+        """One token has been processed by a replayed graph: host-side counters move on."""
+        for cache in self.get_kv_caches():
+            cache.advance_host_counters()
+
     def get_kv_cache_params(self, block_idx: int):
         cache = self.transformer.h[block_idx].attn.kv_cache
         return None if cache is None else cache.get_params()
@@ -395,11 +403,29 @@ class GPT(nn.Module):
         x = self.transformer.ln_f(x)
         return do_softcapping(self.lm_head(x), self.config.final_logit_softcapping)
 
-    def forward(self, idx: torch.Tensor, skip_lm_head: bool = False, chunk_sizes: Optional[Sequence[int]] = None) -> torch.Tensor:
+    # A pass over ``idx (B, T)`` is begin_pass → run_layer for every layer → end_pass; :meth:`forward` and the chunked
+    # prefill (:class:`keys_values_b200.long_context.LongContextInferenceModel`) are written in terms of these.
+    def begin_pass(self, idx: torch.Tensor, counts: Optional[Sequence[int]] = None):
+        """The stream that enters the first layer. ``counts``: real tokens per right-padded row, for models that keep
+        a position per row."""
+        if counts is not None and any(n != idx.shape[1] for n in counts):
+            raise ValueError(f"{type(self).__name__} needs rows of equal length")
+        return self.embed(idx)
+
+    def run_layer(self, block_idx: int, x, idx: torch.Tensor, chunk_sizes: Optional[Sequence[int]] = None):
+        return self.transformer.h[block_idx](x, idx, self.mha, chunk_sizes=chunk_sizes)
+
+    def end_pass(self, x, idx: torch.Tensor):
+        """The stream after the last layer, before ``ln_f``."""
+        return x
+
+    def forward(self, idx: torch.Tensor, skip_lm_head: bool = False, chunk_sizes: Optional[Sequence[int]] = None,
+                counts: Optional[Sequence[int]] = None, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """``idx (B, T)`` token ids. With caches assigned, the first call after
         :meth:`reset` is the prefill, later calls continue the sequence; positions
         are tracked by the caches. Returns logits ``(B, T, padded_vocab)`` or, with
-        ``skip_lm_head``, the final hidden states before ``ln_f``."""
+        ``skip_lm_head``, the final hidden states before ``ln_f``. ``rows``: indices into the
+        ``B · T`` positions; logits ``(len(rows), padded_vocab)`` of these only."""
         if idx.ndim == 1:
             idx = idx.unsqueeze(0)
         T = idx.size(1)
@@ -407,16 +433,19 @@ class GPT(nn.Module):
         input_pos = caches[0].input_pos if caches[0] is not None else 0
         if input_pos + T > self.max_seq_length:
             raise ValueError(f"Cannot forward sequence: input_pos {input_pos} + {T} > max_seq_length {self.max_seq_length}")
-        x = self.embed(idx)
+        x = self.begin_pass(idx, counts)
         hook = self._start_of_layer_hook
-        for block_idx, block in enumerate(self.transformer.h):
+        for block_idx in range(self.config.n_layer):
             if hook is not None:
-                hook(x, block_idx)
-            x = block(x, idx, self.mha, chunk_sizes=chunk_sizes)
+                hook(x.full() if hasattr(x, "full") else x, block_idx)
+            x = self.run_layer(block_idx, x, idx, chunk_sizes)
+        x = self.end_pass(x, idx)
         if hook is not None:
             hook(x, self.config.n_layer)
         if skip_lm_head:
             return x
+        if rows is not None:
+            x = x.reshape(-1, x.shape[-1]).index_select(0, rows)
         return self.head(x)
 
     @classmethod

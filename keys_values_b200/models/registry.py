@@ -1,0 +1,93 @@
+"""Model classes and checkpoint readers by architecture.
+
+A LitGPT-shaped checkpoint (``lit_model.pth`` + ``model_config.yaml``) is a :class:`GPT`. Other architectures register a
+reader here; their checkpoint directories hold ``config.json`` (with an ``"architecture"`` entry) and ``model.safetensors``
+under the architecture's own tensor names.
+"""
+from __future__ import annotations
+
+import json
+from dataclasses import dataclass
+from pathlib import Path
+from typing import Any, Callable, Dict, Mapping, Optional, Union
+
+import torch
+
+from keys_values_b200.config import Config
+
+
+@dataclass(frozen=True)
+class Architecture:
+    name: str
+    config_from_json: Callable[[Dict[str, Any]], Config]
+    # the architecture's tensors (by name) -> state dict of the model class
+    state_dict: Callable[[Mapping[str, torch.Tensor], Config], Dict[str, torch.Tensor]]
+
+
+def _architectures() -> Dict[str, Architecture]:
+    from keys_values_b200.models import mezilix
+
+    return {a.name: a for a in (Architecture("Mezilix", mezilix.config_from_json, mezilix.state_dict),)}
+
+
+def architecture_names():
+    return sorted(_architectures())
+
+
+def get_architecture(name: str) -> Architecture:
+    known = _architectures()
+    if name not in known:
+        raise ValueError(f"architecture {name!r} is not registered; known: {sorted(known)}")
+    return known[name]
+
+
+def config_from_directory(path: Union[str, Path], **kwargs: Any) -> Optional[Config]:
+    """Config of a checkpoint directory with a registered architecture's ``config.json``, else ``None``."""
+    file = Path(path) / "config.json"
+    if not file.is_file():
+        return None
+    content = json.loads(file.read_text(encoding="utf-8"))
+    if not isinstance(content, dict) or "architecture" not in content:
+        return None
+    config = get_architecture(content["architecture"]).config_from_json(content)
+    for k, v in kwargs.items():
+        setattr(config, k, v)
+    return config
+
+
+def model_class(config: Config):
+    from keys_values_b200.models.layered import LayeredGPT
+    from keys_values_b200.models.model import GPT
+
+    return GPT if config.layers is None else LayeredGPT
+
+
+def create_model(config: Config, **mha_kwargs):
+    """The model of ``config``, with whatever class its description needs."""
+    return model_class(config)(config, **mha_kwargs)
+
+
+def default_cache_name(config: Config, name: Optional[str] = None) -> str:
+    """``name``, or for models with described layers the cache that fits them."""
+    if config.layers is None:
+        return name or "h2o-default"
+    return name if name is not None and name.startswith("latent") else "latent-default"
+
+
+def read_safetensors(path: Path) -> Dict[str, torch.Tensor]:
+    from safetensors.torch import load_file
+
+    return load_file(str(path))
+
+
+def load_architecture_weights(model, checkpoint_dir: Union[str, Path]) -> bool:
+    """Weights of a registered architecture's ``*.safetensors`` into ``model``; ``False`` if the directory is not one."""
+    checkpoint_dir = Path(checkpoint_dir)
+    files = sorted(checkpoint_dir.glob("*.safetensors"))
+    if not model.config.architecture or not files:
+        return False
+    tensors: Dict[str, torch.Tensor] = {}
+    for f in files:
+        tensors.update(read_safetensors(f))
+    model.load_state_dict(get_architecture(model.config.architecture).state_dict(tensors, model.config), strict=True)
+    return True
