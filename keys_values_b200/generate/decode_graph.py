@@ -17,6 +17,7 @@ returns ``None`` and falls back to the same eager call otherwise.
 """
 from __future__ import annotations
 
+from contextlib import nullcontext
 from typing import Optional
 
 import torch
@@ -88,19 +89,21 @@ class DecodeGraph:
 
         model = self.model
         dev = tokens.device
-        input_pos = model.get_kv_caches()[0].input_pos
         self.tokens = tokens.clone()
-        self.word = torch.tensor([input_pos], dtype=torch.int32, device=dev)
+        own = model.tracks_positions
+        if not own:
+            self.word = torch.tensor([model.get_kv_caches()[0].input_pos], dtype=torch.int32, device=dev)
         self.graph = torch.cuda.CUDAGraph()
         torch.cuda.synchronize(dev)
         comm = getattr(model, "tp_comm", None)  # tensor-parallel shard: its all-reduce calls take their epochs from a device word
         try:
-            with cu.device_position(self.word):
+            with nullcontext() if own else cu.device_position(self.word):
                 with torch.cuda.graph(self.graph):
                     if comm is not None:
                         comm.begin_capture()
                     self.logits = model(self.tokens)
-                    self.word.add_(1)  # a scalar operand: nothing outside the graph's own memory is read here
+                    if not own:
+                        self.word.add_(1)  # a scalar operand: nothing outside the graph's own memory is read here
                     if comm is not None:
                         comm.end_capture()
         except BaseException:

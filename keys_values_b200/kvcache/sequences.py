@@ -84,11 +84,10 @@ class SequenceTable:
 
     # ----------------------------------------------------------------- passes
     def _const(self, values: Tuple[int, ...]) -> torch.Tensor:
-        """Small int32 tensor; single-token passes find theirs here, so that a captured step copies nothing."""
+        """Small int32 tensor that stays: single-token passes find theirs here, so a captured step copies nothing and its
+        graph can keep reading it."""
         t = self._consts.get(values)
         if t is None:
-            if len(self._consts) > 256:
-                self._consts.clear()
             with torch.inference_mode(False):
                 t = self._consts[values] = torch.tensor(values, dtype=torch.int32, device=self.device)
         return t
@@ -105,7 +104,8 @@ class SequenceTable:
             raise ValueError(f"counts {counts} must give 0 .. {length} tokens for each of {batch_size} rows")
         slots = self.batch
         start = self.pos[:batch_size] if slots == tuple(range(batch_size)) else self.pos.index_select(0, self._const(slots))
-        return SequencePass(self._const(slots), start, self._const(counts), slots, tuple(self.pos_host[s] for s in slots), counts, length)
+        count = self._const(counts) if length == 1 else torch.tensor(counts, dtype=torch.int32, device=self.device)
+        return SequencePass(self._const(slots), start, count, slots, tuple(self.pos_host[s] for s in slots), counts, length)
 
     def finish(self, seq: SequencePass, idx: torch.Tensor) -> None:
         from keys_values_b200.ops import layers as L

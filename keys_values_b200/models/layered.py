@@ -66,7 +66,7 @@ class _Packed(nn.Module):
 
     def packed(self) -> Dict[str, torch.Tensor]:
         if self._pack is None:
-            with torch.no_grad(), torch.inference_mode(False):
+            with torch.inference_mode(False), torch.no_grad():
                 self._pack = self._make_pack()
         return self._pack
 
@@ -235,6 +235,8 @@ class LayeredGPT(GPT):
     """:class:`GPT` for configs with ``layers``. Rows of a batch may have different lengths: ``counts`` of
     :meth:`forward` says how many tokens of each (right-padded) row are real."""
 
+    tracks_positions = True
+
     def __init__(self, config: Config, **mha_kwargs) -> None:
         if config.layers is None or len(config.layers) != config.n_layer:
             raise ValueError("config.layers must describe every layer")
@@ -308,6 +310,9 @@ class LayeredGPT(GPT):
             self.sequences.reset()
 
     def advance_host_counters(self) -> None:
+        end = 1 + max(self.sequences.pos_host[s] for s in self.sequences.batch)
+        for cache in self.get_kv_caches():
+            cache.check_capacity(end)
         self.sequences.advance_host()
 
     def max_pass_tokens(self, batch_size: int) -> int:

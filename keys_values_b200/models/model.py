@@ -263,6 +263,9 @@ StartOfLayerHook = Callable[[torch.Tensor, int], None]
 
 
 class GPT(nn.Module):
+    # True: positions live in device tensors of the model, a captured step needs no position word
+    tracks_positions = False
+
     def __init__(self, config: Config, **mha_kwargs) -> None:
         super().__init__()
         assert config.padded_vocab_size is not None

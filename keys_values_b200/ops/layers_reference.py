@@ -133,7 +133,7 @@ def latent_decode(q_abs, q, ring, seq, s, scale):
 def moe_forward(h, logits, up, down, top, act, renormalize, n_up, n_down):
     n, width = h.shape
     scores = logits.softmax(-1)
-    weight, expert = scores.topk(top, dim=-1)
+    weight, expert = (t[:, :top] for t in torch.sort(scores, dim=-1, descending=True, stable=True))  # ties: lower index
     if renormalize:
         weight = weight / weight.sum(-1, keepdim=True)
     out = torch.zeros(n * top, (n_down + 7) // 8 * 8, dtype=h.dtype)
