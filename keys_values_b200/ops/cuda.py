@@ -87,7 +87,8 @@ def status_word(device) -> torch.Tensor:
     """Per-device int32 word that kernels with bounded waits write their error code to."""
     key = torch.device(device).index or 0
     if key not in _STATUS:
-        _STATUS[key] = torch.zeros(1, dtype=torch.int32, device=device)
+        with torch.inference_mode(False):  # cleared inside and outside of inference mode
+            _STATUS[key] = torch.zeros(1, dtype=torch.int32, device=device)
     return _STATUS[key]
 
 

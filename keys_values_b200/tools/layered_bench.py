@@ -1,0 +1,295 @@
+"""Prefill and decode throughput of a model with described layers beside the closest LitGPT-shaped model of equal size, and the
+time of every kernel of the design beside the like kernel of that model, each against its roofline.
+
+    python -m keys_values_b200.tools.layered_bench [--model Mezilix-2k] [--batch 32] [--prompt 8192] [--decode 128] [--kernels]
+
+Random-init weights, synthetic tokens. The closest model has the same width, depth, heads, window and experts (count, chosen per
+token, expert weights per token): grouped-query attention over a sliding window, SwiGLU experts (``LLaMAMoE``); ``--dense``
+compares with a dense SwiGLU of the width that a token's chosen experts add up to. Kernel times are CUDA-event
+medians with an L2 flush (256 MB write) before every launch.
+"""
+from __future__ import annotations
+
+import argparse
+import json
+from pathlib import Path
+from typing import Callable, Dict, List, Optional
+
+import torch
+
+from keys_values_b200.config import Config
+
+
+def closest_config(config: Config, dense: bool = False) -> Config:
+    """LitGPT-shaped model of the same size: heads of 128, all of them keys and values, the same window; expert (or dense) width
+    such that a token meets the same number of feed-forward weights (three matrices instead of two)."""
+    m, f = config.layers[0]["mixer"], config.layers[0]["mlp"]
+    ff = f["ff"] * 2 // 3 // 8 * 8
+    kw = dict(
+        name=f"closest-to-{config.name}", block_size=1 << 17, vocab_size=config.vocab_size, padded_vocab_size=config.padded_vocab_size,
+        n_layer=config.n_layer, n_embd=config.n_embd, n_head=m["n_head"], n_query_groups=m["n_head"], head_size=128, rotary_percentage=1.0,
+        parallel_residual=False, bias=False, norm_class_name="RMSNorm", norm_eps=config.norm_eps, sliding_window_size=m["window"],
+    )
+    if dense:
+        return Config(mlp_class_name="LLaMAMLP", intermediate_size=ff * f["top"], **kw)
+    return Config(mlp_class_name="LLaMAMoE", intermediate_size=ff, moe_intermediate_size=ff, n_expert=f["n_expert"], n_expert_per_token=f["top"], **kw)
+
+
+def _build(config: Config, batch: int, cache_length: int, dev: torch.device):
+    from keys_values_b200.kvcache.factory import KVCacheFactory
+    from keys_values_b200.models.registry import create_model
+
+    torch.manual_seed(0)
+    with torch.device(dev):
+        model = create_model(config).to(torch.bfloat16).eval()
+    name = "lastrec-default" if config.layers is None else "latent-default"
+    kw = dict(init_grace_tokens=0) if config.layers is None else None
+    model.assign_kv_caches(KVCacheFactory.create(model, name, batch, cache_length, device=dev, dtype=torch.bfloat16, cache_kwargs=kw))
+    return model
+
+
+@torch.inference_mode()
+def throughput(config: Config, batch: int, prompt: int, decode: int, window: int, chunk: int = 2048, repeats: int = 2) -> Dict:
+    """Best of ``repeats`` runs: prompts from pinned host memory, generated tokens read back inside the timed regions."""
+    from keys_values_b200 import ops
+    from keys_values_b200.generate.base import _prefill, batched_sample
+    from keys_values_b200.generate.decode_graph import Decoder
+
+    dev = torch.device("cuda", torch.cuda.current_device())
+    model = _build(config, batch, window, dev)
+    host = torch.randint(0, config.vocab_size, (batch, prompt), generator=torch.Generator().manual_seed(7)).pin_memory()
+    greedy, warm = dict(temperature=0.0), 8
+    total = prompt + decode + warm + 8
+    _prefill(model, host[:, : min(prompt, window + 2 * chunk)].to(dev), chunk, total)
+    best: Optional[Dict] = None
+    for _ in range(repeats):
+        torch.cuda.synchronize(dev)
+        launches = ops.native_launches()
+        e = [torch.cuda.Event(enable_timing=True) for _ in range(4)]
+        e[0].record()
+        logits = _prefill(model, host.to(dev, non_blocking=True), chunk, total)
+        e[1].record()
+        tokens = logits.argmax(-1).view(batch, 1)
+        decoder = Decoder(model, batch)
+        for _ in range(warm):
+            tokens = batched_sample(decoder(tokens)[:, -1:], greedy).view(batch, 1)
+        torch.cuda.synchronize(dev)
+        e[2].record()
+        out = []
+        for _ in range(decode):
+            tokens = batched_sample(decoder(tokens)[:, -1:], greedy).view(batch, 1)
+            out.append(tokens)
+        torch.cat(out, dim=1).cpu()
+        e[3].record()
+        torch.cuda.synchronize(dev)
+        t_pre, t_dec = e[0].elapsed_time(e[1]) / 1e3, e[2].elapsed_time(e[3]) / 1e3
+        if best is None or t_pre + t_dec < best["prefill_s"] + best["decode_s"]:
+            best = dict(
+                model=config.name, batch=batch, prompt=prompt, decode_steps=decode, prefill_s=t_pre, decode_s=t_dec,
+                prefill_tokens_per_s=batch * prompt / t_pre, decode_tokens_per_s=batch * decode / t_dec, ms_per_decode_step=1e3 * t_dec / decode,
+                decode_mode="cuda graph" if decoder.graph is not None else f"eager ({decoder.reason})",
+                native_launches=ops.native_launches() - launches, peak_mem_gb=torch.cuda.max_memory_allocated(dev) / 2**30,
+                parameters=sum(p.numel() for p in model.parameters()),
+            )
+    ops.check_status(dev)
+    return best
+
+
+# ------------------------------------------------------------------------------------------------- kernels
+def _peaks() -> Dict[str, float]:
+    file = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
+    got = json.loads(file.read_text()) if file.is_file() else {}
+    return dict(gbs=got.get("hbm_gbs", 6650.0), tflops=got.get("bf16_tflops", 1590.0))
+
+
+def time_us(fn: Callable[[], None], flush: torch.Tensor, n: int = 15) -> float:
+    times = []
+    for i in range(n + 3):
+        flush.fill_(i & 127)
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        fn()
+        b.record()
+        torch.cuda.synchronize()
+        if i >= 3:
+            times.append(a.elapsed_time(b) * 1e3)
+    return sorted(times)[len(times) // 2]
+
+
+class KernelTable:
+    def __init__(self):
+        self.peaks = _peaks()
+        self.flush = torch.empty(256 * 2**20, dtype=torch.uint8, device="cuda")
+        self.rows: List[Dict] = []
+
+    def add(self, what: str, fn: Callable[[], None], gbytes: float = 0.0, tflop: float = 0.0) -> None:
+        us = time_us(fn, self.flush)
+        roof = 1e6 * max(gbytes / self.peaks["gbs"], tflop / self.peaks["tflops"])
+        self.rows.append(dict(kernel=what, us=round(us, 1), roofline_us=round(roof, 1), fraction=round(roof / us, 3),
+                              bound="memory" if gbytes / self.peaks["gbs"] > tflop / self.peaks["tflops"] else "math"))
+        print(f"{what:64s} {us:9.1f} us   roofline {roof:8.1f} us   {roof / us:6.3f}", flush=True)
+
+
+def _window_pairs(T: int, P: int, window: int) -> int:
+    """Visible (query, key) pairs of T new tokens after P cached ones."""
+    return sum(min(P + t + 1, window) for t in range(T))
+
+
+@torch.inference_mode()
+def kernel_table(config: Config, batch: int, tokens: int = 8192, dense_like: bool = True) -> List[Dict]:
+    """Kernels of one middle layer of ``config``: a pass of ``tokens`` new tokens of one sequence with a full window before them,
+    and a single-token pass of ``batch`` sequences with full rings; like kernels of the closest model after each."""
+    from keys_values_b200 import ops
+    from keys_values_b200.kvcache.sequences import SequenceTable
+    from keys_values_b200.models.layered import latent_shape
+    from keys_values_b200.ops import cuda as cu
+    from keys_values_b200.ops import layers as L
+    from keys_values_b200.ops import layers_cuda as LC
+
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    tab = KernelTable()
+    m, f = config.layers[0]["mixer"], config.layers[0]["mlp"]
+    s, W, win = latent_shape(m), config.n_embd, m["window"]
+    H, E, top, ff = s.heads, f["n_expert"], f["top"], f["ff"]
+    mid, eps = config.n_layer // 2, config.norm_eps
+    rand = lambda *shape: torch.randn(*shape, device=dev, dtype=bf)  # noqa: E731
+
+    def sequences(B, start):
+        t = SequenceTable(B, dev, 1, W)
+        t.set_batch([t.acquire() for _ in range(B)])
+        t.pos.fill_(start)
+        t.pos_host = [start] * B
+        return t
+
+    up, down = 0.02 * rand(E, ff, W), 0.02 * rand(E, W, ff)
+    gain, blend, coef = torch.ones((), device=dev), torch.rand(W, device=dev), torch.rand(mid + 2, device=dev)
+    for B, T in ((1, tokens), (batch, 1)):
+        n = B * T
+        tag = f"prefill {T} tokens" if T > 1 else f"decode {B} rows"
+        seq = sequences(B, 2 * win).begin(B, T)
+        seq.start = seq.start.clone()
+        # ---- layer edge
+        hist = torch.randn(mid + 2, B, T, W, device=dev)
+        x, out, mix = torch.randn(B, T, W, device=dev), torch.empty(B, T, W, device=dev), rand(B, T, W)
+        h, hs = torch.empty_like(mix), torch.empty_like(mix)
+        ex = rand(n * top, W)
+        row = torch.randperm(n * top, device=dev).int().view(n, top)
+        wt = torch.rand(n, top, device=dev)
+        state = torch.zeros(B, W, device=dev)
+        tab.add(f"{tag}: layer edge ({mid + 1} streams, {top} experts)",
+                lambda: LC.layer_edge(x, mix, ex, row, wt, hist, mid + 1, coef, out, gain, blend, state, h, hs, seq, eps),
+                gbytes=n * W * (4 * (mid + 1) + 4 + 2 + 2 * top + 4 + 4 + 2 + 2) / 1e9)
+        a, r, w1 = rand(n, W), rand(n, W), rand(W)
+        if cu.add_rmsnorm_supported(a):
+            tab.add(f"{tag}:   like: add + RMSNorm", lambda: cu.add_rmsnorm_fwd(a, r, w1, eps, False), gbytes=n * W * 8 / 1e9)
+        else:
+            tab.add(f"{tag}:   like: RMSNorm", lambda: cu.rmsnorm_fwd(a, w1, eps, False), gbytes=n * W * 4 / 1e9)
+        del hist, ex
+        # ---- latent prep
+        qkv = rand(B, T, H * (s.dim + s.rot) + s.kv_rank + s.rot)
+        norm, freq = torch.ones(s.kv_rank, device=dev), torch.rand(s.rot_dims // 2, device=dev)
+        ring = rand(B, win, s.row)
+        P = win - 1 if T > 1 else 0
+        lat = rand(B, P + T, s.row)
+        if T > 1:
+            prep = lambda: LC.latent_prep(qkv, norm, freq, lat, None, seq, P, s, eps)  # noqa: E731
+        else:
+            prep = lambda: LC.latent_prep(qkv, norm, freq, None, ring, seq, 0, s, eps)  # noqa: E731
+        tab.add(f"{tag}: split, latent norm, rotation", prep, gbytes=n * 2 * (qkv.shape[2] + H * (s.dimp + s.rp) + s.row) / 1e9)
+        qkv2, cs = rand(B, T, 3 * H * 128), torch.rand(T, 128, device=dev)
+        tab.add(f"{tag}:   like: split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, None, None, H, H, 128, eps, 128, False),
+                gbytes=n * 2 * 2 * qkv2.shape[2] / 1e9)
+        if T > 1:
+            tab.add(f"{tag}: ring gather", lambda: LC.ring_gather(ring, lat, seq, P), gbytes=B * P * s.row * 4 / 1e9)
+            tab.add(f"{tag}: ring append", lambda: LC.ring_append(lat, ring, seq, P), gbytes=B * min(T, win) * s.row * 4 / 1e9)
+            kb, vb, tp = (rand(B, H, win, 128) for _ in range(2)), None, torch.zeros(B, H, win, dtype=torch.int32, device=dev)
+            kb, vb = kb
+            nk, slots = rand(B, H, min(T, win), 128), torch.arange(min(T, win), device=dev).int().view(1, 1, -1).expand(B, H, -1)
+            tab.add(f"{tag}:   like: cache write", lambda: cu.cache_write(kb, vb, tp, slots, nk, nk, 0), gbytes=B * H * min(T, win) * 128 * 8 / 1e9)
+            # ---- attention over expanded keys
+            q, kv = rand(B, T, H, s.dimp + s.rp), rand(B * (P + T), H * (s.dimp + s.vdp))
+            pairs = B * H * _window_pairs(T, P, win)
+            tab.add(f"{tag}: attention {s.dim}+{s.rot} / {s.vdim}, window {win}", lambda: LC.latent_attend(q, kv, lat, seq, P, s, win, 0.07),
+                    tflop=2 * pairs * (s.dim + s.rot + s.vdim) / 1e12)
+            q2, k2 = rand(B, H, T, 128), rand(B, H, P + T, 128)
+            tab.add(f"{tag}:   like: attention 128 / 128, window {win}", lambda: cu.sdpa_fwd(q2, k2, k2, 0.09, P, None, False, win, None),
+                    tflop=2 * pairs * 256 / 1e12)
+            del q, kv, q2, k2, kb, vb
+        else:
+            q, qa = rand(B, 1, H, s.dimp + s.rp), rand(H, B, s.kvp)
+            tab.add(f"{tag}: attention over the ring of {win}", lambda: LC.latent_decode(qa, q, ring, seq, s, 0.07),
+                    gbytes=B * win * s.row * 2 / 1e9, tflop=2 * B * win * H * (2 * s.kv_rank + s.rot) / 1e12)
+            q2, k2, v2 = rand(B, H, 1, 128), rand(B, H, win, 128), rand(B, H, win, 128)
+            tp = torch.arange(win, device=dev, dtype=torch.int32).expand(B, H, win).contiguous()
+            tab.add(f"{tag}:   like: attention over {win} slots", lambda: cu.decode_attention(q2, k2, v2, 0.09, win, False, sliding_window=win,
+                    token_pos=tp, query_pos=win - 1), gbytes=2 * B * H * win * 128 * 2 / 1e9)
+            del k2, v2
+        # ---- routed experts
+        hn = rand(n, W)
+        logits = torch.randn(n, E, device=dev)
+        used = E if n * top >= 4 * E else E * (1 - (1 - 1 / E) ** (n * top))
+        tab.add(f"{tag}: routed experts, all kernels ({E} x {ff}, top {top})",
+                lambda: LC.moe_forward(hn, logits, up, down, top, 1, False, ff, W),
+                gbytes=2 * (used * 2 * ff * W + n * W * (1 + top)) / 1e9, tflop=4 * n * top * ff * W / 1e12)
+        from keys_values_b200.models.model import LLaMAMLP, LLaMAMoE
+
+        for dense in (False, True):
+            cc = closest_config(config, dense)
+            with torch.device(dev):
+                mlp = (LLaMAMLP if dense else LLaMAMoE)(cc).to(bf)
+            x3 = hn.view(1, n, W)
+            fl = 6 * n * cc.intermediate_size * (1 if dense else top) * W / 1e12
+            by = 2 * (3 * cc.intermediate_size * W * (1 if dense else used) + 2 * n * W) / 1e9
+            tab.add(f"{tag}:   like: {'dense SwiGLU' if dense else 'LLaMAMoE'}, all kernels", lambda: mlp(x3), gbytes=by, tflop=fl)
+            del mlp
+        tile = LC.moe_tile(n * top, E, bf)
+        cap = n * top // tile + min(E, n * top)
+        buf, hid = rand(cap * tile, W), torch.empty(cap * tile, ff, device=dev, dtype=bf)
+        ids = torch.randint(0, E, (n * top,), device=dev)
+        cnt = torch.bincount(ids, minlength=E)
+        tiles = ((cnt + tile - 1) // tile)
+        te = torch.repeat_interleave(torch.arange(E, device=dev), tiles).int()
+        plan = torch.tensor([te.numel()], device=dev, dtype=torch.int32)
+        tr = (torch.arange(te.numel(), device=dev) * tile).int()
+        st = cu.status_word(dev)
+        ll, p_ = cu._ll, cu._p
+
+        def grouped(src, w, dst, n_out, k, act):
+            cu._check(LC.lib().kvb_moe_gemm(p_(src), p_(w), p_(dst), p_(plan), p_(te), p_(tr), tile, cap, E, n_out, k, ll(k), ll(n_out), act, 1, 0,
+                                            p_(st), cu._stream(src)), "moe_gemm")
+
+        us_e = int((cnt > 0).sum())
+        tab.add(f"{tag}: grouped product up (tile {tile})", lambda: grouped(buf, up, hid, ff, W, 1),
+                gbytes=2 * (us_e * ff * W + n * top * (W + ff)) / 1e9, tflop=2 * n * top * ff * W / 1e12)
+        tab.add(f"{tag}: grouped product down (tile {tile})", lambda: grouped(hid, down, buf, W, ff, 0),
+                gbytes=2 * (us_e * ff * W + n * top * (W + ff)) / 1e9, tflop=2 * n * top * ff * W / 1e12)
+        w2, a2 = rand(ff * top, W), rand(n, W)
+        tab.add(f"{tag}:   like: library product {n} x {ff * top} x {W}", lambda: torch.mm(a2, w2.t()),
+                gbytes=2 * (ff * top * W + n * (W + ff * top)) / 1e9, tflop=2 * n * ff * top * W / 1e12)
+        del buf, hid
+    ops.check_status(dev)
+    return tab.rows
+
+
+def main() -> None:
+    ap = argparse.ArgumentParser()
+    ap.add_argument("--model", default="Mezilix-2k")
+    ap.add_argument("--batch", type=int, default=32)
+    ap.add_argument("--prompt", type=int, default=8192)
+    ap.add_argument("--decode", type=int, default=128)
+    ap.add_argument("--kernels", action="store_true", help="kernel table instead of model throughput")
+    ap.add_argument("--n-layer", type=int, default=None)
+    args = ap.parse_args()
+    config = Config.from_name(args.model)
+    if args.n_layer is not None:
+        config.layers, config.n_layer = config.layers[: args.n_layer], args.n_layer
+    if args.kernels:
+        kernel_table(config, args.batch)
+        return
+    window = config.layers[0]["mixer"]["window"]
+    for c in (config, closest_config(config), closest_config(config, dense=True)):
+        print(json.dumps(throughput(c, args.batch, args.prompt, args.decode, window)), flush=True)
+
+
+if __name__ == "__main__":
+    main()
