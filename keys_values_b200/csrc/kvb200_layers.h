@@ -57,7 +57,7 @@ int kvb_latent_attend(const void* q, const void* kv, const void* latent, void* o
 long long kvb_latent_decode_scratch_bytes(int B, int heads, int kvp, int ring_len);
 int kvb_latent_decode(const void* q_abs, const void* q, const void* ring, void* out, void* scratch, const int* slots,
                       const int* start, int B, int heads, int dimp, int rp, int kvp, int ring_len, float scale, int dtype,
-                      int simple, void* stream);
+                      int simple, int* status, void* stream);
 
 // ---- latent_sm100.cu: kvb_latent_attend for bf16 on tcgen05
 int kvb_latent_attend_tc_supported(int dimp, int rp, int vdp);

@@ -76,6 +76,8 @@ class DecodeGraph:
             if not cache.kv_buffers.supports_direct_decode() or getattr(cache.kv_buffers, "before_access", None) is not None:
                 return "the cache buffers are not read in place by the decode kernel"
         c = model.config
+        if c.mlp_class_name == "LLaMAMoE":
+            return "the experts of LLaMAMoE are looped over on the host"
         if c.head_size != 128 or c.n_head % c.n_query_groups != 0:
             return "the decode kernel needs head size 128"
         return None

@@ -140,7 +140,7 @@ def latent_decode(q_abs, q, ring, seq, shape, scale) -> torch.Tensor:
     nbytes = int(lib().kvb_latent_decode_scratch_bytes(B, H, kvp, C))
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
     _check(lib().kvb_latent_decode(_p(q_abs), _p(q), _p(ring), _p(out), _p(scratch), _p(seq.slots), _p(seq.start), B, H, s.dimp, s.rp, kvp,
-                                   C, _f(scale), code(q.dtype), int(FORCE_SIMPLE), _stream(q)), "latent_decode")
+                                   C, _f(scale), code(q.dtype), int(FORCE_SIMPLE), _p(status_word(q.device)), _stream(q)), "latent_decode")
     _count()
     return out
 
