@@ -39,25 +39,24 @@ int kvb_sequence_advance(const long long* idx, int* pos, int* prev_token, const 
 // ---- latent_attn.cu
 // One row of the latent storage: [c (kv_rank, padded to kvp) | rotated key part (rot, padded to rp)], kvp and rp
 // multiples of 8, padding zero. Queries: [unrotated (dim padded to dimp) | rotated (rot padded to rp)] per head.
+// prep: latent rows go to latent (B, P+T, kvp+rp) from row P on (NULL: not) and those of the last ring_len real tokens to ring
+// (slots, ring_len, kvp+rp) (NULL: not), position p in row p mod ring_len.
 int kvb_latent_prep(const void* qkv, long long ld, const float* norm_w, const float* freq, void* q, void* latent, void* ring,
                     const int* slots, const int* start, const int* count, int B, int T, int P, int ring_len, int heads, int dim,
                     int dimp, int rot, int rot_dims, int rp, int kv_rank, int kvp, float eps, int dtype, void* stream);
 // latent[b, j] (j < P) = ring row of position start[b] − P + j, zero where there is none
 int kvb_ring_gather(const void* ring, void* latent, const int* slots, const int* start, int B, int T, int P, int ring_len, int lw,
                     int dtype, void* stream);
-// the last min(count, ring_len) new rows of every sequence into its ring
-int kvb_ring_append(const void* latent, void* ring, const int* slots, const int* start, const int* count, int B, int T, int P,
-                    int ring_len, int lw, int dtype, void* stream);
 // Attention of T new tokens over P + T expanded keys: kv (B, P+T, heads, dimp + vdp) = [unrotated key | value],
 // latent (B, P+T, lw) holds the rotated key part at column kvp. out (B, T, heads, vdp).
 int kvb_latent_attend(const void* q, const void* kv, const void* latent, void* out, const int* start, int B, int T, int P, int heads,
                       int dimp, int rp, int kvp, int vdp, int window, float scale, int dtype, void* stream);
 // One new token per sequence over its ring, in latent space: q_abs (heads, B, kvp) = W_uk^T q, q (B, heads, dimp + rp) for
 // the rotated part, out (heads, B, kvp) = weighted latents.
-long long kvb_latent_decode_scratch_bytes(int B, int heads, int kvp, int ring_len);
+long long kvb_latent_decode_scratch_bytes(int B, int heads, int kvp, int rp, int ring_len);
 int kvb_latent_decode(const void* q_abs, const void* q, const void* ring, void* out, void* scratch, const int* slots,
-                      const int* start, int B, int heads, int dimp, int rp, int kvp, int ring_len, float scale, int dtype,
-                      int simple, int* status, void* stream);
+                      const int* start, int B, int n_slots, int heads, int dimp, int rp, int kvp, int ring_len, float scale,
+                      int dtype, int simple, int* status, void* stream);
 
 // ---- latent_sm100.cu: kvb_latent_attend for bf16 on tcgen05
 int kvb_latent_attend_tc_supported(int dimp, int rp, int vdp);

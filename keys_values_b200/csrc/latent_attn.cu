@@ -1,22 +1,27 @@
 // Latent attention: queries of H heads against one latent per token (plus one rotated key part that the heads share).
 //
 //   prep    splits the joint projection, norms the latent, rotates the rotary parts (angles in fp32, computed once per
-//           token), writes padded query and latent rows; a single-token pass writes its latent row straight into the ring;
+//           token), writes padded query and latent rows, the latter to the buffer of the pass and into the ring;
 //   ring    a layer that sees a window of W tokens keeps W latents per sequence: position p lives in slot p mod length;
 //   attend  several new tokens: keys and values of the window before the pass and of the pass itself are expanded from
 //           the latents by a matrix product and swept with an online softmax (here on CUDA cores, for fp32 and for shapes the
 //           tcgen05 kernel of latent_sm100.cu does not take);
 //   decode  one new token per sequence stays in latent space: W_uk is folded into the query and W_uv into the output, so
 //           the ring is read once for all heads and serves as key and value.
+#include <cuda.h>
+
 #include "common.cuh"
 #include "kvb200_layers.h"
+#include "tmap.cuh"
 
 namespace kvb {
 
 // ------------------------------------------------------------------------------------------------ prep
-// One warp per unit of a token: unit h < heads is a query head, unit `heads` the latent row. A CTA has 8 units of one token and
-// computes the token's angles once. V elements per access (16 bytes, or 1 when the sizes do not divide).
-constexpr int LP_WARPS = 8;
+// A CTA has RUN consecutive tokens of a row. First the angles of its tokens and the root mean squares of their latents (one
+// warp per token), then the columns that are only copied or normed, then the rotary ones (V elements per access, 16 bytes; 1 when
+// the sizes do not divide).
+constexpr int LP_THREADS = 256;
+constexpr int LP_RUN = 2;  // tokens of a CTA when there are many
 
 template <typename T, int V>
 struct alignas(sizeof(T) * V) LpVec {
@@ -28,89 +33,153 @@ struct LpParams {
   const float *norm_w, *freq;
   const int *slots, *start, *count;
   int T, P, ring_len, heads, dim, dimp, rot, rot_dims, rp, kv_rank, kvp;
+  unsigned plain_magic, rot_magic;
   float eps;
 };
 
-// the rotary part x (rot elements, the first rot_dims rotated) to dst, zero up to rp
-template <typename T, int V>
-__device__ __forceinline__ void lp_rotate(const T* __restrict__ x, T* __restrict__ dst, const float* cs, const float* sn, const LpParams& p,
-                                          int lane) {
+template <typename T, int V, int RUN>
+__global__ void __launch_bounds__(LP_THREADS, 6)
+latent_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict__ latent, T* __restrict__ ring, const LpParams p) {
   using Vec = LpVec<T, V>;
-  const int half = p.rot_dims / 2;
-  for (int i = lane * V; i < half; i += 32 * V) {
-    const Vec a = *reinterpret_cast<const Vec*>(x + i), b = *reinterpret_cast<const Vec*>(x + half + i);
-    Vec c, d;
-#pragma unroll
-    for (int e = 0; e < V; ++e) {
-      const float u = to_f32(a.v[e]), v = to_f32(b.v[e]);
-      c.v[e] = from_f32<T>(u * cs[i + e] - v * sn[i + e]);
-      d.v[e] = from_f32<T>(v * cs[i + e] + u * sn[i + e]);
-    }
-    *reinterpret_cast<Vec*>(dst + i) = c;
-    *reinterpret_cast<Vec*>(dst + half + i) = d;
+  extern __shared__ float sm[];  // per token: cos | sin (rot_dims / 2 each)
+  __shared__ float inv_rms[RUN];
+  const int t0 = blockIdx.x * RUN, b = blockIdx.y;
+  const int nt = min(RUN, p.T - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int start = p.start[b], half = p.rot_dims / 2;
+  const int c0 = p.heads * (p.dim + p.rot);
+  const long long n0 = (long long)b * p.T + t0;
+  for (int i = threadIdx.x; i < nt * half; i += LP_THREADS) {
+    const int t = i / half, k = i - t * half;
+    sincosf((float)(start + t0 + t) * p.freq[k], &sm[t * p.rot_dims + half + k], &sm[t * p.rot_dims + k]);
   }
-  for (int i = p.rot_dims + lane; i < p.rp; i += 32) dst[i] = i < p.rot ? x[i] : from_f32<T>(0.f);
+  if (warp < nt) {
+    const T* c = qkv + (n0 + warp) * p.ld + c0;
+    float ss = 0.f;
+    for (int i = lane * V; i < p.kv_rank; i += 32 * V) {
+      const Vec a = *reinterpret_cast<const Vec*>(c + i);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(to_f32(a.v[e]), to_f32(a.v[e]), ss);
+    }
+    ss = warp_sum(ss);
+    if (lane == 0) inv_rms[warp] = 1.f / sqrtf(ss / (float)p.kv_rank + p.eps);
+  }
+  __syncthreads();
+  const int dq = p.dimp + p.rp, lw = p.kvp + p.rp;
+  const int last = p.count[b];
+  const T* src0 = qkv + n0 * p.ld;
+  // where token t of this CTA has its latent row in the ring: the last ring_len tokens of the pass, no padding
+  auto ring_row = [&](int t) -> T* {
+    const int tt = t0 + t;
+    if (!ring || tt >= last || tt < last - p.ring_len) return nullptr;
+    return ring + ((long long)p.slots[b] * p.ring_len + (start + tt) % p.ring_len) * lw;
+  };
+  auto put_latent = [&](int t, int col, const Vec& v) {
+    if (latent) *reinterpret_cast<Vec*>(latent + ((long long)b * (p.P + p.T) + p.P + t0 + t) * lw + col) = v;
+    T* r = ring_row(t);
+    if (r) *reinterpret_cast<Vec*>(r + col) = v;
+  };
+  // ---- columns that are not rotated: all tokens are loaded before any is stored
+  const int pu = p.dimp / V, pq = p.heads * pu;
+  for (int i = threadIdx.x; i < pq; i += LP_THREADS) {
+    const int h = pu == 1 ? i : (int)__umulhi((unsigned)i, p.plain_magic), j = (i - h * pu) * V;
+    Vec a[RUN];
+#pragma unroll
+    for (int t = 0; t < RUN; ++t) {
+      if (t < nt && j < p.dim) {
+        a[t] = *reinterpret_cast<const Vec*>(src0 + t * p.ld + h * (p.dim + p.rot) + j);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) a[t].v[e] = from_f32<T>(0.f);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < RUN; ++t)
+      if (t < nt) *reinterpret_cast<Vec*>(q + ((n0 + t) * p.heads + h) * dq + j) = a[t];
+  }
+  for (int i = threadIdx.x; i < p.kvp / V; i += LP_THREADS) {
+    const int j = i * V;
+#pragma unroll
+    for (int t = 0; t < RUN; ++t) {
+      if (t >= nt) break;
+      Vec a;
+      if (j < p.kv_rank) {
+        a = *reinterpret_cast<const Vec*>(src0 + t * p.ld + c0 + j);
+        const float r = inv_rms[t];
+#pragma unroll
+        for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(to_f32(a.v[e]) * r * p.norm_w[j + e]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(0.f);
+      }
+      put_latent(t, j, a);
+    }
+  }
+  // ---- rotary parts of the heads and of the latent row: V pairs per thread, both halves
+  const int ru = half / V, rq = (p.heads + 1) * ru;
+  for (int i = threadIdx.x; i < rq; i += LP_THREADS) {
+    const int h = ru == 1 ? i : (int)__umulhi((unsigned)i, p.rot_magic), k = (i - h * ru) * V;
+    const int x = (h < p.heads ? h * (p.dim + p.rot) + p.dim : c0 + p.kv_rank) + k;
+#pragma unroll
+    for (int t = 0; t < RUN; ++t) {
+      if (t >= nt) break;
+      Vec a = *reinterpret_cast<const Vec*>(src0 + t * p.ld + x), w = *reinterpret_cast<const Vec*>(src0 + t * p.ld + x + half);
+      const float *cs = sm + t * p.rot_dims + k, *sn = cs + half;
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+        const float u = to_f32(a.v[e]), v = to_f32(w.v[e]);
+        a.v[e] = from_f32<T>(u * cs[e] - v * sn[e]);
+        w.v[e] = from_f32<T>(v * cs[e] + u * sn[e]);
+      }
+      if (h < p.heads) {
+        T* d = q + ((n0 + t) * p.heads + h) * dq + p.dimp + k;
+        *reinterpret_cast<Vec*>(d) = a;
+        *reinterpret_cast<Vec*>(d + half) = w;
+      } else {
+        put_latent(t, p.kvp + k, a);
+        put_latent(t, p.kvp + half + k, w);
+      }
+    }
+  }
+  // ---- rotary columns beyond rot_dims pass, padding is zero
+  const int tail = p.rp - p.rot_dims;
+  for (int i = threadIdx.x; i < (p.heads + 1) * tail * nt; i += LP_THREADS) {
+    const int t = i / ((p.heads + 1) * tail), h = i / tail % (p.heads + 1), r = p.rot_dims + i % tail;
+    const T v = r < p.rot ? src0[t * p.ld + (h < p.heads ? h * (p.dim + p.rot) + p.dim : c0 + p.kv_rank) + r] : from_f32<T>(0.f);
+    if (h < p.heads) {
+      q[((n0 + t) * p.heads + h) * dq + p.dimp + r] = v;
+    } else {
+      if (latent) latent[((long long)b * (p.P + p.T) + p.P + t0 + t) * lw + p.kvp + r] = v;
+      T* d = ring_row(t);
+      if (d) d[p.kvp + r] = v;
+    }
+  }
 }
 
 template <typename T, int V>
-__global__ void __launch_bounds__(LP_WARPS * 32)
-latent_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict__ latent, T* __restrict__ ring, const LpParams p) {
-  using Vec = LpVec<T, V>;
-  extern __shared__ float sm[];  // cos | sin (rot_dims / 2 each)
-  const int t = blockIdx.x, b = blockIdx.z;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int unit = blockIdx.y * LP_WARPS + warp;
-  const long long n = (long long)b * p.T + t;
-  const int pos = p.start[b] + t;
-  const int half = p.rot_dims / 2;
-  float *cs = sm, *sn = sm + half;
-  for (int i = threadIdx.x; i < half; i += LP_WARPS * 32) sincosf((float)pos * p.freq[i], &sn[i], &cs[i]);
-  __syncthreads();
-  const T* src = qkv + n * p.ld;
-  if (unit < p.heads) {
-    const T* x = src + unit * (p.dim + p.rot);
-    T* dst = q + (n * p.heads + unit) * (p.dimp + p.rp);
-    for (int i = lane * V; i < p.dim; i += 32 * V) *reinterpret_cast<Vec*>(dst + i) = *reinterpret_cast<const Vec*>(x + i);
-    for (int i = p.dim + lane; i < p.dimp; i += 32) dst[i] = from_f32<T>(0.f);
-    lp_rotate<T, V>(x + p.dim, dst + p.dimp, cs, sn, p, lane);
-    return;
-  }
-  if (unit > p.heads) return;
-  T* dst;
-  if (ring) {
-    if (p.count[b] <= t) return;  // padding never reaches the ring
-    dst = ring + ((long long)p.slots[b] * p.ring_len + pos % p.ring_len) * (p.kvp + p.rp);
-  } else {
-    dst = latent + ((long long)b * (p.P + p.T) + p.P + t) * (p.kvp + p.rp);
-  }
-  const T* c = src + p.heads * (p.dim + p.rot);
-  float ss = 0.f;
-  for (int i = lane * V; i < p.kv_rank; i += 32 * V) {
-    const Vec a = *reinterpret_cast<const Vec*>(c + i);
-#pragma unroll
-    for (int e = 0; e < V; ++e) ss = fmaf(to_f32(a.v[e]), to_f32(a.v[e]), ss);
-  }
-  const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.kv_rank + p.eps);
-  for (int i = lane * V; i < p.kv_rank; i += 32 * V) {
-    Vec a = *reinterpret_cast<const Vec*>(c + i);
-#pragma unroll
-    for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(to_f32(a.v[e]) * r * p.norm_w[i + e]);
-    *reinterpret_cast<Vec*>(dst + i) = a;
-  }
-  for (int i = p.kv_rank + lane; i < p.kvp; i += 32) dst[i] = from_f32<T>(0.f);
-  lp_rotate<T, V>(c + p.kv_rank, dst + p.kvp, cs, sn, p, lane);
+static int lp_launch_run(const void* qkv, void* q, void* latent, void* ring, LpParams& p, int B, cudaStream_t s) {
+  // i / n as a high product, exact for i, n < 2^16
+  auto magic = [](int n) { return n > 1 ? (unsigned)(0x100000000ull / n + 1) : 0u; };
+  p.plain_magic = magic(p.dimp / V);
+  p.rot_magic = magic(p.rot_dims / 2 / V);
+  if ((long long)p.heads * p.dimp >= 65536 || (long long)(p.heads + 1) * p.rot_dims >= 65536) return KVB_ERR_TOO_LARGE;
+  const bool many = (long long)B * p.T >= 148 * 4 * LP_RUN;
+  const int run = many ? LP_RUN : 1;
+  const size_t smem = (size_t)run * p.rot_dims * sizeof(float) + 8;
+  if (smem > 48 * 1024) return KVB_ERR_TOO_LARGE;
+  const dim3 grid((p.T + run - 1) / run, B);
+  if (many)
+    latent_prep_kernel<T, V, LP_RUN><<<grid, LP_THREADS, smem, s>>>((const T*)qkv, (T*)q, (T*)latent, (T*)ring, p);
+  else
+    latent_prep_kernel<T, V, 1><<<grid, LP_THREADS, smem, s>>>((const T*)qkv, (T*)q, (T*)latent, (T*)ring, p);
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
 template <typename T>
-static int lp_launch(const void* qkv, void* q, void* latent, void* ring, const LpParams& p, int B, cudaStream_t s) {
+static int lp_launch(const void* qkv, void* q, void* latent, void* ring, LpParams& p, int B, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
-  const dim3 grid(p.T, (p.heads + LP_WARPS) / LP_WARPS, B);
-  const size_t smem = p.rot_dims * sizeof(float) + 8;
-  if (((p.dim | p.rot | p.kv_rank | (p.rot_dims / 2)) % V) == 0 && p.ld % V == 0)
-    latent_prep_kernel<T, V><<<grid, LP_WARPS * 32, smem, s>>>((const T*)qkv, (T*)q, (T*)latent, (T*)ring, p);
-  else
-    latent_prep_kernel<T, 1><<<grid, LP_WARPS * 32, smem, s>>>((const T*)qkv, (T*)q, (T*)latent, (T*)ring, p);
-  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+  if (((p.dim | p.rot | p.kv_rank | (p.rot_dims / 2)) % V) == 0 && p.ld % V == 0) return lp_launch_run<T, V>(qkv, q, latent, ring, p, B, s);
+  return lp_launch_run<T, 1>(qkv, q, latent, ring, p, B, s);
 }
 
 // ------------------------------------------------------------------------------------------------ ring
@@ -127,17 +196,6 @@ ring_gather_kernel(const uint4* __restrict__ ring, uint4* __restrict__ latent, c
   const bool has = pos >= 0 && pos >= start[b] - ring_len;
   const uint4* src = ring + ((long long)slots[b] * ring_len + (has ? pos % ring_len : 0)) * units;
   for (int i = threadIdx.x & 31; i < units; i += 32) dst[i] = has ? src[i] : make_uint4(0, 0, 0, 0);
-}
-
-__global__ void __launch_bounds__(LR_WARPS * 32)
-ring_append_kernel(const uint4* __restrict__ latent, uint4* __restrict__ ring, const int* __restrict__ slots, const int* __restrict__ start,
-                   const int* __restrict__ count, int Tn, int P, int ring_len, int units) {
-  const int i0 = blockIdx.x * LR_WARPS + (threadIdx.x >> 5), b = blockIdx.y;
-  const int t = count[b] - 1 - i0;  // newest first
-  if (t < 0 || i0 >= ring_len) return;
-  const uint4* src = latent + ((long long)b * (P + Tn) + P + t) * units;
-  uint4* dst = ring + ((long long)slots[b] * ring_len + (start[b] + t) % ring_len) * units;
-  for (int i = threadIdx.x & 31; i < units; i += 32) dst[i] = src[i];
 }
 
 // ------------------------------------------------------------------- attention over expanded keys, CUDA cores
@@ -268,30 +326,41 @@ latent_decode_simple_kernel(const T* __restrict__ q_abs, const T* __restrict__ q
 }
 
 // ------------------------------------------------------------------ single token, bf16 on mma.sync, split over the ring
-// Per CTA: 16 · MT heads of one sequence against tiles of 32 ring rows. A tile is the key AND the value of all heads, so it is
-// fetched once (one bulk copy per row into a ring of stages) and read twice from shared memory: S = Q K^T with the rows as
-// the N operand, O += P C with the same rows transposed by ldmatrix. N is 32 rows and M 16 or 32 heads, far below a
-// tcgen05 tile, and the kernel is bound by the read of the ring.
+// Per CTA: 16 heads of one sequence against tiles of 32 ring rows. A tile is the key AND the value of all heads, so it is
+// fetched once (TMA, 128B-swizzled chunks of 64 columns into a ring of stages, by a warp of its own) and read twice from
+// shared memory: S = Q K^T with the rows as the N operand, O += P C with the same rows transposed by ldmatrix. N is 32
+// rows and M 16 heads, far below a tcgen05 tile. More heads are more CTAs, whose reads of the ring meet in L2.
 //
-// Warps 0..3 and 4..7 take the two halves of the features in S (8 rows each); after one barrier every warp has the whole S tile
-// in the layout of the A operand of the second product, so each keeps maximum and sum of all heads in registers
-// and no second exchange is needed. The barrier of tile t also says that everybody is done with tile t − 1: its
-// stage is refilled then.
-constexpr int LM_THREADS = 256;
+// In S every warp takes an eighth of the columns, with its part of the queries in registers; the eight partial tiles meet in
+// shared memory, where every warp does the softmax of two heads (lane = row); in O it takes its 64 columns. Two groups of
+// eight warps work on alternate tiles of the same ring of stages: one computes while the other waits at its barrier, and
+// enough tiles stay in flight. Each group leaves partial sums, which a second kernel puts together.
+constexpr int LM_WARPS = 8;
+constexpr int LM_GROUPS = 2;
+constexpr int LM_THREADS = 32 * LM_WARPS * LM_GROUPS + 32;
 constexpr int LM_KEYS = 32;
-constexpr int LM_SPITCH = 40;
+constexpr int LM_HEADS = 16;
+constexpr int LM_SPITCH = 40;  // of score rows (fp32) and weight rows (bf16): conflict-free float2 stores and ldmatrix
 constexpr int LM_MAX_STAGES = 6;
+constexpr int LM_CHUNK = LM_KEYS * 128;  // bytes of [32 rows x 64 columns]
+constexpr int LM_GROUP_BYTES = LM_HEADS * (LM_SPITCH * (LM_WARPS * 4 + 2) + 4);
 
 __device__ __forceinline__ void lm_ldsm4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
-__device__ __forceinline__ void lm_ldsm2(uint32_t& r0, uint32_t& r1, uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr) : "memory");
-}
 __device__ __forceinline__ void lm_ldsm4t(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ float lm_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// barrier of the eight warps of one group
+__device__ __forceinline__ void lm_group_sync(int group) {
+  asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "n"(32 * LM_WARPS) : "memory");
 }
 __device__ __forceinline__ void lm_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -300,289 +369,285 @@ __device__ __forceinline__ void lm_mma(float (&d)[4], const uint32_t (&a)[4], ui
 }
 
 struct LmParams {
-  const __nv_bfloat16 *q_abs, *q, *ring;
+  const __nv_bfloat16 *q_abs, *q;
   __nv_bfloat16* out;      // (heads, B, kvp)
-  float* part_o;           // (n_split, B, heads, kvp)
-  float* part_ml;          // (n_split, B, heads, 2)
+  float* part_o;           // (n_part, B, heads, kvp), n_part = n_split · LM_GROUPS
+  float* part_ml;          // (n_part, B, heads, 2)
   const int *slots, *start;
   int* status;
   int B, heads, dimp, rp, kvp, ring_len, n_split, stages;
-  int kv16, ls;            // latent columns rounded up to 16; row pitch in shared memory (elements)
+  int chunks, ksteps;      // chunks of 64 and steps of 16 columns of a row
   float scale_log2;
 };
 
-// MT: tiles of 16 heads; NP: pairs of 8-column tiles per warp in the second product
-template <int MT, int NP>
+// KW: steps of 16 columns per warp in the first product, NP: pairs of 8-column tiles per warp in the second
+template <int KW, int NP>
 __global__ void __launch_bounds__(LM_THREADS, 1)
-latent_decode_mma_kernel(const LmParams p) {
-  extern __shared__ __align__(128) uint8_t lm_smem[];
-  constexpr int HB = 16 * MT;
-  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(lm_smem);
-  __nv_bfloat16* sk = sq + HB * p.ls;
-  float* ss = reinterpret_cast<float*>(sk + p.stages * LM_KEYS * p.ls);  // [2 tiles][2 halves][HB][LM_SPITCH]
-  uint64_t* full = reinterpret_cast<uint64_t*>(ss + 4 * HB * LM_SPITCH);
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(full + LM_MAX_STAGES);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+latent_decode_mma_kernel(const __grid_constant__ CUtensorMap tmR, const LmParams p) {
+  extern __shared__ __align__(1024) uint8_t lm_smem[];
+  constexpr int HB = LM_HEADS;
+  const int stage_bytes = p.chunks * LM_CHUNK;
+  uint8_t* sk = lm_smem;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int group = (tid >> 5) / LM_WARPS, warp = (tid >> 5) % LM_WARPS;  // group LM_GROUPS: the producer
+  // per group: [LM_WARPS][HB][LM_SPITCH] partial scores, [HB][LM_SPITCH] weights, [HB] rescale factors
+  float* ss = reinterpret_cast<float*>(sk + p.stages * stage_bytes + (group % LM_GROUPS) * LM_GROUP_BYTES);
+  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(ss + LM_WARPS * HB * LM_SPITCH);
+  float* sf = reinterpret_cast<float*>(sp + HB * LM_SPITCH);
+  uint64_t* full = reinterpret_cast<uint64_t*>(sk + p.stages * stage_bytes + LM_GROUPS * LM_GROUP_BYTES);
+  uint64_t* empty = full + LM_MAX_STAGES;
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(empty + LM_MAX_STAGES);
   const int b = blockIdx.x, split = blockIdx.y, h0 = blockIdx.z * HB;
   const int lw = p.kvp + p.rp;
   const int nk = min(p.start[b] + 1, p.ring_len);
   const int nT = (nk + LM_KEYS - 1) / LM_KEYS;
   const int per = (nT + p.n_split - 1) / p.n_split;
   const int ta = split * per, tb = min(nT, ta + per);
-  const __nv_bfloat16* base = p.ring + (long long)p.slots[b] * p.ring_len * lw;
-  // zero query rows and the padding columns that no copy writes
-  for (int i = tid; i < (HB + p.stages * LM_KEYS) * p.ls / 8; i += LM_THREADS) reinterpret_cast<uint4*>(lm_smem)[i] = make_uint4(0, 0, 0, 0);
+  if (smem_u32(lm_smem) & 1023u) {
+    if (tid == 0 && p.status) atomicCAS(p.status, 0, STATUS_TIMEOUT_MISC);
+    return;
+  }
   if (tid == 0) {
-    for (int i = 0; i < p.stages; ++i) mbar_init(&full[i], 1);
+    for (int i = 0; i < p.stages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], LM_WARPS);
+    }
     *abort_flag = 0;
     mbar_fence_init();
   }
-  fence_proxy_async_smem();
   __syncthreads();
-  auto load_tile = [&](int t, int stage) {  // warp 0: one row per lane
-    __nv_bfloat16* dst = sk + (stage * LM_KEYS + lane) * p.ls;
-    const int rows = min(LM_KEYS, nk - t * LM_KEYS);
-    const __nv_bfloat16* src = base + (long long)(t * LM_KEYS + lane) * lw;
-    if (lane == 0) mbar_expect_tx(&full[stage], (uint32_t)(rows * lw * 2));
-    __syncwarp();
-    if (lane < rows) {
-      if (p.kv16 == p.kvp) {
-        bulk_load(dst, src, (uint32_t)(lw * 2), &full[stage]);
-      } else {
-        bulk_load(dst, src, (uint32_t)(p.kvp * 2), &full[stage]);
-        bulk_load(dst + p.kv16, src + p.kvp, (uint32_t)(p.rp * 2), &full[stage]);
+  if (group == LM_GROUPS) {
+    // ------------------------------------------------------------ producer
+    if (lane == 0) {
+      tma_prefetch_desc(&tmR);
+      const int row0 = p.slots[b] * p.ring_len;
+      int stage = 0;
+      uint32_t phase = 0;
+      bool ok = true;
+      for (int t = ta; t < tb; ++t) {
+        if (!(ok = mbar_wait_bounded(&empty[stage], phase ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
+        mbar_expect_tx(&full[stage], (uint32_t)stage_bytes);
+        // rows beyond the last visible one belong to nobody or to the next slot: they are hidden below
+        for (int c = 0; c < p.chunks; ++c) tma_load_2d(sk + stage * stage_bytes + c * LM_CHUNK, &tmR, &full[stage], 64 * c, row0 + t * LM_KEYS);
+        if (++stage == p.stages) {
+          stage = 0;
+          phase ^= 1;
+        }
+      }
+      if (!ok) {  // copies in flight get a bounded time to land before the shared memory is released
+        const long long c0 = clock64();
+        while (clock64() - c0 < 2000000LL) {
+        }
       }
     }
-  };
-  if (warp == 0)
-    for (int i = 0; i < p.stages && ta + i < tb; ++i) load_tile(ta + i, i);
-  const int ku = p.kvp / 8, lu = lw / 8;
-  for (int i = tid; i < HB * lu; i += LM_THREADS) {
-    const int h = i / lu, u = i - h * lu;
-    if (h0 + h < p.heads) {
-      const __nv_bfloat16* src = u < ku ? p.q_abs + ((long long)(h0 + h) * p.B + b) * p.kvp + u * 8
-                                        : p.q + ((long long)b * p.heads + h0 + h) * (p.dimp + p.rp) + p.dimp + (u - ku) * 8;
-      *reinterpret_cast<uint4*>(sq + h * p.ls + (u < ku ? u * 8 : p.kv16 + (u - ku) * 8)) = *reinterpret_cast<const uint4*>(src);
+    return;
+  }
+  float acc[2 * NP][4];
+#pragma unroll
+  for (int j = 0; j < 2 * NP; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[j][e] = 0.f;
+  // this warp's columns of the queries as A operands: rows lane / 4 and + 8, columns (lane % 4) · 2 and + 8 of a step;
+  // zero beyond the heads and the columns of a row
+  const int k0 = warp * KW;
+  uint32_t qf[KW][4];
+#pragma unroll
+  for (int i = 0; i < KW; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int h = h0 + (lane >> 2) + 8 * (e & 1), c = (k0 + i) * 16 + (lane & 3) * 2 + 8 * (e >> 1);
+      qf[i][e] = 0u;
+      if (h < p.heads && c < lw)
+        qf[i][e] = *reinterpret_cast<const uint32_t*>(c < p.kvp ? p.q_abs + ((long long)h * p.B + b) * p.kvp + c
+                                                                : p.q + ((long long)b * p.heads + h) * (p.dimp + p.rp) + p.dimp + c - p.kvp);
+    }
+  float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.f, 0.f};  // heads 2 · warp, 2 · warp + 1; sums of this lane's rows
+  const int n_pairs = (p.kvp + 15) / 16;
+  // ldmatrix addresses within a stage: 16 ring rows x 16 columns per load, in the first product rows by columns, in the second
+  // transposed; loads beyond the columns of a row meet zero queries or sums that are not kept, and read the first chunk
+  uint32_t koff[KW], voff[NP];
+  {
+    const int kr = (lane & 7) + ((lane >> 4) << 3), vr = lane & 15;
+#pragma unroll
+    for (int i = 0; i < KW; ++i) {
+      const int k = k0 + i < p.ksteps ? k0 + i : 0;
+      koff[i] = (uint32_t)((k >> 2) * LM_CHUNK + kr * 128 + ((((k & 3) * 2 + ((lane >> 3) & 1)) ^ (kr & 7)) << 4));
+    }
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+      const int np = warp * NP + j < n_pairs ? warp * NP + j : 0;
+      voff[j] = (uint32_t)((np >> 2) * LM_CHUNK + vr * 128 + ((((np & 3) * 2 + (lane >> 4)) ^ (vr & 7)) << 4));
     }
   }
-  float acc[MT][2 * NP][4];
-  float mx[MT][2], sum[MT][2];
-#pragma unroll
-  for (int m = 0; m < MT; ++m) {
-    mx[m][0] = mx[m][1] = -INFINITY;
-    sum[m][0] = sum[m][1] = 0.f;
-#pragma unroll
-    for (int j = 0; j < 2 * NP; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[m][j][e] = 0.f;
-  }
-  __syncthreads();
-  const int ksteps = (p.ls - 8) / 16;
-  const int half = warp >> 2, k_lo = half ? (ksteps + 1) / 2 : 0, k_hi = half ? ksteps : (ksteps + 1) / 2;
-  const int key0 = (warp & 3) * 8;
-  const int n_pairs = p.kv16 / 16;
+  const uint32_t pa0 = smem_u32(sp + (lane & 15) * LM_SPITCH + (lane >> 4) * 8);
+  float* const sd = ss + (warp * HB + (lane >> 2)) * LM_SPITCH + (lane & 3) * 2;
+  const float* const sr = ss + warp * 2 * LM_SPITCH + lane;
   bool ok = true;
-  int stage = 0;
+  int stage = group;  // at least LM_GROUPS + 1 stages
   uint32_t phase = 0;
-  for (int t = ta; t < tb; ++t) {
+  for (int t = ta + group; t < tb; t += LM_GROUPS) {
     // after a wait that ran out the tiles are worked on unseen: the status word tells, and the loop ends
     if (ok) ok = mbar_wait_bounded(&full[stage], phase, abort_flag, p.status, STATUS_TIMEOUT_FULL);
-    const __nv_bfloat16* kt = sk + stage * LM_KEYS * p.ls;
+    const uint32_t kt = smem_u32(sk + stage * stage_bytes);
     {
-      float s[MT][2][4];
+      float s[LM_KEYS / 8][4];
 #pragma unroll
-      for (int m = 0; m < MT; ++m)
+      for (int i = 0; i < LM_KEYS / 8; ++i)
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
+        for (int e = 0; e < 4; ++e) s[i][e] = 0.f;
 #pragma unroll
-          for (int e = 0; e < 4; ++e) s[m][i][e] = 0.f;
-      const uint32_t qa = smem_u32(sq + (lane & 15) * p.ls + (lane >> 4) * 8);
-      const uint32_t kb = smem_u32(kt + (key0 + (lane & 7)) * p.ls + (lane >> 3) * 8);
-      int k = k_lo;
-#pragma unroll 2
-      for (; k + 1 < k_hi; k += 2) {
-        uint32_t bb[4];
-        lm_ldsm4(bb, kb + k * 32);
+      for (int i = 0; i < KW; ++i) {
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          lm_ldsm4(a, qa + m * 16 * p.ls * 2 + k * 32);
-          lm_mma(s[m][0], a, bb[0], bb[1]);
-          lm_ldsm4(a, qa + m * 16 * p.ls * 2 + k * 32 + 32);
-          lm_mma(s[m][1], a, bb[2], bb[3]);
+        for (int g = 0; g < LM_KEYS / 16; ++g) {
+          uint32_t bb[4];
+          lm_ldsm4(bb, kt + koff[i] + g * 16 * 128);
+          lm_mma(s[2 * g], qf[i], bb[0], bb[1]);
+          lm_mma(s[2 * g + 1], qf[i], bb[2], bb[3]);
         }
       }
-      if (k < k_hi) {
-        uint32_t b0, b1;
-        lm_ldsm2(b0, b1, smem_u32(kt + (key0 + (lane & 7)) * p.ls + ((lane >> 3) & 1) * 8) + k * 32);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          lm_ldsm4(a, qa + m * 16 * p.ls * 2 + k * 32);
-          lm_mma(s[m][0], a, b0, b1);
-        }
-      }
-      float* sd = ss + ((t & 1) * 2 + half) * HB * LM_SPITCH;
-#pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const int r = m * 16 + (lane >> 2), c = key0 + (lane & 3) * 2;
-        *reinterpret_cast<float2*>(sd + r * LM_SPITCH + c) = make_float2(s[m][0][0] + s[m][1][0], s[m][0][1] + s[m][1][1]);
-        *reinterpret_cast<float2*>(sd + (r + 8) * LM_SPITCH + c) = make_float2(s[m][0][2] + s[m][1][2], s[m][0][3] + s[m][1][3]);
+      for (int i = 0; i < LM_KEYS / 8; ++i) {
+        *reinterpret_cast<float2*>(sd + 8 * i) = make_float2(s[i][0], s[i][1]);
+        *reinterpret_cast<float2*>(sd + 8 * LM_SPITCH + 8 * i) = make_float2(s[i][2], s[i][3]);
       }
     }
-    __syncthreads();
-    if (warp == 0 && t > ta && t - 1 + p.stages < tb) load_tile(t - 1 + p.stages, stage == 0 ? p.stages - 1 : stage - 1);
-    const int left = nk - t * LM_KEYS;
-    const float* s0 = ss + (t & 1) * 2 * HB * LM_SPITCH;
-    const float* s1 = s0 + HB * LM_SPITCH;
-    uint32_t pa[MT][LM_KEYS / 16][4];
+    lm_group_sync(group);
+    const bool seen = t * LM_KEYS + lane < nk;
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
+    for (int i = 0; i < 2; ++i) {
+      const int r = warp * 2 + i;
+      float part[LM_WARPS];
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {  // rows lane / 4 and lane / 4 + 8
-        const int o = (m * 16 + (lane >> 2) + 8 * e) * LM_SPITCH + (lane & 3) * 2;
-        float x[LM_KEYS / 4];
-        float mn = mx[m][e];
+      for (int g = 0; g < LM_WARPS; ++g) part[g] = sr[(g * HB + i) * LM_SPITCH];
+      const float score = ((part[0] + part[1]) + (part[2] + part[3])) + ((part[4] + part[5]) + (part[6] + part[7]));
+      const float x = seen ? score * p.scale_log2 : -INFINITY;
+      const float mn = fmaxf(mx[i], warp_max(x));
+      const float f = lm_exp2(mx[i] - mn), w = lm_exp2(x - mn);
+      mx[i] = mn;
+      sum[i] = fmaf(sum[i], f, w);
+      sp[r * LM_SPITCH + lane] = __float2bfloat16_rn(w);
+      if (lane == 0) sf[r] = f;
+    }
+    lm_group_sync(group);
+    const float f0 = sf[lane >> 2], f1 = sf[(lane >> 2) + 8];
+    if (__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) {
 #pragma unroll
-        for (int i = 0; i < LM_KEYS / 8; ++i) {
-          const float2 u = *reinterpret_cast<const float2*>(s0 + o + 8 * i), v = *reinterpret_cast<const float2*>(s1 + o + 8 * i);
-          const int c = (lane & 3) * 2 + 8 * i;
-          x[2 * i] = c < left ? (u.x + v.x) * p.scale_log2 : -INFINITY;
-          x[2 * i + 1] = c + 1 < left ? (u.y + v.y) * p.scale_log2 : -INFINITY;
-          mn = fmax3(mn, x[2 * i], x[2 * i + 1]);
-        }
-        mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
-        mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 2));
-        const float f = exp2f(mx[m][e] - mn);
-        mx[m][e] = mn;
-        float l = 0.f;
-#pragma unroll
-        for (int i = 0; i < LM_KEYS / 4; ++i) {
-          x[i] = exp2f(x[i] - mn);
-          l += x[i];
-        }
-        sum[m][e] = sum[m][e] * f + l;  // this lane's columns; the quad is added up at the end
-#pragma unroll
-        for (int i = 0; i < LM_KEYS / 16; ++i) {
-          pa[m][i][e] = pack_bf16x2(x[4 * i], x[4 * i + 1]);
-          pa[m][i][2 + e] = pack_bf16x2(x[4 * i + 2], x[4 * i + 3]);
-        }
-#pragma unroll
-        for (int j = 0; j < 2 * NP; ++j) {
-          acc[m][j][2 * e] *= f;
-          acc[m][j][2 * e + 1] *= f;
-        }
+      for (int j = 0; j < 2 * NP; ++j) {
+        acc[j][0] *= f0;
+        acc[j][1] *= f0;
+        acc[j][2] *= f1;
+        acc[j][3] *= f1;
       }
     }
 #pragma unroll
     for (int k = 0; k < LM_KEYS / 16; ++k) {
-      const uint32_t vb = smem_u32(kt + (k * 16 + (lane & 15)) * p.ls + (lane >> 4) * 8);
+      uint32_t pa[4];
+      lm_ldsm4(pa, pa0 + k * 32);
 #pragma unroll
       for (int j = 0; j < NP; ++j) {
-        const int np = warp * NP + j;
-        if (np < n_pairs) {
-          uint32_t v[4];
-          lm_ldsm4t(v, vb + np * 32);
-#pragma unroll
-          for (int m = 0; m < MT; ++m) {
-            lm_mma(acc[m][2 * j], pa[m][k], v[0], v[1]);
-            lm_mma(acc[m][2 * j + 1], pa[m][k], v[2], v[3]);
-          }
-        }
+        uint32_t v[4];
+        lm_ldsm4t(v, kt + voff[j] + k * 16 * 128);
+        lm_mma(acc[2 * j], pa, v[0], v[1]);
+        lm_mma(acc[2 * j + 1], pa, v[2], v[3]);
       }
     }
-    if (++stage == p.stages) {
-      stage = 0;
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[stage]);
+    stage += LM_GROUPS;
+    if (stage >= p.stages) {
+      stage -= p.stages;
       phase ^= 1;
     }
   }
-  const bool direct = p.n_split == 1;
+  const long long part = ((long long)(split * LM_GROUPS + group) * p.B + b) * p.heads + h0;
 #pragma unroll
-  for (int m = 0; m < MT; ++m) {
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      float l = sum[m][e];
-      l += __shfl_xor_sync(0xffffffffu, l, 1);
-      l += __shfl_xor_sync(0xffffffffu, l, 2);
-      const int r = m * 16 + (lane >> 2) + 8 * e, h = h0 + r;
-      if (h >= p.heads) continue;
-      const float inv = direct ? 1.f / l : 1.f;
-#pragma unroll
-      for (int j = 0; j < 2 * NP; ++j) {
-        const int c = (warp * 2 * NP + j) * 8 + (lane & 3) * 2;
-        if (c >= p.kvp) continue;
-        if (direct)
-          *reinterpret_cast<uint32_t*>(p.out + ((long long)h * p.B + b) * p.kvp + c) =
-              pack_bf16x2(acc[m][j][2 * e] * inv, acc[m][j][2 * e + 1] * inv);
-        else
-          *reinterpret_cast<float2*>(p.part_o + (((long long)split * p.B + b) * p.heads + h) * p.kvp + c) =
-              make_float2(acc[m][j][2 * e], acc[m][j][2 * e + 1]);
-      }
-      if (!direct && warp == 0 && (lane & 3) == 0) {
-        float* ml = p.part_ml + (((long long)split * p.B + b) * p.heads + h) * 2;
-        ml[0] = mx[m][e];
-        ml[1] = l;
-      }
-    }
+  for (int i = 0; i < 2; ++i) {
+    const int r = warp * 2 + i;
+    const float l = warp_sum(sum[i]);
+    if (lane == 0 && h0 + r < p.heads) *reinterpret_cast<float2*>(p.part_ml + (part + r) * 2) = make_float2(mx[i], l);
   }
-  if (!ok) {  // copies in flight get a bounded time to land before the shared memory is released
-    const long long c0 = clock64();
-    while (clock64() - c0 < 2000000LL) {
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int r = (lane >> 2) + 8 * e;
+    if (h0 + r >= p.heads) continue;
+#pragma unroll
+    for (int j = 0; j < 2 * NP; ++j) {
+      const int c = (warp * 2 * NP + j) * 8 + (lane & 3) * 2;
+      if (c < p.kvp) *reinterpret_cast<float2*>(p.part_o + (part + r) * p.kvp + c) = make_float2(acc[j][2 * e], acc[j][2 * e + 1]);
     }
   }
 }
 
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const LmParams p) {
-  const int h = blockIdx.x, b = blockIdx.y;
+  __shared__ float wt[64];
+  const int n_part = p.n_split * LM_GROUPS;
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31;
   const long long bh = (long long)b * p.heads + h, step = (long long)p.B * p.heads;
-  float M = -INFINITY;
-  for (int s = 0; s < p.n_split; ++s) M = fmaxf(M, p.part_ml[(s * step + bh) * 2]);
-  float L = 0.f;
-  for (int s = 0; s < p.n_split; ++s) {
-    const float m = p.part_ml[(s * step + bh) * 2];
-    if (m != -INFINITY) L += p.part_ml[(s * step + bh) * 2 + 1] * exp2f(m - M);
-  }
-  const float inv = 1.f / L;
-  for (int c = threadIdx.x; c < p.kvp; c += 128) {
-    float o = 0.f;
-    for (int s = 0; s < p.n_split; ++s) {
-      const float m = p.part_ml[(s * step + bh) * 2];
-      if (m != -INFINITY) o = fmaf(p.part_o[(s * step + bh) * p.kvp + c], exp2f(m - M), o);
+  if (threadIdx.x < 32) {  // at most 64 parts: two per lane
+    float m[2], l[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int s = lane + 32 * i;
+      const float2 v = s < n_part ? *reinterpret_cast<const float2*>(p.part_ml + (s * step + bh) * 2) : make_float2(-INFINITY, 0.f);
+      m[i] = v.x;
+      l[i] = v.y;
     }
-    p.out[((long long)h * p.B + b) * p.kvp + c] = __float2bfloat16_rn(o * inv);
+    const float M = warp_max(fmaxf(m[0], m[1]));
+    float f[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) f[i] = m[i] == -INFINITY ? 0.f : exp2f(m[i] - M);
+    const float inv = 1.f / warp_sum(f[0] * l[0] + f[1] * l[1]);
+    wt[lane] = f[0] * inv;
+    wt[lane + 32] = f[1] * inv;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * 4; c < p.kvp; c += 512) {
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int s = 0; s < n_part; ++s) {
+      const float4 v = *reinterpret_cast<const float4*>(p.part_o + (s * step + bh) * p.kvp + c);
+      const float w = wt[s];  // 0 for a part that saw no row (its sums are zero)
+      o.x = fmaf(w, v.x, o.x);
+      o.y = fmaf(w, v.y, o.y);
+      o.z = fmaf(w, v.z, o.z);
+      o.w = fmaf(w, v.w, o.w);
+    }
+    *reinterpret_cast<uint2*>(p.out + ((long long)h * p.B + b) * p.kvp + c) = make_uint2(pack_bf16x2(o.x, o.y), pack_bf16x2(o.z, o.w));
   }
 }
 
-static int lm_splits(int B, int heads, int ring_len) {
-  const int hb = heads > 16 ? 32 : 16;
-  const long long ctas = (long long)B * ((heads + hb - 1) / hb);
+static size_t lm_smem_bytes(int chunks, int stages) {
+  return (size_t)stages * chunks * LM_CHUNK + LM_GROUPS * LM_GROUP_BYTES + 2 * LM_MAX_STAGES * 8 + 16;
+}
+
+struct LmPlan {
+  int chunks, ksteps, stages, n_split;
+};
+static LmPlan lm_plan(int B, int heads, int kvp, int rp, int ring_len) {
+  LmPlan pl;
+  pl.chunks = (kvp + rp + 63) / 64;
+  pl.ksteps = (kvp + rp + 15) / 16;
+  pl.stages = 0;
+  for (int st = LM_MAX_STAGES; st >= LM_GROUPS + 1 && !pl.stages; --st)
+    if (lm_smem_bytes(pl.chunks, st) <= 232448) pl.stages = st;
+  const long long ctas = (long long)B * ((heads + LM_HEADS - 1) / LM_HEADS);
   const int tiles = (ring_len + LM_KEYS - 1) / LM_KEYS;
   long long n = 148 / ctas;  // one CTA per SM: a second, partly filled wave would cost as much as the first
-  if (n > (tiles + 3) / 4) n = (tiles + 3) / 4;
-  if (n > 64) n = 64;
-  return n < 1 ? 1 : (int)n;
+  if (n > (tiles + 7) / 8) n = (tiles + 7) / 8;
+  if (n > 64 / LM_GROUPS) n = 64 / LM_GROUPS;
+  pl.n_split = n < 1 ? 1 : (int)n;
+  return pl;
 }
 
-static size_t lm_smem_bytes(int mt, int ls, int stages) {
-  const int hb = 16 * mt;
-  return (size_t)(hb + stages * LM_KEYS) * ls * 2 + (size_t)4 * hb * LM_SPITCH * 4 + LM_MAX_STAGES * 8 + 16;
-}
-
-static int lm_stages(int mt, int ls) {
-  for (int st = LM_MAX_STAGES; st >= 2; --st)
-    if (lm_smem_bytes(mt, ls, st) <= 232448) return st;
-  return 0;
-}
-
-template <int MT, int NP>
-static int lm_launch(const LmParams& p, cudaStream_t s) {
-  const size_t smem = lm_smem_bytes(MT, p.ls, p.stages);
+template <int KW, int NP>
+static int lm_launch(const CUtensorMap& tm, const LmParams& p, cudaStream_t s) {
+  const size_t smem = lm_smem_bytes(p.chunks, p.stages);
   static PerDeviceOnce once;
-  if (once.first()) cudaFuncSetAttribute(latent_decode_mma_kernel<MT, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
-  const dim3 grid(p.B, p.n_split, (p.heads + 16 * MT - 1) / (16 * MT));
-  latent_decode_mma_kernel<MT, NP><<<grid, LM_THREADS, smem, s>>>(p);
-  if (p.n_split > 1) latent_merge_kernel<<<dim3(p.heads, p.B), 128, 0, s>>>(p);
+  if (once.first()) cudaFuncSetAttribute(latent_decode_mma_kernel<KW, NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, 232448);
+  const dim3 grid(p.B, p.n_split, (p.heads + LM_HEADS - 1) / LM_HEADS);
+  latent_decode_mma_kernel<KW, NP><<<grid, LM_THREADS, smem, s>>>(tm, p);
+  latent_merge_kernel<<<dim3(p.heads, p.B), 128, 0, s>>>(p);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
@@ -601,7 +666,7 @@ extern "C" int kvb_latent_prep(const void* qkv, long long ld, const float* norm_
                                void* stream) {
   if (B <= 0 || T_ <= 0 || heads <= 0 || dimp < dim || rp < rot || kvp < kv_rank || rot_dims > rot || rot_dims % 2 || B > 65535)
     return KVB_ERR_ARG;
-  if (ring && (T_ != 1 || ring_len <= 0)) return KVB_ERR_ARG;
+  if (ring && ring_len <= 0) return KVB_ERR_ARG;
   if ((dimp | rp | kvp) % 8) return KVB_ERR_ALIGN;
   kvb::LpParams p;
   p.ld = ld; p.norm_w = norm_w; p.freq = freq; p.slots = slots; p.start = start; p.count = count;
@@ -619,15 +684,6 @@ extern "C" int kvb_ring_gather(const void* ring, void* latent, const int* slots,
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
-extern "C" int kvb_ring_append(const void* latent, void* ring, const int* slots, const int* start, const int* count, int B, int T_,
-                               int P, int ring_len, int lw, int dtype, void* stream) {
-  if (B <= 0 || T_ <= 0 || B > 65535 || ring_len <= 0 || lw % 8 || (dtype != 0 && dtype != 1)) return KVB_ERR_ARG;
-  const int rows = T_ < ring_len ? T_ : ring_len;
-  kvb::ring_append_kernel<<<dim3((rows + kvb::LR_WARPS - 1) / kvb::LR_WARPS, B), kvb::LR_WARPS * 32, 0, (cudaStream_t)stream>>>(
-      (const uint4*)latent, (uint4*)ring, slots, start, count, T_, P, ring_len, lw / (dtype == 0 ? 4 : 8));
-  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
-}
-
 extern "C" int kvb_latent_attend(const void* q, const void* kv, const void* latent, void* out, const int* start, int B, int T_, int P,
                                  int heads, int dimp, int rp, int kvp, int vdp, int window, float scale, int dtype, void* stream) {
   if (B <= 0 || T_ <= 0 || B > 65535 || heads > 65535 || (dimp | rp) & 1) return KVB_ERR_ARG;
@@ -640,34 +696,37 @@ extern "C" int kvb_latent_attend(const void* q, const void* kv, const void* late
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
-extern "C" long long kvb_latent_decode_scratch_bytes(int B, int heads, int kvp, int ring_len) {
-  const int n = kvb::lm_splits(B, heads, ring_len);
-  return n == 1 ? 16 : (long long)n * B * heads * (kvp + 2) * 4;
+extern "C" long long kvb_latent_decode_scratch_bytes(int B, int heads, int kvp, int rp, int ring_len) {
+  const int n = kvb::lm_plan(B, heads, kvp, rp, ring_len).n_split;
+  return (long long)n * kvb::LM_GROUPS * B * heads * (kvp + 2) * 4;
 }
 
 extern "C" int kvb_latent_decode(const void* q_abs, const void* q, const void* ring, void* out, void* scratch, const int* slots,
-                                 const int* start, int B, int heads, int dimp, int rp, int kvp, int ring_len, float scale, int dtype,
-                                 int simple, int* status, void* stream) {
+                                 const int* start, int B, int n_slots, int heads, int dimp, int rp, int kvp, int ring_len,
+                                 float scale, int dtype, int simple, int* status, void* stream) {
   using namespace kvb;
   if (B <= 0 || heads <= 0 || ring_len <= 0 || B > 65535) return KVB_ERR_ARG;
   cudaStream_t s = (cudaStream_t)stream;
   LmParams p;
-  p.kv16 = (kvp + 15) / 16 * 16;
-  p.ls = p.kv16 + (rp + 15) / 16 * 16 + 8;
-  const int mt = heads > 16 ? 2 : 1;
-  p.stages = lm_stages(mt, p.ls);
-  if (dtype == 1 && !simple && kvp % 8 == 0 && rp % 8 == 0 && dimp % 8 == 0 && kvp <= 512 && p.stages > 0) {
-    p.q_abs = (const __nv_bfloat16*)q_abs; p.q = (const __nv_bfloat16*)q; p.ring = (const __nv_bfloat16*)ring;
+  const LmPlan pl = lm_plan(B, heads, kvp, rp, ring_len);
+  p.chunks = pl.chunks; p.ksteps = pl.ksteps; p.stages = pl.stages; p.n_split = pl.n_split;
+  if (dtype == 1 && !simple && kvp % 8 == 0 && rp % 8 == 0 && dimp % 8 == 0 && kvp <= 512 && p.stages > 0 && n_slots > 0 &&
+      p.ksteps <= 40) {
+    CUtensorMap tm;
+    const uint64_t lw = kvp + rp, dims[2] = {lw, (uint64_t)n_slots * ring_len}, st[1] = {lw};
+    const uint32_t box[2] = {64, LM_KEYS};
+    const int rc = tmap_bf16(&tm, ring, 2, dims, st, box);
+    if (rc) return rc;
+    p.q_abs = (const __nv_bfloat16*)q_abs; p.q = (const __nv_bfloat16*)q;
     p.out = (__nv_bfloat16*)out; p.slots = slots; p.start = start;
     p.B = B; p.heads = heads; p.dimp = dimp; p.rp = rp; p.kvp = kvp; p.ring_len = ring_len;
-    p.n_split = lm_splits(B, heads, ring_len);
     p.part_o = (float*)scratch;
-    p.part_ml = p.part_o + (long long)p.n_split * B * heads * kvp;
+    p.part_ml = p.part_o + (long long)p.n_split * LM_GROUPS * B * heads * kvp;
     p.scale_log2 = scale * 1.4426950408889634f;
     p.status = status;
-    const int np = (p.kv16 / 16 + 7) / 8;
-    if (mt == 1) return np <= 1 ? lm_launch<1, 1>(p, s) : (np <= 2 ? lm_launch<1, 2>(p, s) : lm_launch<1, 4>(p, s));
-    return np <= 1 ? lm_launch<2, 1>(p, s) : (np <= 2 ? lm_launch<2, 2>(p, s) : lm_launch<2, 4>(p, s));
+    if (kvp <= 128 && p.ksteps <= 16) return lm_launch<2, 1>(tm, p, s);
+    if (kvp <= 256 && p.ksteps <= 24) return lm_launch<3, 2>(tm, p, s);
+    return lm_launch<5, 4>(tm, p, s);
   }
   if (kvp > 32 * LD_MAX_C) return KVB_ERR_TOO_LARGE;
   const size_t smem = ((size_t)kvp + rp + 4 * kvp + 8) * sizeof(float);

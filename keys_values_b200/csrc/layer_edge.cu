@@ -11,7 +11,7 @@
 
 namespace kvb {
 
-constexpr int EDGE_THREADS = 256;
+constexpr int EDGE_THREADS = 256;  // of the plain norm; the layer edge takes 256 or 512 by width
 
 struct EdgeParams {
   // embedding source
@@ -69,14 +69,15 @@ template <typename T> struct EdgeVec<T, 1> {
   static __device__ __forceinline__ void store(T* p, const float (&v)[1]) { *p = from_f32<T>(v[0]); }
 };
 
-// Sum over the CTA; `red` has one float per warp, alternating between two buffers so that one barrier is enough.
+// Sum over the CTA of TH threads; `red` has one float per warp, alternating between two buffers so that one barrier is enough.
+template <int TH>
 __device__ __forceinline__ float edge_block_sum(float v, float* red) {
   v = warp_sum(v);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
   __syncthreads();
   float s = 0.f;
 #pragma unroll
-  for (int i = 0; i < EDGE_THREADS / 32; ++i) s += red[i];
+  for (int i = 0; i < TH / 32; ++i) s += red[i];
   return s;
 }
 
@@ -98,64 +99,111 @@ __device__ __forceinline__ long long edge_bigram_row(const EdgeParams& p, int b,
   return (prev * p.mul_prev + cur * p.mul_cur) % p.buckets;
 }
 
-// x of token t, columns c .. c + V − 1; `keep`: write the history and the stream
-template <typename T, int V, bool EMBED>
-__device__ __forceinline__ void edge_load(const EdgeParams& p, int b, int t, long long big_row, int c, bool keep, float (&x)[V]) {
+// x of token t for this thread's columns; `keep`: write the history and the stream. All loads of a token are issued before the
+// first store, those of several streams together.
+template <typename T, int V, int TH, int NC, bool EMBED>
+__device__ __forceinline__ void edge_load(const EdgeParams& p, int b, int t, bool keep, float (&x)[NC][V]) {
   const long long n = (long long)b * p.T + t;
-  const long long o = n * p.width + c;
+  const int c0 = threadIdx.x * V;
+  constexpr int STEP = TH * V;
   if (EMBED) {
-    const long long tok = edge_token(p, n);
-    EdgeVec<T, V>::load(static_cast<const T*>(p.embed) + tok * p.width + c, x);
-    if (p.bigram) {
-      float g[V];
-      EdgeVec<T, V>::load(static_cast<const T*>(p.bigram) + big_row * p.width + c, g);
+    const T* e = static_cast<const T*>(p.embed) + edge_token(p, n) * p.width;
+    const T* g = p.bigram ? static_cast<const T*>(p.bigram) + edge_bigram_row(p, b, t) * p.width : nullptr;
 #pragma unroll
-      for (int i = 0; i < V; ++i) x[i] += g[i];
+    for (int i = 0; i < NC; ++i) {
+      const int c = c0 + i * STEP;
+      if (c >= p.width) continue;
+      EdgeVec<T, V>::load(e + c, x[i]);
+      if (g) {
+        float y[V];
+        EdgeVec<T, V>::load(g + c, y);
+#pragma unroll
+        for (int u = 0; u < V; ++u) x[i][u] += y[u];
+      }
     }
-    if (keep) EdgeVec<float, V>::store(p.hist + o, x);
+    if (keep) {
+#pragma unroll
+      for (int i = 0; i < NC; ++i)
+        if (c0 + i * STEP < p.width) EdgeVec<float, V>::store(p.hist + n * p.width + c0 + i * STEP, x[i]);
+    }
     return;
   }
-  float xin[V], sub[V];
-  EdgeVec<float, V>::load(p.x_in + o, xin);
-  EdgeVec<T, V>::load(static_cast<const T*>(p.mix) + o, sub);
-  if (p.expert_out) {
-    for (int k = 0; k < p.top; ++k) {
-      float y[V];
-      const float w = p.expert_w[n * p.top + k];
-      EdgeVec<T, V>::load(static_cast<const T*>(p.expert_out) + (long long)p.expert_row[n * p.top + k] * p.expert_ld + c, y);
+  constexpr int EARLY = 8;  // experts whose rows are looked up first
+  int er[EARLY];
+  float ew[EARLY];
+  const int early = p.expert_out ? min(p.top, EARLY) : 0;
 #pragma unroll
-      for (int i = 0; i < V; ++i) sub[i] = fmaf(w, y[i], sub[i]);
-    }
+  for (int k = 0; k < EARLY; ++k) {
+    er[k] = k < early ? p.expert_row[n * p.top + k] : 0;
+    ew[k] = k < early ? p.expert_w[n * p.top + k] : 0.f;
   }
+  const long long o = n * p.width;
+  float fresh[NC][V], sub[NC][V];
 #pragma unroll
-  for (int i = 0; i < V; ++i) xin[i] += sub[i];
-  if (!p.coef) {
+  for (int i = 0; i < NC; ++i) {
+    const int c = c0 + i * STEP;
 #pragma unroll
-    for (int i = 0; i < V; ++i) x[i] = xin[i];
-  } else {
-#pragma unroll
-    for (int i = 0; i < V; ++i) x[i] = 0.f;
+    for (int u = 0; u < V; ++u) x[i][u] = fresh[i][u] = sub[i][u] = 0.f;
+    if (c >= p.width) continue;
+    EdgeVec<float, V>::load(p.x_in + o + c, fresh[i]);
+    EdgeVec<T, V>::load(static_cast<const T*>(p.mix) + o + c, sub[i]);
+  }
+  if (p.coef) {
 #pragma unroll 4
     for (int j = 0; j < p.n_hist; ++j) {
-      float y[V];
-      EdgeVec<float, V>::load(p.hist + j * p.hist_stride + o, y);
       const float w = p.coef[j];
 #pragma unroll
-      for (int i = 0; i < V; ++i) x[i] = fmaf(w, y[i], x[i]);
-    }
-    const float w = p.coef[p.n_hist];
+      for (int i = 0; i < NC; ++i) {
+        const int c = c0 + i * STEP;
+        if (c >= p.width) continue;
+        float y[V];
+        EdgeVec<float, V>::load(p.hist + j * p.hist_stride + o + c, y);
 #pragma unroll
-    for (int i = 0; i < V; ++i) x[i] = fmaf(w, xin[i], x[i]);
-    if (keep) EdgeVec<float, V>::store(p.hist + p.n_hist * p.hist_stride + o, xin);
+        for (int u = 0; u < V; ++u) x[i][u] = fmaf(w, y[u], x[i][u]);
+      }
+    }
   }
-  if (keep) EdgeVec<float, V>::store(p.x_out + o, x);
+  auto add_expert = [&](int row, float w) {
+    const T* y0 = static_cast<const T*>(p.expert_out) + (long long)row * p.expert_ld;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = c0 + i * STEP;
+      if (c >= p.width) continue;
+      float y[V];
+      EdgeVec<T, V>::load(y0 + c, y);
+#pragma unroll
+      for (int u = 0; u < V; ++u) sub[i][u] = fmaf(w, y[u], sub[i][u]);
+    }
+  };
+#pragma unroll
+  for (int k = 0; k < EARLY; ++k)
+    if (k < early) add_expert(er[k], ew[k]);
+  if (p.expert_out)
+    for (int k = EARLY; k < p.top; ++k) add_expert(p.expert_row[n * p.top + k], p.expert_w[n * p.top + k]);
+  const float w_new = p.coef ? p.coef[p.n_hist] : 1.f;
+#pragma unroll
+  for (int i = 0; i < NC; ++i)
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+      fresh[i][u] += sub[i][u];
+      x[i][u] = fmaf(w_new, fresh[i][u], x[i][u]);
+    }
+  if (keep) {
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = c0 + i * STEP;
+      if (c >= p.width) continue;
+      if (p.coef) EdgeVec<float, V>::store(p.hist + p.n_hist * p.hist_stride + o + c, fresh[i]);
+      EdgeVec<float, V>::store(p.x_out + o + c, x[i]);
+    }
+  }
 }
 
-// NC: column groups (of V columns) per thread held in registers
-template <typename T, int V, int NC, bool EMBED>
-__global__ void __launch_bounds__(EDGE_THREADS)
+// TH threads with NC groups of V columns each
+template <typename T, int V, int TH, int NC, bool EMBED>
+__global__ void __launch_bounds__(TH)
 layer_edge_kernel(const EdgeParams p) {
-  __shared__ float red[2][EDGE_THREADS / 32];
+  __shared__ float red[2][TH / 32];
   const int b = blockIdx.y;
   const int t0 = blockIdx.x * p.run;
   const int t1 = min(t0 + p.run, p.T);
@@ -167,7 +215,7 @@ layer_edge_kernel(const EdgeParams p) {
     const float* st = p.state + (long long)p.slots[b] * p.width;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
-      const int c = (i * EDGE_THREADS + threadIdx.x) * V;
+      const int c = (i * TH + threadIdx.x) * V;
 #pragma unroll
       for (int e = 0; e < V; ++e) hp[i][e] = 0.f;
       if (has && c < p.width) EdgeVec<float, V>::load(st + c, hp[i]);
@@ -176,25 +224,24 @@ layer_edge_kernel(const EdgeParams p) {
   const float gain = p.gain ? *p.gain : 0.f;
   for (int t = first; t < t1; ++t) {
     const bool keep = t >= t0;
-    const long long big = EMBED && p.bigram ? edge_bigram_row(p, b, t) : 0;
     float x[NC][V];
     float ss = 0.f;
+    edge_load<T, V, TH, NC, EMBED>(p, b, t, keep, x);
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
-      const int c = (i * EDGE_THREADS + threadIdx.x) * V;
+      const int c = (i * TH + threadIdx.x) * V;
       if (c < p.width) {
-        edge_load<T, V, EMBED>(p, b, t, big, c, keep, x[i]);
 #pragma unroll
         for (int e = 0; e < V; ++e) ss = fmaf(x[i][e], x[i][e], ss);
       }
     }
     if (!p.gain) continue;
-    ss = edge_block_sum(ss, red[t & 1]);
+    ss = edge_block_sum<TH>(ss, red[t & 1]);
     const float r = gain / sqrtf(ss / (float)p.width + p.eps);
     const long long o = ((long long)b * p.T + t) * p.width;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
-      const int c = (i * EDGE_THREADS + threadIdx.x) * V;
+      const int c = (i * TH + threadIdx.x) * V;
       if (c >= p.width) continue;
       float h[V];
 #pragma unroll
@@ -218,18 +265,18 @@ layer_edge_kernel(const EdgeParams p) {
     float* st = p.state + (long long)p.slots[b] * p.width;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
-      const int c = (i * EDGE_THREADS + threadIdx.x) * V;
+      const int c = (i * TH + threadIdx.x) * V;
       if (c < p.width) EdgeVec<float, V>::store(st + c, hp[i]);
     }
   }
 }
 
 // Passes of several tokens: the state is written after every CTA has read the old one. x: the stream the norm was taken of.
-template <int V, int NC>
-__global__ void __launch_bounds__(EDGE_THREADS)
+template <int V, int TH, int NC>
+__global__ void __launch_bounds__(TH)
 shift_state_kernel(const float* __restrict__ x, const float* __restrict__ gain_p, float* __restrict__ state, const int* __restrict__ slots,
                    const int* __restrict__ count, int T, int width, float eps) {
-  __shared__ float red[EDGE_THREADS / 32];
+  __shared__ float red[TH / 32];
   const int b = blockIdx.x;
   if (count[b] <= 0) return;
   const float* xr = x + ((long long)b * T + count[b] - 1) * width;
@@ -237,19 +284,19 @@ shift_state_kernel(const float* __restrict__ x, const float* __restrict__ gain_p
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < NC; ++i) {
-    const int c = (i * EDGE_THREADS + threadIdx.x) * V;
+    const int c = (i * TH + threadIdx.x) * V;
     if (c < width) {
       EdgeVec<float, V>::load(xr + c, v[i]);
 #pragma unroll
       for (int e = 0; e < V; ++e) ss = fmaf(v[i][e], v[i][e], ss);
     }
   }
-  ss = edge_block_sum(ss, red);
+  ss = edge_block_sum<TH>(ss, red);
   const float r = *gain_p / sqrtf(ss / (float)width + eps);
   float* st = state + (long long)slots[b] * width;
 #pragma unroll
   for (int i = 0; i < NC; ++i) {
-    const int c = (i * EDGE_THREADS + threadIdx.x) * V;
+    const int c = (i * TH + threadIdx.x) * V;
     if (c < width) {
 #pragma unroll
       for (int e = 0; e < V; ++e) v[i][e] *= r;
@@ -272,7 +319,7 @@ scalar_rmsnorm_kernel(const float* __restrict__ x, const long long* __restrict__
 #pragma unroll
     for (int e = 0; e < V; ++e) ss = fmaf(v[e], v[e], ss);
   }
-  ss = edge_block_sum(ss, red);
+  ss = edge_block_sum<EDGE_THREADS>(ss, red);
   const float r = *gain_p / sqrtf(ss / (float)width + eps);
   for (int c = threadIdx.x * V; c < width; c += EDGE_THREADS * V) {
     float v[V];
@@ -302,19 +349,18 @@ template <typename T, int V, bool EMBED>
 static int edge_launch(EdgeParams& p, cudaStream_t s) {
   p.run = edge_run(p.B, p.T);
   const dim3 grid((p.T + p.run - 1) / p.run, p.B);
-  const int groups = (p.width + EDGE_THREADS * V - 1) / (EDGE_THREADS * V);
   const bool late_state = p.gain && p.shift && p.T > 1;
   const float* x = EMBED ? p.hist : p.x_out;
-#define KVB_EDGE(NC)                                                                                                          \
-  do {                                                                                                                        \
-    layer_edge_kernel<T, V, NC, EMBED><<<grid, EDGE_THREADS, 0, s>>>(p);                                                      \
-    if (late_state)                                                                                                           \
-      shift_state_kernel<V, NC><<<p.B, EDGE_THREADS, 0, s>>>(x, p.gain, p.state, p.slots, p.count, p.T, p.width, p.eps);      \
+#define KVB_EDGE(TH, NC)                                                                                                   \
+  do {                                                                                                                     \
+    layer_edge_kernel<T, V, TH, NC, EMBED><<<grid, TH, 0, s>>>(p);                                                         \
+    if (late_state)                                                                                                        \
+      shift_state_kernel<V, TH, NC><<<p.B, TH, 0, s>>>(x, p.gain, p.state, p.slots, p.count, p.T, p.width, p.eps);         \
   } while (0)
-  if (groups <= 1) KVB_EDGE(1);
-  else if (groups <= 2) KVB_EDGE(2);
-  else if (groups <= 4) KVB_EDGE(4);
-  else if (groups <= 8) KVB_EDGE(8);
+  if (p.width <= 256 * V) KVB_EDGE(256, 1);
+  else if (p.width <= 512 * V) KVB_EDGE(512, 1);
+  else if (p.width <= 1024 * V) KVB_EDGE(256, 4);
+  else if (p.width <= 2048 * V) KVB_EDGE(512, 4);
   else return KVB_ERR_TOO_LARGE;
 #undef KVB_EDGE
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;

@@ -142,8 +142,7 @@ class LatentAttention(_Packed):
         P = seq.max_start if self.window == 0 else min(seq.max_start, self.window - 1)
         latent = torch.empty((B, P + T, s.row), dtype=x.dtype, device=x.device)
         L.ring_gather(ring, latent, seq, P)
-        q = L.latent_prep(qkv, w["norm"], w["freq"], latent, None, seq, P, s, self.eps)
-        L.ring_append(latent, ring, seq, P)
+        q = L.latent_prep(qkv, w["norm"], w["freq"], latent, ring, seq, P, s, self.eps)
         kv = torch.mm(latent.view(-1, s.row)[:, : s.kvp], w["key_value"].t())
         y = L.latent_attend(q, kv, latent, seq, P, s, self.window, self.scale)
         return F.linear(y, w["proj"])

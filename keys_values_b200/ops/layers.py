@@ -97,6 +97,9 @@ def linear_fp32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
 
 # ---- latent attention
 def latent_prep(qkv, norm_w, freq, latent, ring, seq, P: int, shape: LatentShape, eps: float) -> torch.Tensor:
+    """Split of the joint projection ``qkv (B, T, ·)``, norm of the latents, rotation. Returns padded queries
+    ``(B, T, heads, dimp + rp)``; latent rows go to ``latent[:, P:]`` and those of the last tokens of every sequence (at most
+    the ring's length) into ``ring``, either of which may be ``None``."""
     return _impl(qkv).latent_prep(qkv, norm_w, freq, latent, ring, seq, P, shape, eps)
 
 
@@ -104,11 +107,6 @@ def ring_gather(ring, latent, seq, P: int) -> None:
     """``latent[:, :P]`` = rows of the ``P`` positions before the pass (zero where a sequence has none)."""
     if P > 0:
         _impl(ring).ring_gather(ring, latent, seq, P)
-
-
-def ring_append(latent, ring, seq, P: int) -> None:
-    """The pass' last rows (at most the ring's length) of every sequence into its ring."""
-    _impl(ring).ring_append(latent, ring, seq, P)
 
 
 def latent_attend(q, kv, latent, seq, P: int, shape: LatentShape, window: int, scale: float) -> torch.Tensor:

@@ -89,7 +89,7 @@ def sequence_advance(idx, pos, prev_token, seq) -> None:
 
 # ------------------------------------------------------------------------------------------- latent attention
 def latent_prep(qkv, norm_w, freq, latent, ring, seq, P, shape, eps) -> torch.Tensor:
-    """``qkv (B, T, ·)`` → padded queries ``(B, T, heads, dimp + rp)``; latent rows go to ``latent`` or straight into ``ring``."""
+    """``qkv (B, T, ·)`` → padded queries ``(B, T, heads, dimp + rp)``; latent rows go to ``latent`` and into ``ring``."""
     B, T, ld = qkv.shape
     s = shape
     q = torch.empty((B, T, s.heads, s.dimp + s.rp), dtype=qkv.dtype, device=qkv.device)
@@ -105,13 +105,6 @@ def ring_gather(ring, latent, seq, P) -> None:
     B, n, lw = latent.shape
     _check(lib().kvb_ring_gather(_p(ring), _p(latent), _p(seq.slots), _p(seq.start), B, n - P, P, ring.shape[1], lw, code(ring.dtype),
                                  _stream(ring)), "ring_gather")
-    _count()
-
-
-def ring_append(latent, ring, seq, P) -> None:
-    B, n, lw = latent.shape
-    _check(lib().kvb_ring_append(_p(latent), _p(ring), _p(seq.slots), _p(seq.start), _p(seq.count), B, n - P, P, ring.shape[1], lw,
-                                 code(ring.dtype), _stream(ring)), "ring_append")
     _count()
 
 
@@ -137,10 +130,10 @@ def latent_decode(q_abs, q, ring, seq, shape, scale) -> torch.Tensor:
     C = ring.shape[1]
     out = torch.empty_like(q_abs)
     _contiguous(q_abs, q, ring)
-    nbytes = int(lib().kvb_latent_decode_scratch_bytes(B, H, kvp, C))
+    nbytes = int(lib().kvb_latent_decode_scratch_bytes(B, H, kvp, s.rp, C))
     scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device)
-    _check(lib().kvb_latent_decode(_p(q_abs), _p(q), _p(ring), _p(out), _p(scratch), _p(seq.slots), _p(seq.start), B, H, s.dimp, s.rp, kvp,
-                                   C, _f(scale), code(q.dtype), int(FORCE_SIMPLE), _p(status_word(q.device)), _stream(q)), "latent_decode")
+    _check(lib().kvb_latent_decode(_p(q_abs), _p(q), _p(ring), _p(out), _p(scratch), _p(seq.slots), _p(seq.start), B,
+                                   ring.shape[0], H, s.dimp, s.rp, kvp, C, _f(scale), code(q.dtype), int(FORCE_SIMPLE), _p(status_word(q.device)), _stream(q)), "latent_decode")
     _count()
     return out
 

@@ -79,12 +79,13 @@ def latent_prep(qkv, norm_w, freq, latent, ring, seq, P, s, eps):
     row = torch.zeros(B, T, s.row, dtype=qkv.dtype)
     row[..., : s.kv_rank] = c / torch.sqrt(c.square().mean(-1, keepdim=True) + eps) * norm_w
     row[..., s.kvp : s.kvp + s.rot] = _rotate(kr, cos, sin, s.rot_dims)
-    if ring is not None:
-        for b, (slot, n) in enumerate(zip(seq.slots.tolist(), seq.count.tolist())):
-            if n > 0:
-                ring[slot, int(pos[b, 0]) % ring.shape[1]] = row[b, 0]
-    else:
+    if latent is not None:
         latent[:, P:] = row
+    if ring is not None:
+        C = ring.shape[1]
+        for b, (slot, n) in enumerate(zip(seq.slots.tolist(), seq.count.tolist())):
+            for t in range(max(0, n - C), n):
+                ring[slot, int(pos[b, t]) % C] = row[b, t]
     return q
 
 
@@ -96,13 +97,6 @@ def ring_gather(ring, latent, seq, P) -> None:
             p = start - P + j
             if p >= max(0, start - C):
                 latent[b, j] = ring[slot, p % C]
-
-
-def ring_append(latent, ring, seq, P) -> None:
-    C = ring.shape[1]
-    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
-        for t in range(max(0, n - C), n):
-            ring[slot, (start + t) % C] = latent[b, P + t]
 
 
 def latent_attend(q, kv, latent, seq, P, s, window, scale):

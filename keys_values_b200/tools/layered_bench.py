@@ -6,7 +6,7 @@ time of every kernel of the design beside the like kernel of that model, each ag
 Random-init weights, synthetic tokens. The closest model has the same width, depth, heads, window and experts (count, chosen per
 token, expert weights per token): grouped-query attention over a sliding window, SwiGLU experts (``LLaMAMoE``); ``--dense``
 compares with a dense SwiGLU of the width that a token's chosen experts add up to. Kernel times are CUDA-event
-medians with an L2 flush (256 MB write) before every launch.
+medians with an L2 flush (256 MB written, another 256 MB read) before every launch.
 """
 from __future__ import annotations
 
@@ -103,9 +103,12 @@ def _peaks() -> Dict[str, float]:
 
 
 def time_us(fn: Callable[[], None], flush: torch.Tensor, n: int = 15) -> float:
+    """Median time. Before every launch a buffer larger than L2 is written and another one read, so that the launch
+    finds L2 full of clean lines (dirty ones would be written back inside the timed region)."""
     times = []
     for i in range(n + 3):
-        flush.fill_(i & 127)
+        flush[0].fill_(i & 127)
+        flush[1].sum()
         a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         a.record()
         fn()
@@ -119,7 +122,7 @@ def time_us(fn: Callable[[], None], flush: torch.Tensor, n: int = 15) -> float:
 class KernelTable:
     def __init__(self):
         self.peaks = _peaks()
-        self.flush = torch.empty(256 * 2**20, dtype=torch.uint8, device="cuda")
+        self.flush = torch.zeros(2, 64 * 2**20, dtype=torch.float32, device="cuda")
         self.rows: List[Dict] = []
 
     def add(self, what: str, fn: Callable[[], None], gbytes: float = 0.0, tflop: float = 0.0) -> None:
@@ -192,16 +195,16 @@ def kernel_table(config: Config, batch: int, tokens: int = 8192, dense_like: boo
         P = win - 1 if T > 1 else 0
         lat = rand(B, P + T, s.row)
         if T > 1:
-            prep = lambda: LC.latent_prep(qkv, norm, freq, lat, None, seq, P, s, eps)  # noqa: E731
+            prep = lambda: LC.latent_prep(qkv, norm, freq, lat, ring, seq, P, s, eps)  # noqa: E731
         else:
             prep = lambda: LC.latent_prep(qkv, norm, freq, None, ring, seq, 0, s, eps)  # noqa: E731
-        tab.add(f"{tag}: split, latent norm, rotation", prep, gbytes=n * 2 * (qkv.shape[2] + H * (s.dimp + s.rp) + s.row) / 1e9)
+        tab.add(f"{tag}: split, latent norm, rotation, into the ring", prep,
+                gbytes=2 * (n * (qkv.shape[2] + H * (s.dimp + s.rp) + s.row) + B * min(T, win) * s.row) / 1e9)
         qkv2, cs = rand(B, T, 3 * H * 128), torch.rand(T, 128, device=dev)
         tab.add(f"{tag}:   like: split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, None, None, H, H, 128, eps, 128, False),
                 gbytes=n * 2 * 2 * qkv2.shape[2] / 1e9)
         if T > 1:
             tab.add(f"{tag}: ring gather", lambda: LC.ring_gather(ring, lat, seq, P), gbytes=B * P * s.row * 4 / 1e9)
-            tab.add(f"{tag}: ring append", lambda: LC.ring_append(lat, ring, seq, P), gbytes=B * min(T, win) * s.row * 4 / 1e9)
             kb, vb, tp = (rand(B, H, win, 128) for _ in range(2)), None, torch.zeros(B, H, win, dtype=torch.int32, device=dev)
             kb, vb = kb
             nk, slots = rand(B, H, min(T, win), 128), torch.arange(min(T, win), device=dev).int().view(1, 1, -1).expand(B, H, -1)

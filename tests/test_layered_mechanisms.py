@@ -229,30 +229,44 @@ def test_latent_prep(env, name):
 
 
 @device_param
-def test_ring_append_and_gather(device):
+def test_rows_into_the_ring_and_back(device):
+    """Several passes of unequal rows: the ring holds the newest positions, a pass finds those before it in order."""
     dev = torch.device(device)
-    B, C, lw = 3, 7, 16
+    s = L.LatentShape(heads=1, dim=8, rot=8, vdim=8, kv_rank=8, rot_dims=8)
+    B, C = 3, 7
     slots = [4, 0, 2]
-    rows = torch.arange(1, 41, dtype=torch.float32)[:, None] * torch.ones(lw) + 100 * torch.arange(B)[:, None, None]  # row p of sequence b
-    ring = torch.zeros(5, C, lw, device=dev)
+    ring = torch.zeros(5, C, s.row, device=dev)
     tab = table(dev, B, [0, 0, 0], slots=slots)
+    g = torch.Generator().manual_seed(0)
+    qkv = torch.randn(B, 40, 16 + 8 + 8, generator=g)
+    rows = torch.zeros(B, 40, s.row)
+    for b in range(B):
+        for p in range(40):
+            rows[b, p, :8] = oracle.unit_rms(qkv[b, p, 16:24].double(), 0.1)
+            rows[b, p, 8:] = oracle.rotate(qkv[b, p, 24:].double(), p, 100.0, 8)
+    norm, freq = torch.ones(8, device=dev), (100.0 ** (torch.arange(4, dtype=torch.float64) * -0.25)).float().to(dev)
     at = [0, 0, 0]
-    for n, cs in ((5, [5, 2, 0]), (9, [9, 1, 9]), (2, [2, 2, 2]), (20, [3, 20, 0])):
+    for n, cs in ((5, [5, 2, 0]), (9, [9, 1, 9]), (1, [1, 0, 1]), (2, [2, 2, 2]), (20, [3, 20, 0])):
         seq = tab.begin(B, n, cs)
         P = min(seq.max_start, C)
-        latent = torch.full((B, P + n, lw), -1.0, device=dev)
+        latent = torch.full((B, P + n, s.row), -1.0, device=dev)
         L.ring_gather(ring, latent, seq, P)
+        part = torch.zeros(B, n, qkv.shape[2])
         for b in range(B):
-            for j in range(P):
-                p = at[b] - P + j
-                assert float(latent[b, j, 3]) == (float(rows[b, p, 3]) if p >= 0 else 0.0), (b, j, p)
-            latent[b, P : P + cs[b]] = rows[b, at[b] : at[b] + cs[b]].to(dev)
-        L.ring_append(latent, ring, seq, P)
+            part[b, : cs[b]] = qkv[b, at[b] : at[b] + cs[b]]
+        L.latent_prep(part.to(dev), norm, freq, latent, ring, seq, P, s, 0.1)
+        for b in range(B):
+            want = torch.zeros(P + cs[b], s.row)
+            for j in range(P + cs[b]):
+                if at[b] - P + j >= 0:
+                    want[j] = rows[b, at[b] - P + j]
+            if len(want):
+                close(latent[b, : P + cs[b]], want, torch.float32)
         tab.finish(seq, torch.zeros(B, n, dtype=torch.int64, device=dev))
         at = [a + c for a, c in zip(at, cs)]
-        for b, s in enumerate(slots):
+        for b, slot in enumerate(slots):
             for p in range(max(0, at[b] - C), at[b]):
-                assert float(ring[s, p % C, 0]) == float(rows[b, p, 0])
+                close(ring[slot, p % C], rows[b, p], torch.float32)
     assert float(ring[1].abs().max()) == 0 and float(ring[3].abs().max()) == 0
 
 
