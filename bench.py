@@ -36,9 +36,11 @@ def parse_args():
     ap.add_argument("--steps", type=int, default=2)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", type=str, default="b200", choices=["b200", "reference"])
-    ap.add_argument("--config", type=str, default="train", choices=["train", "inference"],
+    ap.add_argument("--config", type=str, default="train", choices=["train", "inference", "layered"],
                     help="train: long-context LoRA fine-tuning step, data parallel (the headline); inference: chunked prefill + "
-                         "greedy decoding of Llama-3-8B through an int4 H2O cache, tensor parallel over the launched ranks")
+                         "greedy decoding of Llama-3-8B through an int4 H2O cache, tensor parallel over the launched ranks; layered: "
+                         "prefill and decode of models with described layers (Mezilix) beside the closest LitGPT-shaped models, one GPU")
+    ap.add_argument("--kernels", action="store_true", help="layered: also time every kernel beside the like one (table on stderr, rows in the JSON)")
     ap.add_argument("--batch", type=int, default=4, help="inference: prompts per batch")
     ap.add_argument("--decode", type=int, default=512, help="inference: generated tokens per prompt")
     ap.add_argument("--model", type=str, default="Qwen3-4B")
@@ -250,8 +252,60 @@ def run_inference(args) -> dict:
     }
 
 
+def run_layered(args) -> dict:
+    """Models with described layers at sizes of real layers (random weights): chunked prefill of ``--batch`` prompts and greedy decoding
+    (``--decode`` steps), beside the closest LitGPT-shaped models of equal size (LLaMAMoE and dense feed-forward)."""
+    import contextlib
+
+    import torch
+
+    from keys_values_b200.config import Config
+    from keys_values_b200.tools import layered_bench as lb
+
+    batch = 32 if args.batch == 4 else args.batch
+    prompt = 8192 if args.seq_len == 131072 else args.seq_len
+    decode = 64 if args.decode == 512 else args.decode
+    chunk = 2048 if args.chunk_size == 1024 else args.chunk_size
+    names = ["Mezilix-2k", "Mezilix-4k"] if args.model == "Qwen3-4B" else [args.model]
+    sampler = ClockSampler(0)
+    sampler.start()
+    models, kernels = [], {}
+    for name in names:
+        cfg = Config.from_name(name)
+        if args.n_layer:
+            cfg.layers, cfg.n_layer = cfg.layers[: args.n_layer], args.n_layer
+        window = cfg.layers[0]["mixer"]["window"]
+        for kind, c in (("this design", cfg), ("closest, LLaMAMoE", lb.closest_config(cfg)), ("closest, dense", lb.closest_config(cfg, dense=True))):
+            r = lb.throughput(c, batch, prompt, decode if kind != "closest, LLaMAMoE" else min(decode, 8), window, chunk, max(1, args.steps))
+            models.append(dict(kind=kind, **r))
+            torch.cuda.empty_cache()
+        if args.kernels:
+            with contextlib.redirect_stdout(sys.stderr):
+                kernels[name] = lb.kernel_table(cfg, batch)
+            torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    first = models[0]
+    total = batch * (prompt + decode) / (first["prefill_s"] + first["decode_s"])
+    out = {
+        "metric": "layered model inference tokens/s (prefill + decode)", "value": total, "unit": "tokens/s", "n_gpus": 1, "steps": max(1, args.steps),
+        "warmup": args.warmup, "ms_per_step": 1e3 * (first["prefill_s"] + first["decode_s"]), "higher_is_better": True, "scaling": "strong",
+        "vs_baseline": None, "dtype": "bf16", "data": "synthetic uniform-random token ids, random-init weights", "impl": "b200",
+        "config": {"model": first["model"], "global_batch": batch, "seq_len": prompt, "decode_tokens": decode, "chunk_size": chunk,
+                   "n_layer": args.n_layer, "l2": "weights and caches exceed the 126 MB L2; kernel times after an L2 flush"},
+        "models": models, "clocks": clocks, "gpu_launches": first["native_launches"],
+        "e2e": {"value": total, "unit": "tokens/s", "h2d_bytes_per_step": batch * prompt * 8, "d2h_bytes_per_step": batch * decode * 8},
+    }
+    if kernels:
+        out["kernels"] = kernels
+    return out
+
+
 def main():
     args = parse_args()
+    if args.config == "layered":
+        out = run_layered(args) if args.impl == "b200" else {"impl": "reference", "unavailable": "the reference has no such model"}
+        print(json.dumps(out), flush=True)
+        return
     if args.config == "inference" and args.impl == "reference":
         from baseline.reference_arm import run_reference_inference
 

@@ -269,6 +269,8 @@ class GPT(nn.Module):
     def __init__(self, config: Config, **mha_kwargs) -> None:
         super().__init__()
         assert config.padded_vocab_size is not None
+        if config.layers is not None and not self.tracks_positions:
+            raise ValueError(f"{config.name!r} describes its layers: {type(self).__name__} cannot hold it (use models.registry.create_model)")
         self.config = config
         self.lm_head = nn.Linear(config.n_embd, config.padded_vocab_size, bias=config.lm_head_bias)
         self.transformer = nn.ModuleDict(

@@ -3,7 +3,7 @@
     bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N < steps.jsonl
     python -m keys_values_b200 trace_run ...          (the same)
 
-Every line of standard input is a step, ``{"step": 0, "entries": [{"id": "a", "tokens": [5, 17], "want": [1]}], "end": []}``:
+Every line of standard input is a step, ``{"step": 4, "entries": [{"id": "req7", "tokens": [812, 40], "want": [1]}], "end": ["req7"]}``:
 the next tokens of each request of the batch and the places among them whose logits are wanted; ``end`` names the requests
 that are finished after the step, whose slots are given back. A step with wanted logits writes ``OUT/<step>.f32``
 (little-endian fp32, ``[wanted, vocab]``, in the order of the entries); after every step ``done <step>`` is printed.

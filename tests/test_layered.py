@@ -16,6 +16,7 @@ from keys_values_b200.kvcache.latent import LatentKVCache
 from keys_values_b200.long_context import LongContextInferenceModel
 from keys_values_b200.models.head_model import CrossEntropyOnLogits
 from keys_values_b200.models.layered import LayeredGPT
+from keys_values_b200.models.model import GPT
 from keys_values_b200.models.registry import create_model, default_cache_name
 from keys_values_b200.tools.trace_run import TraceRunner, load_model, run
 
@@ -298,6 +299,8 @@ def test_caches_fit_their_models():
     plain = create_model(Config.from_name("tiny-gpt"))
     with pytest.raises(ValueError, match="does not fit"):
         KVCacheFactory.create(plain, "latent-default", 1, 64)
+    with pytest.raises(ValueError, match="describes its layers"):
+        GPT(Config.from_name("tiny-mezilix"))
     with pytest.raises(ValueError, match="equal length"):
         plain(torch.zeros(2, 3, dtype=torch.int64), counts=[3, 1])
     layered.set_kv_caches(2, max_seq_length=100)
