@@ -23,7 +23,7 @@ CSRC = ROOT / "csrc"
 BUILD = CSRC / "build"
 LIB = ROOT / "libkvb200.so"
 LAYERS_LIB = ROOT / "libkvb200_layers.so"
-LAYERS_SOURCES = ("grouped_attn", "latent_attn", "latent_sm100", "layer_edge", "moe", "moe_sm100", "norm_edge", "ssm", "ssm_sm100")
+LAYERS_SOURCES = ("grouped_attn", "latent_attn", "latent_sm100", "layer_edge", "moe", "moe_sm100", "norm_edge", "retention", "ssm", "ssm_sm100")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

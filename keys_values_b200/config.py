@@ -83,7 +83,7 @@ class Config:
     final_logit_softcapping: Optional[float] = None
     # Models described layer by layer (models/layered.py). Each entry: {"mixer": {"kind": ..., sizes and constants},
     # "mlp": None or {"kind": ..., sizes}}; the kinds and their entries are those of the mixer and feed-forward classes there.
-    # With parallel_residual mixer and feed-forward read one norm's output; without, each has a norm before it and, with
+    # With parallel_residual mixer and feed-forward read one norm's output; without, each has a norm before it (norm_1 / norm_2) and, with
     # post_attention_norm / post_mlp_norm, one after it.
     layers: Optional[List[dict]] = None
     # {"start", "stop", "times"}: layers start .. stop - 1 run `times` times in a row with the same weights. Before each
@@ -93,6 +93,7 @@ class Config:
     bigram: Optional[dict] = None  # {"buckets", "mul_prev", "mul_cur"}: hashed embedding of (previous token, token)
     token_shift: bool = False  # the mixer reads a learned blend of this and the previous token's normed input
     depth_average: bool = False  # learned average over the embedding output and all layers' results
+    tie_embeddings: bool = False  # described layers: the output head is the embedding table
     architecture: str = ""  # entry of models/registry.py the config was read by
     # Added by keys_values (config.py:26-30): use the in-repo RMSNorm
     own_rms_norm_implementation: bool = True
@@ -252,6 +253,43 @@ def _grouped(heads: int, kv_heads: int, dim: int, ff: int, rope_base: float = 50
                 mlp=dict(kind="dense", ff=ff, activation="relu_squared"))
 
 
+def _ladadra(width: int, layers: List[dict], **kwargs: Any) -> dict:
+    """Fields of a model of sequential layers with norms on the sublayers' outputs only; ``layers`` as in ``Config.layers``."""
+    first = next(x["mixer"] for x in layers if x["mixer"]["kind"] == "grouped_attention")
+    return dict(
+        n_embd=width, n_layer=len(layers), layers=layers, n_head=first["n_head"], n_query_groups=first["n_kv_head"], head_size=first["dim"],
+        norm_class_name="StreamRMSNorm", parallel_residual=False, norm_1=False, norm_2=False, post_attention_norm=True, post_mlp_norm=True,
+        bias=False, tie_embeddings=True, architecture="Ladadra", **kwargs,
+    )
+
+
+def _retention(heads: int, dim: int, vdim: int, rope_base: float = 10000.0) -> dict:
+    """Decays 1 − 2^−5, 1 − 2^−6, … over the heads, repeated after 1 − 2^−12."""
+    return dict(kind="retention", n_head=heads, dim=dim, v_dim=vdim, rope_base=rope_base, rope_dims=dim,
+                decay=[1.0 - 2.0 ** -(5 + i % 8) for i in range(heads)])
+
+
+def _chunked(heads: int, kv_heads: int, dim: int, vdim: int, chunk: int, rope_dims: int, softcap: float = 50.0, rope_base: float = 500000.0,
+             bands: Optional[dict] = None) -> dict:
+    return dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=vdim, scale=dim**-0.5, rope_base=rope_base,
+                rope_dims=rope_dims, rope_bands=bands or dict(factor=8.0, low=1.0, high=4.0, original=8192), qkv_bias=True, qk_norm=True,
+                softcap=softcap, chunk=chunk, sink="learned", gate="head")
+
+
+def _differential(heads: int, kv_heads: int, dim: int, vdim: int, window: int, keep_first: int, differential: float) -> dict:
+    return dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=vdim, scale=dim**-0.5, qk_norm="head",
+                window=window, keep_first=keep_first, differential=differential)
+
+
+def _gated(ff: int) -> dict:
+    return dict(kind="gated", ff=ff)
+
+
+def _grouped_experts(n_expert: int, top: int, ff: int, groups: int, keep: int, shared: int) -> dict:
+    return dict(kind="routed", n_expert=n_expert, top=top, ff=ff, activation="silu_gated", score="sigmoid", correction=True, renormalize=True,
+                renormalize_eps=1e-20, groups=dict(count=groups, keep=keep), shared=shared)
+
+
 _llama_like = dict(
     rotary_percentage=1.0,
     parallel_residual=False,
@@ -333,6 +371,34 @@ configs: List[dict] = [
     dict(
         name="Pazenex-4k", block_size=1 << 20, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5,
         **_pazenex(4096, [_mamba2(128, 64, 128, 8, 16384, norm_groups=8), _grouped(32, 8, 128, 16384, rope_scale=4.0)] * 6),
+    ),
+    # Ladadra: retention, differential attention over a window and chunked attention, dense and routed gated feed-forwards, norms on
+    # the sublayers' outputs only
+    dict(
+        name="tiny-ladadra", block_size=1 << 20, vocab_size=416, padded_vocab_size=416, norm_eps=1e-5,
+        **_ladadra(144, [
+            dict(mixer=_retention(3, 40, 24), mlp=_gated(200)),
+            dict(mixer=_differential(4, 1, 24, 40, window=60, keep_first=12, differential=0.4), mlp=_grouped_experts(8, 3, 40, 4, 2, 56)),
+            dict(mixer=_chunked(6, 3, 32, 24, chunk=90, rope_dims=16, bands=dict(factor=2.0, low=1.0, high=4.0, original=512)), mlp=None),
+        ]),
+    ),
+    dict(
+        name="Ladadra-2k", block_size=1 << 20, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5,
+        **_ladadra(2048, [
+            dict(mixer=_retention(16, 128, 128), mlp=_gated(5632)),
+            dict(mixer=_differential(16, 4, 64, 128, window=4096, keep_first=128, differential=0.5), mlp=_grouped_experts(64, 6, 704, 8, 4, 1408)),
+            dict(mixer=_chunked(16, 4, 128, 128, chunk=8192, rope_dims=64), mlp=_gated(5632)),
+            dict(mixer=_chunked(16, 4, 128, 128, chunk=8192, rope_dims=64), mlp=_grouped_experts(64, 6, 704, 8, 4, 1408)),
+        ] * 4),
+    ),
+    dict(
+        name="Ladadra-4k", block_size=1 << 20, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5,
+        **_ladadra(4096, [
+            dict(mixer=_retention(32, 128, 128), mlp=_gated(11008)),
+            dict(mixer=_differential(32, 8, 64, 128, window=4096, keep_first=128, differential=0.5), mlp=_grouped_experts(32, 4, 2048, 4, 2, 2816)),
+            dict(mixer=_chunked(32, 8, 128, 128, chunk=8192, rope_dims=64), mlp=_gated(11008)),
+            dict(mixer=_chunked(32, 8, 128, 128, chunk=8192, rope_dims=64), mlp=_grouped_experts(32, 4, 2048, 4, 2, 2816)),
+        ] * 3),
     ),
     # Qwen 2.5
     dict(

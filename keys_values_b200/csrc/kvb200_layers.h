@@ -37,36 +37,53 @@ int kvb_sequence_advance(const long long* idx, int* pos, int* prev_token, const 
                          void* stream);
 
 // ---- norm_edge.cu
-// Between two sublayers: x = x_in + norm(sub) · after (x_in, sub NULL: without; after NULL: sub as it is) + embed[idx] + step (each
-// unless NULL); x_out = x (NULL: not stored; may be x_in); h = norm(x) · before unless before is NULL. Rows of `width`, x fp32,
-// sub, embed and h of `dtype`, weights and step fp32. center: layer norm, else RMS norm.
-int kvb_norm_edge(const float* x_in, const void* sub, const float* after, float* x_out, const float* before, void* h,
-                  const long long* idx, const void* embed, long long vocab, const float* step, long long n, int width, float eps,
-                  int center, int dtype, int* status, void* stream);
+// Between two sublayers: s = sub + sum_k expert_w[n, k] · expert_out[expert_row[n, k]] (sub, expert_out NULL: without); x = x_in +
+// norm(s) · after (x_in NULL: without; after NULL: s as it is) + embed[idx] + step (each unless NULL); x_out = x (NULL: not stored; may be
+// x_in); h = norm(x) · before, or x (before NULL), unless h is NULL. Rows of `width`, x fp32, sub, expert_out, embed and h of `dtype`,
+// weights and step fp32. center: layer norm, else RMS norm.
+int kvb_norm_edge(const float* x_in, const void* sub, const void* expert_out, const int* expert_row, const float* expert_w, int top,
+                  long long expert_ld, const float* after, float* x_out, const float* before, void* h, const long long* idx,
+                  const void* embed, long long vocab, const float* step, long long n, int width, float eps, int center, int dtype,
+                  int* status, void* stream);
 
 // ---- grouped_attn.cu
-// rows (slots, len, kv_heads, dimp + vdp) = [key | value] of every position. Columns of qkv: queries (heads · dimp), keys
-// (kv_heads · dimp), values from value_col on; value_col = heads · dimp: the values are the keys as they are in qkv. dimp, vdp
-// multiples of 8, padding zero. norm_q / norm_k (heads · dimp / kv_heads · dimp): RMS norm over the whole projection.
+// One grouped-query attention. `maps` queries and keys per head over the same values (1, or 2 for differential attention, whose
+// result is norm(map 1 - lambda · map 2) · post per head, the norm an RMS norm over vdim without a weight). Rows of the cache
+// (slots, len, kv_heads, maps · dimp + vdp) = [keys of the maps | value] of a position; dimp, vdp multiples of 8, padding zero.
+// Position i sees j <= i, and only those with i - j < window or j < keep (window > 0), or in i's own part of `chunk` positions (chunk > 0).
+// ring > 0: the first `head` positions have rows of their own, position p >= head has row head + (p - head) mod ring (both multiples of
+// 128); a pass must not be longer than the ring minus what a position looks back.
+// score = q·k · scale, then softcap · tanh(score / softcap) if softcap > 0. sink: one more term exp(sink_w[head]) in the denominator
+// (sink_w NULL: exp(0)). gate_cols: columns of the gate projection per head, 0 (none), 1 or vdp: out *= sigmoid(gate).
+typedef struct {
+  int heads, kv_heads, maps, dim, dimp, vdim, vdp;
+  int rot_dims, value_col, head_norm;
+  int window, keep, chunk;
+  int head, ring;
+  int sink, gate_cols;
+  float scale, softcap;
+  float lambda, post, eps;
+  const float* sink_w;
+} kvb_attention;
+// Columns of qkv: queries (heads · maps · dimp), keys (kv_heads · maps · dimp), values from value_col on; value_col = heads · dimp: the
+// values are the keys as they are in qkv. RMS norm (norm_q, norm_k NULL: none) over the whole projection with weights of its size, or
+// (head_norm) over every head and map with dimp weights. Rotation of the first rot_dims dimensions by position · freq.
 int kvb_grouped_prep(const void* qkv, long long ld, const float* norm_q, const float* norm_k, const float* freq, void* q, void* rows,
-                     const int* slots, const int* start, const int* count, int B, int T, int len, int heads, int kv_heads, int dim,
-                     int dimp, int vdp, int rot_dims, int value_col, float eps, int dtype, void* stream);
-// Queries (B, T, heads, dimp), the first of row b at position start[b], over the rows of its slot up to their own positions. sink:
-// one more term exp(0) in the denominator. gate (leading dimension gate_ld, NULL: none): out *= sigmoid(gate).
+                     const int* slots, const int* start, const int* count, int B, int T, int len, const kvb_attention* a, int dtype,
+                     void* stream);
+// Queries (B, T, heads · maps, dimp), the first of row b at position start[b], over the rows of its slot. gate: leading dimension
+// gate_ld, NULL: none. out (B, T, heads, vdp).
 int kvb_grouped_attend(const void* q, const void* rows, const void* gate, long long gate_ld, void* out, const int* slots,
-                       const int* start, int B, int T, int len, int heads, int kv_heads, int dimp, int vdp, int sink, float scale,
-                       int dtype, void* stream);
+                       const int* start, int B, int T, int len, const kvb_attention* a, int dtype, void* stream);
 
 // The same in bf16: several tokens on tcgen05 (latent_sm100.cu), one token per sequence split over the positions.
-int kvb_grouped_attend_tc_supported(int dimp, int vdp);
+int kvb_grouped_attend_tc_supported(const kvb_attention* a);
 int kvb_grouped_attend_tc(const void* q, const void* rows, const void* gate, long long gate_ld, void* out, const int* slots,
-                          const int* start, int B, int T, int n_slots, int len, int heads, int kv_heads, int dimp, int vdp, int sink,
-                          float scale, int* status, void* stream);
-int kvb_grouped_decode_supported(int dimp, int vdp);
-long long kvb_grouped_decode_scratch_bytes(int B, int heads, int kv_heads, int dimp, int vdp, int len);
+                          const int* start, int B, int T, int n_slots, int len, const kvb_attention* a, int* status, void* stream);
+int kvb_grouped_decode_supported(const kvb_attention* a);
+long long kvb_grouped_decode_scratch_bytes(int B, int len, const kvb_attention* a);
 int kvb_grouped_decode(const void* q, const void* rows, const void* gate, long long gate_ld, void* out, void* scratch, const int* slots,
-                       const int* start, int B, int n_slots, int len, int heads, int kv_heads, int dimp, int vdp, int sink,
-                       float scale, int* status, void* stream);
+                       const int* start, int B, int n_slots, int len, const kvb_attention* a, int* status, void* stream);
 
 // ---- ssm.cu
 // Columns of u (ld): z (heads · vdp), from `col` on the channels x (heads · vdp) | B (groups · np) | C (groups · np), from
@@ -85,6 +102,28 @@ int kvb_state_scan_tc(const void* u, long long ld, int dt_col, const void* xbc, 
 int kvb_state_step(const void* u, long long ld, int col, int dt_col, const float* w, const float* bias, const float* dt_bias,
                    const float* a_log, const float* skip, void* ring, float* state, void* y, const int* slots, const int* start,
                    const int* count, int B, int heads, int groups, int vdp, int np, int taps, int dtype, void* stream);
+// ---- retention.cu (scans: ssm.cu, ssm_sm100.cu). S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head; state (slots, heads, np, vdp)
+// fp32, np = key size and vdp = value size padded to multiples of 8.
+// in (n, ld) fp32 = [queries heads · np | keys heads · np] -> out (n, 2 · heads · np): both rotated by position · freq, keys times key_scale
+int kvb_retention_prep(const float* in, long long ld, const float* freq, void* out, const int* start, int B, int T, int heads, int np,
+                       int rot_dims, float key_scale, int dtype, void* stream);
+// qk as prep leaves it, v (ldv) heads · vdp columns; y (B, T, heads · vdp), zero in padding
+int kvb_retention_scan(const void* v, long long ldv, const void* qk, long long ldqk, const float* decay, float* state, void* y,
+                       const int* slots, const int* start, const int* count, int B, int T, int heads, int vdp, int np, int dtype,
+                       void* stream);
+// the same in bf16 on tcgen05, sizes and scratch as kvb_state_scan_tc with groups = heads
+int kvb_retention_scan_tc(const void* v, long long ldv, const void* qk, long long ldqk, const float* log2_decay, float* state, void* y,
+                          void* scratch, const int* slots, const int* start, const int* count, int B, int T, int heads, int vdp, int np,
+                          int* status, void* stream);
+// out = y / rms(y) · silu(gate) head by head (the norm without a weight, over vdim columns); gate has leading dimension ld
+int kvb_head_norm_gate(const void* y, const void* gate, long long ld, void* out, long long n, int heads, int vdim, int vdp, float eps,
+                       int dtype, void* stream);
+// One token per sequence, everything between the projections: u (B, ld) fp32 = [queries | keys | values | gate]; out (B, heads · vdp)
+int kvb_retention_step(const float* u, long long ld, const float* freq, const float* decay, float* state, void* out, const int* slots,
+                       const int* start, const int* count, int B, int heads, int vdim, int vdp, int np, int rot_dims, float key_scale,
+                       float eps, int dtype, void* stream);
+
+// ---- ssm.cu
 // out = norm(y · silu(z)) · weight in `parts` equal parts of the heads · vdim unpadded columns
 int kvb_gated_group_norm(const void* y, const void* z, long long ld, const float* weight, void* out, long long n, int heads,
                          int vdim, int vdp, int parts, float eps, int dtype, void* stream);
@@ -119,19 +158,30 @@ int kvb_latent_attend_tc(const void* q, const void* kv, const void* latent, void
                          int heads, int dimp, int rp, int kvp, int vdp, int window, float scale, int* status, void* stream);
 
 // ---- moe.cu
-// Router: softmax over n_expert fp32 logits, the `top` largest (ties: lower index first). weight (n, top) fp32, divided by
-// their sum if renormalize. Every choice gets a row of the buffer sorted by expert: the rows of an expert start at a multiple
-// of `tile`; row (n, top), tile_expert / tile_row (one entry per tile in use), plan[0] = number of tiles. counters: n_expert
-// ints of scratch.
+// Router. score 0: softmax over the experts' fp32 logits, 1: sigmoid of each. correction (n_expert, NULL: none) is added for the choice
+// only. groups > 1: equal groups of neighbouring experts, a group's score is the sum of its two largest choice scores, and only experts
+// of the `keep` best groups can be chosen. renormalize: the chosen scores are divided by their sum + eps.
+typedef struct {
+  int score, groups, keep, renormalize;
+  float eps;
+  const float* correction;
+} kvb_router;
+// The `top` experts with the largest choice scores (ties: lower index first), their scores in weight (n, top) fp32. Every choice gets a
+// row of the buffer sorted by expert: the rows of an expert start at a multiple of `tile`; row (n, top), tile_expert / tile_row (one
+// entry per tile in use), plan[0] = number of tiles. counters: n_expert ints of scratch.
 int kvb_moe_route(const float* logits, int* expert, float* weight, int* row, int* counters, int* plan, int* tile_expert,
-                  int* tile_row, long long n, int n_expert, int top, int tile, int max_tiles, int renormalize, void* stream);
+                  int* tile_row, long long n, int n_expert, int top, int tile, int max_tiles, const kvb_router* router, void* stream);
 // sorted[row[n, k]] = h[n] (columns beyond width zero up to ld)
 int kvb_moe_gather(const void* h, const int* row, void* sorted, long long n, int top, int width, long long ld, int dtype, void* stream);
 // out[r] = act(w[expert of r's tile] · in[r]) for all rows of the tiles in use; in (rows, ldk), w (n_expert, n_out, ldk),
-// out (rows, ldo) with columns n_out .. ldo zero. act 0: none, 1: square of relu.
+// out (rows, ldo) with columns n_out .. ldo zero. act 0: none, 1: square of relu, 2: gated unit, rows 2 f and 2 f + 1 of w are gate and up
+// projection of result f (n_out counts both, out has half as many columns).
 int kvb_moe_gemm(const void* in, const void* w, void* out, const int* plan, const int* tile_expert, const int* tile_row, int tile,
                  int max_tiles, int n_expert, int n_out, int k, long long ldk, long long ldo, int act, int dtype, int simple,
                  int* status, void* stream);
+
+// out (n, ldo) = silu(x[:, :ff]) · x[:, up : up + ff], zero from column ff on
+int kvb_glu(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, int dtype, void* stream);
 
 #ifdef __cplusplus
 }

@@ -4,8 +4,10 @@
 //   S = Q_u K_u^T + Q_r K_r^T (the rotated key part K_r is shared by the heads), P = exp2(S·c − m), O += P V
 //
 // Grouped-query form: no shared part; `group` query heads read one key/value head; keys and values lie in the cache, whose
-// rows are the positions of a slot. Optional: one more term exp(0) in the softmax denominator (the running maximum
-// starts at 0 and the sum at 1), and sigmoid of a gate projection on the output.
+// rows are the positions of a slot (in a ring, if the layer looks back a bounded way). Optional: one more term in the softmax
+// denominator (the running maximum starts at the sink and the sum at 1), soft-capped scores, sigmoid of a gate projection on the output.
+// Two maps per head (DIFF): the two query tiles of a CTA are the two maps of the same 128 tokens; they share the value tiles, and the
+// epilogue takes the difference of both outputs out of TMEM, norms it per head and stores it.
 //
 // The head sizes of keys (unrotated + rotated) and values differ and are run-time values: operands are staged as chunks of
 // 64 features ([128 rows x 128 B], 128B swizzle, TMA fills what lies beyond a tensor's last feature with zero), S sums over
@@ -16,10 +18,12 @@
 //
 // Masks are arithmetic: key row j of sequence b has position start[b] − P + j (P = start[b] in a grouped-query cache), query t sees
 // max(P + t − window + 1, P − start[b], 0) <= j <= P + t. Tiles outside the range of a query tile are skipped, tiles inside
-// the range of all its rows need no mask.
+// the range of all its rows need no mask. A grouped query may also see the first `keep` keys: their tiles come ahead of the others. In
+// a chunked layer its range starts where its chunk does.
 #include <cuda.h>
 #include <limits.h>
 
+#include "attn_spec.cuh"
 #include "common.cuh"
 #include "kvb200_layers.h"
 #include "tmap.cuh"
@@ -45,20 +49,19 @@ struct LfParams {
   int* status;
   const int* slots;          // grouped-query cache: slot of every row; NULL: keys and values of the pass
   int group;                 // query heads per key/value head
-  int sink;
-  const __nv_bfloat16* gate;  // (B, T, gate_ld), vdp columns per head, or NULL
+  const __nv_bfloat16* gate;  // (B, T, gate_ld), or NULL
   long long gate_ld;
+  float cap_in, cap_out;      // cap_out > 0: the score in log2 units is cap_out · tanh(cap_in · q·k), and scale_log2 is 1
+  kvb_attention a;            // masks, rows, sink, gate columns, difference
 };
 
-__device__ __forceinline__ float lf_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
+__device__ __forceinline__ float lf_exp2(float x) { return attn_exp2(x); }
+
+__device__ __forceinline__ void named_barrier(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 
 __device__ __forceinline__ float lf_sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
 
-template <int NQT>
+template <int NQT, bool DIFF>
 __global__ void __launch_bounds__(64 + 128 * NQT, 1)
 latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant__ CUtensorMap tmQr,
                     const __grid_constant__ CUtensorMap tmKu, const __grid_constant__ CUtensorMap tmKr,
@@ -69,9 +72,10 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     return;
   }
   const int nk = p.nu + p.nr;
+  constexpr int MAPS = DIFF ? 2 : 1;  // key tiles of a stage
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + NQT * nk * LF_CHUNK;
-  uint8_t* sV = sK + p.kst * nk * LF_CHUNK;
+  uint8_t* sV = sK + p.kst * MAPS * nk * LF_CHUNK;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sV + p.vst * p.nv * LF_CHUNK);
   uint64_t* q_full = bars;
   uint64_t* o_full = bars + 1;
@@ -91,17 +95,19 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
   const int P = p.slots ? p.start[b] : p.P;
   const int lo_seq = max(0, P - p.start[b]);  // first key row that holds a token
   const int hk = h / p.group, bk = p.slots ? p.slots[b] : b;  // where the keys and values are
+  auto first_query = [&](int u) { return (DIFF ? pair : pair * NQT + u) * LF_T; };
+  // first key that the query at key row hi sees, kept ones aside
+  auto seen = [&](int hi) { return max(lo_seq, p.a.chunk > 0 ? hi / p.a.chunk * p.a.chunk : p.window > 0 ? hi - p.window + 1 : 0); };
   // key tiles [ta, tb] of query tile u (empty if the tile has no query)
   auto range = [&](int u, int& ta, int& tb) {
-    const int t0 = (pair * NQT + u) * LF_T;
+    const int t0 = first_query(u);
     if (t0 >= p.T) {
       ta = INT_MAX;
       tb = -1;
       return;
     }
     const int t1 = min(t0 + LF_T, p.T) - 1;
-    const int lo = max(lo_seq, p.window > 0 ? P + t0 - p.window + 1 : 0);
-    ta = lo / LF_T;
+    ta = seen(P + t0) / LF_T;
     tb = (P + t1) / LF_T;
   };
   int ra[NQT], rb[NQT];
@@ -112,6 +118,21 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     first = min(first, ra[u]);
     last = max(last, rb[u]);
   }
+  // Tiles are counted as they are visited: `kept` ones from the start of the sequence, which every query tile visits, then those from
+  // `first` on; ra, rb, last are of that count from here on.
+  const int keep_tiles = (p.a.keep + LF_T - 1) / LF_T;
+  const int kept = last < 0 ? 0 : min(keep_tiles, first), skipped = first - kept;
+#pragma unroll
+  for (int u = 0; u < NQT; ++u) {
+    if (rb[u] < 0) continue;
+    if (first < keep_tiles) ra[u] = first;  // some of the kept keys lie behind `first`
+    ra[u] -= skipped;
+    rb[u] -= skipped;
+  }
+  if (last >= 0) last -= skipped;
+  auto tile_at = [&](int t) { return t < kept ? t : t + skipped; };
+  auto visits = [&](int u, int t) { return t >= 0 && t <= rb[u] && (t < kept || t >= ra[u]); };
+  auto starts = [&](int u) { return kept > 0 ? 0 : ra[u]; };  // first tile that query tile u visits
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
     mbar_init(o_full, 1);
@@ -143,33 +164,36 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     if (lane == 0) {
       tma_prefetch_desc(&tmQu);
       tma_prefetch_desc(&tmKu);
-      if (p.nr > 0) {
-        tma_prefetch_desc(&tmQr);
-        tma_prefetch_desc(&tmKr);
-      }
+      if (p.nr > 0) tma_prefetch_desc(&tmQr);
+      if (p.nr > 0 || DIFF) tma_prefetch_desc(&tmKr);
       tma_prefetch_desc(&tmV);
       mbar_expect_tx(q_full, (uint32_t)(NQT * nk * LF_CHUNK));
       for (int u = 0; u < NQT; ++u) {
-        const int t0 = (pair * NQT + u) * LF_T;  // beyond T: zero rows
-        for (int c = 0; c < p.nu; ++c) tma_load_4d(sQ + (u * nk + c) * LF_CHUNK, &tmQu, q_full, 64 * c, h, t0, b);
+        const int t0 = first_query(u);  // beyond T: zero rows
+        for (int c = 0; c < p.nu; ++c) tma_load_4d(sQ + (u * nk + c) * LF_CHUNK, &tmQu, q_full, 64 * c, DIFF ? 2 * h + u : h, t0, b);
         for (int c = 0; c < p.nr; ++c) tma_load_4d(sQ + (u * nk + p.nu + c) * LF_CHUNK, &tmQr, q_full, 64 * c, h, t0, b);
       }
       bool ok = true;
       int ks = 0, vs = 0;
       uint32_t kph = 0, vph = 0;
-      for (int t = first; t <= last; ++t) {
+      for (int t = 0; t <= last; ++t) {
+        const int krow = p.slots ? row_of(p.a, tile_at(t) * LF_T) : tile_at(t) * LF_T;
         if (!(ok = mbar_wait_bounded(&k_empty[ks], kph ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
-        mbar_expect_tx(&k_full[ks], (uint32_t)(nk * LF_CHUNK));
-        uint8_t* kd = sK + ks * nk * LF_CHUNK;
-        for (int c = 0; c < p.nu; ++c) tma_load_4d(kd + c * LF_CHUNK, &tmKu, &k_full[ks], 64 * c, hk, t * LF_T, bk);
-        for (int c = 0; c < p.nr; ++c) tma_load_4d(kd + (p.nu + c) * LF_CHUNK, &tmKr, &k_full[ks], 64 * c, 0, t * LF_T, b);
+        mbar_expect_tx(&k_full[ks], (uint32_t)(MAPS * nk * LF_CHUNK));
+        uint8_t* kd = sK + ks * MAPS * nk * LF_CHUNK;
+        for (int c = 0; c < p.nu; ++c) tma_load_4d(kd + c * LF_CHUNK, &tmKu, &k_full[ks], 64 * c, hk, krow, bk);
+        if (DIFF) {  // keys of the second map
+          for (int c = 0; c < p.nu; ++c) tma_load_4d(kd + (p.nu + c) * LF_CHUNK, &tmKr, &k_full[ks], 64 * c, hk, krow, bk);
+        } else {
+          for (int c = 0; c < p.nr; ++c) tma_load_4d(kd + (p.nu + c) * LF_CHUNK, &tmKr, &k_full[ks], 64 * c, 0, krow, b);
+        }
         if (++ks == p.kst) {
           ks = 0;
           kph ^= 1;
         }
         if (!(ok = mbar_wait_bounded(&v_empty[vs], vph ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
         mbar_expect_tx(&v_full[vs], (uint32_t)(p.nv * LF_CHUNK));
-        for (int c = 0; c < p.nv; ++c) tma_load_4d(sV + (vs * p.nv + c) * LF_CHUNK, &tmV, &v_full[vs], 64 * c, hk, t * LF_T, bk);
+        for (int c = 0; c < p.nv; ++c) tma_load_4d(sV + (vs * p.nv + c) * LF_CHUNK, &tmV, &v_full[vs], 64 * c, hk, krow, bk);
         if (++vs == p.vst) {
           vs = 0;
           vph ^= 1;
@@ -195,12 +219,12 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       uint32_t pph[NQT];
 #pragma unroll
       for (int u = 0; u < NQT; ++u) pph[u] = 0;
-      for (int t = first; t <= last + 1 && ok; ++t) {
-        const bool have_k = t <= last, have_v = t > first;
+      for (int t = 0; t <= last + 1 && ok; ++t) {
+        const bool have_k = t <= last, have_v = t > 0;
         bool k_ready = false, v_ready = false;
 #pragma unroll
         for (int u = 0; u < NQT; ++u) {
-          if (have_v && t - 1 >= ra[u] && t - 1 <= rb[u]) {
+          if (visits(u, t - 1)) {
             if (!v_ready) {
               if (!(ok = mbar_wait_bounded(&v_full[vs], vph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
               v_ready = true;
@@ -212,9 +236,9 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
             for (int kk = 0; kk < 8; ++kk)
               umma_f16_ts(tmem_base + (uint32_t)(NQT * LF_T + u * o_cols), tmem_base + (uint32_t)(u * LF_T + 8 * kk),
                           make_smem_desc_sw128(v_addr + (uint32_t)(vs * p.nv * LF_CHUNK + kk * 16 * 128), LF_CHUNK, 1024), idesc_pv,
-                          (t - 1 == ra[u] && kk == 0) ? 0u : 1u);
+                          (t - 1 == starts(u) && kk == 0) ? 0u : 1u);
           }
-          if (have_k && t >= ra[u] && t <= rb[u]) {
+          if (visits(u, t)) {
             if (!k_ready) {
               if (!(ok = mbar_wait_bounded(&k_full[ks], kph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
               k_ready = true;
@@ -225,14 +249,14 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
               const int kk = s < su ? (s & 3) : ((s - su) & 3);
               const uint32_t off = (uint32_t)(c * LF_CHUNK + kk * 32);
               umma_f16_ss(tmem_base + (uint32_t)(u * LF_T), make_smem_desc_sw128(q_addr + (uint32_t)(u * nk * LF_CHUNK) + off, 16, 1024),
-                          make_smem_desc_sw128(k_addr + (uint32_t)(ks * nk * LF_CHUNK) + off, 16, 1024), idesc_qk, s != 0 ? 1u : 0u);
+                          make_smem_desc_sw128(k_addr + (uint32_t)((ks * MAPS + (DIFF ? u : 0)) * nk * LF_CHUNK) + off, 16, 1024), idesc_qk, s != 0 ? 1u : 0u);
             }
             umma_commit(&s_full[u]);
           }
         }
         if (!ok) break;
         if (have_v) {
-          // a stage that no query tile of this CTA reads cannot occur between first and last: the ranges overlap or touch
+          // a tile that no query tile of this CTA visits cannot occur: the ranges overlap or touch
           umma_commit(&v_empty[vs]);
           if (!v_ready && !(ok = mbar_wait_bounded(&v_full[vs], vph, abort_flag, p.status, STATUS_TIMEOUT_FULL))) break;
           if (++vs == p.vst) {
@@ -256,22 +280,25 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     const int u = NQT == 1 ? 0 : (warp - 2) >> 2;
     const int quarter = warp & 3;
     const int row = quarter * 32 + lane;
-    const int t0 = (pair * NQT + u) * LF_T;
+    const int t0 = first_query(u);
     const int tq = t0 + row;
     const int my_ra = u == 0 ? ra[0] : ra[NQT - 1], my_rb = u == 0 ? rb[0] : rb[NQT - 1];
+    const int my_start = kept > 0 ? 0 : my_ra;
     const int hi = P + tq;
-    const int lo = max(lo_seq, p.window > 0 ? hi - p.window + 1 : 0);
-    // rows of the tile: all see keys in [lo of the last row, hi of the first row]
-    const int lo_max = max(lo_seq, p.window > 0 ? P + t0 + LF_T - 1 - p.window + 1 : 0), hi_min = P + t0;
+    const int lo = seen(hi);
+    // rows of the tile: all see keys in [lo of the last row, hi of the first row] and the kept ones up to the first row
+    const int lo_max = seen(P + t0 + LF_T - 1), hi_min = P + t0;
+    const int keep = min(p.a.keep, hi + 1);
     const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
     const uint32_t tmem_S = tmem_base + (uint32_t)(u * LF_T) + lane_base;
     const uint32_t tmem_O = tmem_base + (uint32_t)(NQT * LF_T + u * o_cols) + lane_base;
     const float c = p.scale_log2;
     const float2 c2 = make_float2(c, c);
-    float m_used = p.sink ? 0.f : -1e30f, l = p.sink ? 1.f : 0.f;
+    float m_used = !p.a.sink ? -1e30f : p.a.sink_w ? p.a.sink_w[h] * ATTN_LOG2E : 0.f, l = p.a.sink ? 1.f : 0.f;
     bool ok = true;
     uint32_t ph = 0;
-    for (int t = my_ra; t <= my_rb; ++t) {
+    for (int t = my_start; t <= my_rb; ++t) {
+      if (t >= kept && t < my_ra) continue;
       if (!(ok = mbar_wait_bounded(&s_full[u], ph, abort_flag, p.status, STATUS_TIMEOUT_TMEM_FULL))) break;
       ph ^= 1;
       tc_fence_after();
@@ -279,13 +306,38 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
 #pragma unroll
       for (int w = 0; w < 4; ++w) tmem_ld_32x32b_x32(tmem_S + (uint32_t)(32 * w), x + 32 * w);
       tmem_ld_wait();
-      const int j0 = t * LF_T;
-      if (j0 < lo_max || j0 + LF_T - 1 > hi_min) {
+      if (p.cap_out > 0.f) {
+        // scores well below the cap take the series, others (any of the warp's) the exponential
+        const float2 ci = make_float2(p.cap_in, p.cap_in), co = make_float2(p.cap_out, p.cap_out);
+        float top = 0.f;
+#pragma unroll
+        for (int e = 0; e < LF_T; e += 2) top = fmax3(top, fabsf(__uint_as_float(x[e])), fabsf(__uint_as_float(x[e + 1])));
+        if (__any_sync(0xffffffffu, !(top * p.cap_in <= CAP_SERIES))) {
+#pragma unroll
+          for (int e = 0; e < LF_T; ++e) x[e] = __float_as_uint(p.cap_out * cap_tanh(__uint_as_float(x[e]) * p.cap_in));
+        } else {
+#pragma unroll
+          for (int e = 0; e < LF_T; e += 2) {
+            const float2 y = fmul2(cap_tanh_series(fmul2(make_float2(__uint_as_float(x[e]), __uint_as_float(x[e + 1])), ci)), co);
+            x[e] = __float_as_uint(y.x);
+            x[e + 1] = __float_as_uint(y.y);
+          }
+        }
+      }
+      const int j0 = tile_at(t) * LF_T;
+      if (j0 + LF_T - 1 > hi_min || (j0 < lo_max && j0 + LF_T > p.a.keep)) {
         const uint32_t span = (uint32_t)(hi - lo);
         const uint32_t off = (uint32_t)(j0 - lo);
+        const int keep_here = keep - j0;
+        if (keep_here <= 0) {
 #pragma unroll
-        for (int e = 0; e < LF_T; ++e)
-          if (off + (uint32_t)e > span) x[e] = 0xff800000u;
+          for (int e = 0; e < LF_T; ++e)
+            if (off + (uint32_t)e > span) x[e] = 0xff800000u;
+        } else {
+#pragma unroll
+          for (int e = 0; e < LF_T; ++e)
+            if (off + (uint32_t)e > span && e >= keep_here) x[e] = 0xff800000u;
+        }
       }
       float a8[8];
 #pragma unroll
@@ -300,7 +352,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       // the PV product of the previous tile was issued before this tile's scores: it is complete, O is quiet
       const float f = raise ? lf_exp2(m_used - m_new) : 1.f;
       l *= f;  // at the first tile the sink, if there is one
-      if (t > my_ra && __any_sync(0xffffffffu, raise)) {
+      if (t > my_start && __any_sync(0xffffffffu, raise)) {
 #pragma unroll 1
         for (int c0 = 0; c0 < o_cols; c0 += 16) {
           uint32_t o[16];
@@ -339,9 +391,50 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       if (lane == 0) mbar_arrive(&p_full[u]);
     }
     if (ok) ok = mbar_wait_bounded(o_full, 0, abort_flag, p.status, STATUS_TIMEOUT_TMEM_FULL);
-    if (ok && my_rb >= my_ra) {
+    if (DIFF) {
+      // both warpgroups: half of the columns each, of the same rows of both outputs
+      __shared__ float s_l[2][LF_T], s_ss[2][LF_T];
+      s_l[u][row] = l;
+      named_barrier(1, 256);
       tc_fence_after();
-      const float inv_l = l > 0.f ? 1.f / l : 0.f;
+      const uint32_t o0 = tmem_base + (uint32_t)(NQT * LF_T) + lane_base, o1 = o0 + (uint32_t)o_cols;
+      const float f0 = 1.f / s_l[0][row], f1 = -p.a.lambda / s_l[1][row];
+      const int half = o_cols / 2, c_begin = u * half;  // 32 or 64 columns
+      float d[64];
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        if (16 * k >= half) break;
+        uint32_t y0[16], y1[16];
+        tmem_ld_32x32b_x16(o0 + (uint32_t)(c_begin + 16 * k), y0);
+        tmem_ld_32x32b_x16(o1 + (uint32_t)(c_begin + 16 * k), y1);
+        tmem_ld_wait();
+#pragma unroll
+        for (int e = 0; e < 16; ++e) {
+          d[16 * k + e] = fmaf(__uint_as_float(y1[e]), f1, __uint_as_float(y0[e]) * f0);  // zero in the padding
+          ss = fmaf(d[16 * k + e], d[16 * k + e], ss);
+        }
+      }
+      s_ss[u][row] = ss;
+      named_barrier(1, 256);
+      const float r = p.a.post / sqrtf((s_ss[0][row] + s_ss[1][row]) / (float)p.a.vdim + p.a.eps);
+      __nv_bfloat16* dst = p.out + (((long long)b * p.T + (tq < p.T ? tq : 0)) * p.heads + h) * p.vdp;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int c = c_begin + 8 * k;
+        if (8 * k >= half || c >= p.vdp || tq >= p.T || !ok) break;
+        uint4 v;
+        v.x = pack_bf16x2(d[8 * k + 0] * r, d[8 * k + 1] * r);
+        v.y = pack_bf16x2(d[8 * k + 2] * r, d[8 * k + 3] * r);
+        v.z = pack_bf16x2(d[8 * k + 4] * r, d[8 * k + 5] * r);
+        v.w = pack_bf16x2(d[8 * k + 6] * r, d[8 * k + 7] * r);
+        *reinterpret_cast<uint4*>(dst + c) = v;
+      }
+    } else if (ok && my_rb >= my_ra) {
+      tc_fence_after();
+      float inv_l = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate && p.a.gate_cols == 1 && tq < p.T)  // one number per head
+        inv_l *= lf_sigmoid(__bfloat162float(p.gate[((long long)b * p.T + tq) * p.gate_ld + h]));
       __nv_bfloat16* dst = p.out + (((long long)b * p.T + (tq < p.T ? tq : 0)) * p.heads + h) * p.vdp;
 #pragma unroll 1
       for (int c0 = 0; c0 < p.vdp; c0 += 16) {
@@ -352,7 +445,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
 #pragma unroll
           for (int i = 0; i < 2; ++i) {
             if (c0 + 8 * i >= p.vdp) break;
-            if (p.gate) {
+            if (p.gate && p.a.gate_cols > 1) {
               const uint4 g = *reinterpret_cast<const uint4*>(p.gate + ((long long)b * p.T + tq) * p.gate_ld + h * p.vdp + c0 + 8 * i);
               const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
@@ -387,7 +480,7 @@ struct LfPlan {
 };
 
 // query tiles per CTA and stages that fit into shared and tensor memory; nqt = 0: not supported
-static LfPlan lf_plan(int dimp, int rp, int vdp) {
+static LfPlan lf_plan(int dimp, int rp, int vdp, int maps = 1) {
   LfPlan pl;
   pl.nqt = 0;
   pl.nu = (dimp + 63) / 64;
@@ -395,13 +488,13 @@ static LfPlan lf_plan(int dimp, int rp, int vdp) {
   pl.nv = (vdp + 63) / 64;
   const int nk = pl.nu + pl.nr;
   if (dimp <= 0 || rp < 0 || vdp <= 0 || pl.nv > 4) return pl;
-  const int limit = LF_SMEM_LIMIT - 512;
+  const int limit = LF_SMEM_LIMIT - 512 - (maps == 2 ? 2048 : 0);
   for (int nqt = 2; nqt >= 1; --nqt) {
-    if (nqt * (LF_T + 64 * pl.nv) > 512) continue;
-    static const int stages[][2] = {{3, 3}, {2, 2}, {2, 1}, {1, 1}};
+    if (nqt * (LF_T + 64 * pl.nv) > 512 || nqt < maps) continue;
+    static const int stages[][2] = {{3, 3}, {2, 2}, {2, 1}, {1, 2}, {1, 1}};
     for (auto& st : stages) {
-      const int bytes = (nqt * nk + st[0] * nk + st[1] * pl.nv) * LF_CHUNK;
-      if (bytes > limit || (nqt == 2 && st[0] == 1)) continue;
+      const int bytes = (nqt * nk + st[0] * maps * nk + st[1] * pl.nv) * LF_CHUNK;
+      if (bytes > limit || (nqt == 2 && maps == 1 && st[0] == 1)) continue;
       pl.nqt = nqt;
       pl.kst = st[0];
       pl.vst = st[1];
@@ -412,12 +505,13 @@ static LfPlan lf_plan(int dimp, int rp, int vdp) {
   return pl;
 }
 
-template <int NQT>
+template <int NQT, bool DIFF>
 static int lf_launch(const CUtensorMap* tm, LfParams& p, int smem, cudaStream_t s) {
   static PerDeviceOnce once;
-  if (once.first()) cudaFuncSetAttribute(latent_flash_kernel<NQT>, cudaFuncAttributeMaxDynamicSharedMemorySize, LF_SMEM_LIMIT);
-  p.n_pair = (p.nQ + NQT - 1) / NQT;
-  latent_flash_kernel<NQT><<<p.B * p.heads * p.n_pair, 64 + 128 * NQT, smem, s>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  if (once.first())
+    cudaFuncSetAttribute(latent_flash_kernel<NQT, DIFF>, cudaFuncAttributeMaxDynamicSharedMemorySize, LF_SMEM_LIMIT - (DIFF ? 2048 : 0));
+  p.n_pair = DIFF ? p.nQ : (p.nQ + NQT - 1) / NQT;
+  latent_flash_kernel<NQT, DIFF><<<p.B * p.heads * p.n_pair, 64 + 128 * NQT, smem, s>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
@@ -460,26 +554,27 @@ extern "C" int kvb_latent_attend_tc(const void* q, const void* kv, const void* l
   p.ksu_last = (dimp - 64 * (pl.nu - 1) + 15) / 16;
   p.ksr = (rp + 15) / 16;
   p.vdp = vdp; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
-  p.slots = nullptr; p.group = 1; p.sink = 0; p.gate = nullptr; p.gate_ld = 0;
-  return pl.nqt == 2 ? lf_launch<2>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1>(tm, p, pl.smem, (cudaStream_t)stream);
+  p.slots = nullptr; p.group = 1; p.gate = nullptr; p.gate_ld = 0; p.cap_in = p.cap_out = 0.f; p.a = kvb_attention{};
+  return pl.nqt == 2 ? lf_launch<2, false>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1, false>(tm, p, pl.smem, (cudaStream_t)stream);
 }
 
-extern "C" int kvb_grouped_attend_tc_supported(int dimp, int vdp) {
-  return (dimp % 8 == 0 && vdp % 8 == 0 && kvb::lf_plan(dimp, 0, vdp).nqt > 0) ? 1 : 0;
+extern "C" int kvb_grouped_attend_tc_supported(const kvb_attention* a) {
+  return (a->dimp % 8 == 0 && a->vdp % 8 == 0 && kvb::lf_plan(a->dimp, 0, a->vdp, a->maps).nqt > 0) ? 1 : 0;
 }
 
 extern "C" int kvb_grouped_attend_tc(const void* q, const void* rows, const void* gate, long long gate_ld, void* out, const int* slots,
-                                     const int* start, int B, int T, int n_slots, int len, int heads, int kv_heads, int dimp, int vdp,
-                                     int sink, float scale, int* status, void* stream) {
+                                     const int* start, int B, int T, int n_slots, int len, const kvb_attention* a, int* status, void* stream) {
   using namespace kvb;
-  if (B <= 0 || T <= 0 || n_slots <= 0 || len <= 0 || kv_heads <= 0 || heads % kv_heads || !(scale > 0.f)) return KVB_ERR_ARG;
-  if ((dimp | vdp) % 8 || (gate && gate_ld % 8)) return KVB_ERR_ALIGN;
-  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(gate) |
-       reinterpret_cast<uintptr_t>(out)) & 15)
-    return KVB_ERR_ALIGN;
-  const LfPlan pl = lf_plan(dimp, 0, vdp);
+  if (!a || B <= 0 || T <= 0 || n_slots <= 0 || len <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || !(a->scale > 0.f) ||
+      (a->maps != 1 && a->maps != 2) || (a->maps == 2 && (a->sink || gate)) || (a->window && a->chunk) || (a->keep && !a->window) ||
+      a->head % LF_T || a->ring % LF_T || (a->ring && (a->head < a->keep || a->head + a->ring > len)))
+    return KVB_ERR_ARG;
+  const int dimp = a->dimp, vdp = a->vdp, maps = a->maps;
+  if ((dimp | vdp) % 8 || (gate && a->gate_cols > 1 && (gate_ld % 8 || reinterpret_cast<uintptr_t>(gate) & 15))) return KVB_ERR_ALIGN;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(out)) & 15) return KVB_ERR_ALIGN;
+  const LfPlan pl = lf_plan(dimp, 0, vdp, maps);
   if (!pl.nqt) return KVB_ERR_UNSUPPORTED;
-  const uint64_t dq = dimp, row = dimp + vdp, H = heads, G = kv_heads;
+  const uint64_t dq = dimp, row = maps * dimp + vdp, H = a->heads * maps, G = a->kv_heads;
   const uint32_t box[4] = {64, 1, LF_T, 1};
   CUtensorMap tm[5];
   int rc;
@@ -490,16 +585,21 @@ extern "C" int kvb_grouped_attend_tc(const void* q, const void* rows, const void
   const uint64_t dku[4] = {dq, G, (uint64_t)len, (uint64_t)n_slots}, dv[4] = {(uint64_t)vdp, G, (uint64_t)len, (uint64_t)n_slots};
   if ((rc = tmap_bf16(&tm[0], q, 4, dqu, sq, box))) return rc;
   if ((rc = tmap_bf16(&tm[2], kb, 4, dku, sk, box))) return rc;
-  if ((rc = tmap_bf16(&tm[4], kb + dimp, 4, dv, sk, box))) return rc;
+  if ((rc = tmap_bf16(&tm[3], kb + (maps - 1) * dimp, 4, dku, sk, box))) return rc;  // one map: never used
+  if ((rc = tmap_bf16(&tm[4], kb + maps * dimp, 4, dv, sk, box))) return rc;
   tm[1] = tm[0];  // no shared part: never used
-  tm[3] = tm[2];
   LfParams p;
   p.out = (__nv_bfloat16*)out; p.start = start;
-  p.B = B; p.heads = heads; p.T = T; p.P = 0; p.nQ = (T + LF_T - 1) / LF_T;
+  p.B = B; p.heads = a->heads; p.T = T; p.P = 0; p.nQ = (T + LF_T - 1) / LF_T;
   p.nu = pl.nu; p.nr = 0; p.nv = pl.nv; p.kst = pl.kst; p.vst = pl.vst;
   p.ksu_last = (dimp - 64 * (pl.nu - 1) + 15) / 16;
   p.ksr = 0;
-  p.vdp = vdp; p.window = 0; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
-  p.slots = slots; p.group = heads / kv_heads; p.sink = sink; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld;
-  return pl.nqt == 2 ? lf_launch<2>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1>(tm, p, pl.smem, (cudaStream_t)stream);
+  p.vdp = vdp; p.window = a->window; p.status = status;
+  p.cap_in = a->softcap > 0.f ? a->scale / a->softcap : 0.f;
+  p.cap_out = a->softcap * ATTN_LOG2E;
+  p.scale_log2 = a->softcap > 0.f ? 1.f : a->scale * ATTN_LOG2E;
+  p.slots = slots; p.group = a->heads / a->kv_heads; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld; p.a = *a;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (maps == 2) return lf_launch<2, true>(tm, p, pl.smem, s);
+  return pl.nqt == 2 ? lf_launch<2, false>(tm, p, pl.smem, s) : lf_launch<1, false>(tm, p, pl.smem, s);
 }

@@ -1,9 +1,11 @@
-// Routed experts: softmax router with top-k choice, rows sorted by expert, grouped products.
+// Routed experts: softmax or sigmoid router with top-k choice, rows sorted by expert, grouped products.
 //
-//   route  one warp per token: softmax over the fp32 router logits, the k largest, a rank within every chosen expert;
+//   route  one warp per token: scores from the fp32 router logits; the k largest, with a correction that only the choice sees and out of
+//          the best groups of neighbouring experts, if the router has these; a rank within every chosen expert;
 //   plan   one CTA: rows of an expert start at a multiple of the row tile; table of tiles for the grouped products;
 //   gather rows of the chosen tokens into the sorted buffer;
-//   gemm   out = act(W_e · in) per tile of rows of one expert. bf16: tcgen05 with the expert's weight rows as the
+//   gemm   out = act(W_e · in) per tile of rows of one expert; a gated unit has the rows of gate and up projection in turns, so
+//          that silu(gate) · up is part of the product. bf16: tcgen05 with the expert's weight rows as the
 //          M = 128 operand and the tokens as N (16 .. 256 columns), so that a decode step with a handful of tokens per
 //          expert streams the weights without padding the token side to 128; fp32: CUDA cores.
 // The weighted sum over a token's experts is part of the kernel that closes the layer (layer_edge.cu).
@@ -19,35 +21,53 @@ constexpr int ROUTE_MAX_EXPERTS = 2048;
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ logits, int* __restrict__ expert, float* __restrict__ weight, int* __restrict__ row,
-                 int* __restrict__ counters, long long n, int E, int top, int renormalize) {
+                 int* __restrict__ counters, long long n, int E, int top, const kvb_router r) {
   extern __shared__ float sc_all[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* sc = sc_all + warp * E;
+  float* sc = sc_all + warp * (E + r.groups);  // choice scores; scores of the groups
+  float* gs = sc + E;
   const long long tok = (long long)blockIdx.x * ROUTE_WARPS + warp;
   if (tok >= n) return;
   const float* z = logits + tok * E;
-  float m = -INFINITY;
-  for (int e = lane; e < E; e += 32) {
-    const float v = z[e];
-    sc[e] = v;
-    m = fmaxf(m, v);
+  float m = 0.f, l = 1.f;  // softmax: score = exp(z - m) / l
+  if (r.score == 0) {
+    m = -INFINITY;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    l = 0.f;
+    for (int e = lane; e < E; e += 32) l += expf(z[e] - m);
+    l = warp_sum(l);
   }
-  m = warp_max(m);
-  float l = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float v = expf(sc[e] - m);
-    sc[e] = v;
-    l += v;
-  }
-  l = warp_sum(l);
+  auto score = [&](int e) { return r.score == 0 ? expf(z[e] - m) / l : 1.f / (1.f + expf(-z[e])); };
+  for (int e = lane; e < E; e += 32) sc[e] = score(e) + (r.correction ? r.correction[e] : 0.f);
   __syncwarp();
+  if (r.groups > 1) {
+    const int size = E / r.groups;
+    for (int g = lane; g < r.groups; g += 32) {  // sum of the two largest
+      float a = -INFINITY, b = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float v = sc[e];
+        b = fmaxf(b, fminf(a, v));
+        a = fmaxf(a, v);
+      }
+      gs[g] = size > 1 ? a + b : a;
+    }
+    __syncwarp();
+    for (int g = lane; g < r.groups; g += 32) {
+      int ahead = 0;  // groups that come before this one; ties: lower index first
+      for (int o = 0; o < r.groups; ++o) ahead += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+      if (ahead >= r.keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) sc[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
   float chosen = 0.f;
   for (int k = 0; k < top; ++k) {
-    float best = -2.f;
+    float best = -INFINITY;
     int bi = 0x7fffffff;
     for (int e = lane; e < E; e += 32) {
       const float v = sc[e];
-      if (v > best) {
+      if (v > best) {  // those that cannot be chosen are at minus infinity
         best = v;
         bi = e;
       }
@@ -62,18 +82,18 @@ moe_route_kernel(const float* __restrict__ logits, int* __restrict__ expert, flo
       }
     }
     if (bi >= E) bi = 0;  // scores that are not numbers: any expert
-    const float w = best / l;
+    const float w = score(bi);
     chosen += w;
     if (lane == 0) {
       expert[tok * top + k] = bi;
       weight[tok * top + k] = w;
       row[tok * top + k] = atomicAdd(&counters[bi], 1);
-      sc[bi] = -1.f;
+      sc[bi] = -INFINITY;
     }
     __syncwarp();
   }
-  if (renormalize && lane < top)
-    for (int k = lane; k < top; k += 32) weight[tok * top + k] = weight[tok * top + k] / chosen;
+  if (r.renormalize)
+    for (int k = lane; k < top; k += 32) weight[tok * top + k] = weight[tok * top + k] / (chosen + r.eps);
 }
 
 // Exclusive prefix over the experts' tile counts, tile table. One CTA of 1024 threads.
@@ -143,6 +163,8 @@ moe_gather_kernel(const T* __restrict__ h, const int* __restrict__ row, T* __res
   }
 }
 
+__device__ __forceinline__ float moe_glu(float gate, float up) { return gate / (1.f + expf(-gate)) * up; }
+
 __device__ __forceinline__ float moe_act(float v, int act) {
   if (act == 1) {
     v = fmaxf(v, 0.f);
@@ -151,7 +173,7 @@ __device__ __forceinline__ float moe_act(float v, int act) {
   return v;
 }
 
-// ---- CUDA-core product: 32 rows x 64 features per CTA
+// ---- CUDA-core product: 32 rows x 64 features per CTA. act 2: features 2 f and 2 f + 1 are gate and up of result f
 constexpr int MS_R = 32, MS_F = 64, MS_K = 32;
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -167,7 +189,7 @@ moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __r
   const long long e = tile_expert[ti];
   const int f0 = blockIdx.y * MS_F;
   const T* we = w + e * n_out * ldk;
-  const int tr = threadIdx.x / 32, tf = threadIdx.x % 32;  // rows tr + 8 i, features tf and tf + 32
+  const int tr = threadIdx.x / 32, tf = threadIdx.x % 32;  // rows tr + 8 i, features 2 tf and 2 tf + 1
   float acc[4][2] = {};
   for (int k0 = 0; k0 < k; k0 += MS_K) {
     for (int i = threadIdx.x; i < MS_R * MS_K; i += 256) {
@@ -181,7 +203,7 @@ moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __r
     __syncthreads();
 #pragma unroll 8
     for (int kk = 0; kk < MS_K; ++kk) {
-      const float w0 = sw[kk][tf], w1 = sw[kk][tf + 32];
+      const float w0 = sw[kk][2 * tf], w1 = sw[kk][2 * tf + 1];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const float a = sa[kk][tr + 8 * i];
@@ -191,13 +213,54 @@ moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __r
     }
     __syncthreads();
   }
+  if (act == 2) {
+    const int f = f0 / 2 + tf;
+    if (f < ldo) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) out[(r0 + tr + 8 * i) * ldo + f] = from_f32<T>(2 * f < n_out ? moe_glu(acc[i][0], acc[i][1]) : 0.f);
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
-      const int f = f0 + tf + 32 * j;
+      const int f = f0 + 2 * tf + j;
       if (f < ldo) out[(r0 + tr + 8 * i) * ldo + f] = from_f32<T>(f < n_out ? moe_act(acc[i][j], act) : 0.f);
     }
+}
+
+// out[n, c] = silu(x[n, c]) · x[n, up + c], zero in the columns from ff to ldo
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long n, long long ldx, int up, int ff, int ldo) {
+  struct alignas(sizeof(T) * V) Vec { T v[V]; };
+  const int per = ldo / V;
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  const long long r = i / per;
+  if (r >= n) return;
+  const int c = (int)(i - r * per) * V;
+  Vec y;
+  if (c < ff) {
+    const Vec g = *reinterpret_cast<const Vec*>(x + r * ldx + c), u = *reinterpret_cast<const Vec*>(x + r * ldx + up + c);
+#pragma unroll
+    for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(moe_glu(to_f32(g.v[e]), to_f32(u.v[e])));
+  } else {
+#pragma unroll
+    for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(0.f);
+  }
+  *reinterpret_cast<Vec*>(out + r * ldo + c) = y;
+}
+
+template <typename T>
+static int glu_launch(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  if (ff % V == 0 && up % V == 0 && ldx % V == 0 && ldo % V == 0) {
+    glu_kernel<T, V><<<(unsigned)((n * (ldo / V) + 255) / 256), 256, 0, s>>>((const T*)x, (T*)out, n, ldx, up, ff, ldo);
+  } else {
+    glu_kernel<T, 1><<<(unsigned)((n * ldo + 255) / 256), 256, 0, s>>>((const T*)x, (T*)out, n, ldx, up, ff, ldo);
+  }
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
 int moe_gemm_tc(const void* in, const void* w, void* out, const int* plan, const int* tile_expert, const int* tile_row, int tile,
@@ -206,14 +269,17 @@ int moe_gemm_tc(const void* in, const void* w, void* out, const int* plan, const
 }  // namespace kvb
 
 extern "C" int kvb_moe_route(const float* logits, int* expert, float* weight, int* row, int* counters, int* plan, int* tile_expert,
-                             int* tile_row, long long n, int n_expert, int top, int tile, int max_tiles, int renormalize, void* stream) {
+                             int* tile_row, long long n, int n_expert, int top, int tile, int max_tiles, const kvb_router* router, void* stream) {
   using namespace kvb;
-  if (n <= 0 || n_expert <= 0 || top <= 0 || top > n_expert || tile <= 0) return KVB_ERR_ARG;
+  if (n <= 0 || n_expert <= 0 || top <= 0 || top > n_expert || tile <= 0 || !router) return KVB_ERR_ARG;
+  const kvb_router r = *router;
+  if (r.groups < 1 || n_expert % r.groups || r.keep < 1 || r.keep > r.groups || r.keep * (n_expert / r.groups) < top || r.score < 0 || r.score > 1)
+    return KVB_ERR_ARG;
   if (n_expert > ROUTE_MAX_EXPERTS) return KVB_ERR_TOO_LARGE;
   cudaStream_t s = (cudaStream_t)stream;
   if (cudaMemsetAsync(counters, 0, sizeof(int) * n_expert, s) != cudaSuccess) return KVB_ERR_CUDA;
-  moe_route_kernel<<<(unsigned)((n + ROUTE_WARPS - 1) / ROUTE_WARPS), ROUTE_WARPS * 32, ROUTE_WARPS * n_expert * sizeof(float), s>>>(
-      logits, expert, weight, row, counters, n, n_expert, top, renormalize);
+  moe_route_kernel<<<(unsigned)((n + ROUTE_WARPS - 1) / ROUTE_WARPS), ROUTE_WARPS * 32, ROUTE_WARPS * (n_expert + r.groups) * sizeof(float), s>>>(
+      logits, expert, weight, row, counters, n, n_expert, top, r);
   moe_plan_kernel<<<1, 1024, 0, s>>>(counters, plan, tile_expert, tile_row, n_expert, tile, max_tiles);
   const long long m = n * top;
   moe_rows_kernel<<<(unsigned)((m + 255) / 256), 256, 0, s>>>(expert, counters, row, m);
@@ -243,12 +309,14 @@ extern "C" int kvb_moe_gemm(const void* in, const void* w, void* out, const int*
                             int tile, int max_tiles, int n_expert, int n_out, int k, long long ldk, long long ldo, int act, int dtype,
                             int simple, int* status, void* stream) {
   using namespace kvb;
-  if (max_tiles <= 0 || n_out <= 0 || k <= 0 || ldk < k || ldo < n_out || tile <= 0) return KVB_ERR_ARG;
+  if (max_tiles <= 0 || n_out <= 0 || k <= 0 || ldk < k || ldo < (act == 2 ? n_out / 2 : n_out) || tile <= 0 || (act == 2 && n_out % 2))
+    return KVB_ERR_ARG;
   cudaStream_t s = (cudaStream_t)stream;
   if (dtype == 1 && !simple)
     return moe_gemm_tc(in, w, out, plan, tile_expert, tile_row, tile, max_tiles, n_expert, n_out, k, ldk, ldo, act, status, s);
   if (tile % MS_R) return KVB_ERR_ARG;
-  const dim3 grid(max_tiles * (tile / MS_R), (unsigned)((ldo + MS_F - 1) / MS_F));
+  const long long features = act == 2 ? 2 * ldo : ldo;
+  const dim3 grid(max_tiles * (tile / MS_R), (unsigned)((features + MS_F - 1) / MS_F));
   if (dtype == 0)
     moe_gemm_simple_kernel<float><<<grid, 256, 0, s>>>((const float*)in, (const float*)w, (float*)out, plan, tile_expert, tile_row, tile,
                                                        n_out, k, ldk, ldo, act);
@@ -257,4 +325,11 @@ extern "C" int kvb_moe_gemm(const void* in, const void* w, void* out, const int*
                                                                plan, tile_expert, tile_row, tile, n_out, k, ldk, ldo, act);
   else return KVB_ERR_ARG;
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+extern "C" int kvb_glu(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, int dtype, void* stream) {
+  if (n <= 0 || ff <= 0 || up < ff || ldx < up + ff || ldo < ff || n * ldo > 0x7fffffffLL * 256) return KVB_ERR_ARG;
+  if (dtype == 0) return kvb::glu_launch<float>(x, out, n, ldx, up, ff, ldo, (cudaStream_t)stream);
+  if (dtype == 1) return kvb::glu_launch<__nv_bfloat16>(x, out, n, ldx, up, ff, ldo, (cudaStream_t)stream);
+  return KVB_ERR_ARG;
 }

@@ -5,7 +5,8 @@
 // tiles, a decode step with a few tokens per expert streams each weight once without padding the tokens to 128 rows.
 // Persistent CTAs over a device-side tile table (token tile, expert), the structure of the plain GEMM of this package:
 // warp 0 TMA producer (ring of 128B-swizzled stages), warp 1 MMA issuer with a double-buffered accumulator in TMEM,
-// warps 2..5 epilogue (activation, bf16, stores of two tokens per instruction).
+// warps 2..5 epilogue (activation, bf16, stores of two tokens per instruction). In a gated unit (act 2) weight rows 2 f and 2 f + 1 are
+// gate and up projection of result f: neighbouring lanes exchange what the other needs and each has silu(gate) · up of every other token.
 #include <cuda.h>
 
 #include "common.cuh"
@@ -138,7 +139,31 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
       const int f = f0 + quarter * 32 + lane;       // this lane's feature
       const int fp = f & ~1;                        // feature pair it stores: even lanes token c, odd lanes token c + 1
       __nv_bfloat16* dst = p.out + (row0 + (lane & 1)) * p.ldo + fp;
-      if (f0 + quarter * 32 < p.ldo) {
+      if (p.act == 2) {
+        const int fo = ((f0 + quarter * 32 + lane) >> 2) * 2;  // pair of results that four lanes make; of 4 tokens, this lane stores one
+        if ((f0 + quarter * 32) / 2 < p.ldo) {
+          __nv_bfloat16* d2 = p.out + (row0 + (lane & 1) + (lane & 2)) * p.ldo + fo;
+          for (int c0 = 0; c0 < p.tile; c0 += 16) {
+            uint32_t r[16];
+            tmem_ld_32x32b_x16(taddr + (uint32_t)c0, r);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; i += 4) {
+              float y[2];  // of tokens i and i + 2, odd lanes i + 1 and i + 3
+#pragma unroll
+              for (int k = 0; k < 2; ++k) {
+                const float a = __uint_as_float(r[i + 2 * k]), b = __uint_as_float(r[i + 2 * k + 1]);
+                const float got = __shfl_xor_sync(0xffffffffu, (lane & 1) ? a : b, 1);
+                const float gate = (lane & 1) ? got : a, up = (lane & 1) ? b : got;
+                y[k] = f < p.n_out ? __fdividef(gate, 1.f + __expf(-gate)) * up : 0.f;
+              }
+              const float got = __shfl_xor_sync(0xffffffffu, (lane & 2) ? y[0] : y[1], 2);
+              const uint32_t w = (lane & 2) ? pack_bf16x2(got, y[1]) : pack_bf16x2(y[0], got);
+              if (fo < p.ldo) *reinterpret_cast<uint32_t*>(d2 + (long long)(c0 + i) * p.ldo) = w;
+            }
+          }
+        }
+      } else if (f0 + quarter * 32 < p.ldo) {
         for (int c0 = 0; c0 < p.tile; c0 += 16) {
           uint32_t r[16];
           tmem_ld_32x32b_x16(taddr + (uint32_t)c0, r);

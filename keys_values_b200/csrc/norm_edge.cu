@@ -1,7 +1,7 @@
-// What happens between two sublayers of a model whose layers have a norm before and after each sublayer, in one pass over
-// the fp32 residual stream: norm of the sublayer's output, residual sum, what a loop adds ahead of a pass (embedding row of
-// the token, a vector), norm for the next sublayer. Also the entry into the stack (embedding rows only) and the norm of
-// rows in front of the output head.
+// What happens between two sublayers of a model whose layers have norms before and / or after each sublayer, in one pass over
+// the fp32 residual stream: weighted sum of a token's routed experts, norm of the sublayer's output, residual sum, what a loop adds
+// ahead of a pass (embedding row of the token, a vector), norm for the next sublayer (or the stream itself, where sublayers read
+// that). Also the entry into the stack (embedding rows only) and the norm of rows in front of the output head.
 //
 // A CTA has one row, which stays in registers; means and squared deviations are separate sums (no cancellation).
 #include "common.cuh"
@@ -20,6 +20,11 @@ struct NormEdgeParams {
   const void* embed;
   long long vocab;
   const float* step;
+  const void* expert_out;
+  const int* expert_row;
+  const float* expert_w;
+  long long expert_ld;
+  int top;
   int width;
   float eps, inv_width;
   int* status;
@@ -102,6 +107,19 @@ norm_edge_kernel(const NormEdgeParams p) {
     if (p.sub) RowVec<T, V>::load(static_cast<const T*>(p.sub) + o + c, y[i]);
     if (p.x_in) RowVec<float, V>::load(p.x_in + o + c, x[i]);
   }
+  for (int k = 0; k < p.top; ++k) {
+    const T* src = static_cast<const T*>(p.expert_out) + (long long)p.expert_row[n * p.top + k] * p.expert_ld;
+    const float w = p.expert_w[n * p.top + k];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = (i * TH + threadIdx.x) * V;
+      if (c >= p.width) continue;
+      float e[V];
+      RowVec<T, V>::load(src + c, e);
+#pragma unroll
+      for (int j = 0; j < V; ++j) y[i][j] = fmaf(w, e[j], y[i][j]);
+    }
+  }
   long long tok = 0;
   if (p.embed) {
     tok = p.idx[n];
@@ -137,7 +155,15 @@ norm_edge_kernel(const NormEdgeParams p) {
     }
     if (p.x_out) RowVec<float, V>::store(p.x_out + o + c, x[i]);
   }
-  if (!p.before) return;
+  if (!p.before) {
+    if (!p.h) return;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = (i * TH + threadIdx.x) * V;
+      if (c < p.width) RowVec<T, V>::store(static_cast<T*>(p.h) + o + c, x[i]);
+    }
+    return;
+  }
   r = row_norm_factor<TH, NC, V, CENTER>(x, p, red + 2);
 #pragma unroll
   for (int i = 0; i < NC; ++i) {
@@ -172,13 +198,18 @@ static int norm_edge_type(const NormEdgeParams& p, long long n, int center, cuda
 
 }  // namespace kvb
 
-extern "C" int kvb_norm_edge(const float* x_in, const void* sub, const float* after, float* x_out, const float* before, void* h,
-                             const long long* idx, const void* embed, long long vocab, const float* step, long long n, int width,
-                             float eps, int center, int dtype, int* status, void* stream) {
-  if (n <= 0 || n > 0x7fffffffLL || width <= 0 || (before && !h) || (embed && !idx) || (after && !sub)) return KVB_ERR_ARG;
+extern "C" int kvb_norm_edge(const float* x_in, const void* sub, const void* expert_out, const int* expert_row, const float* expert_w, int top,
+                             long long expert_ld, const float* after, float* x_out, const float* before, void* h, const long long* idx,
+                             const void* embed, long long vocab, const float* step, long long n, int width, float eps, int center,
+                             int dtype, int* status, void* stream) {
+  if (n <= 0 || n > 0x7fffffffLL || width <= 0 || (before && !h) || (embed && !idx) || (after && !sub && !expert_out) ||
+      (expert_out && (!expert_row || !expert_w || top <= 0 || expert_ld < width)))
+    return KVB_ERR_ARG;
+  if (expert_out && width % 4 == 0 && expert_ld % 4) return KVB_ERR_ALIGN;
   kvb::NormEdgeParams p;
   p.x_in = x_in; p.sub = sub; p.after = after; p.x_out = x_out; p.before = before; p.h = h; p.idx = idx; p.embed = embed;
   p.vocab = vocab; p.step = step; p.width = width; p.eps = eps; p.inv_width = 1.f / (float)width; p.status = status;
+  p.expert_out = expert_out; p.expert_row = expert_row; p.expert_w = expert_w; p.expert_ld = expert_ld; p.top = expert_out ? top : 0;
   if (dtype == 0) return kvb::norm_edge_type<float>(p, n, center, (cudaStream_t)stream);
   if (dtype == 1) return kvb::norm_edge_type<__nv_bfloat16>(p, n, center, (cudaStream_t)stream);
   return KVB_ERR_ARG;

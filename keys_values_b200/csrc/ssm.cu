@@ -139,7 +139,8 @@ constexpr int SN_CHUNK = 8;   // tokens staged at a time
 // NR: rows of the state per thread; thread (p, r) has column p of rows r, r + SN_ROWS, ...
 template <typename T, int NR>
 __global__ void __launch_bounds__(SN_COLS * SN_ROWS)
-state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ xbc, T* __restrict__ y, const ScanParams p) {
+state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long long ldx, const T* __restrict__ bm, const T* __restrict__ cm,
+                         long long ldb, T* __restrict__ y, const ScanParams p) {
   constexpr int NP = NR * SN_ROWS;
   __shared__ float sb[SN_CHUNK][NP], sc[SN_CHUNK][NP], sx[SN_CHUNK][SN_COLS], sdt[SN_CHUNK], sa[SN_CHUNK];
   __shared__ float part[SN_CHUNK][SN_ROWS][SN_COLS];
@@ -154,21 +155,26 @@ state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ xbc, T* 
     const int row = r + i * SN_ROWS;
     s[i] = p.start[b] > 0 && mine && row < p.np ? st[(long long)row * p.vdp] : 0.f;
   }
-  const float rate = -expf(p.a_log[h]), skip = p.skip[h], bias = p.dt_bias[h];
-  const T* xr = xbc + (long long)b * p.T * p.channels;
+  const float rate = p.decay ? 0.f : -expf(p.a_log[h]), skip = p.decay ? 0.f : p.skip[h], bias = p.decay ? 0.f : p.dt_bias[h];
+  x += (long long)b * p.T * ldx;
+  bm += (long long)b * p.T * ldb;
+  cm += (long long)b * p.T * ldb;
   for (int t0 = 0; t0 < p.T; t0 += SN_CHUNK) {
     const int nt = min(SN_CHUNK, p.T - t0);
     for (int i = tid; i < nt * NP; i += SN_COLS * SN_ROWS) {
       const int t = i / NP, k = i - t * NP;
-      const T* src = xr + (long long)(t0 + t) * p.channels + p.inner + g * p.np + k;
-      sb[t][k] = k < p.np ? to_f32(src[0]) : 0.f;
-      sc[t][k] = k < p.np ? to_f32(src[p.groups * p.np]) : 0.f;
+      const long long at = (long long)(t0 + t) * ldb + g * p.np + k;
+      sb[t][k] = k < p.np ? to_f32(bm[at]) : 0.f;
+      sc[t][k] = k < p.np ? to_f32(cm[at]) : 0.f;
     }
     for (int i = tid; i < nt * SN_COLS; i += SN_COLS * SN_ROWS) {
       const int t = i / SN_COLS, k = i - t * SN_COLS;
-      sx[t][k] = p0 + k < p.vdp ? to_f32(xr[(long long)(t0 + t) * p.channels + h * p.vdp + p0 + k]) : 0.f;
+      sx[t][k] = p0 + k < p.vdp ? to_f32(x[(long long)(t0 + t) * ldx + h * p.vdp + p0 + k]) : 0.f;
     }
-    if (tid < nt) {
+    if (tid < nt && p.decay) {
+      sdt[tid] = 1.f;
+      sa[tid] = p.decay[h];
+    } else if (tid < nt) {
       const float dt = ss_softplus(to_f32(u[((long long)b * p.T + t0 + tid) * p.ld + p.dt_col + h]) + bias);
       sdt[tid] = dt;
       sa[tid] = ss_decay(rate * dt);
@@ -206,9 +212,11 @@ state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ xbc, T* 
 }
 
 template <typename T>
-static int scan_simple_launch(const void* u, const void* xbc, void* y, const ScanParams& p, int B, cudaStream_t s) {
+static int scan_simple_launch(const void* u, const void* x, long long ldx, const void* bm, const void* cm, long long ldb, void* y,
+                              const ScanParams& p, int B, cudaStream_t s) {
   const dim3 grid((p.vdp + SN_COLS - 1) / SN_COLS, p.heads, B);
-#define KVB_SCAN(NR) state_scan_simple_kernel<T, NR><<<grid, SN_COLS * SN_ROWS, 0, s>>>((const T*)u, (const T*)xbc, (T*)y, p)
+#define KVB_SCAN(NR) state_scan_simple_kernel<T, NR><<<grid, SN_COLS * SN_ROWS, 0, s>>>( \
+    (const T*)u, (const T*)x, ldx, (const T*)bm, (const T*)cm, ldb, (T*)y, p)
   if (p.np <= 4 * SN_ROWS) KVB_SCAN(4);
   else if (p.np <= 16 * SN_ROWS) KVB_SCAN(16);
   else if (p.np <= 32 * SN_ROWS) KVB_SCAN(32);
@@ -455,10 +463,22 @@ extern "C" int kvb_state_scan(const void* u, long long ld, int dt_col, const voi
                               int T_, int heads, int groups, int vdp, int np, int dtype, void* stream) {
   if (B <= 0 || B > 65535 || T_ <= 0 || heads <= 0 || heads > 65535 || groups <= 0 || heads % groups || vdp <= 0 || np <= 0) return KVB_ERR_ARG;
   kvb::ScanParams p;
-  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.slots = slots; p.start = start; p.count = count; p.state = state; p.ld = ld;
-  p.T = T_; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
+  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.decay = nullptr; p.slots = slots; p.start = start; p.count = count;
+  p.state = state; p.ld = ld; p.T = T_; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
   p.channels = heads * vdp + 2 * groups * np;
-  KVB_SSM_TYPES(dtype, return kvb::scan_simple_launch<T>(u, xbc, y, p, B, (cudaStream_t)stream));
+  KVB_SSM_TYPES(dtype, const T* x = (const T*)xbc; const T* bm = x + p.inner;
+                return kvb::scan_simple_launch<T>(u, x, p.channels, bm, bm + groups * np, p.channels, y, p, B, (cudaStream_t)stream));
+}
+
+extern "C" int kvb_retention_scan(const void* v, long long ldv, const void* qk, long long ldqk, const float* decay, float* state, void* y,
+                                  const int* slots, const int* start, const int* count, int B, int T_, int heads, int vdp, int np,
+                                  int dtype, void* stream) {
+  if (B <= 0 || B > 65535 || T_ <= 0 || heads <= 0 || heads > 65535 || vdp <= 0 || np <= 0 || !decay) return KVB_ERR_ARG;
+  kvb::ScanParams p;
+  p.dt_bias = p.a_log = p.skip = nullptr; p.decay = decay; p.slots = slots; p.start = start; p.count = count; p.state = state; p.ld = 0;
+  p.T = T_; p.dt_col = 0; p.heads = heads; p.groups = heads; p.vdp = vdp; p.np = np; p.inner = heads * vdp; p.channels = 0;
+  KVB_SSM_TYPES(dtype, const T* q = (const T*)qk;
+                return kvb::scan_simple_launch<T>(nullptr, v, ldv, q + heads * np, q, ldqk, y, p, B, (cudaStream_t)stream));
 }
 
 extern "C" int kvb_state_step(const void* u, long long ld, int col, int dt_col, const float* w, const float* bias, const float* dt_bias,
@@ -472,8 +492,8 @@ extern "C" int kvb_state_step(const void* u, long long ld, int col, int dt_col, 
   if (smem > 48 * 1024) return KVB_ERR_TOO_LARGE;
   kvb::StepParams q;
   kvb::ScanParams& p = q.s;
-  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.slots = slots; p.start = start; p.count = count; p.state = state; p.ld = ld;
-  p.T = 1; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
+  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.decay = nullptr; p.slots = slots; p.start = start; p.count = count;
+  p.state = state; p.ld = ld; p.T = 1; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
   p.channels = heads * vdp + 2 * groups * np;
   q.w = w; q.bias = bias; q.taps = taps; q.col = col;
   KVB_SSM_TYPES(dtype, (kvb::state_step_kernel<T><<<dim3(heads, B), kvb::SS_THREADS, smem, (cudaStream_t)stream>>>(

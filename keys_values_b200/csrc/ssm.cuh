@@ -13,8 +13,11 @@ __device__ __forceinline__ float ss_softplus(float x) { return fmaxf(x, 0.f) + l
 // exp(x) of a small negative number: what it lacks to 1 keeps its relative precision (a decay is taken to high powers)
 __device__ __forceinline__ float ss_decay(float x) { return 1.f + expm1f(x); }
 
+// The recurrence S_t = a_t S_(t-1) + dt_t B_t x_t^T, y_t = S_t^T C_t + skip x_t, with a_t = exp(-exp(a_log) dt_t) and dt_t from the joint
+// projection, or (decay not NULL) with a fixed decay per head and step 1, without skip.
 struct ScanParams {
   const float *dt_bias, *a_log, *skip;  // (heads)
+  const float* decay;                   // (heads): the decay, in the chunked kernel its log2; NULL: from step sizes
   const int *slots, *start, *count;
   float* state;                         // (slots, heads, np, vdp)
   long long ld;                         // of the joint projection, whose step sizes start at column dt_col

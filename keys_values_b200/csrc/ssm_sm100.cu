@@ -15,6 +15,9 @@
 // columns. TMEM per head: G (128 columns, P takes its place), Y and S (64 or
 // 128 each).
 //
+// With a fixed decay per head (retention: B the keys, C the queries, x the values) the step size is 1, the running sums are multiples
+// of its logarithm and there is no D.
+//
 // Long passes of few heads are cut into segments: a first launch (STATES) finds what each segment adds to the state and its total
 // decay, a small kernel chains them, and the segments then run side by side from their own starting states.
 #include <cuda.h>
@@ -261,17 +264,17 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
     float rate[NH], bias[NH];
 #pragma unroll
     for (int u = 0; u < NH; ++u) {
-      rate[u] = -expf(p.a_log[h0 + u]) * SD_LOG2E;
-      bias[u] = p.dt_bias[h0 + u];
+      rate[u] = p.decay ? p.decay[h0 + u] : -expf(p.a_log[h0 + u]) * SD_LOG2E;
+      bias[u] = p.decay ? 0.f : p.dt_bias[h0 + u];
     }
-    const __nv_bfloat16* raw_dt = q.u + (long long)b * p.T * p.ld + p.dt_col + h0;
+    const __nv_bfloat16* raw_dt = p.decay ? nullptr : q.u + (long long)b * p.T * p.ld + p.dt_col + h0;
     float raw[NH][4];
     auto fetch = [&](int i) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int t = chunk_of(i) * SD_T + 4 * lane + j;
 #pragma unroll
-        for (int u = 0; u < NH; ++u) raw[u][j] = t < n ? __bfloat162float(raw_dt[(long long)t * p.ld + u]) : 0.f;
+        for (int u = 0; u < NH; ++u) raw[u][j] = raw_dt && t < n ? __bfloat162float(raw_dt[(long long)t * p.ld + u]) : 0.f;
       }
     };
     if (n_chunks > 0) fetch(0);
@@ -282,7 +285,7 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
 #pragma unroll
       for (int u = 0; u < NH; ++u)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) dt[u][j] = t0 + j < n ? sd_softplus(raw[u][j] + bias[u]) : 0.f;
+        for (int j = 0; j < 4; ++j) dt[u][j] = t0 + j >= n ? 0.f : p.decay ? 1.f : sd_softplus(raw[u][j] + bias[u]);
       if (i + 1 < n_chunks) fetch(i + 1);
       if (ok) ok = mbar_wait_bounded(&sh.d_empty[i & 1], (uint32_t)((i >> 1) & 1) ^ 1, abort_flag, q.status, STATUS_TIMEOUT_EMPTY);
 #pragma unroll
@@ -321,7 +324,7 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
     float* const seg_base = q.seg_state ? q.seg_state + ((long long)b * p.heads + h) * p.np * p.vdp : nullptr;
     // starting state of this CTA, NULL: zero
     const float* from = STATES ? nullptr : (q.n_seg > 1 ? seg_base + seg * seg_step : (p.start[b] > 0 ? own : nullptr));
-    const float skip = p.skip[h];
+    const float skip = p.decay ? 0.f : p.skip[h];
     bool ok = true;  // after a wait that ran out the work goes on unseen: the status word tells, and the loop ends
     float decay_log2 = 0.f;
     auto state_at = [&](const float* base, int c) {  // four columns of this row, zero beyond the sizes
@@ -639,40 +642,67 @@ extern "C" long long kvb_state_scan_tc_scratch_bytes(int B, int T, int heads, in
   return pl.n_seg > 1 ? (long long)pl.n_seg * B * heads * ((long long)np * vdp + 1) * 4 : 0;
 }
 
+namespace kvb {
+
+// What both recurrences hand over: values x (ldx), keys B and queries C (ldb) of every token, heads in groups that share B and C.
+static int sd_run(SdParams& q, const __nv_bfloat16* x, long long ldx, const __nv_bfloat16* bm, const __nv_bfloat16* cm, long long ldb,
+                  float* scratch, cudaStream_t s) {
+  const ScanParams& p = q.s;
+  const int B = q.B, T = p.T;
+  if (B <= 0 || B > 65535 || T <= 0) return KVB_ERR_ARG;
+  if (!kvb_state_scan_tc_supported(p.heads, p.groups, p.vdp, p.np)) return KVB_ERR_UNSUPPORTED;
+  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(bm) | reinterpret_cast<uintptr_t>(cm) | reinterpret_cast<uintptr_t>(q.y) |
+       reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(scratch)) & 15 || ldx % 8 || ldb % 8)
+    return KVB_ERR_ALIGN;
+  const SdPlan pl = sd_plan(B, T, p.heads, p.groups, p.vdp, p.np);
+  if (pl.smem > SD_SMEM_LIMIT) return KVB_ERR_TOO_LARGE;
+  if (pl.n_seg > 1 && !scratch) return KVB_ERR_ARG;
+  q.n_seg = pl.n_seg;
+  q.seg_chunks = pl.seg_chunks;
+  q.seg_state = pl.n_seg > 1 ? scratch : nullptr;
+  q.seg_decay = pl.n_seg > 1 ? scratch + (long long)pl.n_seg * B * p.heads * p.np * p.vdp : nullptr;
+  const uint32_t box[4] = {64, 1, SD_T, 1};
+  CUtensorMap tm[4];
+  int rc;
+  const uint64_t lx = ldx, lb = ldb;
+  const uint64_t dx[4] = {(uint64_t)p.vdp, (uint64_t)p.heads, (uint64_t)T, (uint64_t)B}, sx[3] = {(uint64_t)p.vdp, lx, T * lx};
+  const uint64_t db[4] = {(uint64_t)p.np, (uint64_t)p.groups, (uint64_t)T, (uint64_t)B}, sb[3] = {(uint64_t)p.np, lb, T * lb};
+  if ((rc = tmap_bf16(&tm[0], x, 4, dx, sx, box))) return rc;
+  if ((rc = tmap_bf16(&tm[1], bm, 4, db, sb, box))) return rc;
+  if ((rc = tmap_bf16(&tm[2], cm, 4, db, sb, box))) return rc;
+  const uint64_t sy[3] = {(uint64_t)p.vdp, (uint64_t)p.inner, (uint64_t)T * p.inner};
+  if ((rc = tmap_bf16(&tm[3], q.y, 4, dx, sy, box))) return rc;
+  if (pl.nh == 2) return pl.kc == 1 ? sd_launch<2, 1, 1>(tm, q, pl.smem, s) : sd_launch<2, 1, 2>(tm, q, pl.smem, s);
+  if (pl.nv == 1) return pl.kc == 1 ? sd_launch<1, 1, 1>(tm, q, pl.smem, s) : sd_launch<1, 1, 2>(tm, q, pl.smem, s);
+  return pl.kc == 1 ? sd_launch<1, 2, 1>(tm, q, pl.smem, s) : sd_launch<1, 2, 2>(tm, q, pl.smem, s);
+}
+
+}  // namespace kvb
+
 extern "C" int kvb_state_scan_tc(const void* u, long long ld, int dt_col, const void* xbc, const float* dt_bias, const float* a_log,
                                  const float* skip, float* state, void* y, void* scratch, const int* slots, const int* start,
                                  const int* count, int B, int T, int heads, int groups, int vdp, int np, int* status, void* stream) {
   using namespace kvb;
-  if (B <= 0 || B > 65535 || T <= 0) return KVB_ERR_ARG;
-  if (!kvb_state_scan_tc_supported(heads, groups, vdp, np)) return KVB_ERR_UNSUPPORTED;
-  if ((reinterpret_cast<uintptr_t>(xbc) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(state) |
-       reinterpret_cast<uintptr_t>(scratch)) & 15)
-    return KVB_ERR_ALIGN;
-  const SdPlan pl = sd_plan(B, T, heads, groups, vdp, np);
-  if (pl.smem > SD_SMEM_LIMIT) return KVB_ERR_TOO_LARGE;
-  if (pl.n_seg > 1 && !scratch) return KVB_ERR_ARG;
   SdParams q;
   ScanParams& p = q.s;
-  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.slots = slots; p.start = start; p.count = count; p.state = state; p.ld = ld;
-  p.T = T; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
+  p.dt_bias = dt_bias; p.a_log = a_log; p.skip = skip; p.decay = nullptr; p.slots = slots; p.start = start; p.count = count;
+  p.state = state; p.ld = ld; p.T = T; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
   p.channels = heads * vdp + 2 * groups * np;
-  q.u = (const __nv_bfloat16*)u; q.y = (__nv_bfloat16*)y; q.status = status; q.B = B; q.n_seg = pl.n_seg; q.seg_chunks = pl.seg_chunks;
-  q.seg_state = pl.n_seg > 1 ? (float*)scratch : nullptr;
-  q.seg_decay = pl.n_seg > 1 ? (float*)scratch + (long long)pl.n_seg * B * heads * np * vdp : nullptr;
-  const uint64_t ch = p.channels, st[3] = {0, ch, (uint64_t)T * ch};
-  const uint32_t box[4] = {64, 1, SD_T, 1};
-  CUtensorMap tm[4];
-  int rc;
-  const __nv_bfloat16* base = (const __nv_bfloat16*)xbc;
-  const uint64_t dx[4] = {(uint64_t)vdp, (uint64_t)heads, (uint64_t)T, (uint64_t)B}, sx[3] = {(uint64_t)vdp, st[1], st[2]};
-  const uint64_t db[4] = {(uint64_t)np, (uint64_t)groups, (uint64_t)T, (uint64_t)B}, sb[3] = {(uint64_t)np, st[1], st[2]};
-  if ((rc = tmap_bf16(&tm[0], base, 4, dx, sx, box))) return rc;
-  if ((rc = tmap_bf16(&tm[1], base + p.inner, 4, db, sb, box))) return rc;
-  if ((rc = tmap_bf16(&tm[2], base + p.inner + groups * np, 4, db, sb, box))) return rc;
-  const uint64_t sy[3] = {(uint64_t)vdp, (uint64_t)p.inner, (uint64_t)T * p.inner};
-  if ((rc = tmap_bf16(&tm[3], y, 4, dx, sy, box))) return rc;
-  cudaStream_t s = (cudaStream_t)stream;
-  if (pl.nh == 2) return pl.kc == 1 ? sd_launch<2, 1, 1>(tm, q, pl.smem, s) : sd_launch<2, 1, 2>(tm, q, pl.smem, s);
-  if (pl.nv == 1) return pl.kc == 1 ? sd_launch<1, 1, 1>(tm, q, pl.smem, s) : sd_launch<1, 1, 2>(tm, q, pl.smem, s);
-  return pl.kc == 1 ? sd_launch<1, 2, 1>(tm, q, pl.smem, s) : sd_launch<1, 2, 2>(tm, q, pl.smem, s);
+  q.u = (const __nv_bfloat16*)u; q.y = (__nv_bfloat16*)y; q.status = status; q.B = B;
+  const __nv_bfloat16* x = (const __nv_bfloat16*)xbc;
+  return sd_run(q, x, p.channels, x + p.inner, x + p.inner + groups * np, p.channels, (float*)scratch, (cudaStream_t)stream);
+}
+
+extern "C" int kvb_retention_scan_tc(const void* v, long long ldv, const void* qk, long long ldqk, const float* log2_decay, float* state,
+                                     void* y, void* scratch, const int* slots, const int* start, const int* count, int B, int T, int heads,
+                                     int vdp, int np, int* status, void* stream) {
+  using namespace kvb;
+  if (!log2_decay) return KVB_ERR_ARG;
+  SdParams q;
+  ScanParams& p = q.s;
+  p.dt_bias = p.a_log = p.skip = nullptr; p.decay = log2_decay; p.slots = slots; p.start = start; p.count = count; p.state = state;
+  p.ld = 0; p.T = T; p.dt_col = 0; p.heads = heads; p.groups = heads; p.vdp = vdp; p.np = np; p.inner = heads * vdp; p.channels = 0;
+  q.u = nullptr; q.y = (__nv_bfloat16*)y; q.status = status; q.B = B;
+  const __nv_bfloat16* c = (const __nv_bfloat16*)qk;
+  return sd_run(q, (const __nv_bfloat16*)v, ldv, c + heads * np, c, ldqk, (float*)scratch, (cudaStream_t)stream);
 }

@@ -59,6 +59,10 @@ class LayerCache(KVCache):
     def check_capacity(self, end: int) -> None:
         """Raises if positions up to ``end`` cannot all be kept as long as the layer needs them."""
 
+    def check_pass(self, seq) -> None:
+        """Raises if the pass cannot be worked on."""
+        self.check_capacity(seq.max_end)
+
     # ---------------------------------------------------------------- storage
     def _shapes(self, dtype: torch.dtype) -> Dict[str, Tuple[Tuple[int, ...], torch.dtype]]:
         """Name, shape (of one turn) and type of every buffer."""
@@ -111,9 +115,9 @@ def layer_cache_class(kind: Optional[str]) -> Type[LayerCache]:
     """The cache class that serves mixers of ``kind``."""
     from keys_values_b200.kvcache.grouped import GroupedKVCache
     from keys_values_b200.kvcache.latent import LatentKVCache
-    from keys_values_b200.kvcache.recurrent import StateSpaceCache
+    from keys_values_b200.kvcache.recurrent import RetentionCache, StateSpaceCache
 
-    classes = {c.kind: c for c in (LatentKVCache, GroupedKVCache, StateSpaceCache)}
+    classes = {c.kind: c for c in (LatentKVCache, GroupedKVCache, StateSpaceCache, RetentionCache)}
     if kind not in classes:
         raise ValueError(f"no cache for mixers of kind {kind!r}")
     return classes[kind]

@@ -1,4 +1,5 @@
-"""State of a recurrent layer: per sequence the fp32 state of every head and the last inputs of the short convolution.
+"""State of a recurrent layer: per sequence the fp32 state of every head and, where the layer has a short convolution, its last
+inputs.
 
 The state ``(heads, state, vdim)`` has its sizes padded to multiples of 8 (padding stays zero). The convolution's inputs lie in
 a ring of ``taps`` rows, position p in row ``p mod taps``: one row more than the convolution looks back, so that a step
@@ -14,7 +15,37 @@ from keys_values_b200.config import Config
 from keys_values_b200.kvcache.layer_cache import LayerCache
 
 
-class StateSpaceCache(LayerCache):
+class RecurrentCache(LayerCache):
+    """Holds a state per sequence and no tokens."""
+
+    @property
+    def state(self) -> Optional[torch.Tensor]:
+        """``(turns, max_batch_size, heads, np, vdp)`` fp32."""
+        return None if self.buffers_ is None else self.buffers_[0]
+
+    @property
+    def current_length(self) -> int:
+        return self.input_pos
+
+    def _shapes(self, dtype):
+        s = self.shape
+        return {"state": ((self.max_batch_size, s.heads, s.np, s.vdp), torch.float32)}
+
+    def token_positions(self) -> torch.Tensor:
+        raise NotImplementedError("a recurrent state holds no tokens")
+
+
+class RetentionCache(RecurrentCache):
+    kind = "retention"
+
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
+        from keys_values_b200.models.retention import retention_shape
+
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device)
+        self.shape = retention_shape(config.layers[block_idx]["mixer"])
+
+
+class StateSpaceCache(RecurrentCache):
     kind = "mamba2"
 
     def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
@@ -24,23 +55,9 @@ class StateSpaceCache(LayerCache):
         self.shape = state_shape(config.layers[block_idx]["mixer"])
 
     @property
-    def state(self) -> Optional[torch.Tensor]:
-        """``(turns, max_batch_size, heads, np, vdp)`` fp32."""
-        return None if self.buffers_ is None else self.buffers_[0]
-
-    @property
     def conv(self) -> Optional[torch.Tensor]:
         """``(turns, max_batch_size, taps, channels)``."""
         return None if self.buffers_ is None else self.buffers_[1]
 
-    @property
-    def current_length(self) -> int:
-        return self.input_pos
-
     def _shapes(self, dtype):
-        s = self.shape
-        return {"state": ((self.max_batch_size, s.heads, s.np, s.vdp), torch.float32),
-                "conv": ((self.max_batch_size, s.taps, s.channels), dtype)}
-
-    def token_positions(self) -> torch.Tensor:
-        raise NotImplementedError("a recurrent state holds no tokens")
+        return {**super()._shapes(dtype), "conv": ((self.max_batch_size, self.shape.taps, self.shape.channels), dtype)}

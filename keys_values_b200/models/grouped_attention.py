@@ -1,17 +1,28 @@
 """Grouped-query attention of models described layer by layer, with its variants as entries of the description:
 
-* ``qk_norm``: RMS norm over the whole query and the whole key projection, before the split into heads and the rotation;
+* ``qkv_bias``: the projections of queries, keys and values have biases;
+* ``qk_norm``: RMS norm over the whole query and the whole key projection (``True``), or over every head with one weight for all heads
+  (``"head"``), before the rotation;
 * ``rope_base``, ``rope_dims``, ``rope_scale``: rotation of the first ``rope_dims`` dimensions of every head (pairs i and
-  i + rope_dims / 2), angles position · base^(−2i / rope_dims) / rope_scale;
+  i + rope_dims / 2), angles position · base^(−2i / rope_dims) / rope_scale; ``rope_bands``: frequencies stretched by their wavelength,
+  see :func:`band_frequencies`;
 * ``shared_value``: the values are the keys as projected (no norm, no rotation, no value projection);
-* ``sink``: one more term exp(0) in the denominator of the softmax;
-* ``gate``: the heads' outputs are multiplied with sigmoid of one more projection of the mixer's input.
+* ``softcap``: scores become softcap · tanh(score / softcap);
+* ``window`` and ``keep_first``: a position sees the last ``window`` positions and the first ``keep_first`` of the sequence;
+  ``chunk``: it sees its own part of ``chunk`` positions;
+* ``sink``: one more term in the denominator of the softmax, exp(0) (``True``) or learned per head (``"learned"``);
+* ``gate``: the heads' outputs are multiplied with sigmoid of one more projection of the mixer's input, one number per coordinate
+  (``True``) or per head (``"head"``);
+* ``differential``: every head has two queries and two keys over the same values; the result is the first map less lambda times the
+  second, RMS-normed per head and times 1 − differential. lambda = exp(lq1 · lk1) − exp(lq2 · lk2) + differential.
 
 Queries, keys, values and gate are one library product; one kernel norms, rotates and writes keys and values to the cache;
-attention reads the cache as it lies and applies the gate.
+attention reads the cache as it lies and applies masks, difference and gate.
 """
 from __future__ import annotations
 
+import math
+from dataclasses import replace
 from typing import Any, Dict, Optional
 
 import torch
@@ -24,17 +35,43 @@ from keys_values_b200.models.packed import Packed, pad_groups, pad_last
 from keys_values_b200.ops import layers as L
 
 
+def band_frequencies(freq: torch.Tensor, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """Frequencies for contexts longer than the ``original`` one: wavelengths above original / low are stretched by ``factor``, those below
+    original / high are left, between them the two are blended linearly in original / wavelength."""
+    turns = original * freq / (2 * math.pi)  # of a pair over the original context
+    share = (turns - low) / (high - low)
+    blend = torch.where(turns < low, torch.zeros_like(share), torch.where(turns > high, torch.ones_like(share), share))
+    return freq * (blend + (1 - blend) / factor)
+
+
+def rotation_frequencies(spec: Dict[str, Any]) -> torch.Tensor:
+    """Angle per position of every rotated pair, float64."""
+    dims = spec.get("rope_dims") or 0
+    if not dims:
+        return torch.empty(0, dtype=torch.float64)
+    freq = float(spec["rope_base"]) ** (torch.arange(dims // 2, dtype=torch.float64) * (-2.0 / dims)) / float(spec.get("rope_scale") or 1.0)
+    return band_frequencies(freq, **spec["rope_bands"]) if spec.get("rope_bands") else freq
+
+
 def grouped_shape(spec: Dict[str, Any]) -> L.GroupedShape:
+    diff = spec.get("differential")
     s = L.GroupedShape(
-        heads=spec["n_head"], kv_heads=spec["n_kv_head"], dim=spec["dim"], vdim=spec["v_dim"], rot_dims=spec["rope_dims"],
+        heads=spec["n_head"], kv_heads=spec["n_kv_head"], dim=spec["dim"], vdim=spec["v_dim"], rot_dims=spec.get("rope_dims") or 0,
         shared_value=bool(spec.get("shared_value")), gate=bool(spec.get("gate")), sink=bool(spec.get("sink")), scale=float(spec["scale"]),
+        maps=1 if diff is None else 2, head_norm=spec.get("qk_norm") == "head", gate_per_head=spec.get("gate") == "head",
+        softcap=float(spec.get("softcap") or 0.0), window=spec.get("window") or 0, keep=spec.get("keep_first") or 0 if spec.get("window") else 0,
+        chunk=spec.get("chunk") or 0, post=1.0 if diff is None else 1.0 - float(diff),
     )
     if s.heads % s.kv_heads or s.rot_dims % 2 or s.rot_dims > s.dim:
         raise ValueError(f"attention of {s.heads} heads on {s.kv_heads} with {s.rot_dims} of {s.dim} dimensions rotated")
-    if s.shared_value and s.vdim != s.dim:
-        raise ValueError(f"values that are the keys have {s.dim} dimensions, not {s.vdim}")
-    if not s.scale > 0:
-        raise ValueError("attention scale must be positive")
+    if s.shared_value and (s.vdim != s.dim or s.maps != 1):
+        raise ValueError(f"values that are the keys have one map and {s.dim} dimensions, not {s.vdim}")
+    if not s.scale > 0 or s.softcap < 0:
+        raise ValueError("attention scale must be positive, a soft cap not negative")
+    if s.window and s.chunk:
+        raise ValueError("a layer has a window or chunks, not both")
+    if s.maps == 2 and (s.sink or s.gate):
+        raise NotImplementedError("differential attention with a sink or a gate")
     return s
 
 
@@ -45,43 +82,66 @@ class GroupedAttention(Packed):
         s = self.shape = grouped_shape(spec)
         self.spec = spec
         self.eps = config.norm_eps
-        # rows: queries, keys, values (unless they are the keys), gate
-        rows = (s.heads + s.kv_heads) * s.dim + (0 if s.shared_value else s.kv_heads * s.vdim) + (s.heads * s.vdim if s.gate else 0)
-        self.qkv = nn.Linear(config.n_embd, rows, bias=False)
-        self.norm_q = nn.Parameter(torch.ones(s.heads * s.dim)) if spec.get("qk_norm") else None
-        self.norm_k = nn.Parameter(torch.ones(s.kv_heads * s.dim)) if spec.get("qk_norm") else None
+        # rows: queries, keys (head by head, the maps of a head in a row), values (unless they are the keys), gate
+        H, G = s.heads * s.maps, s.kv_heads * s.maps
+        self.parts = [H * s.dim, G * s.dim] + ([] if s.shared_value else [s.kv_heads * s.vdim])
+        self.gate_rows = 0 if not s.gate else s.heads if s.gate_per_head else s.heads * s.vdim
+        self.qkv = nn.Linear(config.n_embd, sum(self.parts) + self.gate_rows, bias=False)
+        self.qkv_bias = nn.Parameter(torch.zeros(sum(self.parts))) if spec.get("qkv_bias") else None
+        norm = spec.get("qk_norm")
+        self.norm_q = nn.Parameter(torch.ones(s.dim if norm == "head" else H * s.dim)) if norm else None
+        self.norm_k = nn.Parameter(torch.ones(s.dim if norm == "head" else G * s.dim)) if norm else None
+        self.sink = nn.Parameter(torch.zeros(s.heads)) if spec.get("sink") == "learned" else None
+        # rows lq1, lk1, lq2, lk2
+        self.map_weights = nn.Parameter(torch.zeros(4, s.dim)) if s.maps == 2 else None
         self.proj = nn.Linear(s.heads * s.vdim, config.n_embd, bias=False)
         self.kv_cache = kv_cache
         self.config = config
         self.block_idx = block_idx
 
-    def _make_pack(self) -> Dict[str, Optional[torch.Tensor]]:
+    def _pad_rows(self, w: torch.Tensor, gate: bool) -> torch.Tensor:
+        """Rows of the joint projection, every head padded and the whole padded to its leading dimension."""
         s = self.shape
-        w = self.qkv.weight
-        sizes = [s.heads * s.dim, s.kv_heads * s.dim] + ([] if s.shared_value else [s.kv_heads * s.vdim]) + ([s.heads * s.vdim] if s.gate else [])
-        parts = list(torch.split(w, sizes))
-        out = [pad_groups(parts[0], s.heads, s.dimp), pad_groups(parts[1], s.kv_heads, s.dimp)]
+        parts = list(torch.split(w, self.parts + ([self.gate_rows] if gate and self.gate_rows else [])))
+        out = [pad_groups(parts[0], s.heads * s.maps, s.dimp), pad_groups(parts[1], s.kv_heads * s.maps, s.dimp)]
         if not s.shared_value:
             out.append(pad_groups(parts[2], s.kv_heads, s.vdp))
-        if s.gate:
-            out.append(pad_groups(parts[-1], s.heads, s.vdp))
-        exps = torch.arange(s.rot_dims // 2, dtype=torch.float64) * (-2.0 / max(s.rot_dims, 1))
-        freq = float(self.spec["rope_base"]) ** exps / float(self.spec.get("rope_scale", 1.0))
+        if gate and self.gate_rows:
+            out.append(pad_groups(parts[-1], s.heads, s.gate_cols))
+        out = torch.cat(out)
+        return F.pad(out, (0, 0) * (out.ndim - 1) + (0, s.ld - out.shape[0])).contiguous()
+
+    def _pad_norm(self, w: Optional[torch.Tensor], heads: int) -> Optional[torch.Tensor]:
+        if w is None:
+            return None
+        return pad_last(w.float(), self.shape.dimp) if self.shape.head_norm else pad_groups(w.float(), heads * self.shape.maps, self.shape.dimp)
+
+    def _make_pack(self) -> Dict[str, Any]:
+        s = self.shape
+        if s.maps == 2:
+            a = self.map_weights.double()
+            lam = float(torch.exp((a[0] * a[1]).sum()) - torch.exp((a[2] * a[3]).sum())) + float(self.spec["differential"])
+            s = replace(s, lam=lam, eps=self.eps)
+        w = self.qkv.weight
         return {
-            "qkv": torch.cat(out).contiguous(),
-            "norm_q": None if self.norm_q is None else pad_groups(self.norm_q.float(), s.heads, s.dimp),
-            "norm_k": None if self.norm_k is None else pad_groups(self.norm_k.float(), s.kv_heads, s.dimp),
-            "freq": freq.to(device=w.device, dtype=torch.float32),
+            "shape": s,
+            "qkv": self._pad_rows(w, True),
+            "bias": None if self.qkv_bias is None else self._pad_rows(self.qkv_bias, False),
+            "norm_q": self._pad_norm(self.norm_q, s.heads),
+            "norm_k": self._pad_norm(self.norm_k, s.kv_heads),
+            "sink": None if self.sink is None else self.sink.float().contiguous(),
+            "freq": rotation_frequencies(self.spec).to(device=w.device, dtype=torch.float32),
             "proj": pad_last(self.proj.weight.view(-1, s.heads, s.vdim), s.vdp).view(-1, s.heads * s.vdp),
         }
 
     def forward(self, x: torch.Tensor, seq: SequencePass, turn: int = 0) -> torch.Tensor:
         """``x (B, T, width)`` → ``(B, T, width)``; the cache takes the keys and values of the pass."""
-        s, w = self.shape, self.packed()
-        qkv = F.linear(x, w["qkv"])
+        w = self.packed()
+        s, plan = w["shape"], self.kv_cache.plan
+        qkv = F.linear(x, w["qkv"], w["bias"])
         rows = self.kv_cache.allocate(x.device, x.dtype)[0][turn]
-        q = L.grouped_prep(qkv, w["norm_q"], w["norm_k"], w["freq"], rows, seq, s, self.eps)
-        return F.linear(L.grouped_attend(q, qkv, rows, seq, s), w["proj"])
+        q = L.grouped_prep(qkv, w["norm_q"], w["norm_k"], w["freq"], rows, seq, s, self.eps, plan)
+        return F.linear(L.grouped_attend(q, qkv, rows, seq, s, w["sink"], plan), w["proj"])
 
     def check_kv_cache(self, cache) -> None:
         from keys_values_b200.kvcache.grouped import GroupedKVCache

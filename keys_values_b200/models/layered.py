@@ -6,9 +6,11 @@ differ. The mechanisms are modules of their own, picked by the description:
 * :class:`LatentAttention`: low-rank keys and values (one latent per token plus one rotated key part that the heads
   share), optional sliding window, ring cache of latents (:class:`keys_values_b200.kvcache.latent.LatentKVCache`);
 * :class:`keys_values_b200.models.grouped_attention.GroupedAttention`: grouped-query attention with optional norm of queries and
-  keys, values shared with the keys, softmax sink and output gate;
+  keys, windows or chunks, values shared with the keys, soft cap, softmax sink, output gate and differential maps;
 * :class:`keys_values_b200.models.state_space.Mamba2Mixer`: state-space recurrence;
-* :class:`RoutedMLP`: softmax router, top-k experts without gates; :class:`DenseMLP`: two matrices and an activation;
+* :class:`keys_values_b200.models.retention.Retention`: linear attention with a fixed decay per head;
+* :class:`RoutedMLP`: softmax or sigmoid router, top-k experts with or without gates, optionally a shared expert;
+  :class:`DenseMLP`: two matrices and an activation; :class:`GatedMLP`: three matrices;
 * :class:`ScalarRMSNorm`: RMS norm with one gain for all coordinates; :class:`StreamNorm`: layer or RMS norm of the fp32 stream;
 * token shift (``config.token_shift``): the mixer reads a learned blend of the token's normed input and the previous token's;
 * depth average (``config.depth_average``): what goes on to the next layer is a learned average of the embedding output
@@ -17,7 +19,7 @@ differ. The mechanisms are modules of their own, picked by the description:
 * loop (``config.loop``): a run of layers is passed several times, with a cache or state of its own each time.
 
 Two kinds of layers: :class:`ParallelBlock` (mixer and feed-forward read one norm's output) and :class:`SequentialBlock` (one
-after the other, each between norms). The residual stream and the depth history are fp32. What lies between two sublayers
+after the other, each with a norm before it, after it or both). The residual stream and the depth history are fp32. What lies between two sublayers
 that depend on each other (residual sum, norms, weighted expert outputs, depth average, token shift, what a loop adds) is one
 kernel, :func:`keys_values_b200.ops.layers.layer_edge` or :func:`keys_values_b200.ops.layers.norm_edge`; therefore the stream
 that :meth:`LayeredGPT.run_layer` hands on is a :class:`LayerStream`, which carries the next layer's normed inputs along.
@@ -36,7 +38,8 @@ from keys_values_b200.kvcache.layer_cache import LayerCache
 from keys_values_b200.kvcache.sequences import SequencePass, SequenceTable
 from keys_values_b200.models.grouped_attention import GroupedAttention
 from keys_values_b200.models.model import GPT
-from keys_values_b200.models.packed import Packed, pad_last
+from keys_values_b200.models.packed import Packed, pad_groups, pad_last
+from keys_values_b200.models.retention import Retention
 from keys_values_b200.models.state_space import Mamba2Mixer
 from keys_values_b200.ops import layers as L
 
@@ -161,34 +164,72 @@ class LatentAttention(Packed):
 
 
 class RoutedMLP(Packed):
-    """``Σ over the chosen experts of score_e · down_e(act(up_e(x)))``. Returns the experts' outputs unsummed (the sum is
-    part of the kernel that closes the layer)."""
+    """``Σ over the chosen experts of weight_e · down_e(act(up_e(x)))``. Returns the experts' outputs unsummed (the sum is
+    part of the kernel that closes the sublayer).
+
+    Entries of the description: ``n_expert``, ``top``, ``ff``; ``activation`` (``"silu_gated"``: the rows of ``up`` are those of
+    the gate projection, then those of the up projection); ``score`` ``"softmax"`` or ``"sigmoid"``; ``renormalize`` (the chosen scores
+    are divided by their sum + ``renormalize_eps``); ``correction``: a learned number per expert that is added to the scores for the choice
+    only; ``groups`` ``{"count", "keep"}``: only experts of the best groups can be chosen; ``shared``: width of a gated
+    feed-forward that every token passes (``self.shared``, summed by the caller)."""
 
     def __init__(self, config: Config, spec: Dict[str, Any]) -> None:
         super().__init__()
         E, ff, width = spec["n_expert"], spec["ff"], config.n_embd
+        groups = spec.get("groups") or dict(count=1, keep=1)
         if not 0 < spec["top"] <= E:
             raise ValueError(f"top = {spec['top']} of {E} experts")
-        if spec.get("activation", "relu_squared") not in L.ACTIVATIONS:
+        if E % groups["count"] or not 0 < groups["keep"] <= groups["count"] or spec["top"] > groups["keep"] * (E // groups["count"]):
+            raise ValueError(f"top = {spec['top']} of {E} experts in groups {groups}")
+        self.activation = spec.get("activation", "relu_squared")
+        if self.activation not in L.ACTIVATIONS:
             raise ValueError(f"activation {spec['activation']!r}")
+        if spec.get("score", "softmax") not in ("softmax", "sigmoid"):
+            raise ValueError(f"score {spec['score']!r}")
         self.spec = spec
+        self.rule = L.RouterRule(score=spec.get("score", "softmax"), groups=groups["count"], keep=groups["keep"],
+                                 renormalize=bool(spec.get("renormalize", False)), eps=float(spec.get("renormalize_eps", 0.0)))
+        self.ff = ff
         self.gate = nn.Linear(width, E, bias=False)
-        self.up = nn.Parameter(torch.empty(E, ff, width))
+        self.correction = nn.Parameter(torch.zeros(E)) if spec.get("correction") else None
+        self.up = nn.Parameter(torch.empty(E, 2 * ff if self.activation == "silu_gated" else ff, width))
         self.down = nn.Parameter(torch.empty(E, width, ff))
+        self.shared = GatedMLP(config, dict(ff=spec["shared"])) if spec.get("shared") else None
         for p in (self.up, self.down):
             nn.init.normal_(p, mean=0.0, std=0.02)
 
-    def _make_pack(self) -> Dict[str, torch.Tensor]:
-        E, ff, width = self.up.shape
-        return {"up": pad_last(self.up.detach(), L.round8(width)), "down": pad_last(self.down.detach(), L.round8(ff))}
+    def _make_pack(self) -> Dict[str, Optional[torch.Tensor]]:
+        E, rows, width = self.up.shape
+        up = self.up.detach()
+        if self.activation == "silu_gated":  # gate and up projection of a result in neighbouring rows
+            up = up.view(E, 2, self.ff, width).transpose(1, 2).reshape(E, rows, width)
+        return {"up": pad_last(up, L.round8(width)), "down": pad_last(self.down.detach(), L.round8(self.ff)),
+                "correction": None if self.correction is None else self.correction.float().contiguous()}
 
     def forward(self, x: torch.Tensor):
-        _, ff, width = self.up.shape
+        width = self.up.shape[2]
         w = self.packed()
         x = x.reshape(-1, width)
         logits = L.linear_fp32(x, self.gate.weight)
-        return L.routed_experts(x, logits, w["up"], w["down"], self.spec["top"], self.spec.get("activation", "relu_squared"),
-                                bool(self.spec.get("renormalize", False)), ff, width)
+        return L.routed_experts(x, logits, w["up"], w["down"], self.spec["top"], self.activation, self.rule, self.ff, width, w["correction"])
+
+
+class GatedMLP(Packed):
+    """``down(silu(gate x) · up x)``; gate and up projection are one product, rows ``[gate | up]``."""
+
+    def __init__(self, config: Config, spec: Dict[str, Any]) -> None:
+        super().__init__()
+        self.ff = spec["ff"]
+        self.up = nn.Linear(config.n_embd, 2 * self.ff, bias=False)
+        self.down = nn.Linear(self.ff, config.n_embd, bias=False)
+
+    def _make_pack(self) -> Dict[str, torch.Tensor]:
+        n = L.round8(self.ff)
+        return {"up": pad_groups(self.up.weight.detach(), 2, n), "down": pad_last(self.down.weight.detach(), n)}
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        w = self.packed()
+        return F.linear(L.glu(F.linear(x, w["up"]), self.ff), w["down"])
 
 
 class DenseMLP(nn.Module):
@@ -196,9 +237,9 @@ class DenseMLP(nn.Module):
 
     def __init__(self, config: Config, spec: Dict[str, Any]) -> None:
         super().__init__()
-        if spec.get("activation", "relu_squared") not in L.ACTIVATIONS:
-            raise ValueError(f"activation {spec['activation']!r}")
         self.activation = spec.get("activation", "relu_squared")
+        if self.activation not in ("none", "relu_squared"):
+            raise ValueError(f"activation {self.activation!r}")
         self.up = nn.Linear(config.n_embd, spec["ff"], bias=False)
         self.down = nn.Linear(spec["ff"], config.n_embd, bias=False)
 
@@ -206,8 +247,8 @@ class DenseMLP(nn.Module):
         return F.linear(L.activate(F.linear(x, self.up.weight), self.activation), self.down.weight)
 
 
-MIXERS = {"latent_attention": LatentAttention, "grouped_attention": GroupedAttention, "mamba2": Mamba2Mixer}
-FEED_FORWARDS = {"routed": RoutedMLP, "dense": DenseMLP}
+MIXERS = {"latent_attention": LatentAttention, "grouped_attention": GroupedAttention, "mamba2": Mamba2Mixer, "retention": Retention}
+FEED_FORWARDS = {"routed": RoutedMLP, "dense": DenseMLP, "gated": GatedMLP}
 
 
 class ParallelBlock(Packed):
@@ -223,8 +264,10 @@ class ParallelBlock(Packed):
         self.depth = None
         if config.depth_average:  # the identity: all weight on the layer's own result
             self.depth = nn.Parameter(F.one_hot(torch.tensor(block_idx + 1), block_idx + 2).float())
-        if config.loop is not None or isinstance(self.mlp, DenseMLP):
-            raise NotImplementedError("parallel layers are not run in loops and have routed feed-forwards")
+        if config.loop is not None or not (self.mlp is None or isinstance(self.mlp, RoutedMLP) and self.mlp.shared is None):
+            raise NotImplementedError("parallel layers are not run in loops and have routed feed-forwards without a shared expert")
+        if not (config.norm_1 and config.norm_2) or config.post_attention_norm or config.post_mlp_norm:
+            raise NotImplementedError("parallel layers have one norm, ahead of mixer and feed-forward")
         self.config = config
         self.block_idx = block_idx
 
@@ -270,23 +313,25 @@ class ParallelBlock(Packed):
 
 
 class SequentialBlock(Packed):
-    """Norm, mixer, norm, residual sum; then the same with the feed-forward. The norms after the sublayers are optional."""
+    """Norm, mixer, norm, residual sum; then the same with the feed-forward. The norms before the sublayers (``config.norm_1``,
+    ``norm_2``; without them a sublayer reads the stream itself) and after them (``post_attention_norm``, ``post_mlp_norm``) are
+    optional."""
 
     def __init__(self, config: Config, block_idx: int, kv_cache=None) -> None:
         super().__init__()
         spec = config.layers[block_idx]
+        if config.norm_class_name not in ("StreamLayerNorm", "StreamRMSNorm"):
+            raise ValueError(f"norm {config.norm_class_name!r}: sequential layers take StreamLayerNorm or StreamRMSNorm")
         norm = partial(config.norm_class, config.n_embd, eps=config.norm_eps)
-        self.norm_1 = norm()
+        self.norm_1 = norm() if config.norm_1 else None
         self.attn = MIXERS[spec["mixer"]["kind"]](config, block_idx, kv_cache)
         self.post_attention_norm = norm() if config.post_attention_norm else None
         self.mlp = None if spec.get("mlp") is None else FEED_FORWARDS[spec["mlp"]["kind"]](config, spec["mlp"])
-        self.norm_2 = None if self.mlp is None else norm()
+        self.norm_2 = norm() if self.mlp is not None and config.norm_2 else None
         self.post_mlp_norm = norm() if self.mlp is not None and config.post_mlp_norm else None
-        if config.token_shift or config.depth_average or config.bigram is not None or isinstance(self.mlp, RoutedMLP):
-            raise NotImplementedError("token shift, depth average, bigram embedding and routed experts go with parallel layers")
-        if not isinstance(self.norm_1, StreamNorm):
-            raise ValueError(f"norm {config.norm_class_name!r}: sequential layers take StreamLayerNorm or StreamRMSNorm")
-        self.center = self.norm_1.center
+        if config.token_shift or config.depth_average or config.bigram is not None:
+            raise NotImplementedError("token shift, depth average and bigram embedding go with parallel layers")
+        self.center = config.norm_class_name == "StreamLayerNorm"
         self.config = config
         self.block_idx = block_idx
 
@@ -304,16 +349,21 @@ class SequentialBlock(Packed):
 
     def run(self, model: "LayeredGPT", run: int, x: "LayerStream", idx: torch.Tensor) -> "LayerStream":
         w, eps = self.packed(), self.config.norm_eps
-        y, after = self.attn(x.h, x.seq, model.runs[run][1]), w["after_1"]
+        y, after, experts = self.attn(x.h, x.seq, model.runs[run][1]), w["after_1"], None
         if self.mlp is not None:
             L.norm_edge(x.x, y, after, x.x, w["norm_2"], x.h, None, None, None, eps, self.center)
-            y, after = self.mlp(x.h), w["after_2"]
+            after = w["after_2"]
+            if isinstance(self.mlp, RoutedMLP):
+                y = None if self.mlp.shared is None else self.mlp.shared(x.h)
+                experts = self.mlp(x.h)
+            else:
+                y = self.mlp(x.h)
         last = run + 1 == model.n_runs
         before = None if last else model.transformer.h[model.runs[run + 1][0]].packed()["norm_1"]
         add_embedding, step = (False, None) if last else model.ahead_of_run(run + 1)
         wte = model.transformer.wte.weight
-        L.norm_edge(x.x, y, after, x.x, before, x.h, idx.contiguous() if add_embedding else None, wte if add_embedding else None, step, eps,
-                    self.center)
+        L.norm_edge(x.x, y, after, x.x, before, None if last else x.h, idx.contiguous() if add_embedding else None, wte if add_embedding else None,
+                    step, eps, self.center, experts)
         return x
 
 
@@ -353,6 +403,8 @@ class LayeredGPT(GPT):
         if config.bigram is not None:  # the last row is for tokens without a predecessor
             self.bigram = nn.Embedding(config.bigram["buckets"] + 1, config.n_embd)
         self.sequences: Optional[SequenceTable] = None
+        if config.tie_embeddings:
+            self.lm_head.weight = self.transformer.wte.weight
 
     def _make_block(self, config: Config, block_idx: int) -> nn.Module:
         return (ParallelBlock if config.parallel_residual else SequentialBlock)(config, block_idx)
@@ -467,7 +519,7 @@ class LayeredGPT(GPT):
             raise NotImplementedError("models with described layers run in inference only (use torch.inference_mode())")
         seq = self.sequences.begin(*idx.shape, counts)
         for cache in self.get_kv_caches():
-            cache.check_capacity(seq.max_end)
+            cache.check_pass(seq)
         return self.transformer.h[0].enter(self, idx.contiguous(), seq)
 
     def run_layer(self, run: int, x: LayerStream, idx: torch.Tensor, chunk_sizes: Optional[Sequence[int]] = None) -> LayerStream:

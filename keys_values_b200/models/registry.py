@@ -25,9 +25,10 @@ class Architecture:
 
 
 def _architectures() -> Dict[str, Architecture]:
-    from keys_values_b200.models import mezilix, pazenex
+    from keys_values_b200.models import ladadra, mezilix, pazenex
 
     known = (
+        Architecture("Ladadra", ladadra.config_from_json, ladadra.state_dict),
         Architecture("Mezilix", mezilix.config_from_json, mezilix.state_dict),
         Architecture("Pazenex", pazenex.config_from_json, pazenex.state_dict),
     )

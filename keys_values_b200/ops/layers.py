@@ -10,7 +10,7 @@ token counts of its rows.
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -55,8 +55,13 @@ class LatentShape:
 @dataclass(frozen=True)
 class GroupedShape:
     """Sizes and constants of one grouped-query attention; padded sizes are multiples of 8. The joint projection has the
-    columns ``[queries: heads · dimp | keys: kv_heads · dimp | values: kv_heads · vdp (not with shared_value) |
-    gate: heads · vdp (with gate)]``, every head padded with zeros."""
+    columns ``[queries: heads · maps · dimp | keys: kv_heads · maps · dimp | values: kv_heads · vdp (not with shared_value) |
+    gate: heads · vdp, or heads (gate_per_head)]``, every head padded with zeros, the whole to a multiple of 8.
+
+    ``maps = 2``: differential attention, every head has two queries and two keys over the same values; the result is
+    ``norm(map 1 − lam · map 2) · post``, the norm an RMS norm of the head without a weight.
+    Position i sees j <= i, and only ``i − j < window`` or ``j < keep`` (``window > 0``), or its own part of ``chunk`` positions
+    (``chunk > 0``). ``softcap > 0``: scores become softcap · tanh(score / softcap)."""
 
     heads: int
     kv_heads: int
@@ -67,6 +72,16 @@ class GroupedShape:
     gate: bool
     sink: bool
     scale: float
+    maps: int = 1
+    head_norm: bool = False
+    gate_per_head: bool = False
+    softcap: float = 0.0
+    window: int = 0
+    keep: int = 0
+    chunk: int = 0
+    lam: float = 0.0
+    post: float = 1.0
+    eps: float = 0.0
 
     @property
     def dimp(self) -> int:
@@ -77,13 +92,86 @@ class GroupedShape:
         return round8(self.vdim)
 
     @property
+    def row(self) -> int:
+        """Width of a cache row: the keys of all maps and the value of one key/value head."""
+        return self.maps * self.dimp + self.vdp
+
+    @property
     def value_col(self) -> int:
         """First value column of the joint projection."""
-        return (self.heads + (0 if self.shared_value else self.kv_heads)) * self.dimp
+        return (self.heads + (0 if self.shared_value else self.kv_heads)) * self.maps * self.dimp
 
     @property
     def gate_col(self) -> int:
-        return (self.heads + self.kv_heads) * self.dimp + (0 if self.shared_value else self.kv_heads * self.vdp)
+        return (self.heads + self.kv_heads) * self.maps * self.dimp + (0 if self.shared_value else self.kv_heads * self.vdp)
+
+    @property
+    def gate_cols(self) -> int:
+        """Gate columns per head."""
+        return 0 if not self.gate else 1 if self.gate_per_head else self.vdp
+
+    @property
+    def ld(self) -> int:
+        """Columns of the joint projection."""
+        return round8(self.gate_col + self.heads * self.gate_cols)
+
+    @property
+    def span(self) -> int:
+        """Positions a query looks back at most, itself included and kept ones aside; 0: all."""
+        return self.chunk or self.window
+
+
+class RowPlan(NamedTuple):
+    """Where the positions of a sequence lie: ``ring = 0`` position p in row p; else the first ``head`` positions have rows of
+    their own and position p >= head has row ``head + (p − head) mod ring``. Both are multiples of 128."""
+
+    head: int = 0
+    ring: int = 0
+
+
+@dataclass(frozen=True)
+class RetentionShape:
+    """Sizes of one retention mixer; padded sizes are multiples of 8. The projection has the columns ``[queries: heads · np |
+    keys: heads · np | values: heads · vdp | gate: heads · vdp]``, every head padded with zeros."""
+
+    heads: int
+    dim: int
+    vdim: int
+    rot_dims: int
+
+    @property
+    def np(self) -> int:
+        return round8(self.dim)
+
+    @property
+    def vdp(self) -> int:
+        return round8(self.vdim)
+
+    @property
+    def qk(self) -> int:
+        """Columns of queries and keys."""
+        return 2 * self.heads * self.np
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdp
+
+    @property
+    def key_scale(self) -> float:
+        return self.dim**-0.5
+
+
+@dataclass(frozen=True)
+class RouterRule:
+    """How a router scores and chooses: ``score`` ``"softmax"`` or ``"sigmoid"``; ``groups`` of neighbouring experts, of which the
+    ``keep`` best (by the sum of their two largest choice scores) stay in the choice; ``renormalize``: the chosen scores are divided by
+    their sum + ``eps``."""
+
+    score: str = "softmax"
+    groups: int = 1
+    keep: int = 1
+    renormalize: bool = False
+    eps: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -156,11 +244,12 @@ def scalar_rmsnorm(x: torch.Tensor, gain: torch.Tensor, eps: float, dtype: torch
     return _impl(x).scalar_rmsnorm(x, rows, gain, eps, dtype)
 
 
-def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps: float, center: bool) -> None:
-    """``x = x_in + norm(sub) · after`` (``x_in`` or ``sub`` ``None``: without it; ``after`` ``None``: ``sub`` as it is), then
-    ``x += embed[idx] + step`` (each unless ``None``); ``x_out = x`` (fp32, may be ``x_in``) and, unless ``before`` is
-    ``None``, ``h = norm(x) · before``. The norm takes the mean off if ``center``."""
-    _impl(x_out).norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center)
+def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps: float, center: bool, experts=None) -> None:
+    """``x = x_in + norm(s) · after`` with ``s = sub + Σ_k weight_k · expert output_k`` (``x_in``, ``sub`` or ``experts`` ``None``:
+    without it; ``after`` ``None``: ``s`` as it is), then ``x += embed[idx] + step`` (each unless ``None``); ``x_out = x`` (fp32, may be
+    ``x_in``) and, unless ``h`` is ``None``, ``h = norm(x) · before`` (``before`` ``None``: ``h = x``). The norm takes the mean off if
+    ``center``. ``experts``: ``(out, row, weight)`` of :func:`routed_experts`."""
+    _impl(x_out).norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts)
 
 
 def row_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, center: bool, dtype: torch.dtype) -> torch.Tensor:
@@ -208,17 +297,40 @@ def latent_decode(q_abs, q, ring, seq, shape: LatentShape, scale: float) -> torc
 
 
 # ---- grouped-query attention
-def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape: GroupedShape, eps: float) -> torch.Tensor:
-    """Norm (unless ``norm_q`` is ``None``) and rotation of queries and keys of the joint projection ``qkv (B, T, ·)``. Returns
-    queries ``(B, T, heads, dimp)``; ``[key | value]`` of every real token goes to its position in ``rows (slots, length,
-    kv_heads, dimp + vdp)``."""
-    return _impl(qkv).grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape, eps)
+def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape: GroupedShape, eps: float, plan: RowPlan = RowPlan()) -> torch.Tensor:
+    """Norm (unless ``norm_q`` is ``None``) and rotation of queries and keys of the joint projection ``qkv (B, T, ·)``. The norm goes over
+    a whole projection or (``head_norm``) over every head and map with weights of one head. Returns queries ``(B, T, heads · maps,
+    dimp)``; ``[keys of the maps | value]`` of every real token goes to its place in ``rows (slots, length, kv_heads, row)``."""
+    return _impl(qkv).grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape, eps, plan)
 
 
-def grouped_attend(q, qkv, rows, seq, shape: GroupedShape) -> torch.Tensor:
-    """Causal attention of ``q (B, T, heads, dimp)`` over ``rows``, which hold the pass already; with the gate of ``qkv``
-    applied. Returns ``(B, T, heads · vdp)``."""
-    return _impl(q).grouped_attend(q, qkv, rows, seq, shape)
+def grouped_attend(q, qkv, rows, seq, shape: GroupedShape, sink=None, plan: RowPlan = RowPlan()) -> torch.Tensor:
+    """Causal attention of ``q (B, T, heads · maps, dimp)`` over ``rows``, which hold the pass already; with the gate of ``qkv``
+    applied. ``sink (heads,)`` fp32: logarithms of what shapes with a sink add to the denominators (``None``: zeros). Returns
+    ``(B, T, heads · vdp)``."""
+    return _impl(q).grouped_attend(q, qkv, rows, seq, shape, sink, plan)
+
+
+# ---- retention
+def retention_prep(qk, freq, seq, shape: RetentionShape, dtype: torch.dtype) -> torch.Tensor:
+    """``qk (B, T, shape.qk)`` fp32, queries and keys as projected → the same rotated, keys times dim^(−1/2), as ``dtype``."""
+    return _impl(qk).retention_prep(qk, freq, seq, shape, dtype)
+
+
+def retention_scan(qk, v, decay, log2_decay, state, seq, shape: RetentionShape) -> torch.Tensor:
+    """``S_t = decay S_(t−1) + k_t v_t^T``, ``o_t = S_t^T q_t`` per head over the tokens of a pass, from and to ``state (slots, heads, np,
+    vdp)`` fp32. ``v``: rows of any leading dimension whose first ``inner`` columns are the values. Returns ``(B, T, inner)``."""
+    return _impl(qk).retention_scan(qk, v, decay, log2_decay, state, seq, shape)
+
+
+def head_norm_gate(y, gate, shape: RetentionShape, eps: float) -> torch.Tensor:
+    """``y (B, T, inner)`` divided by every head's root mean square, times silu of ``gate`` (rows of any leading dimension)."""
+    return _impl(y).head_norm_gate(y, gate, shape, eps)
+
+
+def retention_step(u, freq, decay, state, seq, shape: RetentionShape, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """The three above for one token per sequence, from the fp32 projections ``u (B, 1, qk + 2 inner)``; all of it in fp32."""
+    return _impl(u).retention_step(u, freq, decay, state, seq, shape, eps, dtype)
 
 
 # ---- state-space recurrence
@@ -249,11 +361,17 @@ def activate(x: torch.Tensor, activation: str) -> torch.Tensor:
     return x if activation == "none" else _impl(x).activate(x, ACTIVATIONS[activation])
 
 
-# ---- routed experts
-ACTIVATIONS = {"none": 0, "relu_squared": 1}
+def glu(x: torch.Tensor, ff: int) -> torch.Tensor:
+    """``x (n, 2 · round8(ff))`` = ``[gate | up]`` → ``silu(gate) · up (n, round8(ff))``, zero in the padding."""
+    return _impl(x).glu(x, ff)
 
 
-def routed_experts(h, logits, up, down, top: int, activation: str, renormalize: bool, n_up: int, n_down: int):
-    """Softmax over all experts' ``logits (n, E)``, the ``top`` largest per token, ``down_e · act(up_e · h)`` of each.
-    Returns ``(out, row (n, top), weight (n, top))``; choice ``k`` of token ``n`` is ``weight[n, k] · out[row[n, k]]``."""
-    return _impl(h).moe_forward(h, logits, up, down, top, ACTIVATIONS[activation], renormalize, n_up, n_down)
+# ---- routed experts. silu_gated: the rows of gate and up projection in turns, act(up h) = silu(gate h) · (up h)
+ACTIVATIONS = {"none": 0, "relu_squared": 1, "silu_gated": 2}
+
+
+def routed_experts(h, logits, up, down, top: int, activation: str, rule: RouterRule, n_up: int, n_down: int, correction=None):
+    """Scores of all experts from ``logits (n, E)``, the ``top`` of every token by score + ``correction (E,)``, ``down_e · act(up_e · h)`` of
+    each; ``n_up`` results of the activation, ``n_down`` outputs. Returns ``(out, row (n, top), weight (n, top))``; choice ``k`` of token
+    ``n`` is ``weight[n, k] · out[row[n, k]]``."""
+    return _impl(h).moe_forward(h, logits, up, down, top, ACTIVATIONS[activation], rule, n_up, n_down, correction)

@@ -7,6 +7,7 @@ the same status word.
 from __future__ import annotations
 
 import ctypes
+import functools
 from typing import Optional
 
 import torch
@@ -19,6 +20,26 @@ LIB_PATH = _base._ROOT / "libkvb200_layers.so"
 _CODE = {torch.float32: 0, torch.bfloat16: 1}
 # True: the CUDA-core kernels serve bf16 too (comparisons in tests and benchmarks)
 FORCE_SIMPLE = False
+
+
+class _Attention(ctypes.Structure):
+    """``kvb_attention`` of ``kvb200_layers.h``."""
+
+    _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "maps", "dim", "dimp", "vdim", "vdp", "rot_dims", "value_col", "head_norm",
+                                            "window", "keep", "chunk", "head", "ring", "sink", "gate_cols")]
+    _fields_ += [(n, ctypes.c_float) for n in ("scale", "softcap", "lam", "post", "eps")] + [("sink_w", ctypes.c_void_p)]
+
+
+class _Router(ctypes.Structure):
+    """``kvb_router`` of ``kvb200_layers.h``."""
+
+    _fields_ = [(n, ctypes.c_int) for n in ("score", "groups", "keep", "renormalize")] + [("eps", ctypes.c_float), ("correction", ctypes.c_void_p)]
+
+
+@functools.lru_cache(maxsize=512)
+def _attention(s, plan, eps: float, sink: Optional[int]) -> _Attention:
+    return _Attention(s.heads, s.kv_heads, s.maps, s.dim, s.dimp, s.vdim, s.vdp, s.rot_dims, s.value_col, int(s.head_norm), s.window, s.keep,
+                      s.chunk, plan.head, plan.ring, int(s.sink), s.gate_cols, s.scale, s.softcap, s.lam, s.post, eps, sink)
 
 
 def lib():
@@ -141,11 +162,13 @@ def latent_decode(q_abs, q, ring, seq, shape, scale) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------------------------ sequential layers
-def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center) -> None:
+def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None) -> None:
     width = x_out.shape[-1]
-    _contiguous(x_in, sub, after, x_out, before, h, idx, embed, step)
-    dtype = next((t.dtype for t in (sub, h, embed) if t is not None), torch.float32)
-    _check(lib().kvb_norm_edge(_p(x_in), _p(sub), _p(after), _p(x_out), _p(before), _p(h), _p(idx), _p(embed),
+    out, row, weight = experts if experts is not None else (None, None, None)
+    _contiguous(x_in, sub, after, x_out, before, h, idx, embed, step, out, row, weight)
+    dtype = next((t.dtype for t in (sub, out, h, embed) if t is not None), torch.float32)
+    _check(lib().kvb_norm_edge(_p(x_in), _p(sub), _p(out), _p(row), _p(weight), 0 if weight is None else weight.shape[1],
+                               _ll(0 if out is None else out.shape[1]), _p(after), _p(x_out), _p(before), _p(h), _p(idx), _p(embed),
                                _ll(0 if embed is None else embed.shape[0]), _p(step), _ll(x_out.numel() // width), width, _f(eps), int(center),
                                code(dtype), _p(status_word(x_out.device)), _stream(x_out)), "norm_edge")
     _count()
@@ -155,7 +178,7 @@ def row_norm(x, weight, eps, center, dtype) -> torch.Tensor:
     n, width = x.shape
     y = torch.empty((n, width), dtype=dtype, device=x.device)
     _contiguous(x, weight)
-    _check(lib().kvb_norm_edge(_p(x), None, None, None, _p(weight), _p(y), None, None, _ll(0), None, _ll(n), width, _f(eps), int(center),
+    _check(lib().kvb_norm_edge(_p(x), None, None, None, None, 0, _ll(0), None, None, _p(weight), _p(y), None, None, _ll(0), None, _ll(n), width, _f(eps), int(center),
                                code(dtype), _p(status_word(x.device)), _stream(x)), "row_norm")
     _count()
     return y
@@ -169,39 +192,94 @@ def activate(x, act: int) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------------------------ grouped attention
-def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps) -> torch.Tensor:
+def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan) -> torch.Tensor:
     B, T, ld = qkv.shape
-    q = torch.empty((B, T, s.heads, s.dimp), dtype=qkv.dtype, device=qkv.device)
+    q = torch.empty((B, T, s.heads * s.maps, s.dimp), dtype=qkv.dtype, device=qkv.device)
     _contiguous(qkv, norm_q, norm_k, freq, rows)
+    a = _attention(s, plan, eps, None)
     _check(lib().kvb_grouped_prep(_p(qkv), _ll(ld), _p(norm_q), _p(norm_k), _p(freq), _p(q), _p(rows), _p(seq.slots), _p(seq.start),
-                                  _p(seq.count), B, T, rows.shape[1], s.heads, s.kv_heads, s.dim, s.dimp, s.vdp, s.rot_dims, s.value_col,
-                                  _f(eps), code(qkv.dtype), _stream(qkv)), "grouped_prep")
+                                  _p(seq.count), B, T, rows.shape[1], ctypes.byref(a), code(qkv.dtype), _stream(qkv)), "grouped_prep")
     _count()
     return q
 
 
-def grouped_attend(q, qkv, rows, seq, s) -> torch.Tensor:
+def grouped_attend(q, qkv, rows, seq, s, sink, plan) -> torch.Tensor:
     B, T = q.shape[:2]
     out = torch.empty((B, T, s.heads * s.vdp), dtype=q.dtype, device=q.device)
-    _contiguous(q, qkv, rows)
+    _contiguous(q, qkv, rows, sink)
     gate = qkv.data_ptr() + s.gate_col * qkv.element_size() if s.gate else None
     gate_args = (ctypes.c_void_p(gate), _ll(qkv.shape[-1]))
     where = (_p(seq.slots), _p(seq.start))
     length = rows.shape[1]
-    sizes = (s.heads, s.kv_heads, s.dimp, s.vdp, int(s.sink), _f(s.scale))
+    a = ctypes.byref(_attention(s, plan, s.eps, None if sink is None else sink.data_ptr()))
     fast = q.dtype == torch.bfloat16 and not FORCE_SIMPLE
-    if fast and T == 1 and lib().kvb_grouped_decode_supported(s.dimp, s.vdp):
-        nbytes = int(lib().kvb_grouped_decode_scratch_bytes(B, s.heads, s.kv_heads, s.dimp, s.vdp, length))
+    if fast and T == 1 and lib().kvb_grouped_decode_supported(a):
+        nbytes = int(lib().kvb_grouped_decode_scratch_bytes(B, length, a))
         scratch = torch.empty(nbytes, dtype=torch.uint8, device=q.device) if nbytes else None
-        _check(lib().kvb_grouped_decode(_p(q), _p(rows), *gate_args, _p(out), _p(scratch), *where, B, rows.shape[0], length, *sizes,
+        _check(lib().kvb_grouped_decode(_p(q), _p(rows), *gate_args, _p(out), _p(scratch), *where, B, rows.shape[0], length, a,
                                         _p(status_word(q.device)), _stream(q)), "grouped_decode")
         _count(2 if nbytes else 1)
         return out
-    if fast and T > 1 and lib().kvb_grouped_attend_tc_supported(s.dimp, s.vdp):
-        _check(lib().kvb_grouped_attend_tc(_p(q), _p(rows), *gate_args, _p(out), *where, B, T, rows.shape[0], length, *sizes,
+    if fast and T > 1 and lib().kvb_grouped_attend_tc_supported(a):
+        _check(lib().kvb_grouped_attend_tc(_p(q), _p(rows), *gate_args, _p(out), *where, B, T, rows.shape[0], length, a,
                                            _p(status_word(q.device)), _stream(q)), "grouped_attend_tc")
     else:
-        _check(lib().kvb_grouped_attend(_p(q), _p(rows), *gate_args, _p(out), *where, B, T, length, *sizes, code(q.dtype), _stream(q)), "grouped_attend")
+        _check(lib().kvb_grouped_attend(_p(q), _p(rows), *gate_args, _p(out), *where, B, T, length, a, code(q.dtype), _stream(q)), "grouped_attend")
+    _count()
+    return out
+
+
+# --------------------------------------------------------------------------------------------------- retention
+def _rows_of(t: torch.Tensor) -> int:
+    """Leading dimension of a view of equal columns of contiguous rows ``(B, T, ·)``."""
+    B, T, _ = t.shape
+    if t.stride(2) != 1 or (B > 1 and t.stride(0) != T * t.stride(1)):
+        raise NativeError("rows must lie one behind the other")
+    return t.stride(1)
+
+
+def retention_prep(qk, freq, seq, s, dtype) -> torch.Tensor:
+    B, T, _ = qk.shape
+    out = torch.empty((B, T, s.qk), dtype=dtype, device=qk.device)
+    _check(lib().kvb_retention_prep(_p(qk), _ll(_rows_of(qk)), _p(freq), _p(out), _p(seq.start), B, T, s.heads, s.np, s.rot_dims, _f(s.key_scale),
+                                    code(dtype), _stream(qk)), "retention_prep")
+    _count()
+    return out
+
+
+def retention_scan(qk, v, decay, log2_decay, state, seq, s) -> torch.Tensor:
+    B, T, ldqk = qk.shape
+    y = torch.empty((B, T, s.inner), dtype=qk.dtype, device=qk.device)
+    _contiguous(qk, state)
+    where = (_p(seq.slots), _p(seq.start), _p(seq.count), B, T, s.heads, s.vdp, s.np)
+    if qk.dtype == torch.bfloat16 and not FORCE_SIMPLE and lib().kvb_state_scan_tc_supported(s.heads, s.heads, s.vdp, s.np):
+        nbytes = int(lib().kvb_state_scan_tc_scratch_bytes(B, T, s.heads, s.heads, s.vdp, s.np))
+        scratch = torch.empty(nbytes, dtype=torch.uint8, device=qk.device) if nbytes else None
+        _check(lib().kvb_retention_scan_tc(_p(v), _ll(_rows_of(v)), _p(qk), _ll(ldqk), _p(log2_decay), _p(state), _p(y), _p(scratch), *where,
+                                           _p(status_word(qk.device)), _stream(qk)), "retention_scan_tc")
+        _count(3 if nbytes else 1)
+        return y
+    _check(lib().kvb_retention_scan(_p(v), _ll(_rows_of(v)), _p(qk), _ll(ldqk), _p(decay), _p(state), _p(y), *where, code(qk.dtype), _stream(qk)),
+           "retention_scan")
+    _count()
+    return y
+
+
+def head_norm_gate(y, gate, s, eps) -> torch.Tensor:
+    out = torch.empty_like(y)
+    _contiguous(y)
+    _check(lib().kvb_head_norm_gate(_p(y), _p(gate), _ll(_rows_of(gate)), _p(out), _ll(y.numel() // s.inner), s.heads, s.vdim, s.vdp, _f(eps),
+                                    code(y.dtype), _stream(y)), "head_norm_gate")
+    _count()
+    return out
+
+
+def retention_step(u, freq, decay, state, seq, s, eps, dtype) -> torch.Tensor:
+    B, _, ld = u.shape
+    out = torch.empty((B, 1, s.inner), dtype=dtype, device=u.device)
+    _contiguous(u, state)
+    _check(lib().kvb_retention_step(_p(u), _ll(ld), _p(freq), _p(decay), _p(state), _p(out), _p(seq.slots), _p(seq.start), _p(seq.count), B,
+                                    s.heads, s.vdim, s.vdp, s.np, s.rot_dims, _f(s.key_scale), _f(eps), code(dtype), _stream(u)), "retention_step")
     _count()
     return out
 
@@ -255,6 +333,15 @@ def gated_group_norm(y, u, weight, s, eps) -> torch.Tensor:
     return out
 
 
+def glu(x, ff) -> torch.Tensor:
+    half = x.shape[-1] // 2
+    out = torch.empty((*x.shape[:-1], half), dtype=x.dtype, device=x.device)
+    _contiguous(x)
+    _check(lib().kvb_glu(_p(x), _p(out), _ll(x.numel() // (2 * half)), _ll(2 * half), half, ff, half, code(x.dtype), _stream(x)), "glu")
+    _count()
+    return out
+
+
 # ---------------------------------------------------------------------------------------------- routed experts
 def moe_tile(n_choices: int, n_expert: int, dtype: torch.dtype) -> int:
     """Rows per tile of the grouped products: the expected number of tokens per expert, 16 … 256."""
@@ -267,27 +354,29 @@ def moe_tile(n_choices: int, n_expert: int, dtype: torch.dtype) -> int:
     return tile
 
 
-def moe_forward(h, logits, up, down, top: int, act: int, renormalize: bool, n_up: int, n_down: int):
-    """``h (n, width)``, fp32 router ``logits (n, E)``, ``up (E, ff, ldw)``, ``down (E, width, ldf)`` (rows padded to
-    multiples of 8). Returns ``(expert_out, row (n, top), weight (n, top))``: row of every choice in ``expert_out``."""
+def moe_forward(h, logits, up, down, top: int, act: int, rule, n_up: int, n_down: int, correction=None):
+    """``h (n, width)``, fp32 router ``logits (n, E)``, ``up (E, ff, ldw)`` (gated: ``(E, 2 ff, ldw)``, rows of gate and up in turns),
+    ``down (E, width, ldf)`` (rows padded to multiples of 8). Returns ``(expert_out, row (n, top), weight (n, top))``: row of every choice in ``expert_out``."""
     n, width = h.shape
     E = logits.shape[1]
     dev, dt = h.device, h.dtype
-    _contiguous(h, logits, up, down)
+    _contiguous(h, logits, up, down, correction)
+    router = _Router(int(rule.score == "sigmoid"), rule.groups, rule.keep, int(rule.renormalize), rule.eps,
+                     None if correction is None else correction.data_ptr())
     tile = moe_tile(n * top, E, dt)
     max_tiles = n * top // tile + min(E, n * top)
     ints = torch.empty(E + 2 * n * top + 1 + 2 * max_tiles, dtype=torch.int32, device=dev)
     counters, expert, row, plan, tile_expert, tile_row = torch.split(ints, [E, n * top, n * top, 1, max_tiles, max_tiles])
     weight = torch.empty((n, top), dtype=torch.float32, device=dev)
     _check(lib().kvb_moe_route(_p(logits), _p(expert), _p(weight), _p(row), _p(counters), _p(plan), _p(tile_expert), _p(tile_row), _ll(n), E,
-                               top, tile, max_tiles, int(renormalize), _stream(h)), "moe_route")
+                               top, tile, max_tiles, ctypes.byref(router), _stream(h)), "moe_route")
     ldw, ldf = up.shape[2], down.shape[2]
     ldo = (n_down + 7) // 8 * 8
     sorted_h = torch.empty((max_tiles * tile, ldw), dtype=dt, device=dev)
     _check(lib().kvb_moe_gather(_p(h), _p(row), _p(sorted_h), _ll(n), top, width, _ll(ldw), code(dt), _stream(h)), "moe_gather")
     hidden = torch.empty((max_tiles * tile, ldf), dtype=dt, device=dev)
     st = _p(status_word(dev))
-    _check(lib().kvb_moe_gemm(_p(sorted_h), _p(up), _p(hidden), _p(plan), _p(tile_expert), _p(tile_row), tile, max_tiles, E, n_up, width,
+    _check(lib().kvb_moe_gemm(_p(sorted_h), _p(up), _p(hidden), _p(plan), _p(tile_expert), _p(tile_row), tile, max_tiles, E, up.shape[1], width,
                               _ll(ldw), _ll(ldf), act, code(dt), int(FORCE_SIMPLE), st, _stream(h)), "moe_gemm (up)")
     out = torch.empty((max_tiles * tile, ldo), dtype=dt, device=dev)
     _check(lib().kvb_moe_gemm(_p(hidden), _p(down), _p(out), _p(plan), _p(tile_expert), _p(tile_row), tile, max_tiles, E, n_down, n_up,

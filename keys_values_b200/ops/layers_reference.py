@@ -125,21 +125,43 @@ def latent_decode(q_abs, q, ring, seq, s, scale):
     return out
 
 
-def moe_forward(h, logits, up, down, top, act, renormalize, n_up, n_down):
+def _choose(score, correction, top, rule):
+    choice = score if correction is None else score + correction
+    if rule.groups > 1:
+        n, E = choice.shape
+        parts = choice.view(n, rule.groups, -1)
+        group = parts.topk(min(2, parts.shape[-1]), dim=-1).values.sum(-1)
+        best = torch.sort(group, dim=-1, descending=True, stable=True)[1][:, : rule.keep]
+        seen = torch.zeros_like(group, dtype=torch.bool).scatter_(1, best, True)
+        choice = parts.masked_fill(~seen[..., None], float("-inf")).reshape(n, E)
+    return torch.sort(choice, dim=-1, descending=True, stable=True)[1][:, :top]  # ties: lower index
+
+
+def moe_forward(h, logits, up, down, top, act, rule, n_up, n_down, correction=None):
     n, width = h.shape
-    scores = logits.softmax(-1)
-    weight, expert = (t[:, :top] for t in torch.sort(scores, dim=-1, descending=True, stable=True))  # ties: lower index
-    if renormalize:
-        weight = weight / weight.sum(-1, keepdim=True)
+    scores = logits.softmax(-1) if rule.score == "softmax" else torch.sigmoid(logits)
+    expert = _choose(scores, correction, top, rule)
+    weight = scores.gather(1, expert)
+    if rule.renormalize:
+        weight = weight / (weight.sum(-1, keepdim=True) + rule.eps)
     out = torch.zeros(n * top, (n_down + 7) // 8 * 8, dtype=h.dtype)
     for e in range(logits.shape[1]):
         t, k = torch.where(expert == e)
         if t.numel():
-            z = h[t].float() @ up[e, :n_up, :width].float().t()
+            z = h[t].float() @ up[e, : 2 * n_up if act == 2 else n_up, :width].float().t()
             if act == 1:
                 z = z.relu().square()
+            elif act == 2:
+                z = F.silu(z[:, ::2]) * z[:, 1::2]
             out[t * top + k, :n_down] = (z.to(h.dtype).float() @ down[e, :n_down, :n_up].float().t()).to(h.dtype)
     return out, torch.arange(n * top, dtype=torch.int32).view(n, top), weight
+
+
+def glu(x, ff):
+    n = x.shape[-1] // 2
+    y = F.silu(x[..., :n].float()) * x[..., n:].float()
+    y[..., ff:] = 0
+    return y.to(x.dtype)
 
 
 # ---- sequential layers
@@ -149,10 +171,16 @@ def _norm(x, weight, eps, center):
     return x / torch.sqrt(x.square().mean(-1, keepdim=True) + eps) * weight
 
 
-def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center) -> None:
+def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None) -> None:
     x = torch.zeros_like(x_out) if x_in is None else x_in
-    if sub is not None:
-        x = x + (sub.float() if after is None else _norm(sub.float(), after, eps, center))
+    s = None if sub is None else sub.float()
+    if experts is not None:
+        out, row, weight = experts
+        width = x_out.shape[-1]
+        add = (weight[:, :, None] * out[row.long()][:, :, :width].float()).sum(1).view_as(x_out)
+        s = add if s is None else s + add
+    if s is not None:
+        x = x + (s if after is None else _norm(s, after, eps, center))
     if embed is not None:
         if int(idx.min()) < 0 or int(idx.max()) >= embed.shape[0]:
             raise IndexError("token id outside of the vocabulary")
@@ -160,8 +188,8 @@ def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center)
     if step is not None:
         x = x + step
     x_out.copy_(x)
-    if before is not None:
-        h.copy_(_norm(x, before, eps, center))
+    if h is not None:
+        h.copy_(x if before is None else _norm(x, before, eps, center))
 
 
 def row_norm(x, weight, eps, center, dtype):
@@ -173,38 +201,108 @@ def activate(x, act):
 
 
 # ---- grouped-query attention
-def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps):
+def _places(plan, positions):
+    p = torch.as_tensor(positions)
+    return p if plan.ring == 0 else torch.where(p < plan.head, p, plan.head + (p - plan.head) % plan.ring)
+
+
+def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan):
     B, T, _ = qkv.shape
-    nq, nk = s.heads * s.dimp, s.kv_heads * s.dimp
+    H, G = s.heads * s.maps, s.kv_heads * s.maps
+    nq, nk = H * s.dimp, G * s.dimp
     q, k = qkv[..., :nq].float(), qkv[..., nq : nq + nk].float()
-    if norm_q is not None:  # padding adds nothing to the sums of squares
-        q = q / torch.sqrt(q.square().sum(-1, keepdim=True) / (s.heads * s.dim) + eps) * norm_q
-        k = k / torch.sqrt(k.square().sum(-1, keepdim=True) / (s.kv_heads * s.dim) + eps) * norm_k
+    if norm_q is not None and s.head_norm:
+        q, k = (x.view(B, T, -1, s.dimp) for x in (q, k))
+        q, k = (x / torch.sqrt(x.square().sum(-1, keepdim=True) / s.dim + eps) * w for x, w in ((q, norm_q), (k, norm_k)))
+    elif norm_q is not None:  # padding adds nothing to the sums of squares
+        q = q / torch.sqrt(q.square().sum(-1, keepdim=True) / (H * s.dim) + eps) * norm_q
+        k = k / torch.sqrt(k.square().sum(-1, keepdim=True) / (G * s.dim) + eps) * norm_k
     angle = (seq.start[:, None] + torch.arange(T)).float()[..., None] * freq
     cos, sin = angle.cos()[:, :, None], angle.sin()[:, :, None]
-    q = _rotate(q.view(B, T, s.heads, s.dimp), cos, sin, s.rot_dims).to(qkv.dtype)
-    k = _rotate(k.view(B, T, s.kv_heads, s.dimp), cos, sin, s.rot_dims).to(qkv.dtype)
+    q = _rotate(q.reshape(B, T, H, s.dimp), cos, sin, s.rot_dims).to(qkv.dtype)
+    k = _rotate(k.reshape(B, T, G, s.dimp), cos, sin, s.rot_dims).to(qkv.dtype).reshape(B, T, s.kv_heads, s.maps * s.dimp)
     v = qkv[..., s.value_col : s.value_col + s.kv_heads * s.vdp].view(B, T, s.kv_heads, s.vdp)
     for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
-        rows[slot, start : start + n, :, : s.dimp] = k[b, :n]
-        rows[slot, start : start + n, :, s.dimp :] = v[b, :n]
+        at = _places(plan, torch.arange(start, start + n))
+        rows[slot, at] = torch.cat((k[b, :n], v[b, :n]), -1)
     return q
 
 
-def grouped_attend(q, qkv, rows, seq, s):
+def _seen(s, query, key):
+    """Which of the positions ``key (N,)`` each of ``query (T,)`` sees."""
+    i, j = query[:, None], key[None]
+    seen = j <= i
+    if s.chunk:
+        return seen & (i // s.chunk == j // s.chunk)
+    return seen & ((i - j < s.window) | (j < s.keep)) if s.window else seen
+
+
+def grouped_attend(q, qkv, rows, seq, s, sink, plan):
     B, T = q.shape[:2]
     out = torch.zeros(B, T, s.heads, s.vdp)
     for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
-        kv = rows[slot, : start + n].float().repeat_interleave(s.heads // s.kv_heads, dim=1)
-        score = torch.einsum("thd,jhd->htj", q[b, :n].float(), kv[..., : s.dimp]) * s.scale
-        score = score.masked_fill(torch.arange(start + n) > start + torch.arange(n)[:, None], float("-inf"))
-        if s.sink:
-            score = torch.cat((score, torch.zeros(s.heads, n, 1)), dim=-1)
-        out[b, :n] = torch.einsum("htj,jhv->thv", score.softmax(-1)[..., : start + n], kv[..., s.dimp :])
-    out = out.view(B, T, -1)
+        if n == 0:
+            continue
+        key = torch.arange(start + n)
+        if plan.ring:  # positions that are seen no more have lost their rows
+            key = key[(key < plan.head) | (key > start - s.span)]
+        kv = rows[slot, _places(plan, key)].float().repeat_interleave(s.heads // s.kv_heads, dim=1)
+        hidden = ~_seen(s, start + torch.arange(n), key)
+        maps = []
+        for u in range(s.maps):
+            score = torch.einsum("thd,jhd->htj", q[b, :n, u :: s.maps].float(), kv[..., u * s.dimp : (u + 1) * s.dimp]) * s.scale
+            if s.softcap:
+                score = s.softcap * torch.tanh(score / s.softcap)
+            score = score.masked_fill(hidden, float("-inf"))
+            if s.sink:
+                add = torch.zeros(s.heads) if sink is None else sink
+                score = torch.cat((score, add.view(-1, 1, 1).expand(-1, n, 1)), dim=-1)
+            maps.append(torch.einsum("htj,jhv->thv", score.softmax(-1)[..., : len(key)], kv[..., s.maps * s.dimp :]))
+        if s.maps == 2:
+            d = maps[0] - s.lam * maps[1]
+            maps[0] = d / torch.sqrt(d.square().sum(-1, keepdim=True) / s.vdim + s.eps) * s.post
+        out[b, :n] = maps[0]
     if s.gate:
-        out = out * torch.sigmoid(qkv[..., s.gate_col :].float())
-    return out.to(q.dtype)
+        gate = torch.sigmoid(qkv[..., s.gate_col : s.gate_col + s.heads * s.gate_cols].float())
+        out = out * gate.view(B, T, s.heads, s.gate_cols)
+    return out.view(B, T, -1).to(q.dtype)
+
+
+# ---- retention
+def retention_prep(qk, freq, seq, s, dtype):
+    B, T, _ = qk.shape
+    x = qk[..., : s.qk].view(B, T, 2 * s.heads, s.np)
+    angle = (seq.start[:, None] + torch.arange(T)).float()[..., None] * freq
+    x = _rotate(x, angle.cos()[:, :, None], angle.sin()[:, :, None], s.rot_dims).clone()
+    x[:, :, s.heads :] *= s.key_scale
+    return x.reshape(B, T, s.qk).to(dtype)
+
+
+def retention_scan(qk, v, decay, log2_decay, state, seq, s):
+    B, T = qk.shape[:2]
+    q, k = qk.float().view(B, T, 2, s.heads, s.np).unbind(2)
+    v = v[..., : s.inner].float().reshape(B, T, s.heads, s.vdp)
+    y = torch.zeros(B, T, s.heads, s.vdp)
+    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
+        S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+        for t in range(n):
+            S = decay[:, None, None] * S + k[b, t, :, :, None] * v[b, t, :, None]
+            y[b, t] = torch.einsum("hnp,hn->hp", S, q[b, t])
+        if n > 0:
+            state[slot] = S
+    return y.view(B, T, -1).to(qk.dtype)
+
+
+def head_norm_gate(y, gate, s, eps):
+    x = y.float().view(*y.shape[:-1], s.heads, s.vdp)
+    x = x / torch.sqrt(x.square().sum(-1, keepdim=True) / s.vdim + eps)
+    return (x.view(y.shape) * F.silu(gate[..., : s.inner].float())).to(y.dtype)
+
+
+def retention_step(u, freq, decay, state, seq, s, eps, dtype):
+    qk = retention_prep(u, freq, seq, s, torch.float32)
+    y = retention_scan(qk, u[..., s.qk :], decay, None, state, seq, s)
+    return head_norm_gate(y, u[..., s.qk + s.inner :], s, eps).to(dtype)
 
 
 # ---- state-space recurrence

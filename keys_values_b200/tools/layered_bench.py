@@ -275,7 +275,7 @@ def kernel_table(config: Config, batch: int, tokens: int = 8192, dense_like: boo
         logits = torch.randn(n, E, device=dev)
         used = E if n * top >= 4 * E else E * (1 - (1 - 1 / E) ** (n * top))
         tab.add(f"{tag}: routed experts, all kernels ({E} x {ff}, top {top})",
-                lambda: LC.moe_forward(hn, logits, up, down, top, 1, False, ff, W),
+                lambda: LC.moe_forward(hn, logits, up, down, top, 1, L.RouterRule(), ff, W),
                 gbytes=2 * (used * 2 * ff * W + n * W * (1 + top)) / 1e9, tflop=4 * n * top * ff * W / 1e12)
         from keys_values_b200.models.model import LLaMAMLP, LLaMAMoE
 

@@ -381,7 +381,7 @@ def experts(env, n, E, top, width, ff, seed, renormalize=False, spread=2.0):
     down = pad(torch.stack([w[f"e{e}.down"] for e in range(E)]), L.round8(ff)).to(dev)
     logits = L.linear_fp32(h.to(dev), w["router"].to(dev))
     assert logits.dtype == torch.float32
-    out, row, weight = L.routed_experts(h.to(dev), logits, up, down, top, "relu_squared", renormalize, ff, width)
+    out, row, weight = L.routed_experts(h.to(dev), logits, up, down, top, "relu_squared", L.RouterRule(renormalize=renormalize), ff, width)
     y = (weight[..., None] * out[row.long()][..., :width].float()).sum(1)
     return h.double(), {k: v.double() for k, v in w.items()}, y, weight, logits
 
@@ -418,15 +418,15 @@ def test_routing_weights_ties_and_unused_experts(env):
     logits[:, 4] = 2.0
     logits[:, 6] = 2.0
     logits[:, 2] = 0.5
-    out, row, weight = L.routed_experts(h.to(dev), logits.to(dev), up.to(dev), down.to(dev), 3, "relu_squared", False, ff, width)
+    out, row, weight = L.routed_experts(h.to(dev), logits.to(dev), up.to(dev), down.to(dev), 3, "relu_squared", L.RouterRule(), ff, width)
     s = torch.softmax(logits.double(), -1)
     close(weight, s[:, [4, 6, 2]], torch.float32)
     relu2 = h.double().clamp(min=0) ** 2
     for k, e in enumerate((4, 6, 2)):
         close(out[row[:, k].long()][:, :width], (e + 1) * relu2, dtype)
     assert len(set(row.view(-1).tolist())) == 3 * n
-    _, _, weight = L.routed_experts(h.to(dev), logits.to(dev), up.to(dev), down.to(dev), 3, "relu_squared", True, ff, width)
+    _, _, weight = L.routed_experts(h.to(dev), logits.to(dev), up.to(dev), down.to(dev), 3, "relu_squared", L.RouterRule(renormalize=True), ff, width)
     close(weight.sum(-1), torch.ones(n), torch.float32)
     # all scores equal
-    _, _, weight = L.routed_experts(h.to(dev), torch.zeros(n, E, device=dev), up.to(dev), down.to(dev), 2, "none", False, ff, width)
+    _, _, weight = L.routed_experts(h.to(dev), torch.zeros(n, E, device=dev), up.to(dev), down.to(dev), 2, "none", L.RouterRule(), ff, width)
     close(weight, torch.full((n, 2), 1 / 9), torch.float32)
