@@ -387,8 +387,8 @@ configs: List[dict] = [
         **_ladadra(2048, [
             dict(mixer=_retention(16, 128, 128), mlp=_gated(5632)),
             dict(mixer=_differential(16, 4, 64, 128, window=4096, keep_first=128, differential=0.5), mlp=_grouped_experts(64, 6, 704, 8, 4, 1408)),
-            dict(mixer=_chunked(16, 4, 128, 128, chunk=8192, rope_dims=64), mlp=_gated(5632)),
-            dict(mixer=_chunked(16, 4, 128, 128, chunk=8192, rope_dims=64), mlp=_grouped_experts(64, 6, 704, 8, 4, 1408)),
+            dict(mixer=_chunked(16, 4, 128, 128, chunk=16384, rope_dims=64), mlp=_gated(5632)),
+            dict(mixer=_chunked(16, 4, 128, 128, chunk=16384, rope_dims=64), mlp=_grouped_experts(64, 6, 704, 8, 4, 1408)),
         ] * 4),
     ),
     dict(
@@ -396,8 +396,8 @@ configs: List[dict] = [
         **_ladadra(4096, [
             dict(mixer=_retention(32, 128, 128), mlp=_gated(11008)),
             dict(mixer=_differential(32, 8, 64, 128, window=4096, keep_first=128, differential=0.5), mlp=_grouped_experts(32, 4, 2048, 4, 2, 2816)),
-            dict(mixer=_chunked(32, 8, 128, 128, chunk=8192, rope_dims=64), mlp=_gated(11008)),
-            dict(mixer=_chunked(32, 8, 128, 128, chunk=8192, rope_dims=64), mlp=_grouped_experts(32, 4, 2048, 4, 2, 2816)),
+            dict(mixer=_chunked(32, 8, 128, 128, chunk=16384, rope_dims=64), mlp=_gated(11008)),
+            dict(mixer=_chunked(32, 8, 128, 128, chunk=16384, rope_dims=64), mlp=_grouped_experts(32, 4, 2048, 4, 2, 2816)),
         ] * 3),
     ),
     # Qwen 2.5

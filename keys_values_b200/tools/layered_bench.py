@@ -5,8 +5,9 @@ time of every kernel of the design beside the like kernel of that model, each ag
 
 Random-init weights, synthetic tokens. For Mezilix the closest model has the same width, depth, heads, window and experts
 (count, chosen per token, expert weights per token): grouped-query attention over a sliding window, SwiGLU experts
-(``LLaMAMoE``), or a dense SwiGLU of the width that a token's chosen experts add up to. For Pazenex it has the same width, depth,
-heads and key/value heads, attention in every layer and a dense SwiGLU that makes the number of weights equal. Kernel times are
+(``LLaMAMoE``), or a dense SwiGLU of the width that a token's chosen experts add up to. For Pazenex and Ladadra it has the same width,
+depth, heads and key/value heads, attention in every layer and a dense SwiGLU that makes the number of weights that a token meets
+equal. Kernel times are
 CUDA-event medians with an L2 flush (256 MB written, another 256 MB read) before every launch.
 """
 from __future__ import annotations
@@ -38,19 +39,31 @@ def closest_config(config: Config, dense: bool = False) -> Config:
     return Config(mlp_class_name="LLaMAMoE", intermediate_size=ff, moe_intermediate_size=ff, n_expert=f["n_expert"], n_expert_per_token=f["top"], **kw)
 
 
+def layer_weights(layer: Dict, width: int) -> int:
+    """Weights of the products that a token meets in one sequential layer."""
+    x, f = layer["mixer"], layer["mlp"]
+    if x["kind"] == "mamba2":
+        inner, bc = x["n_head"] * x["v_dim"], x["groups"] * x["state"]
+        n = width * (3 * inner + 2 * bc + x["n_head"])
+    elif x["kind"] == "retention":
+        n = width * x["n_head"] * (2 * x["dim"] + 3 * x["v_dim"])
+    else:
+        maps = 1 if x.get("differential") is None else 2
+        H, G = x["n_head"], x["n_kv_head"]
+        n = width * ((H + G) * maps * x["dim"] + H * x["v_dim"])
+        n += width * ((0 if x.get("shared_value") else G * x["v_dim"]) + {True: H * x["v_dim"], "head": H}.get(x.get("gate"), 0))
+    if f is None:
+        return n
+    if f["kind"] == "routed":
+        return n + width * (f["n_expert"] + 3 * (f["top"] * f["ff"] + (f.get("shared") or 0)))
+    return n + (3 if f["kind"] == "gated" else 2) * width * f["ff"]
+
+
 def closest_attention_config(config: Config) -> Config:
-    """Llama-shaped model of the same depth, width, heads and number of layer weights."""
+    """Llama-shaped model of the same depth, width, heads and number of layer weights that a token meets."""
     m = next(x["mixer"] for x in config.layers if x["mixer"]["kind"] == "grouped_attention")
     H, G, W, n = m["n_head"], m["n_kv_head"], config.n_embd, config.n_layer
-    weights = 0
-    for layer in config.layers:
-        x = layer["mixer"]
-        if x["kind"] == "mamba2":
-            inner, bc = x["n_head"] * x["v_dim"], x["groups"] * x["state"]
-            weights += W * (3 * inner + 2 * bc + x["n_head"])
-        else:
-            weights += W * (3 * x["n_head"] + x["n_kv_head"]) * x["dim"]
-        weights += 2 * W * layer["mlp"]["ff"]
+    weights = sum(layer_weights(layer, W) for layer in config.layers)
     ff = (weights // n - W * (2 * H + 2 * G) * 128) // (3 * W) // 8 * 8
     return Config(
         name=f"closest-to-{config.name}", block_size=1 << 17, vocab_size=config.vocab_size, padded_vocab_size=config.padded_vocab_size, n_layer=n,
@@ -183,6 +196,8 @@ def _window_pairs(T: int, P: int, window: int) -> int:
 def kernel_table(config: Config, batch: int, tokens: int = 8192, dense_like: bool = True) -> List[Dict]:
     """Kernels of one middle layer of ``config`` (Pazenex: of one layer of each kind): a pass of ``tokens`` new tokens of one sequence with a full window before them,
     and a single-token pass of ``batch`` sequences with full rings; like kernels of the closest model after each."""
+    if any(x["mixer"]["kind"] == "retention" for x in config.layers):
+        return output_norm_kernel_table(config, batch, tokens)
     if any(x["mixer"]["kind"] != "latent_attention" for x in config.layers):
         return sequential_kernel_table(config, batch, tokens)
     from keys_values_b200 import ops
@@ -326,6 +341,7 @@ def sequential_kernel_table(config: Config, batch: int, tokens: int = 8192) -> L
     from keys_values_b200.models.grouped_attention import grouped_shape
     from keys_values_b200.models.state_space import state_shape
     from keys_values_b200.ops import cuda as cu
+    from keys_values_b200.ops import layers as L
     from keys_values_b200.ops import layers_cuda as LC
 
     dev, bf = torch.device("cuda"), torch.bfloat16
@@ -362,7 +378,7 @@ def sequential_kernel_table(config: Config, batch: int, tokens: int = 8192) -> L
         length = tokens + 64
         rows = rand(B, length, G, D + s.vdp)
         kv_bytes = 2 * n * G * (D + s.vdp)
-        tab.add(f"{tag}: norm, rotation, into the cache", lambda: LC.grouped_prep(qkv, nq, nk, freq, rows, seq, s, eps),
+        tab.add(f"{tag}: norm, rotation, into the cache", lambda: LC.grouped_prep(qkv, nq, nk, freq, rows, seq, s, eps, L.RowPlan()),
                 gbytes=(2 * n * (2 * H * D + G * D) + kv_bytes) / 1e9)
         qkv2, cs, wq = rand(B, T, (H + 2 * G) * D), f32(T, D), rand(D)
         tab.add(f"{tag}:   like: QK norm, split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, H, G, D, eps, D, False),
@@ -371,12 +387,12 @@ def sequential_kernel_table(config: Config, batch: int, tokens: int = 8192) -> L
         q2, k2 = rand(B, H, T, D), rand(B, G, tokens, D)
         if T > 1:
             flop = B * H * (T * (T + 1) // 2) * 2 * (s.dim + s.vdim) / 1e12
-            tab.add(f"{tag}: attention, {H} heads on {G}, sink and gate", lambda: LC.grouped_attend(q, qkv, rows, seq, s), tflop=flop)
+            tab.add(f"{tag}: attention, {H} heads on {G}, sink and gate", lambda: LC.grouped_attend(q, qkv, rows, seq, s, None, L.RowPlan()), tflop=flop)
             tab.add(f"{tag}:   like: attention, {H} heads on {G}", lambda: cu.sdpa_fwd(q2, k2, k2, 0.09, 0), tflop=flop)
         else:
             by = 2 * B * G * tokens * (s.dim + s.vdim) / 1e9
             v2 = rand(B, G, tokens, D)
-            tab.add(f"{tag}: attention over {tokens} positions, {H} heads on {G}", lambda: LC.grouped_attend(q, qkv, rows, seq, s), gbytes=by)
+            tab.add(f"{tag}: attention over {tokens} positions, {H} heads on {G}", lambda: LC.grouped_attend(q, qkv, rows, seq, s, None, L.RowPlan()), gbytes=by)
             tab.add(f"{tag}:   like: attention over {tokens} slots", lambda: cu.decode_attention(q2, k2, v2, 0.09, tokens), gbytes=by)
         del rows, k2, q2, q, qkv2
         # ---- state space
@@ -403,6 +419,155 @@ def sequential_kernel_table(config: Config, batch: int, tokens: int = 8192) -> L
             tab.add(f"{tag}: library product {what} {n} x {cols_out} x {k}", lambda: torch.mm(a2, w3.t()), gbytes=2 * (n * (k + cols_out) + k * cols_out) / 1e9,
                     tflop=2 * n * k * cols_out / 1e12)
         del u, y, a2, w3, x, sub, h
+    ops.check_status(dev)
+    return tab.rows
+
+
+def _like_mlp(width: int, ff: int, dev, dtype):
+    from keys_values_b200.models.model import LLaMAMLP
+
+    c = Config(name="like", n_layer=1, n_embd=width, n_head=1, head_size=width, vocab_size=8, padded_vocab_size=8, bias=False, norm_class_name="RMSNorm",
+               mlp_class_name="LLaMAMLP", intermediate_size=ff)
+    with torch.device(dev):
+        return LLaMAMLP(c).to(dtype)
+
+
+@torch.inference_mode()
+def output_norm_kernel_table(config: Config, batch: int, tokens: int = 8192) -> List[Dict]:
+    """Kernels of one layer of each kind of a model with retention, differential and chunked attention: prompts of ``tokens`` tokens, and a
+    single-token pass of ``batch`` sequences at that position; like kernels of the closest model after each."""
+    from keys_values_b200 import ops
+    from keys_values_b200.kvcache.sequences import SequenceTable
+    from keys_values_b200.models.grouped_attention import grouped_shape
+    from keys_values_b200.models.layered import RoutedMLP
+    from keys_values_b200.models.retention import retention_shape
+    from keys_values_b200.ops import cuda as cu
+    from keys_values_b200.ops import layers as L
+    from keys_values_b200.ops import layers_cuda as LC
+
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    tab = KernelTable()
+    mixers = [x["mixer"] for x in config.layers]
+    diff = grouped_shape(next(x for x in mixers if x.get("differential") is not None))
+    diff = L.GroupedShape(**{**diff.__dict__, "lam": 0.4, "eps": config.norm_eps})
+    chunked = grouped_shape(next(x for x in mixers if x.get("chunk")))
+    r = retention_shape(next(x for x in mixers if x["kind"] == "retention"))
+    mlps = [x["mlp"] for x in config.layers if x["mlp"]]
+    ff, f = next(x["ff"] for x in mlps if x["kind"] == "gated"), next(x for x in mlps if x["kind"] == "routed")
+    W, eps = config.n_embd, config.norm_eps
+    plan = L.RowPlan()
+    rand = lambda *shape: torch.randn(*shape, device=dev, dtype=bf)  # noqa: E731
+    f32 = lambda *shape: torch.rand(*shape, device=dev)  # noqa: E731
+    with torch.device(dev):
+        routed = RoutedMLP(config, {**f, "shared": None}).to(bf)
+        torch.nn.init.normal_(routed.gate.weight, std=0.02)
+    shared_mlp, active_mlp = _like_mlp(W, f["shared"], dev, bf), _like_mlp(W, f["top"] * f["ff"], dev, bf)
+    for B, T, start in ((1, tokens, 0), (4, tokens, 0), (batch, 1, tokens - 1)):
+        n = B * T
+        tag = f"prefill {B} x {T} tokens" if T > 1 else f"decode {B} rows"
+        table = SequenceTable(B, dev)
+        table.set_batch([table.acquire() for _ in range(B)])
+        table.pos.fill_(start)
+        table.pos_host = [start] * B
+        seq = table.begin(B, T)
+        seq.start = seq.start.clone()
+        # ---- between sublayers
+        x, sub, h, w1 = torch.randn(B, T, W, device=dev), rand(B, T, W), rand(B, T, W), f32(W)
+        tab.add(f"{tag}: norm, residual sum", lambda: LC.norm_edge(x, sub, w1, x, None, h, None, None, None, eps, False), gbytes=n * W * 12 / 1e9)
+        a, rr, w = rand(n, W), rand(n, W), rand(W)
+        fused = cu.add_rmsnorm_supported(a)
+        like_norm = lambda: cu.add_rmsnorm_fwd(a, rr, w, eps, False) if fused else cu.rmsnorm_fwd(a, w, eps, False)  # noqa: E731
+        norm_bytes = n * W * (8 if fused else 4) / 1e9
+        tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+        top = f["top"]
+        experts = (rand(n * top, W), torch.randperm(n * top, device=dev).int().view(n, top), f32(n, top))
+        tab.add(f"{tag}: sum of {top} experts and shared, norm, residual sum",
+                lambda: LC.norm_edge(x, sub, w1, x, None, h, None, None, None, eps, False, experts), gbytes=n * W * (12 + 2 * top) / 1e9)
+        del experts
+        up = rand(n, 2 * ff)
+        tab.add(f"{tag}: SwiGLU", lambda: LC.glu(up, ff), gbytes=n * ff * 6 / 1e9)
+        u1 = up.view(2, n, ff)
+        tab.add(f"{tag}:   like: SwiGLU", lambda: cu.swiglu_fwd(u1[0], u1[1]), gbytes=n * ff * 6 / 1e9)
+        del up, u1
+        # ---- attentions
+        length = tokens + 64
+        for what, s in (("chunked", chunked), ("differential", diff)):
+            H, G, D, V = s.heads, s.kv_heads, s.dim, s.vdim
+            qkv = rand(B, T, s.ld)
+            if s.head_norm:
+                nq, nk = f32(s.dimp), f32(s.dimp)
+            else:
+                nq, nk = f32(H * s.dimp), f32(G * s.dimp)
+            freq, sink = f32(s.rot_dims // 2), torch.zeros(H, device=dev) if s.sink else None
+            rows = rand(B, length, G, s.row)
+            tab.add(f"{tag}: {what}: norm, rotation, into the cache", lambda: LC.grouped_prep(qkv, nq, nk, freq, rows, seq, s, eps, plan),
+                    gbytes=2 * n * (2 * H * s.maps * D + 2 * G * (s.maps * D + V)) / 1e9)
+            qkv2, cs, wq = rand(B, T, (H + 2 * G) * 128), f32(T, 128), rand(128)
+            tab.add(f"{tag}:   like: QK norm, split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, H, G, 128, eps, 128, False),
+                    gbytes=2 * 2 * n * (H + 2 * G) * 128 / 1e9)
+            q = rand(B, T, H * s.maps, s.dimp)
+            seen = s.window or 1 << 40
+            q2, k2 = rand(B, H, T, 128), rand(B, G, tokens, 128)
+            win = s.window if s.window and s.window < tokens else 0
+            if T > 1:
+                pairs = B * H * (_window_pairs(T, 0, seen) + (min(s.keep, T) * max(0, T - seen) if s.window else 0))
+                tab.add(f"{tag}: {what} attention, {H} heads on {G}" + (f", window {s.window} + {s.keep}" if s.window else ", soft cap, sink, gate"),
+                        lambda: LC.grouped_attend(q, qkv, rows, seq, s, sink, plan), tflop=2 * pairs * s.maps * (D + V) / 1e12)
+                like = B * H * _window_pairs(T, 0, seen)
+                tab.add(f"{tag}:   like: attention 128 / 128" + (f", window {win}" if win else ""),
+                        lambda: cu.sdpa_fwd(q2, k2, k2, 0.09, 0, None, False, win, None) if win else cu.sdpa_fwd(q2, k2, k2, 0.09, 0), tflop=2 * like * 256 / 1e12)
+            else:
+                m = min(tokens, seen) + (s.keep if win else 0)
+                tab.add(f"{tag}: {what} attention over {m} positions, {H} heads on {G}", lambda: LC.grouped_attend(q, qkv, rows, seq, s, sink, plan),
+                        gbytes=2 * B * G * m * (s.maps * D + V) / 1e9)
+                m2 = min(tokens, seen)
+                k3, v3 = rand(B, G, m2, 128), rand(B, G, m2, 128)
+                tab.add(f"{tag}:   like: attention over {m2} slots", lambda: cu.decode_attention(q2, k3, v3, 0.09, m2), gbytes=2 * B * G * m2 * 256 / 1e9)
+                del k3, v3
+            del rows, k2, q2, q, qkv2, qkv
+        # ---- retention
+        state, decay = 0.01 * torch.randn(B, r.heads, r.np, r.vdp, device=dev), 1 - 0.05 * f32(r.heads)
+        log2, freq = decay.log2(), f32(r.rot_dims // 2)
+        state_bytes = B * r.heads * r.np * r.vdp * 8
+        if T > 1:
+            qk32, vg = torch.randn(B, T, r.qk, device=dev), rand(B, T, 2 * r.inner)
+            tab.add(f"{tag}: retention: rotation", lambda: LC.retention_prep(qk32, freq, seq, r, bf), gbytes=6 * n * r.qk / 1e9)
+            qkv2, cs, wq = rand(B, T, 2 * r.qk), f32(T, 128), rand(128)
+            tab.add(f"{tag}:   like: QK norm, split + RoPE",
+                    lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, 2 * r.qk // 384, r.qk // 384, 128, eps, 128, False) if r.qk % 384 == 0
+                    else cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, 2 * r.qk // 128 - 16, 8, 128, eps, 128, False), gbytes=8 * n * r.qk / 1e9)
+            qk = rand(B, T, r.qk)
+            flop = n * r.heads * (4 * r.np * r.vdp + 128 * (r.np + r.vdp)) / 1e12
+            tab.add(f"{tag}: retention scan, {r.heads} heads of {r.np} x {r.vdp}", lambda: LC.retention_scan(qk, vg, decay, log2, state, seq, r),
+                    gbytes=(2 * n * (r.qk + 2 * r.inner) + state_bytes) / 1e9, tflop=flop)
+            q2 = rand(B, r.heads, T, 128)
+            tab.add(f"{tag}:   like: attention 128 / 128, {r.heads} heads", lambda: cu.sdpa_fwd(q2, q2, q2, 0.09, 0),
+                    tflop=2 * B * r.heads * (T * (T + 1) // 2) * 256 / 1e12)
+            y = rand(B, T, r.inner)
+            tab.add(f"{tag}: retention: norm per head, gate", lambda: LC.head_norm_gate(y, vg[..., r.inner :], r, eps), gbytes=6 * n * r.inner / 1e9)
+            tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+            del qk32, vg, qk, q2, qkv2, y
+        else:
+            u = torch.randn(B, 1, r.qk + 2 * r.inner, device=dev)
+            tab.add(f"{tag}: retention step, {r.heads} heads of {r.np} x {r.vdp}", lambda: LC.retention_step(u, freq, decay, state, seq, r, eps, bf),
+                    gbytes=(state_bytes + 4 * n * u.shape[-1]) / 1e9)
+        del state
+        # ---- feed-forwards
+        hn = rand(n, W)
+        E = f["n_expert"]
+        used = E if n * top >= 4 * E else E * (1 - (1 - 1 / E) ** (n * top))
+        tab.add(f"{tag}: routed experts, all kernels ({E} x {f['ff']}, top {top})", lambda: routed(hn),
+                gbytes=2 * (used * 3 * f["ff"] * W + n * W * (1 + top)) / 1e9, tflop=6 * n * top * f["ff"] * W / 1e12)
+        tab.add(f"{tag}:   like: dense SwiGLU of {top * f['ff']}, all kernels", lambda: active_mlp(hn.view(1, n, W)),
+                gbytes=2 * (3 * top * f["ff"] * W + 2 * n * W) / 1e9, tflop=6 * n * top * f["ff"] * W / 1e12)
+        tab.add(f"{tag}: shared expert (library products, SwiGLU)", lambda: shared_mlp(hn.view(1, n, W)),
+                gbytes=2 * (3 * f["shared"] * W + 2 * n * W) / 1e9, tflop=6 * n * f["shared"] * W / 1e12)
+        w3 = rand(r.qk, W)
+        tab.add(f"{tag}: library product with fp32 result {n} x {r.qk} x {W}", lambda: L.linear_fp32(hn, w3),
+                gbytes=(2 * n * W + 2 * r.qk * W + 4 * n * r.qk) / 1e9, tflop=2 * n * r.qk * W / 1e12)
+        tab.add(f"{tag}:   like: with bf16 result", lambda: torch.mm(hn, w3.t()), gbytes=2 * (n * W + r.qk * W + n * r.qk) / 1e9, tflop=2 * n * r.qk * W / 1e12)
+        del hn, w3, x, sub, h, a, rr
+        torch.cuda.empty_cache()
     ops.check_status(dev)
     return tab.rows
 

@@ -241,8 +241,9 @@ def content(layers, width=40, vocab=61, eps=1e-4):
     return {"architecture": "Ladadra", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": layers}
 
 
-def tensors(c, seed=0):
-    """Random bf16 tensors. Norm weights, sinks, biases and corrections differ from what would hide them."""
+def tensors(c, seed=0, decided=False):
+    """Random bf16 tensors. Norm weights, sinks, biases and corrections differ from what would hide them. ``decided``: corrections so far
+    apart that rounding changes no choice of experts."""
     g = torch.Generator().manual_seed(seed)
 
     def mat(*shape, gain=1.0):
@@ -284,6 +285,8 @@ def tensors(c, seed=0):
         for e in range(E):
             glu(f"{p}mlp.e{e}.", f["expert"]["ff"])
         w.update({p + "mlp.router": mat(E, W, gain=2.0), p + "mlp.correction": near(-0.4, E, spread=0.5)})
+        if decided:
+            w[p + "mlp.correction"] = 3 * 1.8 ** torch.randperm(E, generator=g).float()
         if f.get("shared"):
             glu(p + "mlp.shared.", f["shared"]["ff"])
     return {k: v.to(torch.bfloat16) for k, v in w.items()}
