@@ -33,14 +33,30 @@ __device__ __forceinline__ float attn_rcp(float x) {
 // tanh z = 1 - 2 / (1 + e^2z): absolute error of the order of 1e-7, which is what a soft cap wants (cap · tanh(score / cap) is a sum's exponent)
 __device__ __forceinline__ float cap_tanh(float z) { return fmaf(-2.f, attn_rcp(1.f + attn_exp2(2.f * ATTN_LOG2E * z)), 1.f); }
 
-// The same by the Taylor series up to z^9 for |z| <= 0.3 (what it leaves out is below 1e-7 of the result), two values at a time.
+// Below CAP_SERIES tanh z = z (1 - z^2/3 + 2 z^4/15 - 17 z^6/315 + 62 z^8/2835), which leaves out less than 1e-7 of the result. A score that is
+// capped that way is a polynomial in its square times the score: the coefficients take the factors on both sides.
 constexpr float CAP_SERIES = 0.3f;
-__device__ __forceinline__ float2 cap_tanh_series(float2 z) {
-  const float2 q = fmul2(z, z);
-  float2 r = ffma2(q, make_float2(62.f / 2835.f, 62.f / 2835.f), make_float2(-17.f / 315.f, -17.f / 315.f));
-  r = ffma2(q, r, make_float2(2.f / 15.f, 2.f / 15.f));
-  r = ffma2(q, r, make_float2(-1.f / 3.f, -1.f / 3.f));
-  return ffma2(fmul2(q, r), z, z);
+struct CapSeries {
+  float c0, c1, c2, c3, c4;
+  __host__ __device__ __forceinline__ CapSeries(float in, float out) {
+    const float q = in * in;
+    c0 = in * out;
+    c1 = c0 * q * (-1.f / 3.f);
+    c2 = c0 * q * q * (2.f / 15.f);
+    c3 = c0 * q * q * q * (-17.f / 315.f);
+    c4 = c0 * q * q * q * q * (62.f / 2835.f);
+  }
+  // with a last coefficient that has underflowed, minus infinity would not stay what it is
+  __host__ __device__ __forceinline__ bool usable() const { return c4 > 1e-37f; }
+};
+// out · tanh(in · x) + add, two values at a time; minus infinity stays
+__device__ __forceinline__ float2 cap_series(const CapSeries& s, float2 x, float2 add) {
+  const float2 q = fmul2(x, x);
+  float2 r = ffma2(q, make_float2(s.c4, s.c4), make_float2(s.c3, s.c3));
+  r = ffma2(q, r, make_float2(s.c2, s.c2));
+  r = ffma2(q, r, make_float2(s.c1, s.c1));
+  r = ffma2(q, r, make_float2(s.c0, s.c0));
+  return ffma2(x, r, add);
 }
 
 }  // namespace kvb

@@ -48,6 +48,50 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
   const T* src = qkv + n * p.ld;
   const int nq = p.heads * p.dimp, nk = p.kv_heads * p.dimp;
   for (int k = threadIdx.x; k < half; k += GP_THREADS) sincosf((float)pos * p.freq[k], &cs_sm[half + k], &cs_sm[k]);
+  const int maps = p.a.maps, row = maps * p.dimp + p.vdp, place = row_of(p.a, pos);
+  // where the token's keys and values go; padding goes nowhere
+  T* const dst = (t < p.count[b] && place < p.len) ? rows + ((long long)p.slots[b] * p.len + place) * p.a.kv_heads * row : nullptr;
+  const bool shared = p.value_col == nq;
+  // one piece of a head: the key part of the cache or the query
+  auto put = [&](int h, int col, const Vec& v) {
+    if (h < p.heads) *reinterpret_cast<Vec*>(q + (n * p.heads + h) * p.dimp + col) = v;
+    else if (dst) {
+      const int k = h - p.heads, g = maps == 1 ? k : k / maps;
+      *reinterpret_cast<Vec*>(dst + g * row + (k - g * maps) * p.dimp + col) = v;
+    }
+  };
+  auto put_values = [&]() {
+    for (int i = threadIdx.x * V; i < p.a.kv_heads * p.vdp; i += GP_THREADS * V) {
+      const int g = i / p.vdp;
+      *reinterpret_cast<Vec*>(dst + g * row + maps * p.dimp + i - g * p.vdp) = *reinterpret_cast<const Vec*>(src + p.value_col + i);
+    }
+  };
+  const int per_head = p.dimp / V;
+  if (p.norm_q && p.a.head_norm && half == 0 && !shared && per_head <= 32 && (per_head & (per_head - 1)) == 0) {
+    // nothing is rotated and a head lies in neighbouring lanes: one pass without shared memory
+    if (dst) put_values();
+    const int total = (nq + nk) / V;
+#pragma unroll 4
+    for (int i0 = 0; i0 < total; i0 += GP_THREADS) {
+      const int i = i0 + threadIdx.x;
+      Vec a;
+      float s = 0.f;
+      if (i < total) {
+        a = *reinterpret_cast<const Vec*>(src + i * V);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s = fmaf(to_f32(a.v[e]), to_f32(a.v[e]), s);
+      }
+      for (int o = per_head >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      if (i >= total) continue;
+      const float r = 1.f / sqrtf(s / (float)p.dim + p.a.eps);
+      const int h = i / per_head, col = (i - h * per_head) * V;
+      const float* w = (h < p.heads ? p.norm_q : p.norm_k) + col;
+#pragma unroll
+      for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(to_f32(a.v[e]) * r * w[e]);
+      put(h, col, a);
+    }
+    return;
+  }
   float rq = 1.f, rk = 1.f;
   const bool whole = p.norm_q && !p.a.head_norm;
   float* const head_r = cs_sm + p.rot_dims;
@@ -90,18 +134,6 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
     rq = 1.f / sqrtf(s0 / (float)(p.heads * p.dim) + p.a.eps);  // padding adds nothing to the sums
     rk = 1.f / sqrtf(s1 / (float)(p.kv_heads * p.dim) + p.a.eps);
   }
-  const int maps = p.a.maps, row = maps * p.dimp + p.vdp, place = row_of(p.a, pos);
-  // where the token's keys and values go; padding goes nowhere
-  T* const dst = (t < p.count[b] && place < p.len) ? rows + ((long long)p.slots[b] * p.len + place) * p.a.kv_heads * row : nullptr;
-  const bool shared = p.value_col == nq;
-  // one piece of a head: the key part of the cache or the query
-  auto put = [&](int h, int col, const Vec& v) {
-    if (h < p.heads) *reinterpret_cast<Vec*>(q + (n * p.heads + h) * p.dimp + col) = v;
-    else if (dst) {
-      const int k = h - p.heads, g = maps == 1 ? k : k / maps;
-      *reinterpret_cast<Vec*>(dst + g * row + (k - g * maps) * p.dimp + col) = v;
-    }
-  };
   auto normed = [&](int h, int col, const Vec& a, float (&x)[V]) {
     const float r = p.norm_q && !whole ? head_r[h] : (h < p.heads ? rq : rk);
     const float* w = p.norm_q ? (h < p.heads ? p.norm_q + (whole ? h * p.dimp : 0) : p.norm_k + (whole ? (h - p.heads) * p.dimp : 0)) + col : nullptr;
@@ -142,12 +174,7 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
     for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(x[e]);
     put(h, k, a);
   }
-  if (!shared && dst) {
-    for (int i = threadIdx.x * V; i < p.a.kv_heads * p.vdp; i += GP_THREADS * V) {
-      const int g = i / p.vdp;
-      *reinterpret_cast<Vec*>(dst + g * row + maps * p.dimp + i - g * p.vdp) = *reinterpret_cast<const Vec*>(src + p.value_col + i);
-    }
-  }
+  if (!shared && dst) put_values();
 }
 
 template <typename T, int V>

@@ -23,6 +23,8 @@
 #include <cuda.h>
 #include <limits.h>
 
+#include <type_traits>
+
 #include "attn_spec.cuh"
 #include "common.cuh"
 #include "kvb200_layers.h"
@@ -61,7 +63,7 @@ __device__ __forceinline__ void named_barrier(int id, int threads) { asm volatil
 
 __device__ __forceinline__ float lf_sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
 
-template <int NQT, bool DIFF>
+template <int NQT, bool DIFF, bool CAP>
 __global__ void __launch_bounds__(64 + 128 * NQT, 1)
 latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_constant__ CUtensorMap tmQr,
                     const __grid_constant__ CUtensorMap tmKu, const __grid_constant__ CUtensorMap tmKr,
@@ -294,6 +296,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     const uint32_t tmem_O = tmem_base + (uint32_t)(NQT * LF_T + u * o_cols) + lane_base;
     const float c = p.scale_log2;
     const float2 c2 = make_float2(c, c);
+    const CapSeries cap(p.cap_in, p.cap_out);
     float m_used = !p.a.sink ? -1e30f : p.a.sink_w ? p.a.sink_w[h] * ATTN_LOG2E : 0.f, l = p.a.sink ? 1.f : 0.f;
     bool ok = true;
     uint32_t ph = 0;
@@ -306,22 +309,16 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
 #pragma unroll
       for (int w = 0; w < 4; ++w) tmem_ld_32x32b_x32(tmem_S + (uint32_t)(32 * w), x + 32 * w);
       tmem_ld_wait();
-      if (p.cap_out > 0.f) {
-        // scores well below the cap take the series, others (any of the warp's) the exponential
-        const float2 ci = make_float2(p.cap_in, p.cap_in), co = make_float2(p.cap_out, p.cap_out);
+      bool series = false;
+      if (CAP) {
+        // scores well below the cap are capped in the exponent by a series, others (any of the warp's) here by the exponential
         float top = 0.f;
 #pragma unroll
         for (int e = 0; e < LF_T; e += 2) top = fmax3(top, fabsf(__uint_as_float(x[e])), fabsf(__uint_as_float(x[e + 1])));
-        if (__any_sync(0xffffffffu, !(top * p.cap_in <= CAP_SERIES))) {
+        series = cap.usable() && __all_sync(0xffffffffu, top * p.cap_in <= CAP_SERIES);
+        if (!series) {
 #pragma unroll
           for (int e = 0; e < LF_T; ++e) x[e] = __float_as_uint(p.cap_out * cap_tanh(__uint_as_float(x[e]) * p.cap_in));
-        } else {
-#pragma unroll
-          for (int e = 0; e < LF_T; e += 2) {
-            const float2 y = fmul2(cap_tanh_series(fmul2(make_float2(__uint_as_float(x[e]), __uint_as_float(x[e + 1])), ci)), co);
-            x[e] = __float_as_uint(y.x);
-            x[e + 1] = __float_as_uint(y.y);
-          }
         }
       }
       const int j0 = tile_at(t) * LF_T;
@@ -346,7 +343,8 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       for (int e = 16; e < LF_T; e += 16)
 #pragma unroll
         for (int i = 0; i < 8; ++i) a8[i] = fmax3(a8[i], __uint_as_float(x[e + 2 * i]), __uint_as_float(x[e + 2 * i + 1]));
-      const float m_tile = fmax3(fmax3(a8[0], a8[1], a8[2]), fmax3(a8[3], a8[4], a8[5]), fmaxf(a8[6], a8[7])) * c;
+      float m_tile = fmax3(fmax3(a8[0], a8[1], a8[2]), fmax3(a8[3], a8[4], a8[5]), fmaxf(a8[6], a8[7]));
+      m_tile = CAP && series ? cap_series(cap, make_float2(m_tile, m_tile), make_float2(0.f, 0.f)).x : m_tile * c;
       const bool raise = m_tile > m_used + LF_RESCALE_STEP;
       const float m_new = raise ? m_tile : m_used;
       // the PV product of the previous tile was issued before this tile's scores: it is complete, O is quiet
@@ -366,23 +364,27 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       m_used = m_new;
       const float2 neg_m2 = make_float2(-m_used, -m_used);
       float2 s0 = make_float2(0.f, 0.f), s1 = s0;
+      auto weights = [&](auto exponent) {
 #pragma unroll
-      for (int w = 0; w < 4; ++w) {
-        uint32_t pk[16];
+        for (int w = 0; w < 4; ++w) {
+          uint32_t pk[16];
 #pragma unroll
-        for (int e = 0; e < 32; e += 4) {
-          const uint32_t* xe = x + 32 * w + e;
-          const float2 x0 = ffma2(make_float2(__uint_as_float(xe[0]), __uint_as_float(xe[1])), c2, neg_m2);
-          const float2 x1 = ffma2(make_float2(__uint_as_float(xe[2]), __uint_as_float(xe[3])), c2, neg_m2);
-          const float2 y0 = make_float2(lf_exp2(x0.x), lf_exp2(x0.y));
-          const float2 y1 = make_float2(lf_exp2(x1.x), lf_exp2(x1.y));
-          s0 = fadd2(s0, y0);
-          s1 = fadd2(s1, y1);
-          pk[e >> 1] = pack_bf16x2(y0.x, y0.y);
-          pk[(e >> 1) + 1] = pack_bf16x2(y1.x, y1.y);
+          for (int e = 0; e < 32; e += 4) {
+            const uint32_t* xe = x + 32 * w + e;
+            const float2 x0 = exponent(make_float2(__uint_as_float(xe[0]), __uint_as_float(xe[1])));
+            const float2 x1 = exponent(make_float2(__uint_as_float(xe[2]), __uint_as_float(xe[3])));
+            const float2 y0 = make_float2(lf_exp2(x0.x), lf_exp2(x0.y));
+            const float2 y1 = make_float2(lf_exp2(x1.x), lf_exp2(x1.y));
+            s0 = fadd2(s0, y0);
+            s1 = fadd2(s1, y1);
+            pk[e >> 1] = pack_bf16x2(y0.x, y0.y);
+            pk[(e >> 1) + 1] = pack_bf16x2(y1.x, y1.y);
+          }
+          tmem_st_32x32b_x16(tmem_S + (uint32_t)(16 * w), pk);
         }
-        tmem_st_32x32b_x16(tmem_S + (uint32_t)(16 * w), pk);
-      }
+      };
+      if (CAP && series) weights([&](float2 v) { return cap_series(cap, v, neg_m2); });
+      else weights([&](float2 v) { return ffma2(v, c2, neg_m2); });
       s0 = fadd2(s0, s1);
       l += s0.x + s0.y;
       tmem_st_wait();
@@ -505,13 +507,13 @@ static LfPlan lf_plan(int dimp, int rp, int vdp, int maps = 1) {
   return pl;
 }
 
-template <int NQT, bool DIFF>
+template <int NQT, bool DIFF, bool CAP>
 static int lf_launch(const CUtensorMap* tm, LfParams& p, int smem, cudaStream_t s) {
   static PerDeviceOnce once;
   if (once.first())
-    cudaFuncSetAttribute(latent_flash_kernel<NQT, DIFF>, cudaFuncAttributeMaxDynamicSharedMemorySize, LF_SMEM_LIMIT - (DIFF ? 2048 : 0));
+    cudaFuncSetAttribute(latent_flash_kernel<NQT, DIFF, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, LF_SMEM_LIMIT - (DIFF ? 2048 : 0));
   p.n_pair = DIFF ? p.nQ : (p.nQ + NQT - 1) / NQT;
-  latent_flash_kernel<NQT, DIFF><<<p.B * p.heads * p.n_pair, 64 + 128 * NQT, smem, s>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
+  latent_flash_kernel<NQT, DIFF, CAP><<<p.B * p.heads * p.n_pair, 64 + 128 * NQT, smem, s>>>(tm[0], tm[1], tm[2], tm[3], tm[4], p);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
@@ -555,7 +557,7 @@ extern "C" int kvb_latent_attend_tc(const void* q, const void* kv, const void* l
   p.ksr = (rp + 15) / 16;
   p.vdp = vdp; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.slots = nullptr; p.group = 1; p.gate = nullptr; p.gate_ld = 0; p.cap_in = p.cap_out = 0.f; p.a = kvb_attention{};
-  return pl.nqt == 2 ? lf_launch<2, false>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1, false>(tm, p, pl.smem, (cudaStream_t)stream);
+  return pl.nqt == 2 ? lf_launch<2, false, false>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1, false, false>(tm, p, pl.smem, (cudaStream_t)stream);
 }
 
 extern "C" int kvb_grouped_attend_tc_supported(const kvb_attention* a) {
@@ -600,6 +602,10 @@ extern "C" int kvb_grouped_attend_tc(const void* q, const void* rows, const void
   p.scale_log2 = a->softcap > 0.f ? 1.f : a->scale * ATTN_LOG2E;
   p.slots = slots; p.group = a->heads / a->kv_heads; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld; p.a = *a;
   cudaStream_t s = (cudaStream_t)stream;
-  if (maps == 2) return lf_launch<2, true>(tm, p, pl.smem, s);
-  return pl.nqt == 2 ? lf_launch<2, false>(tm, p, pl.smem, s) : lf_launch<1, false>(tm, p, pl.smem, s);
+  auto launch = [&](auto capped) {
+    constexpr bool CAP = decltype(capped)::value;
+    if (maps == 2) return lf_launch<2, true, CAP>(tm, p, pl.smem, s);
+    return pl.nqt == 2 ? lf_launch<2, false, CAP>(tm, p, pl.smem, s) : lf_launch<1, false, CAP>(tm, p, pl.smem, s);
+  };
+  return a->softcap > 0.f ? launch(std::true_type{}) : launch(std::false_type{});
 }

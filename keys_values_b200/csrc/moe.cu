@@ -16,84 +16,100 @@
 
 namespace kvb {
 
-constexpr int ROUTE_WARPS = 4;
+constexpr int ROUTE_WARPS = 8;
+constexpr int ROUTE_TOKENS = 4;  // tokens of a warp, at most; a CTA counts its choices first and takes its rows of every expert at once
 constexpr int ROUTE_MAX_EXPERTS = 2048;
 
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ logits, int* __restrict__ expert, float* __restrict__ weight, int* __restrict__ row,
-                 int* __restrict__ counters, long long n, int E, int top, const kvb_router r) {
+                 int* __restrict__ counters, long long n, int E, int top, int per_warp, const kvb_router r) {
   extern __shared__ float sc_all[];
+  int* const local = reinterpret_cast<int*>(sc_all + ROUTE_WARPS * (E + r.groups));  // choices of this CTA per expert, then their first rows
+  for (int e = threadIdx.x; e < E; e += ROUTE_WARPS * 32) local[e] = 0;
+  __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* sc = sc_all + warp * (E + r.groups);  // choice scores; scores of the groups
   float* gs = sc + E;
-  const long long tok = (long long)blockIdx.x * ROUTE_WARPS + warp;
-  if (tok >= n) return;
-  const float* z = logits + tok * E;
-  float m = 0.f, l = 1.f;  // softmax: score = exp(z - m) / l
-  if (r.score == 0) {
-    m = -INFINITY;
-    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
-    m = warp_max(m);
-    l = 0.f;
-    for (int e = lane; e < E; e += 32) l += expf(z[e] - m);
-    l = warp_sum(l);
-  }
-  auto score = [&](int e) { return r.score == 0 ? expf(z[e] - m) / l : 1.f / (1.f + expf(-z[e])); };
-  for (int e = lane; e < E; e += 32) sc[e] = score(e) + (r.correction ? r.correction[e] : 0.f);
-  __syncwarp();
-  if (r.groups > 1) {
-    const int size = E / r.groups;
-    for (int g = lane; g < r.groups; g += 32) {  // sum of the two largest
-      float a = -INFINITY, b = -INFINITY;
-      for (int e = g * size; e < (g + 1) * size; ++e) {
+  const long long tok0 = (long long)blockIdx.x * ROUTE_WARPS * per_warp;
+  for (int i = 0; i < per_warp; ++i) {
+    const long long tok = tok0 + i * ROUTE_WARPS + warp;
+    if (tok >= n) break;
+    const float* z = logits + tok * E;
+    float m = 0.f, l = 1.f;  // softmax: score = exp(z - m) / l
+    if (r.score == 0) {
+      m = -INFINITY;
+      for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+      m = warp_max(m);
+      l = 0.f;
+      for (int e = lane; e < E; e += 32) l += expf(z[e] - m);
+      l = warp_sum(l);
+    }
+    auto score = [&](int e) { return r.score == 0 ? expf(z[e] - m) / l : 1.f / (1.f + expf(-z[e])); };
+    for (int e = lane; e < E; e += 32) sc[e] = score(e) + (r.correction ? r.correction[e] : 0.f);
+    __syncwarp();
+    if (r.groups > 1) {
+      const int size = E / r.groups;
+      for (int g = lane; g < r.groups; g += 32) {  // sum of the two largest
+        float a = -INFINITY, b = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) {
+          const float v = sc[e];
+          b = fmaxf(b, fminf(a, v));
+          a = fmaxf(a, v);
+        }
+        gs[g] = size > 1 ? a + b : a;
+      }
+      __syncwarp();
+      for (int g = lane; g < r.groups; g += 32) {
+        int ahead = 0;  // groups that come before this one; ties: lower index first
+        for (int o = 0; o < r.groups; ++o) ahead += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+        if (ahead >= r.keep)
+          for (int e = g * size; e < (g + 1) * size; ++e) sc[e] = -INFINITY;
+      }
+      __syncwarp();
+    }
+    float chosen = 0.f;
+    for (int k = 0; k < top; ++k) {
+      float best = -INFINITY;
+      int bi = 0x7fffffff;
+      for (int e = lane; e < E; e += 32) {
         const float v = sc[e];
-        b = fmaxf(b, fminf(a, v));
-        a = fmaxf(a, v);
+        if (v > best) {  // those that cannot be chosen are at minus infinity
+          best = v;
+          bi = e;
+        }
       }
-      gs[g] = size > 1 ? a + b : a;
-    }
-    __syncwarp();
-    for (int g = lane; g < r.groups; g += 32) {
-      int ahead = 0;  // groups that come before this one; ties: lower index first
-      for (int o = 0; o < r.groups; ++o) ahead += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
-      if (ahead >= r.keep)
-        for (int e = g * size; e < (g + 1) * size; ++e) sc[e] = -INFINITY;
-    }
-    __syncwarp();
-  }
-  float chosen = 0.f;
-  for (int k = 0; k < top; ++k) {
-    float best = -INFINITY;
-    int bi = 0x7fffffff;
-    for (int e = lane; e < E; e += 32) {
-      const float v = sc[e];
-      if (v > best) {  // those that cannot be chosen are at minus infinity
-        best = v;
-        bi = e;
-      }
-    }
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > best || (ov == best && oi < bi)) {
-        best = ov;
-        bi = oi;
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > best || (ov == best && oi < bi)) {
+          best = ov;
+          bi = oi;
+        }
       }
+      if (bi >= E) bi = 0;  // scores that are not numbers: any expert
+      const float w = score(bi);
+      chosen += w;
+      if (lane == 0) {
+        expert[tok * top + k] = bi;
+        weight[tok * top + k] = w;
+        row[tok * top + k] = atomicAdd(&local[bi], 1);
+        sc[bi] = -INFINITY;
+      }
+      __syncwarp();
     }
-    if (bi >= E) bi = 0;  // scores that are not numbers: any expert
-    const float w = score(bi);
-    chosen += w;
-    if (lane == 0) {
-      expert[tok * top + k] = bi;
-      weight[tok * top + k] = w;
-      row[tok * top + k] = atomicAdd(&counters[bi], 1);
-      sc[bi] = -INFINITY;
-    }
+    if (r.renormalize)
+      for (int k = lane; k < top; k += 32) weight[tok * top + k] = weight[tok * top + k] / (chosen + r.eps);
     __syncwarp();
   }
-  if (r.renormalize)
-    for (int k = lane; k < top; k += 32) weight[tok * top + k] = weight[tok * top + k] / (chosen + r.eps);
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += ROUTE_WARPS * 32)
+    if (local[e] > 0) local[e] = atomicAdd(&counters[e], local[e]);
+  __syncthreads();
+  for (int i = threadIdx.x; i < ROUTE_WARPS * per_warp * top; i += ROUTE_WARPS * 32) {
+    const long long at = tok0 * top + i;
+    if (at < n * top) row[at] += local[expert[at]];
+  }
 }
 
 // Exclusive prefix over the experts' tile counts, tile table. One CTA of 1024 threads.
@@ -163,7 +179,10 @@ moe_gather_kernel(const T* __restrict__ h, const int* __restrict__ row, T* __res
   }
 }
 
-__device__ __forceinline__ float moe_glu(float gate, float up) { return gate / (1.f + expf(-gate)) * up; }
+// silu(gate) · up; for results that are rounded to 16 bits with the fast exponential and quotient
+template <typename T> __device__ __forceinline__ float moe_glu(float gate, float up) {
+  return sizeof(T) == 2 ? __fdividef(gate, 1.f + __expf(-gate)) * up : gate / (1.f + expf(-gate)) * up;
+}
 
 __device__ __forceinline__ float moe_act(float v, int act) {
   if (act == 1) {
@@ -217,7 +236,7 @@ moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __r
     const int f = f0 / 2 + tf;
     if (f < ldo) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) out[(r0 + tr + 8 * i) * ldo + f] = from_f32<T>(2 * f < n_out ? moe_glu(acc[i][0], acc[i][1]) : 0.f);
+      for (int i = 0; i < 4; ++i) out[(r0 + tr + 8 * i) * ldo + f] = from_f32<T>(2 * f < n_out ? moe_glu<T>(acc[i][0], acc[i][1]) : 0.f);
     }
     return;
   }
@@ -230,36 +249,36 @@ moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __r
     }
 }
 
-// out[n, c] = silu(x[n, c]) · x[n, up + c], zero in the columns from ff to ldo
+// out[n, c] = silu(x[n, c]) · x[n, up + c], zero in the columns from ff to ldo. A CTA has one row.
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
-glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long n, long long ldx, int up, int ff, int ldo) {
+glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long ldx, int up, int ff, int ldo) {
   struct alignas(sizeof(T) * V) Vec { T v[V]; };
-  const int per = ldo / V;
-  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
-  const long long r = i / per;
-  if (r >= n) return;
-  const int c = (int)(i - r * per) * V;
-  Vec y;
-  if (c < ff) {
-    const Vec g = *reinterpret_cast<const Vec*>(x + r * ldx + c), u = *reinterpret_cast<const Vec*>(x + r * ldx + up + c);
+  x += blockIdx.x * ldx;
+  out += (long long)blockIdx.x * ldo;
+#pragma unroll 4
+  for (int c = threadIdx.x * V; c < ldo; c += blockDim.x * V) {
+    Vec y;
+    if (c < ff) {
+      const Vec g = *reinterpret_cast<const Vec*>(x + c), u = *reinterpret_cast<const Vec*>(x + up + c);
 #pragma unroll
-    for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(moe_glu(to_f32(g.v[e]), to_f32(u.v[e])));
-  } else {
+      for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(moe_glu<T>(to_f32(g.v[e]), to_f32(u.v[e])));
+    } else {
 #pragma unroll
-    for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(0.f);
+      for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(0.f);
+    }
+    *reinterpret_cast<Vec*>(out + c) = y;
   }
-  *reinterpret_cast<Vec*>(out + r * ldo + c) = y;
 }
 
 template <typename T>
 static int glu_launch(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
-  if (ff % V == 0 && up % V == 0 && ldx % V == 0 && ldo % V == 0) {
-    glu_kernel<T, V><<<(unsigned)((n * (ldo / V) + 255) / 256), 256, 0, s>>>((const T*)x, (T*)out, n, ldx, up, ff, ldo);
-  } else {
-    glu_kernel<T, 1><<<(unsigned)((n * ldo + 255) / 256), 256, 0, s>>>((const T*)x, (T*)out, n, ldx, up, ff, ldo);
-  }
+  const bool vec = ff % V == 0 && up % V == 0 && ldx % V == 0 && ldo % V == 0;
+  int threads = ((vec ? ldo / V : ldo) + 31) / 32 * 32;
+  if (threads > 256) threads = 256;
+  if (vec) glu_kernel<T, V><<<(unsigned)n, threads, 0, s>>>((const T*)x, (T*)out, ldx, up, ff, ldo);
+  else glu_kernel<T, 1><<<(unsigned)n, threads, 0, s>>>((const T*)x, (T*)out, ldx, up, ff, ldo);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
@@ -278,8 +297,13 @@ extern "C" int kvb_moe_route(const float* logits, int* expert, float* weight, in
   if (n_expert > ROUTE_MAX_EXPERTS) return KVB_ERR_TOO_LARGE;
   cudaStream_t s = (cudaStream_t)stream;
   if (cudaMemsetAsync(counters, 0, sizeof(int) * n_expert, s) != cudaSuccess) return KVB_ERR_CUDA;
-  moe_route_kernel<<<(unsigned)((n + ROUTE_WARPS - 1) / ROUTE_WARPS), ROUTE_WARPS * 32, ROUTE_WARPS * (n_expert + r.groups) * sizeof(float), s>>>(
-      logits, expert, weight, row, counters, n, n_expert, top, r);
+  const int per_warp = n >= 148LL * 8 * ROUTE_WARPS * ROUTE_TOKENS / 4 ? ROUTE_TOKENS : 1;
+  const int tokens = ROUTE_WARPS * per_warp;
+  const size_t smem = (size_t)ROUTE_WARPS * (n_expert + r.groups) * sizeof(float) + (size_t)n_expert * sizeof(int);
+  static PerDeviceOnce once;
+  if (once.first()) cudaFuncSetAttribute(moe_route_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+  moe_route_kernel<<<(unsigned)((n + tokens - 1) / tokens), ROUTE_WARPS * 32, smem, s>>>(logits, expert, weight, row, counters, n, n_expert, top,
+                                                                                       per_warp, r);
   moe_plan_kernel<<<1, 1024, 0, s>>>(counters, plan, tile_expert, tile_row, n_expert, tile, max_tiles);
   const long long m = n * top;
   moe_rows_kernel<<<(unsigned)((m + 255) / 256), 256, 0, s>>>(expert, counters, row, m);
@@ -328,7 +352,7 @@ extern "C" int kvb_moe_gemm(const void* in, const void* w, void* out, const int*
 }
 
 extern "C" int kvb_glu(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, int dtype, void* stream) {
-  if (n <= 0 || ff <= 0 || up < ff || ldx < up + ff || ldo < ff || n * ldo > 0x7fffffffLL * 256) return KVB_ERR_ARG;
+  if (n <= 0 || ff <= 0 || up < ff || ldx < up + ff || ldo < ff || n > 0x7fffffffLL) return KVB_ERR_ARG;
   if (dtype == 0) return kvb::glu_launch<float>(x, out, n, ldx, up, ff, ldo, (cudaStream_t)stream);
   if (dtype == 1) return kvb::glu_launch<__nv_bfloat16>(x, out, n, ldx, up, ff, ldo, (cudaStream_t)stream);
   return KVB_ERR_ARG;

@@ -4,6 +4,8 @@
 // that). Also the entry into the stack (embedding rows only) and the norm of rows in front of the output head.
 //
 // A CTA has one row, which stays in registers; means and squared deviations are separate sums (no cancellation).
+#include <type_traits>
+
 #include "common.cuh"
 #include "kvb200_layers.h"
 
@@ -92,7 +94,7 @@ __device__ __forceinline__ float row_norm_factor(float (&x)[NC][V], const NormEd
   return 1.f / sqrtf(row_sum<TH>(ss, red[1]) * p.inv_width + p.eps);
 }
 
-template <typename T, int V, int TH, int NC, bool CENTER>
+template <typename T, int V, int TH, int NC, bool CENTER, bool EXPERTS>
 __global__ void __launch_bounds__(TH)
 norm_edge_kernel(const NormEdgeParams p) {
   __shared__ float red[4][TH / 32];
@@ -107,17 +109,30 @@ norm_edge_kernel(const NormEdgeParams p) {
     if (p.sub) RowVec<T, V>::load(static_cast<const T*>(p.sub) + o + c, y[i]);
     if (p.x_in) RowVec<float, V>::load(p.x_in + o + c, x[i]);
   }
-  for (int k = 0; k < p.top; ++k) {
-    const T* src = static_cast<const T*>(p.expert_out) + (long long)p.expert_row[n * p.top + k] * p.expert_ld;
-    const float w = p.expert_w[n * p.top + k];
+  // up to four experts at a time, so that their rows are on their way together
+  for (int k0 = 0; EXPERTS && k0 < p.top; k0 += 4) {
+    const T* src[4];
+    float w[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const bool in = k0 + k < p.top;
+      src[k] = static_cast<const T*>(p.expert_out) + (long long)p.expert_row[n * p.top + (in ? k0 + k : k0)] * p.expert_ld;
+      w[k] = in ? p.expert_w[n * p.top + k0 + k] : 0.f;
+    }
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
       const int c = (i * TH + threadIdx.x) * V;
       if (c >= p.width) continue;
-      float e[V];
-      RowVec<T, V>::load(src + c, e);
+      float e[4][V];
 #pragma unroll
-      for (int j = 0; j < V; ++j) y[i][j] = fmaf(w, e[j], y[i][j]);
+      for (int k = 0; k < 4; ++k)
+        if (k0 + k < p.top) RowVec<T, V>::load(src[k] + c, e[k]);
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        if (k0 + k < p.top) {
+#pragma unroll
+          for (int j = 0; j < V; ++j) y[i][j] = fmaf(w[k], e[k][j], y[i][j]);
+        }
     }
   }
   long long tok = 0;
@@ -177,23 +192,36 @@ norm_edge_kernel(const NormEdgeParams p) {
   }
 }
 
-template <typename T, int V, bool CENTER>
+template <typename T, int V, bool CENTER, bool EXPERTS>
 static int norm_edge_launch(const NormEdgeParams& p, long long n, cudaStream_t s) {
   const unsigned g = (unsigned)n;
-  if (p.width <= 128 * V) norm_edge_kernel<T, V, 128, 1, CENTER><<<g, 128, 0, s>>>(p);
-  else if (p.width <= 256 * V) norm_edge_kernel<T, V, 128, 2, CENTER><<<g, 128, 0, s>>>(p);
-  else if (p.width <= 512 * V) norm_edge_kernel<T, V, 128, 4, CENTER><<<g, 128, 0, s>>>(p);
-  else if (p.width <= 1024 * V) norm_edge_kernel<T, V, 256, 4, CENTER><<<g, 256, 0, s>>>(p);
-  else if (p.width <= 2048 * V) norm_edge_kernel<T, V, 512, 4, CENTER><<<g, 512, 0, s>>>(p);
-  else if (p.width <= 8192 * V) norm_edge_kernel<T, V, 1024, 8, CENTER><<<g, 1024, 0, s>>>(p);
+  if (n <= 148 && p.width > 128 * V) {  // few rows: latency counts, every thread has one access
+    if (p.width <= 256 * V) norm_edge_kernel<T, V, 256, 1, CENTER, EXPERTS><<<g, 256, 0, s>>>(p);
+    else if (p.width <= 512 * V) norm_edge_kernel<T, V, 512, 1, CENTER, EXPERTS><<<g, 512, 0, s>>>(p);
+    else if (p.width <= 1024 * V) norm_edge_kernel<T, V, 1024, 1, CENTER, EXPERTS><<<g, 1024, 0, s>>>(p);
+    else if (p.width <= 8192 * V) norm_edge_kernel<T, V, 1024, 8, CENTER, EXPERTS><<<g, 1024, 0, s>>>(p);
+    else return KVB_ERR_TOO_LARGE;
+  } else if (p.width <= 128 * V) norm_edge_kernel<T, V, 128, 1, CENTER, EXPERTS><<<g, 128, 0, s>>>(p);
+  else if (p.width <= 256 * V) norm_edge_kernel<T, V, 128, 2, CENTER, EXPERTS><<<g, 128, 0, s>>>(p);
+  else if (p.width <= 512 * V) norm_edge_kernel<T, V, 128, 4, CENTER, EXPERTS><<<g, 128, 0, s>>>(p);
+  else if (p.width <= 1024 * V) norm_edge_kernel<T, V, 256, 4, CENTER, EXPERTS><<<g, 256, 0, s>>>(p);
+  else if (p.width <= 2048 * V) norm_edge_kernel<T, V, 512, 4, CENTER, EXPERTS><<<g, 512, 0, s>>>(p);
+  else if (p.width <= 8192 * V) norm_edge_kernel<T, V, 1024, 8, CENTER, EXPERTS><<<g, 1024, 0, s>>>(p);
   else return KVB_ERR_TOO_LARGE;
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
 template <typename T>
 static int norm_edge_type(const NormEdgeParams& p, long long n, int center, cudaStream_t s) {
-  if (p.width % 4 == 0) return center ? norm_edge_launch<T, 4, true>(p, n, s) : norm_edge_launch<T, 4, false>(p, n, s);
-  return center ? norm_edge_launch<T, 1, true>(p, n, s) : norm_edge_launch<T, 1, false>(p, n, s);
+  auto launch = [&](auto vec, auto experts) {
+    constexpr int V = decltype(vec)::value;
+    constexpr bool E = decltype(experts)::value;
+    return center ? norm_edge_launch<T, V, true, E>(p, n, s) : norm_edge_launch<T, V, false, E>(p, n, s);
+  };
+  using One = std::integral_constant<int, 1>;
+  using Four = std::integral_constant<int, 4>;
+  if (p.top > 0) return p.width % 4 == 0 ? launch(Four{}, std::true_type{}) : launch(One{}, std::true_type{});
+  return p.width % 4 == 0 ? launch(Four{}, std::false_type{}) : launch(One{}, std::false_type{});
 }
 
 }  // namespace kvb

@@ -2,7 +2,7 @@
 // o normed per head and gated. The recurrence over several tokens is the one of state-space mixers (ssm.cu, ssm_sm100.cu); here are
 //
 //   prep   rotation of the fp32 projections of queries and keys, rounded once to the type of the scan's operands;
-//   norm   y / rms(y) · silu(gate), a warp per head of a token;
+//   norm   y / rms(y) · silu(gate), a few lanes per head of a token;
 //   step   one new token per sequence: rotation, decay, state, output, norm and gate of a head in one kernel, all in fp32, bound by
 //          reading and writing the state once.
 #include "common.cuh"
@@ -67,41 +67,89 @@ retention_prep_kernel(const float* __restrict__ in, T* __restrict__ out, const R
 
 // ------------------------------------------------------------------------------------------------ norm
 constexpr int HN_WARPS = 8;
-constexpr int HN_MAX = 16;  // accesses per lane
+constexpr int HN_ROWS = 4;  // rows (heads of tokens) that a group of lanes works on side by side
+constexpr int HN_MAX = 16;  // accesses per lane and row
 
-template <typename T, int V>
+struct HeadNormParams {
+  long long ld, rows;
+  int heads, vdim, vdp;
+  float eps;
+};
+
+// LANES lanes have a row; NC accesses of V columns per lane.
+template <typename T, int V, int LANES, int NC, int ROWS>
 __global__ void __launch_bounds__(HN_WARPS * 32)
-head_norm_gate_kernel(const T* __restrict__ y, const T* __restrict__ gate, T* __restrict__ out, long long ld, long long rows, int heads,
-                      int vdim, int vdp, float eps) {
+head_norm_gate_kernel(const T* __restrict__ y, const T* __restrict__ gate, T* __restrict__ out, const HeadNormParams p) {
   using Vec = RtVec<T, V>;
-  const int lane = threadIdx.x & 31;
-  const long long r = (long long)blockIdx.x * HN_WARPS + (threadIdx.x >> 5);
-  if (r >= rows) return;
-  const long long n = r / heads;
-  const int h = (int)(r - n * heads);
-  const T* src = y + r * vdp;
-  const T* g = gate + n * ld + (long long)h * vdp;
-  Vec v[HN_MAX];
-  float ss = 0.f;
+  constexpr int PER = HN_WARPS * 32 / LANES;  // rows that a CTA works on at a time
+  const int lane = threadIdx.x % LANES;
+  const unsigned r0 = blockIdx.x * (unsigned)(PER * ROWS) + threadIdx.x / LANES, rows = (unsigned)p.rows, heads = (unsigned)p.heads;
+  unsigned n = r0 / heads, h = r0 - n * heads;  // token and head
+  Vec v[ROWS][NC], z[ROWS][NC];
+  float ss[ROWS];
 #pragma unroll
-  for (int i = 0; i < HN_MAX; ++i) {
-    const int c = (i * 32 + lane) * V;
-    if (c >= vdp) break;
-    v[i] = *reinterpret_cast<const Vec*>(src + c);
+  for (int i = 0; i < ROWS; ++i) {
+    const unsigned r = r0 + i * PER;
+    const bool in = r < rows;
+    const T* g = gate + n * p.ld + h * (unsigned)p.vdp;
+    for (h += PER; h >= heads; h -= heads) ++n;
 #pragma unroll
-    for (int e = 0; e < V; ++e) ss = fmaf(to_f32(v[i].v[e]), to_f32(v[i].v[e]), ss);  // padding is zero
+    for (int k = 0; k < NC; ++k) {
+      const int c = (k * LANES + lane) * V;
+      if (in && c < p.vdp) {
+        v[i][k] = *reinterpret_cast<const Vec*>(y + (long long)r * p.vdp + c);
+        z[i][k] = *reinterpret_cast<const Vec*>(g + c);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) v[i][k].v[e] = z[i][k].v[e] = from_f32<T>(0.f);
+      }
+    }
   }
-  const float f = 1.f / sqrtf(warp_sum(ss) / (float)vdim + eps);
 #pragma unroll
-  for (int i = 0; i < HN_MAX; ++i) {
-    const int c = (i * 32 + lane) * V;
-    if (c >= vdp) break;
-    const Vec z = *reinterpret_cast<const Vec*>(g + c);
-    Vec o;
+  for (int i = 0; i < ROWS; ++i) {
+    ss[i] = 0.f;
 #pragma unroll
-    for (int e = 0; e < V; ++e) o.v[e] = from_f32<T>(to_f32(v[i].v[e]) * f * ss_silu_for<T>(to_f32(z.v[e])));
-    *reinterpret_cast<Vec*>(out + r * vdp + c) = o;
+    for (int k = 0; k < NC; ++k)
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss[i] = fmaf(to_f32(v[i][k].v[e]), to_f32(v[i][k].v[e]), ss[i]);  // padding is zero
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
   }
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const unsigned r = r0 + i * PER;
+    if (r >= rows) break;
+    const float f = 1.f / sqrtf(ss[i] / (float)p.vdim + p.eps);
+#pragma unroll
+    for (int k = 0; k < NC; ++k) {
+      const int c = (k * LANES + lane) * V;
+      if (c >= p.vdp) break;
+      Vec o;
+#pragma unroll
+      for (int e = 0; e < V; ++e) o.v[e] = from_f32<T>(to_f32(v[i][k].v[e]) * f * ss_silu_for<T>(to_f32(z[i][k].v[e])));
+      *reinterpret_cast<Vec*>(out + (long long)r * p.vdp + c) = o;
+    }
+  }
+}
+
+template <typename T, int V, int LANES, int NC, int ROWS>
+static int hn_launch(const void* y, const void* gate, void* out, const HeadNormParams& p, cudaStream_t s) {
+  constexpr int per = HN_WARPS * 32 / LANES * ROWS;
+  const long long blocks = (p.rows + per - 1) / per;
+  if (blocks > 0x7fffffffLL) return KVB_ERR_TOO_LARGE;
+  head_norm_gate_kernel<T, V, LANES, NC, ROWS><<<(unsigned)blocks, HN_WARPS * 32, 0, s>>>((const T*)y, (const T*)gate, (T*)out, p);
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+template <typename T>
+static int hn_type(const void* y, const void* gate, void* out, const HeadNormParams& p, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  if (p.vdp <= 8 * V) return hn_launch<T, V, 8, 1, HN_ROWS>(y, gate, out, p, s);
+  if (p.vdp <= 16 * V) return hn_launch<T, V, 16, 1, HN_ROWS>(y, gate, out, p, s);
+  if (p.vdp <= 32 * V) return hn_launch<T, V, 32, 1, HN_ROWS>(y, gate, out, p, s);
+  if (p.vdp <= 64 * V) return hn_launch<T, V, 32, 2, 2>(y, gate, out, p, s);
+  if (p.vdp <= 32 * V * HN_MAX) return hn_launch<T, V, 32, HN_MAX, 1>(y, gate, out, p, s);
+  return KVB_ERR_TOO_LARGE;
 }
 
 // ------------------------------------------------------------------------------------------------ step
@@ -235,14 +283,12 @@ extern "C" int kvb_retention_prep(const float* in, long long ld, const float* fr
 
 extern "C" int kvb_head_norm_gate(const void* y, const void* gate, long long ld, void* out, long long n, int heads, int vdim, int vdp,
                                   float eps, int dtype, void* stream) {
-  const long long rows = n * heads, blocks = (rows + kvb::HN_WARPS - 1) / kvb::HN_WARPS;
-  if (n <= 0 || heads <= 0 || vdim <= 0 || vdp < vdim || blocks > 0x7fffffffLL) return KVB_ERR_ARG;
-  if (vdp % 8 || ld % 4 || (reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15)
+  if (n <= 0 || heads <= 0 || vdim <= 0 || vdp < vdim || n * heads > 0x7f000000LL) return KVB_ERR_ARG;
+  if (vdp % 8 || ld % 8 || (reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15)
     return KVB_ERR_ALIGN;
-  if (vdp > 32 * 4 * kvb::HN_MAX) return KVB_ERR_TOO_LARGE;
-  KVB_RETENTION_TYPES(dtype, (kvb::head_norm_gate_kernel<T, 4><<<(unsigned)blocks, kvb::HN_WARPS * 32, 0, (cudaStream_t)stream>>>(
-      (const T*)y, (const T*)gate, (T*)out, ld, rows, heads, vdim, vdp, eps)));
-  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+  kvb::HeadNormParams p;
+  p.ld = ld; p.rows = n * heads; p.heads = heads; p.vdim = vdim; p.vdp = vdp; p.eps = eps;
+  KVB_RETENTION_TYPES(dtype, return kvb::hn_type<T>(y, gate, out, p, (cudaStream_t)stream));
 }
 
 extern "C" int kvb_retention_step(const float* u, long long ld, const float* freq, const float* decay, float* state, void* out,
