@@ -1,7 +1,7 @@
 """Builds the CUDA/C++ sources under ``csrc/`` for sm_100a, in-tree, into two libraries:
 ``libkvb200.so`` (caches, attention, GEMM, collectives of the LitGPT-shaped models) and
 ``libkvb200_layers.so`` (kernels of models described layer by layer: latent and grouped attention,
-state-space recurrence, routed experts, token shift, depth averages, norms). Each loads on its own, so a command that needs one
+state-space recurrence, retention, routed experts, token shift, depth averages, norms). Each loads on its own, so a command that needs one
 of them compiles no more than that.
 
 Usage: ``python -m keys_values_b200.build_ext [--force] [--verbose]``. nvcc

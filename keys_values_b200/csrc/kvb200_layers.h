@@ -1,6 +1,7 @@
 // C API of libkvb200_layers: kernels of models whose layers are described one by one (latent attention over a
-// ring of latents, grouped attention, state-space recurrence, routed experts, token shift, averages over the depth, norms). Conventions as in kvb200.h: launches on
-// the given stream, returns KVB_OK or a negative code, dtype 0 = fp32, 1 = bf16; nothing synchronises the device.
+// ring of latents, grouped attention, state-space recurrence, retention, routed experts, token shift, averages over the depth,
+// norms). Conventions as in kvb200.h: launches on the given stream, returns KVB_OK or a negative code, dtype 0 = fp32, 1 = bf16;
+// nothing synchronises the device.
 //
 // A pass works on B rows of T tokens (right padded). Row b belongs to the sequence in slot slots[b]; its first
 // token has position start[b], and count[b] <= T of its tokens are real. Padding is computed like tokens but never

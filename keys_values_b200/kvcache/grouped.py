@@ -13,7 +13,7 @@ from typing import Optional
 import torch
 
 from keys_values_b200.config import Config
-from keys_values_b200.kvcache.layer_cache import LayerCache
+from keys_values_b200.kvcache.layer_cache import MAX_PASS_TOKENS, LayerCache
 from keys_values_b200.ops.layers import RowPlan
 
 
@@ -27,7 +27,7 @@ def tiles(n: int) -> int:
 class GroupedKVCache(LayerCache):
     kind = "grouped_attention"
     # tokens of a pass that a ring takes besides the span of its layer
-    max_pass = 16384
+    max_pass = MAX_PASS_TOKENS
 
     def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
         from keys_values_b200.models.grouped_attention import grouped_shape

@@ -14,6 +14,10 @@ from keys_values_b200.config import Config
 from keys_values_b200.kvcache.base import KVCache, KVCacheParams, bits_for_torch_dtype
 
 
+# tokens that one pass of a chunked prefill takes at most, all rows together; rings of bounded layers have room for as many
+MAX_PASS_TOKENS = 16384
+
+
 class LayerCache(KVCache):
     kind: str  # of the mixer that the cache serves
 

@@ -34,7 +34,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from keys_values_b200.config import Config
-from keys_values_b200.kvcache.layer_cache import LayerCache
+from keys_values_b200.kvcache.layer_cache import MAX_PASS_TOKENS, LayerCache
 from keys_values_b200.kvcache.sequences import SequencePass, SequenceTable
 from keys_values_b200.models.grouped_attention import GroupedAttention
 from keys_values_b200.models.model import GPT
@@ -45,7 +45,6 @@ from keys_values_b200.ops import layers as L
 
 # fp32 bytes of residual streams (depth history included) that one pass of a chunked prefill may hold
 MAX_STREAM_BYTES = 4 * 2**30
-MAX_PASS_TOKENS = 16384
 
 
 def latent_shape(spec: Dict[str, Any]) -> L.LatentShape:

@@ -1,5 +1,5 @@
 """Ops of models that are described layer by layer (fp32 residual stream, latent and grouped attention, state-space
-recurrence, routed experts).
+recurrence, retention, routed experts).
 
 A CUDA tensor is always served by the kernels of ``libkvb200_layers.so`` (bf16 or fp32; anything else
 raises), a CPU tensor by the PyTorch restatement in :mod:`keys_values_b200.ops.layers_reference`.
