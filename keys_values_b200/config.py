@@ -16,6 +16,14 @@ from typing import Any, Dict, List, Optional, Tuple, Type, Union
 import yaml
 
 
+# norms of an fp32 residual stream by their names in `norm_class_name`: the mean taken off or not, weights stored around one or zero
+STREAM_NORMS = {
+    "StreamLayerNorm": dict(center=True),
+    "StreamRMSNorm": dict(center=False),
+    "StreamOffsetRMSNorm": dict(center=False, unit_offset=True),
+}
+
+
 def find_multiple(n: int, k: int) -> int:
     """Smallest multiple of ``k`` that is ``>= n``."""
     if n % k == 0:
@@ -94,6 +102,10 @@ class Config:
     token_shift: bool = False  # the mixer reads a learned blend of this and the previous token's normed input
     depth_average: bool = False  # learned average over the embedding output and all layers' results
     tie_embeddings: bool = False  # described layers: the output head is the embedding table
+    # Sequential layers: what a sublayer reads, h, becomes h + a causal convolution over time of h, this many taps (0: none)
+    input_conv: int = 0
+    residual_mult: float = 1.0  # sequential layers: factor of what a sublayer adds to the stream
+    position_table: bool = False  # described layers: a learned vector per position (block_size of them) is added to the embedding
     architecture: str = ""  # entry of models/registry.py the config was read by
     # Added by keys_values (config.py:26-30): use the in-repo RMSNorm
     own_rms_norm_implementation: bool = True
@@ -205,10 +217,10 @@ class Config:
             from keys_values_b200.models.layered import ScalarRMSNorm
 
             return ScalarRMSNorm
-        if self.norm_class_name in ("StreamLayerNorm", "StreamRMSNorm"):
+        if self.norm_class_name in STREAM_NORMS:
             from keys_values_b200.models.layered import StreamNorm
 
-            return partial(StreamNorm, center=self.norm_class_name == "StreamLayerNorm")
+            return partial(StreamNorm, **STREAM_NORMS[self.norm_class_name])
         if self.norm_class_name == "RMSNorm":
             return partial(RMSNorm, add_unit_offset="Gemma" in self.name)
         if self.norm_class_name == "LayerNorm" and "OLMo" in self.name:

@@ -5,10 +5,15 @@ tokens attend over the cache as it lies. A layer that sees every earlier positio
 of that slot. A layer that looks back a bounded way (a window or chunks) needs the rows of that span and of the pass at hand: if
 the cache is longer, the first positions that stay visible have rows of their own and the others share a ring
 (:class:`keys_values_b200.ops.layers.RowPlan`), in tiles of the attention kernels, so that a tile never wraps.
+
+A window with pooled blocks has the rows of the blocks ahead of a ring of tokens: row b of the first ones holds the means of keys and values
+of block b, written by the pass that brings the block's last token.
+
+A layer that takes the keys and values of an earlier layer holds none (:class:`BorrowedKVCache`).
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -29,13 +34,15 @@ class GroupedKVCache(LayerCache):
     # tokens of a pass that a ring takes besides the span of its layer
     max_pass = MAX_PASS_TOKENS
 
-    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
         from keys_values_b200.models.grouped_attention import grouped_shape
 
-        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device)
-        s = self.shape = grouped_shape(config.layers[block_idx]["mixer"])
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        s = self.shape = grouped_shape(self.spec)
         self.plan = RowPlan()
-        if s.span:
+        if s.pool:
+            self.plan = RowPlan(tiles(cache_length // s.pool), min(tiles(s.span + self.max_pass), tiles(cache_length)))
+        elif s.span:
             head, ring = tiles(s.keep), tiles(s.span + self.max_pass)
             if head + ring < cache_length:
                 self.plan = RowPlan(head, ring)
@@ -50,13 +57,18 @@ class GroupedKVCache(LayerCache):
     def current_length(self) -> int:
         return min(self.input_pos, self.length)
 
+    @property
+    def wraps(self) -> bool:
+        """Whether positions of a sequence share rows."""
+        return self.plan.ring > 0 and (not self.shape.pool or self.plan.ring < self.cache_length)
+
     def check_capacity(self, end: int) -> None:
-        if end > self.cache_length and not self.plan.ring:
+        if end > self.cache_length and (self.shape.pool or not self.plan.ring):
             raise IndexError(f"layer {self.block_idx}: {end} tokens exceed the cache of {self.cache_length}")
 
     def check_pass(self, seq) -> None:
         super().check_pass(seq)
-        if self.plan.ring and seq.length > self.plan.ring - self.shape.span:
+        if self.wraps and seq.length > self.plan.ring - self.shape.span:
             raise IndexError(f"layer {self.block_idx}: a pass of {seq.length} tokens exceeds the ring of {self.plan.ring} (take smaller portions)")
 
     def _shapes(self, dtype):
@@ -68,8 +80,48 @@ class GroupedKVCache(LayerCache):
         seq = self.sequences
         pos = torch.tensor([seq.pos_host[s] for s in seq.batch], dtype=torch.int32)[:, None]
         row = torch.arange(self.current_length, dtype=torch.int32)[None]
-        if self.plan.ring:
+        if self.shape.pool:  # of the tokens; the rows of blocks hold none
+            row = pos - 1 - (pos - 1 - torch.arange(min(self.input_pos, self.plan.ring), dtype=torch.int32)[None]) % self.plan.ring
+            row = torch.where(row >= 0, row, torch.full_like(row, -1))
+        elif self.plan.ring:
             head, ring = self.plan
             row = torch.where(row < head, row, pos - 1 - (pos - 1 - row) % ring)
             row = torch.where((row >= 0) & ((row >= head) | (torch.arange(row.shape[1])[None] < head)), row, torch.full_like(row, -1))
         return torch.where(row < pos, row, torch.full_like(row, -1))[:, None].to(self.device or "cpu")
+
+
+class BorrowedKVCache(LayerCache):
+    """Stands for the cache of an earlier layer (``kv_from``), which this layer reads and never writes."""
+
+    kind = "grouped_attention"
+
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        if self.spec.get("kv_from") is None:
+            raise ValueError(f"layer {block_idx} has keys and values of its own")
+        self._source: Tuple[GroupedKVCache, ...] = ()
+
+    def get_source(self) -> GroupedKVCache:
+        if not self._source:
+            raise ValueError(f"the cache of layer {self.block_idx} stands for that of layer {self.spec['kv_from']}: assign both to a model")
+        return self._source[0]
+
+    def set_source(self, cache: GroupedKVCache) -> None:
+        self._source = (cache,)  # not a module of this one
+
+    @property
+    def plan(self) -> RowPlan:
+        return self.get_source().plan
+
+    @property
+    def current_length(self) -> int:
+        return self.get_source().current_length
+
+    def allocate(self, device, dtype):
+        return self.get_source().allocate(device, dtype)
+
+    def _shapes(self, dtype):
+        return {}
+
+    def token_positions(self) -> torch.Tensor:
+        return self.get_source().token_positions()

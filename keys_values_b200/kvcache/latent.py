@@ -19,11 +19,11 @@ from keys_values_b200.kvcache.layer_cache import LayerCache
 class LatentKVCache(LayerCache):
     kind = "latent_attention"
 
-    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
         from keys_values_b200.models.layered import latent_shape
 
-        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device)
-        spec = config.layers[block_idx]["mixer"]
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        spec = self.spec
         self.window: Optional[int] = spec.get("window")
         self.shape = latent_shape(spec)
         self.ring_length = cache_length if self.window is None else min(cache_length, self.window)

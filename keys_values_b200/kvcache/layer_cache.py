@@ -6,7 +6,7 @@ several times in a pass (``config.loop``) has one region per run (``turns``) in 
 """
 from __future__ import annotations
 
-from typing import Dict, Optional, Tuple, Type
+from typing import Any, Dict, Optional, Tuple, Type
 
 import torch
 
@@ -21,8 +21,10 @@ MAX_PASS_TOKENS = 16384
 class LayerCache(KVCache):
     kind: str  # of the mixer that the cache serves
 
-    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
-        if config.layers is None or config.layers[block_idx]["mixer"]["kind"] != self.kind:
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, spec=None, **_ignored):
+        """``spec``: description of the mixer, if it is a part of the layer's."""
+        self.spec: Dict[str, Any] = (None if config.layers is None else config.layers[block_idx]["mixer"]) if spec is None else spec
+        if self.spec is None or self.spec["kind"] != self.kind:
             raise ValueError(f"layer {block_idx} of {config.name!r} has no {self.kind.replace('_', ' ')} mixer")
         super().__init__(config, max_batch_size, cache_length, block_idx, dtype)
         self.turns = config.layer_turns(block_idx)
@@ -33,9 +35,9 @@ class LayerCache(KVCache):
 
     @classmethod
     def from_config(cls, config: Config, max_batch_size: int, cache_length: int, block_idx: int, device=None, dtype=None, **kwargs):
-        kind = None if config.layers is None else config.layers[block_idx]["mixer"]["kind"]
         if cls is LayerCache:
-            return layer_cache_class(kind)(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+            spec = {"kind": None} if config.layers is None else config.layers[block_idx]["mixer"]
+            return layer_cache_class(spec)(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
         return cls(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
 
     # ------------------------------------------------------------- properties
@@ -109,19 +111,80 @@ class LayerCache(KVCache):
         raise NotImplementedError("sizes of these caches depend on the layer; create them and call size_estimate")
 
     def clone(self, device=None) -> "LayerCache":
-        other = type(self)(self.config, self.max_batch_size, self.cache_length, self.block_idx, dtype=self._dtype, device=device or self._device)
+        other = type(self)(self.config, self.max_batch_size, self.cache_length, self.block_idx, dtype=self._dtype, device=device or self._device,
+                           spec=self.spec)
         if self.buffers_ is not None:
             other.buffers_ = tuple(t.clone() if device is None else t.to(device, copy=True) for t in self.buffers_)
         return other
 
 
-def layer_cache_class(kind: Optional[str]) -> Type[LayerCache]:
-    """The cache class that serves mixers of ``kind``."""
-    from keys_values_b200.kvcache.grouped import GroupedKVCache
-    from keys_values_b200.kvcache.latent import LatentKVCache
-    from keys_values_b200.kvcache.recurrent import RetentionCache, StateSpaceCache
+class SideBySideCache(LayerCache):
+    """Caches of two mixers that read the same input, each of the class that its mixer needs."""
 
-    classes = {c.kind: c for c in (LatentKVCache, GroupedKVCache, StateSpaceCache, RetentionCache)}
-    if kind not in classes:
-        raise ValueError(f"no cache for mixers of kind {kind!r}")
-    return classes[kind]
+    kind = "side_by_side"
+
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, spec=None, **kwargs):
+        self.parts: Tuple[LayerCache, ...] = ()
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, spec=spec)
+        self.parts = tuple(layer_cache_class(s)(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, spec=s, **kwargs)
+                           for s in (self.spec["left"], self.spec["right"]))
+
+    @property
+    def sequences(self):
+        return self._sequences
+
+    @sequences.setter
+    def sequences(self, value) -> None:
+        self._sequences = value
+        for p in self.parts:
+            p.sequences = value
+
+    @property
+    def device(self):
+        return self.parts[0].device
+
+    @property
+    def current_length(self) -> int:
+        return max(p.current_length for p in self.parts)
+
+    def check_capacity(self, end: int) -> None:
+        for p in self.parts:
+            p.check_capacity(end)
+
+    def check_pass(self, seq) -> None:
+        for p in self.parts:
+            p.check_pass(seq)
+
+    def deallocate_buffers(self) -> None:
+        for p in self.parts:
+            p.deallocate_buffers()
+
+    def token_positions(self) -> torch.Tensor:
+        return self.parts[0].token_positions()
+
+    def size_estimate(self) -> Tuple[int, Dict[str, int]]:
+        total, sizes = 0, {}
+        for side, p in zip(("left", "right"), self.parts):
+            n, detail = p.size_estimate()
+            total += n
+            sizes.update({f"{side}.{k}": v for k, v in detail.items()})
+        return total, sizes
+
+    def clone(self, device=None) -> "SideBySideCache":
+        other = super().clone(device)
+        other.parts = tuple(p.clone(device) for p in self.parts)
+        return other
+
+
+def layer_cache_class(spec: Dict[str, Any]) -> Type[LayerCache]:
+    """The cache class that serves the mixer described by ``spec``."""
+    from keys_values_b200.kvcache.grouped import BorrowedKVCache, GroupedKVCache
+    from keys_values_b200.kvcache.latent import LatentKVCache
+    from keys_values_b200.kvcache.recurrent import GatedLinearCache, GatedRecurrenceCache, RetentionCache, StateSpaceCache
+
+    if spec.get("kv_from") is not None:
+        return BorrowedKVCache
+    classes = {c.kind: c for c in (LatentKVCache, GroupedKVCache, StateSpaceCache, RetentionCache, GatedLinearCache, GatedRecurrenceCache, SideBySideCache)}
+    if spec["kind"] not in classes:
+        raise ValueError(f"no cache for mixers of kind {spec['kind']!r}")
+    return classes[spec["kind"]]

@@ -38,21 +38,52 @@ class RecurrentCache(LayerCache):
 class RetentionCache(RecurrentCache):
     kind = "retention"
 
-    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
         from keys_values_b200.models.retention import retention_shape
 
-        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device)
-        self.shape = retention_shape(config.layers[block_idx]["mixer"])
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        self.shape = retention_shape(self.spec)
+
+
+class GatedLinearCache(RecurrentCache):
+    kind = "gated_linear_attention"
+
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
+        from keys_values_b200.models.gated_linear import gated_linear_shape
+
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        self.shape = gated_linear_shape(self.spec)
+
+
+class GatedRecurrenceCache(RecurrentCache):
+    """One number per channel instead of a matrix per head: state ``(turns, max_batch_size, channels)``."""
+
+    kind = "gated_recurrence"
+
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
+        from keys_values_b200.models.gated_recurrence import recurrence_shape
+
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        self.shape = recurrence_shape(self.spec)
+
+    @property
+    def conv(self) -> Optional[torch.Tensor]:
+        """``(turns, max_batch_size, taps, channels)``."""
+        return None if self.buffers_ is None else self.buffers_[1]
+
+    def _shapes(self, dtype):
+        s = self.shape
+        return {"state": ((self.max_batch_size, s.channels), torch.float32), "conv": ((self.max_batch_size, s.taps, s.channels), dtype)}
 
 
 class StateSpaceCache(RecurrentCache):
     kind = "mamba2"
 
-    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **_ignored):
+    def __init__(self, config: Config, max_batch_size: int, cache_length: int, block_idx: int, dtype=None, device=None, **kwargs):
         from keys_values_b200.models.state_space import state_shape
 
-        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device)
-        self.shape = state_shape(config.layers[block_idx]["mixer"])
+        super().__init__(config, max_batch_size, cache_length, block_idx, dtype=dtype, device=device, **kwargs)
+        self.shape = state_shape(self.spec)
 
     @property
     def conv(self) -> Optional[torch.Tensor]:

@@ -6,16 +6,22 @@ differ. The mechanisms are modules of their own, picked by the description:
 * :class:`LatentAttention`: low-rank keys and values (one latent per token plus one rotated key part that the heads
   share), optional sliding window, ring cache of latents (:class:`keys_values_b200.kvcache.latent.LatentKVCache`);
 * :class:`keys_values_b200.models.grouped_attention.GroupedAttention`: grouped-query attention with optional norm of queries and
-  keys, windows or chunks, values shared with the keys, soft cap, softmax sink, output gate and differential maps;
+  keys, windows (also with pooled blocks before them) or chunks, keys and values of another layer, values shared with the keys, soft cap, softmax
+  sink, output gate and differential maps;
 * :class:`keys_values_b200.models.state_space.Mamba2Mixer`: state-space recurrence;
 * :class:`keys_values_b200.models.retention.Retention`: linear attention with a fixed decay per head;
+* :class:`keys_values_b200.models.gated_linear.GatedLinearAttention`: linear attention with a decay per token and key channel;
+* :class:`keys_values_b200.models.gated_recurrence.GatedRecurrence`: short convolution and a gated recurrence per channel;
+* :class:`keys_values_b200.models.side_by_side.SideBySide`: two mixers on the same input;
 * :class:`RoutedMLP`: softmax or sigmoid router, top-k experts with or without gates, optionally a shared expert;
-  :class:`DenseMLP`: two matrices and an activation; :class:`GatedMLP`: three matrices;
+  :class:`DenseMLP`: two matrices and an activation; :class:`GatedMLP`: three matrices, silu or a clamped unit;
 * :class:`ScalarRMSNorm`: RMS norm with one gain for all coordinates; :class:`StreamNorm`: layer or RMS norm of the fp32 stream;
 * token shift (``config.token_shift``): the mixer reads a learned blend of the token's normed input and the previous token's;
 * depth average (``config.depth_average``): what goes on to the next layer is a learned average of the embedding output
   and all layers' results so far;
 * bigram embedding (``config.bigram``): a hashed row for the pair (previous token, token) is added to the embedding;
+* position table (``config.position_table``): a learned vector per position is added to the embedding;
+* input convolution (``config.input_conv``): what a sublayer reads becomes itself plus a causal convolution of itself;
 * loop (``config.loop``): a run of layers is passed several times, with a cache or state of its own each time.
 
 Two kinds of layers: :class:`ParallelBlock` (mixer and feed-forward read one norm's output) and :class:`SequentialBlock` (one
@@ -33,13 +39,17 @@ import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
-from keys_values_b200.config import Config
+from keys_values_b200.config import STREAM_NORMS, Config
+from keys_values_b200.kvcache.grouped import BorrowedKVCache
 from keys_values_b200.kvcache.layer_cache import MAX_PASS_TOKENS, LayerCache
 from keys_values_b200.kvcache.sequences import SequencePass, SequenceTable
+from keys_values_b200.models.gated_linear import GatedLinearAttention
+from keys_values_b200.models.gated_recurrence import GatedRecurrence
 from keys_values_b200.models.grouped_attention import GroupedAttention
 from keys_values_b200.models.model import GPT
 from keys_values_b200.models.packed import Packed, pad_groups, pad_last
 from keys_values_b200.models.retention import Retention
+from keys_values_b200.models.side_by_side import SideBySide
 from keys_values_b200.models.state_space import Mamba2Mixer
 from keys_values_b200.ops import layers as L
 
@@ -70,23 +80,26 @@ class ScalarRMSNorm(nn.Module):
 
 
 class StreamNorm(Packed):
-    """Layer norm (``center``) or RMS norm of fp32 rows with one weight per coordinate and no bias."""
+    """Layer norm (``center``) or RMS norm of fp32 rows with one weight per coordinate and no bias. ``unit_offset``: the weight is stored
+    around zero, the norm is multiplied by 1 + weight."""
 
-    def __init__(self, size: int, eps: float = 1e-5, center: bool = True) -> None:
+    def __init__(self, size: int, eps: float = 1e-5, center: bool = True, unit_offset: bool = False) -> None:
         super().__init__()
-        self.weight = nn.Parameter(torch.ones(size))
+        self.weight = nn.Parameter(torch.zeros(size) if unit_offset else torch.ones(size))
         self.eps = eps
         self.center = center
+        self.unit_offset = unit_offset
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         rows = x.reshape(-1, self.weight.numel()).float().contiguous()
         return L.row_norm(rows, self.packed()["weight"], self.eps, self.center, self.weight.dtype).view(x.shape)
 
     def _make_pack(self) -> Dict[str, torch.Tensor]:
-        return {"weight": self.weight.float().contiguous()}
+        w = self.weight.float()
+        return {"weight": (1.0 + w if self.unit_offset else w).contiguous()}
 
     def reset_parameters(self) -> None:
-        nn.init.ones_(self.weight)
+        nn.init.constant_(self.weight, 0.0 if self.unit_offset else 1.0)
 
 
 class LatentAttention(Packed):
@@ -214,11 +227,15 @@ class RoutedMLP(Packed):
 
 
 class GatedMLP(Packed):
-    """``down(silu(gate x) · up x)``; gate and up projection are one product, rows ``[gate | up]``."""
+    """``down(silu(gate x) · up x)``; gate and up projection are one product, rows ``[gate | up]``. With a ``limit``: the clamped unit of
+    :func:`keys_values_b200.ops.layers.glu` instead."""
 
     def __init__(self, config: Config, spec: Dict[str, Any]) -> None:
         super().__init__()
         self.ff = spec["ff"]
+        self.limit = None if spec.get("limit") is None else float(spec["limit"])
+        if self.limit is not None and not self.limit > 0:
+            raise ValueError(f"limit = {self.limit} of a gated feed-forward must be positive")
         self.up = nn.Linear(config.n_embd, 2 * self.ff, bias=False)
         self.down = nn.Linear(self.ff, config.n_embd, bias=False)
 
@@ -228,7 +245,7 @@ class GatedMLP(Packed):
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         w = self.packed()
-        return F.linear(L.glu(F.linear(x, w["up"]), self.ff), w["down"])
+        return F.linear(L.glu(F.linear(x, w["up"]), self.ff, self.limit), w["down"])
 
 
 class DenseMLP(nn.Module):
@@ -246,7 +263,10 @@ class DenseMLP(nn.Module):
         return F.linear(L.activate(F.linear(x, self.up.weight), self.activation), self.down.weight)
 
 
-MIXERS = {"latent_attention": LatentAttention, "grouped_attention": GroupedAttention, "mamba2": Mamba2Mixer, "retention": Retention}
+MIXERS = {
+    "latent_attention": LatentAttention, "grouped_attention": GroupedAttention, "mamba2": Mamba2Mixer, "retention": Retention,
+    "gated_linear_attention": GatedLinearAttention, "gated_recurrence": GatedRecurrence, "side_by_side": SideBySide,
+}
 FEED_FORWARDS = {"routed": RoutedMLP, "dense": DenseMLP, "gated": GatedMLP}
 
 
@@ -263,6 +283,8 @@ class ParallelBlock(Packed):
         self.depth = None
         if config.depth_average:  # the identity: all weight on the layer's own result
             self.depth = nn.Parameter(F.one_hot(torch.tensor(block_idx + 1), block_idx + 2).float())
+        if config.input_conv or config.residual_mult != 1.0 or config.position_table:
+            raise NotImplementedError("input convolution, residual factor and position table go with sequential layers")
         if config.loop is not None or not (self.mlp is None or isinstance(self.mlp, RoutedMLP) and self.mlp.shared is None):
             raise NotImplementedError("parallel layers are not run in loops and have routed feed-forwards without a shared expert")
         if not (config.norm_1 and config.norm_2) or config.post_attention_norm or config.post_mlp_norm:
@@ -319,8 +341,8 @@ class SequentialBlock(Packed):
     def __init__(self, config: Config, block_idx: int, kv_cache=None) -> None:
         super().__init__()
         spec = config.layers[block_idx]
-        if config.norm_class_name not in ("StreamLayerNorm", "StreamRMSNorm"):
-            raise ValueError(f"norm {config.norm_class_name!r}: sequential layers take StreamLayerNorm or StreamRMSNorm")
+        if config.norm_class_name not in STREAM_NORMS:
+            raise ValueError(f"norm {config.norm_class_name!r}: sequential layers take one of {sorted(STREAM_NORMS)}")
         norm = partial(config.norm_class, config.n_embd, eps=config.norm_eps)
         self.norm_1 = norm() if config.norm_1 else None
         self.attn = MIXERS[spec["mixer"]["kind"]](config, block_idx, kv_cache)
@@ -330,27 +352,53 @@ class SequentialBlock(Packed):
         self.post_mlp_norm = norm() if self.mlp is not None and config.post_mlp_norm else None
         if config.token_shift or config.depth_average or config.bigram is not None:
             raise NotImplementedError("token shift, depth average and bigram embedding go with parallel layers")
-        self.center = config.norm_class_name == "StreamLayerNorm"
+        self.conv_1 = self.conv_2 = None
+        if config.input_conv:  # (width, taps), the last column meets the token itself
+            self.conv_1 = nn.Parameter(torch.zeros(config.n_embd, config.input_conv))
+            self.conv_2 = None if self.mlp is None else nn.Parameter(torch.zeros(config.n_embd, config.input_conv))
+            if isinstance(self.mlp, RoutedMLP):
+                raise NotImplementedError("routed experts and an input convolution")
+        if config.residual_mult != 1.0 and (self.post_attention_norm is None or self.mlp is not None and self.post_mlp_norm is None):
+            raise NotImplementedError("a residual factor goes with norms after the sublayers, whose weights take it")
+        self.center = STREAM_NORMS[config.norm_class_name]["center"]
         self.config = config
         self.block_idx = block_idx
 
     def _make_pack(self) -> Dict[str, Optional[torch.Tensor]]:
-        norms = dict(norm_1=self.norm_1, after_1=self.post_attention_norm, norm_2=self.norm_2, after_2=self.post_mlp_norm)
-        return {k: None if n is None else n.packed()["weight"] for k, n in norms.items()}
+        mult = self.config.residual_mult
+        norms = dict(norm_1=(self.norm_1, 1.0), after_1=(self.post_attention_norm, mult), norm_2=(self.norm_2, 1.0), after_2=(self.post_mlp_norm, mult))
+        pack = {k: None if n is None else n.packed()["weight"] * f for k, (n, f) in norms.items()}
+        for k, w in dict(conv_1=self.conv_1, conv_2=self.conv_2).items():
+            pack[k] = None if w is None else w.float().t().contiguous()
+        return pack
+
+    def _edge(self, model: "LayeredGPT", x: "LayerStream", y, after, before, conv, edge: int, want_h: bool = True, **kw: Any) -> None:
+        """From a sublayer's result to the next one's input, the ``edge``-th in the pass; ``conv``: what that input passes. A convolution over
+        several tokens reads a token's neighbours again, so the stream changes its place."""
+        ring = None if conv is None else model.sequences.conv[edge]
+        moves = conv is not None and x.x.shape[1] > 1
+        out = x.x if not moves else x.spare if x.spare is not None else torch.empty_like(x.x)
+        L.norm_edge(x.x, y, after, out, before, x.h if want_h else None, kw.get("idx"), kw.get("embed"), kw.get("step"), self.config.norm_eps, self.center,
+                    kw.get("experts"), None if conv is None else L.EdgeTokens(x.seq, None, conv, ring))
+        if moves:
+            x.x, x.spare = out, x.x
 
     def enter(self, model: "LayeredGPT", idx: torch.Tensor, seq: SequencePass) -> "LayerStream":
         """The stream in front of this (the first) layer."""
         wte = model.transformer.wte.weight
         x = torch.empty((*idx.shape, self.config.n_embd), dtype=torch.float32, device=wte.device)
         h = torch.empty(x.shape, dtype=wte.dtype, device=wte.device)
-        L.norm_edge(None, None, None, x, self.packed()["norm_1"], h, idx, wte, model.ahead_of_run(0)[1], self.config.norm_eps, self.center)
+        w, table = self.packed(), None if model.positions is None else model.positions.weight
+        ring = None if w["conv_1"] is None else model.sequences.conv[0]
+        tokens = None if table is None and ring is None else L.EdgeTokens(seq, table, w["conv_1"], ring)
+        L.norm_edge(None, None, None, x, w["norm_1"], h, idx, wte, model.ahead_of_run(0)[1], self.config.norm_eps, self.center, None, tokens)
         return LayerStream(seq, x, None, h, None)
 
     def run(self, model: "LayeredGPT", run: int, x: "LayerStream", idx: torch.Tensor) -> "LayerStream":
-        w, eps = self.packed(), self.config.norm_eps
+        w = self.packed()
         y, after, experts = self.attn(x.h, x.seq, model.runs[run][1]), w["after_1"], None
         if self.mlp is not None:
-            L.norm_edge(x.x, y, after, x.x, w["norm_2"], x.h, None, None, None, eps, self.center)
+            self._edge(model, x, y, after, w["norm_2"], w["conv_2"], 2 * run + 1)
             after = w["after_2"]
             if isinstance(self.mlp, RoutedMLP):
                 y = None if self.mlp.shared is None else self.mlp.shared(x.h)
@@ -358,11 +406,10 @@ class SequentialBlock(Packed):
             else:
                 y = self.mlp(x.h)
         last = run + 1 == model.n_runs
-        before = None if last else model.transformer.h[model.runs[run + 1][0]].packed()["norm_1"]
+        nxt = {"norm_1": None, "conv_1": None} if last else model.transformer.h[model.runs[run + 1][0]].packed()
         add_embedding, step = (False, None) if last else model.ahead_of_run(run + 1)
-        wte = model.transformer.wte.weight
-        L.norm_edge(x.x, y, after, x.x, before, None if last else x.h, idx.contiguous() if add_embedding else None, wte if add_embedding else None,
-                    step, eps, self.center, experts)
+        self._edge(model, x, y, after, nxt["norm_1"], nxt["conv_1"], 2 * run + 2, not last, idx=idx.contiguous() if add_embedding else None,
+                   embed=model.transformer.wte.weight if add_embedding else None, step=step, experts=experts)
         return x
 
 
@@ -401,6 +448,7 @@ class LayeredGPT(GPT):
         self.bigram = None
         if config.bigram is not None:  # the last row is for tokens without a predecessor
             self.bigram = nn.Embedding(config.bigram["buckets"] + 1, config.n_embd)
+        self.positions = nn.Embedding(config.block_size, config.n_embd) if config.position_table else None
         self.sequences: Optional[SequenceTable] = None
         if config.tie_embeddings:
             self.lm_head.weight = self.transformer.wte.weight
@@ -444,7 +492,7 @@ class LayeredGPT(GPT):
         if isinstance(module, RoutedMLP):
             nn.init.normal_(module.up, mean=0.0, std=0.02)
             nn.init.normal_(module.down, mean=0.0, std=0.02)
-        if isinstance(module, Mamba2Mixer):
+        if isinstance(module, (Mamba2Mixer, GatedLinearAttention, GatedRecurrence)):
             module.reset_parameters()
         if isinstance(module, Packed):
             module.drop_pack()
@@ -482,9 +530,11 @@ class LayeredGPT(GPT):
             return
         c = self.config
         self.sequences = SequenceTable(min(x.max_batch_size for x in caches), self.lm_head.weight.device,
-                                       c.n_layer if c.token_shift else 0, c.n_embd)
+                                       c.n_layer if c.token_shift else 0, c.n_embd, 2 * self.n_runs if c.input_conv else 0, c.input_conv)
         for x in caches:
             x.sequences = self.sequences
+            if isinstance(x, BorrowedKVCache):
+                x.set_source(caches[x.spec["kv_from"]])
 
     def clear_kv_caches(self) -> None:
         super().clear_kv_caches()
@@ -497,9 +547,14 @@ class LayeredGPT(GPT):
 
     def advance_host_counters(self) -> None:
         end = 1 + max(self.sequences.pos_host[s] for s in self.sequences.batch)
+        self._check_positions(end)
         for cache in self.get_kv_caches():
             cache.check_capacity(end)
         self.sequences.advance_host()
+
+    def _check_positions(self, end: int) -> None:
+        if self.positions is not None and end > self.positions.num_embeddings:
+            raise IndexError(f"{end} tokens exceed the table of {self.positions.num_embeddings} positions")
 
     def max_pass_tokens(self, batch_size: int) -> int:
         """Tokens per row that one pass of a chunked prefill may take."""
@@ -517,6 +572,7 @@ class LayeredGPT(GPT):
         if torch.is_grad_enabled():
             raise NotImplementedError("models with described layers run in inference only (use torch.inference_mode())")
         seq = self.sequences.begin(*idx.shape, counts)
+        self._check_positions(seq.max_end)
         for cache in self.get_kv_caches():
             cache.check_pass(seq)
         return self.transformer.h[0].enter(self, idx.contiguous(), seq)

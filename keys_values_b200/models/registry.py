@@ -9,7 +9,7 @@ from __future__ import annotations
 import json
 from dataclasses import dataclass
 from pathlib import Path
-from typing import Any, Callable, Dict, Mapping, Optional, Union
+from typing import Any, Callable, Dict, Mapping, Optional, Sequence, Union
 
 import torch
 
@@ -19,18 +19,25 @@ from keys_values_b200.config import Config
 @dataclass(frozen=True)
 class Architecture:
     name: str
-    config_from_json: Callable[[Dict[str, Any]], Config]
+    # content of config.json and shapes of the checkpoint's tensors by name (some sizes may stand there only)
+    config_from_json: Callable[[Dict[str, Any], Mapping[str, Sequence[int]]], Config]
     # the architecture's tensors (by name) -> state dict of the model class
     state_dict: Callable[[Mapping[str, torch.Tensor], Config], Dict[str, torch.Tensor]]
 
 
+def _from_content(reader: Callable[[Dict[str, Any]], Config]):
+    """Reader of a design whose configuration gives every size."""
+    return lambda content, shapes: reader(content)
+
+
 def _architectures() -> Dict[str, Architecture]:
-    from keys_values_b200.models import ladadra, mezilix, pazenex
+    from keys_values_b200.models import dotorax, ladadra, mezilix, pazenex
 
     known = (
-        Architecture("Ladadra", ladadra.config_from_json, ladadra.state_dict),
-        Architecture("Mezilix", mezilix.config_from_json, mezilix.state_dict),
-        Architecture("Pazenex", pazenex.config_from_json, pazenex.state_dict),
+        Architecture("Dotorax", dotorax.config_from_json, dotorax.state_dict),
+        Architecture("Ladadra", _from_content(ladadra.config_from_json), ladadra.state_dict),
+        Architecture("Mezilix", _from_content(mezilix.config_from_json), mezilix.state_dict),
+        Architecture("Pazenex", _from_content(pazenex.config_from_json), pazenex.state_dict),
     )
     return {a.name: a for a in known}
 
@@ -54,7 +61,7 @@ def config_from_directory(path: Union[str, Path], **kwargs: Any) -> Optional[Con
     content = json.loads(file.read_text(encoding="utf-8"))
     if not isinstance(content, dict) or "architecture" not in content:
         return None
-    config = get_architecture(content["architecture"]).config_from_json(content)
+    config = get_architecture(content["architecture"]).config_from_json(content, tensor_shapes(path))
     for k, v in kwargs.items():
         setattr(config, k, v)
     return config
@@ -78,6 +85,16 @@ def default_cache_name(config: Config, name: Optional[str] = None) -> str:
         return name or "h2o-default"
     fits = "latent-default" if all(x["mixer"]["kind"] == "latent_attention" for x in config.layers) else "layered-default"
     return name if name in ("layered-default", fits) else fits
+
+
+def tensor_shapes(checkpoint_dir: Union[str, Path]) -> Dict[str, Sequence[int]]:
+    """Shapes of a directory's ``*.safetensors`` by tensor name, from the files' headers."""
+    shapes: Dict[str, Sequence[int]] = {}
+    for file in sorted(Path(checkpoint_dir).glob("*.safetensors")):
+        with open(file, "rb") as f:
+            header = json.loads(f.read(int.from_bytes(f.read(8), "little")))
+        shapes.update({name: tuple(x["shape"]) for name, x in header.items() if name != "__metadata__"})
+    return shapes
 
 
 def read_safetensors(path: Path) -> Dict[str, torch.Tensor]:

@@ -87,7 +87,7 @@ class Mamba2Mixer(Packed):
         if x.shape[1] == 1:
             y = L.state_step(u, w["conv"], w["conv_bias"], w["dt_bias"], w["a_log"], w["skip"], ring, state, seq, s)
         else:
-            xbc = L.short_conv(u, w["conv"], w["conv_bias"], ring, seq, s)
+            xbc = L.short_conv(u, s.inner, w["conv"], w["conv_bias"], ring, seq)
             y = L.state_scan(u, xbc, w["dt_bias"], w["a_log"], w["skip"], state, seq, s)
         return F.linear(L.gated_group_norm(y, u, w["norm"], s, self.eps), w["proj"])
 

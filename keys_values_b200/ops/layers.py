@@ -1,5 +1,5 @@
 """Ops of models that are described layer by layer (fp32 residual stream, latent and grouped attention, state-space
-recurrence, retention, routed experts).
+recurrence, retention, gated linear attention, gated recurrence per channel, routed experts).
 
 A CUDA tensor is always served by the kernels of ``libkvb200_layers.so`` (bf16 or fp32; anything else
 raises), a CPU tensor by the PyTorch restatement in :mod:`keys_values_b200.ops.layers_reference`.
@@ -61,7 +61,10 @@ class GroupedShape:
     ``maps = 2``: differential attention, every head has two queries and two keys over the same values; the result is
     ``norm(map 1 − lam · map 2) · post``, the norm an RMS norm of the head without a weight.
     Position i sees j <= i, and only ``i − j < window`` or ``j < keep`` (``window > 0``), or its own part of ``chunk`` positions
-    (``chunk > 0``). ``softcap > 0``: scores become softcap · tanh(score / softcap)."""
+    (``chunk > 0``). ``pool > 0``: it also sees, as one key and one value each, the means of all blocks of ``pool`` positions that end
+    before its window. ``softcap > 0``: scores become softcap · tanh(score / softcap). One map: the result is multiplied by ``post``.
+
+    ``borrowed``: the keys and values are those of another layer; the projection has columns for queries and gate only."""
 
     heads: int
     kv_heads: int
@@ -82,6 +85,8 @@ class GroupedShape:
     lam: float = 0.0
     post: float = 1.0
     eps: float = 0.0
+    pool: int = 0
+    borrowed: bool = False
 
     @property
     def dimp(self) -> int:
@@ -99,11 +104,11 @@ class GroupedShape:
     @property
     def value_col(self) -> int:
         """First value column of the joint projection."""
-        return (self.heads + (0 if self.shared_value else self.kv_heads)) * self.maps * self.dimp
+        return (self.heads + (0 if self.shared_value or self.borrowed else self.kv_heads)) * self.maps * self.dimp
 
     @property
     def gate_col(self) -> int:
-        return (self.heads + self.kv_heads) * self.maps * self.dimp + (0 if self.shared_value else self.kv_heads * self.vdp)
+        return self.value_col if self.borrowed else (self.heads + self.kv_heads) * self.maps * self.dimp + (0 if self.shared_value else self.kv_heads * self.vdp)
 
     @property
     def gate_cols(self) -> int:
@@ -117,13 +122,20 @@ class GroupedShape:
 
     @property
     def span(self) -> int:
-        """Positions a query looks back at most, itself included and kept ones aside; 0: all."""
-        return self.chunk or self.window
+        """Positions a query looks back at most, itself included, kept ones and means of blocks aside (but a block's positions stay until its
+        mean is taken); 0: all."""
+        return max(self.chunk or self.window, self.pool)
+
+    @property
+    def inner(self) -> int:
+        """Columns of the result."""
+        return self.heads * self.vdp
 
 
 class RowPlan(NamedTuple):
     """Where the positions of a sequence lie: ``ring = 0`` position p in row p; else the first ``head`` positions have rows of
-    their own and position p >= head has row ``head + (p − head) mod ring``. Both are multiples of 128."""
+    their own and position p >= head has row ``head + (p − head) mod ring``; with pooled blocks the first ``head`` rows are those of the
+    blocks, and position p has row ``head + p mod ring``. Both are multiples of 128."""
 
     head: int = 0
     ring: int = 0
@@ -159,6 +171,105 @@ class RetentionShape:
     @property
     def key_scale(self) -> float:
         return self.dim**-0.5
+
+
+@dataclass(frozen=True)
+class GatedLinearShape:
+    """Sizes of one gated linear attention; padded sizes are multiples of 8. The projection has the columns ``[queries: heads · np |
+    keys: heads · np | low-rank input of the decays: rp | values: heads · vdp | gate: heads · vdp]``, every head padded with zeros."""
+
+    heads: int
+    dim: int
+    vdim: int
+    rank: int
+    tau: float
+
+    @property
+    def np(self) -> int:
+        return round8(self.dim)
+
+    @property
+    def vdp(self) -> int:
+        return round8(self.vdim)
+
+    @property
+    def rp(self) -> int:
+        return round8(self.rank)
+
+    @property
+    def qk(self) -> int:
+        """Columns of queries and keys."""
+        return 2 * self.heads * self.np
+
+    @property
+    def keys(self) -> int:
+        """Key channels of all heads, each with a decay of its own."""
+        return self.heads * self.np
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdp
+
+    @property
+    def query_scale(self) -> float:
+        return self.dim**-0.5
+
+
+class DecayWeights(NamedTuple):
+    """Second half of the decays' projection: ``weight (rank, keys)`` and ``bias (keys,)``, fp32."""
+
+    weight: torch.Tensor
+    bias: torch.Tensor
+
+
+@dataclass(frozen=True)
+class RecurrenceShape:
+    """Sizes of one gated recurrence per channel. ``blocks`` equal parts of the channels, each padded to a multiple of 8, with gates that are
+    square products within a part. The projection has the columns ``[y: channels | x: channels]``."""
+
+    width: int
+    blocks: int
+    taps: int
+
+    @property
+    def part(self) -> int:
+        return self.width // self.blocks
+
+    @property
+    def pp(self) -> int:
+        return round8(self.part)
+
+    @property
+    def channels(self) -> int:
+        """Padded width."""
+        return self.blocks * self.pp
+
+    @property
+    def inner(self) -> int:
+        return self.channels
+
+
+class RecurrenceWeights(NamedTuple):
+    """``conv (taps, channels)``, ``conv_bias``, ``bias_r``, ``bias_i`` and ``rate`` (log2 of the decay at an open gate) ``(channels,)``, all fp32;
+    ``gates (blocks, pp, 2 · pp)`` in the model's type: columns of the decay gates, then of the input gates of a part."""
+
+    conv: torch.Tensor
+    conv_bias: torch.Tensor
+    gates: torch.Tensor
+    bias_r: torch.Tensor
+    bias_i: torch.Tensor
+    rate: torch.Tensor
+
+
+class EdgeTokens(NamedTuple):
+    """What an edge between sublayers needs to know of its tokens: the pass; ``table`` (a vector per position is added to the stream); ``conv
+    (taps, width)`` fp32 and its ``ring (slots, taps, width)`` fp32 (what the sublayer reads, h, becomes h + a causal convolution of h; the ring
+    keeps the last h of every sequence, position p in row p mod taps)."""
+
+    seq: object
+    table: Optional[torch.Tensor] = None
+    conv: Optional[torch.Tensor] = None
+    ring: Optional[torch.Tensor] = None
 
 
 @dataclass(frozen=True)
@@ -244,12 +355,13 @@ def scalar_rmsnorm(x: torch.Tensor, gain: torch.Tensor, eps: float, dtype: torch
     return _impl(x).scalar_rmsnorm(x, rows, gain, eps, dtype)
 
 
-def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps: float, center: bool, experts=None) -> None:
+def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps: float, center: bool, experts=None, tokens: Optional[EdgeTokens] = None) -> None:
     """``x = x_in + norm(s) · after`` with ``s = sub + Σ_k weight_k · expert output_k`` (``x_in``, ``sub`` or ``experts`` ``None``:
     without it; ``after`` ``None``: ``s`` as it is), then ``x += embed[idx] + step`` (each unless ``None``); ``x_out = x`` (fp32, may be
     ``x_in``) and, unless ``h`` is ``None``, ``h = norm(x) · before`` (``before`` ``None``: ``h = x``). The norm takes the mean off if
-    ``center``. ``experts``: ``(out, row, weight)`` of :func:`routed_experts`."""
-    _impl(x_out).norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts)
+    ``center``. ``experts``: ``(out, row, weight)`` of :func:`routed_experts`. ``tokens``: see :class:`EdgeTokens`; with a convolution over
+    several tokens ``x_out`` must not be ``x_in`` (a token's neighbours are read again)."""
+    _impl(x_out).norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts, tokens)
 
 
 def row_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, center: bool, dtype: torch.dtype) -> torch.Tensor:
@@ -297,18 +409,19 @@ def latent_decode(q_abs, q, ring, seq, shape: LatentShape, scale: float) -> torc
 
 
 # ---- grouped-query attention
-def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape: GroupedShape, eps: float, plan: RowPlan = RowPlan()) -> torch.Tensor:
+def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape: GroupedShape, eps: float, plan: RowPlan = RowPlan(), q_scale=None) -> torch.Tensor:
     """Norm (unless ``norm_q`` is ``None``) and rotation of queries and keys of the joint projection ``qkv (B, T, ·)``. The norm goes over
-    a whole projection or (``head_norm``) over every head and map with weights of one head. Returns queries ``(B, T, heads · maps,
-    dimp)``; ``[keys of the maps | value]`` of every real token goes to its place in ``rows (slots, length, kv_heads, row)``."""
-    return _impl(qkv).grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape, eps, plan)
+    a whole projection or (``head_norm``) over every head and map with weights of one head; ``q_scale (heads,)`` multiplies queries. Returns
+    queries ``(B, T, heads · maps, dimp)``; ``[keys of the maps | value]`` of every real token goes to its place in ``rows (slots, length,
+    kv_heads, row)`` (unless they are ``borrowed``), and the means of blocks that the pass completes to theirs."""
+    return _impl(qkv).grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, shape, eps, plan, q_scale)
 
 
-def grouped_attend(q, qkv, rows, seq, shape: GroupedShape, sink=None, plan: RowPlan = RowPlan()) -> torch.Tensor:
+def grouped_attend(q, qkv, rows, seq, shape: GroupedShape, sink=None, plan: RowPlan = RowPlan(), out=None) -> torch.Tensor:
     """Causal attention of ``q (B, T, heads · maps, dimp)`` over ``rows``, which hold the pass already; with the gate of ``qkv``
     applied. ``sink (heads,)`` fp32: logarithms of what shapes with a sink add to the denominators (``None``: zeros). Returns
-    ``(B, T, heads · vdp)``."""
-    return _impl(q).grouped_attend(q, qkv, rows, seq, shape, sink, plan)
+    ``(B, T, heads · vdp)``, in ``out`` if that is given (rows of any leading dimension)."""
+    return _impl(q).grouped_attend(q, qkv, rows, seq, shape, sink, plan, out)
 
 
 # ---- retention
@@ -323,9 +436,10 @@ def retention_scan(qk, v, decay, log2_decay, state, seq, shape: RetentionShape) 
     return _impl(qk).retention_scan(qk, v, decay, log2_decay, state, seq, shape)
 
 
-def head_norm_gate(y, gate, shape: RetentionShape, eps: float) -> torch.Tensor:
-    """``y (B, T, inner)`` divided by every head's root mean square, times silu of ``gate`` (rows of any leading dimension)."""
-    return _impl(y).head_norm_gate(y, gate, shape, eps)
+def head_norm_gate(y, gate, shape, eps: float, weight=None) -> torch.Tensor:
+    """``y (B, T, inner)`` divided by every head's root mean square, times ``weight (vdp,)`` (``None``: without), times silu of ``gate`` (rows of
+    any leading dimension)."""
+    return _impl(y).head_norm_gate(y, gate, shape, eps, weight)
 
 
 def retention_step(u, freq, decay, state, seq, shape: RetentionShape, eps: float, dtype: torch.dtype) -> torch.Tensor:
@@ -333,11 +447,33 @@ def retention_step(u, freq, decay, state, seq, shape: RetentionShape, eps: float
     return _impl(u).retention_step(u, freq, decay, state, seq, shape, eps, dtype)
 
 
+# ---- gated linear attention
+def gated_linear_scan(qka, v, decay: DecayWeights, state, seq, shape: GatedLinearShape) -> torch.Tensor:
+    """``S_t = diag(alpha_t) S_(t−1) + k_t v_t^T``, ``o_t = S_t^T q_t · query_scale`` per head over the tokens of a pass, from and to ``state
+    (slots, heads, np, vdp)`` fp32. ``qka (B, T, qk + rp)`` fp32: queries, keys and input a of the decays ``alpha = sigmoid(weight^T a +
+    bias)^(1 / tau)``; ``v``: rows of any leading dimension whose first ``inner`` columns are the values. Returns ``(B, T, inner)``."""
+    return _impl(qka).gated_linear_scan(qka, v, decay, state, seq, shape)
+
+
+def gated_linear_step(u, decay: DecayWeights, weight, state, seq, shape: GatedLinearShape, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """The scan, norm (times ``weight (vdp,)``) and gate for one token per sequence, from the fp32 projections ``u (B, 1, qk + rp + 2 inner)``; all
+    of it in fp32."""
+    return _impl(u).gated_linear_step(u, decay, weight, state, seq, shape, eps, dtype)
+
+
+# ---- gated recurrence per channel
+def gated_recurrence(u, w: RecurrenceWeights, ring, state, seq, shape: RecurrenceShape, scale: float, out) -> torch.Tensor:
+    """``u (B, T, 2 · channels)``: y and x. x passes a causal convolution (its inputs before the pass come from ``ring``), gives gates r and i, and
+    ``S_t = a S_(t−1) + sqrt(1 − a²) i x`` with ``log2 a = rate · r``, from and to ``state (slots, channels)`` fp32. Returns ``out (B, T, channels)``
+    = S · gelu(y) · ``scale``, zero in padding. u and out: rows of any leading dimension."""
+    return _impl(u).gated_recurrence(u, w, ring, state, seq, shape, scale, out)
+
+
 # ---- state-space recurrence
-def short_conv(u, w, bias, ring, seq, shape: StateShape) -> torch.Tensor:
-    """Causal convolution ``w (taps, channels)`` with bias and silu over the channels of ``u (B, T, ld)``; the inputs before the
+def short_conv(u, col: int, w, bias, ring, seq, silu: bool = True) -> torch.Tensor:
+    """Causal convolution ``w (taps, channels)`` with bias (and silu) over the channels of ``u (B, T, ·)`` from ``col`` on; the inputs before the
     pass come from ``ring (slots, taps, channels)``, which takes the last ones of the pass. Returns ``(B, T, channels)``."""
-    return _impl(u).short_conv(u, w, bias, ring, seq, shape)
+    return _impl(u).short_conv(u, col, w, bias, ring, seq, silu)
 
 
 def state_scan(u, xbc, dt_bias, a_log, skip, state, seq, shape: StateShape) -> torch.Tensor:
@@ -361,9 +497,10 @@ def activate(x: torch.Tensor, activation: str) -> torch.Tensor:
     return x if activation == "none" else _impl(x).activate(x, ACTIVATIONS[activation])
 
 
-def glu(x: torch.Tensor, ff: int) -> torch.Tensor:
-    """``x (n, 2 · round8(ff))`` = ``[gate | up]`` → ``silu(gate) · up (n, round8(ff))``, zero in the padding."""
-    return _impl(x).glu(x, ff)
+def glu(x: torch.Tensor, ff: int, limit: Optional[float] = None) -> torch.Tensor:
+    """``x (n, 2 · round8(ff))`` = ``[gate | up]`` → ``silu(gate) · up (n, round8(ff))``, zero in the padding. With a ``limit``: the clamped unit
+    ``g · sigmoid(1.702 g) · (u + 1)`` with ``g = min(gate, limit)`` and u = up clamped to ±limit."""
+    return _impl(x).glu(x, ff, limit)
 
 
 # ---- routed experts. silu_gated: the rows of gate and up projection in turns, act(up h) = silu(gate h) · (up h)

@@ -1,6 +1,8 @@
 """PyTorch restatement of :mod:`keys_values_b200.ops.layers` for CPU tensors (same layouts, same padding)."""
 from __future__ import annotations
 
+import math
+
 import torch
 import torch.nn.functional as F
 
@@ -157,9 +159,14 @@ def moe_forward(h, logits, up, down, top, act, rule, n_up, n_down, correction=No
     return out, torch.arange(n * top, dtype=torch.int32).view(n, top), weight
 
 
-def glu(x, ff):
+def glu(x, ff, limit=None):
     n = x.shape[-1] // 2
-    y = F.silu(x[..., :n].float()) * x[..., n:].float()
+    g, u = x[..., :n].float(), x[..., n:].float()
+    if limit is None:
+        y = F.silu(g) * u
+    else:
+        g = g.clamp(max=limit)
+        y = g * torch.sigmoid(1.702 * g) * (u.clamp(-limit, limit) + 1)
     y[..., ff:] = 0
     return y.to(x.dtype)
 
@@ -171,7 +178,21 @@ def _norm(x, weight, eps, center):
     return x / torch.sqrt(x.square().mean(-1, keepdim=True) + eps) * weight
 
 
-def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None) -> None:
+def _input_conv(h, w, ring, seq):
+    """h + causal convolution of h; the ring takes the last ones of every sequence."""
+    taps = w.shape[0]
+    B, T, _ = h.shape
+    out = h.clone()
+    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
+        before = [ring[slot, p % taps] if p >= 0 else torch.zeros_like(h[b, 0]) for p in range(start - taps + 1, start)]
+        rows = torch.cat((torch.stack(before), h[b])) if before else h[b]
+        out[b] += sum(w[k] * rows[k : k + T] for k in range(taps))
+        for t in range(max(0, n - taps), n):
+            ring[slot, (start + t) % taps] = h[b, t]
+    return out
+
+
+def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None, tokens=None) -> None:
     x = torch.zeros_like(x_out) if x_in is None else x_in
     s = None if sub is None else sub.float()
     if experts is not None:
@@ -185,11 +206,15 @@ def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center,
         if int(idx.min()) < 0 or int(idx.max()) >= embed.shape[0]:
             raise IndexError("token id outside of the vocabulary")
         x = x + embed[idx].float()
+    if tokens is not None and tokens.table is not None:
+        at = (tokens.seq.start[:, None] + torch.arange(x_out.shape[1])).clamp(max=tokens.table.shape[0] - 1)  # padding may lie beyond
+        x = x + tokens.table[at.long()].float()
     if step is not None:
         x = x + step
     x_out.copy_(x)
     if h is not None:
-        h.copy_(x if before is None else _norm(x, before, eps, center))
+        y = x if before is None else _norm(x, before, eps, center)
+        h.copy_(y if tokens is None or tokens.conv is None else _input_conv(y, tokens.conv, tokens.ring, tokens.seq))
 
 
 def row_norm(x, weight, eps, center, dtype):
@@ -201,14 +226,16 @@ def activate(x, act):
 
 
 # ---- grouped-query attention
-def _places(plan, positions):
+def _places(s, plan, positions):
     p = torch.as_tensor(positions)
+    if s.pool:
+        return plan.head + p % plan.ring
     return p if plan.ring == 0 else torch.where(p < plan.head, p, plan.head + (p - plan.head) % plan.ring)
 
 
-def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan):
+def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan, q_scale=None):
     B, T, _ = qkv.shape
-    H, G = s.heads * s.maps, s.kv_heads * s.maps
+    H, G = s.heads * s.maps, 0 if s.borrowed else s.kv_heads * s.maps
     nq, nk = H * s.dimp, G * s.dimp
     q, k = qkv[..., :nq].float(), qkv[..., nq : nq + nk].float()
     if norm_q is not None and s.head_norm:
@@ -219,12 +246,21 @@ def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan):
         k = k / torch.sqrt(k.square().sum(-1, keepdim=True) / (G * s.dim) + eps) * norm_k
     angle = (seq.start[:, None] + torch.arange(T)).float()[..., None] * freq
     cos, sin = angle.cos()[:, :, None], angle.sin()[:, :, None]
-    q = _rotate(q.reshape(B, T, H, s.dimp), cos, sin, s.rot_dims).to(qkv.dtype)
+    q = _rotate(q.reshape(B, T, H, s.dimp), cos, sin, s.rot_dims)
+    if q_scale is not None:
+        q = q * q_scale.repeat_interleave(s.maps)[:, None]
+    q = q.to(qkv.dtype)
+    if s.borrowed:
+        return q
     k = _rotate(k.reshape(B, T, G, s.dimp), cos, sin, s.rot_dims).to(qkv.dtype).reshape(B, T, s.kv_heads, s.maps * s.dimp)
     v = qkv[..., s.value_col : s.value_col + s.kv_heads * s.vdp].view(B, T, s.kv_heads, s.vdp)
     for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
-        at = _places(plan, torch.arange(start, start + n))
+        at = _places(s, plan, torch.arange(start, start + n))
         rows[slot, at] = torch.cat((k[b, :n], v[b, :n]), -1)
+        if s.pool:
+            for block in range(start // s.pool, (start + n) // s.pool):
+                held = _places(s, plan, torch.arange(block * s.pool, (block + 1) * s.pool))
+                rows[slot, block] = rows[slot, held].float().mean(0).to(rows.dtype)
     return q
 
 
@@ -237,7 +273,7 @@ def _seen(s, query, key):
     return seen & ((i - j < s.window) | (j < s.keep)) if s.window else seen
 
 
-def grouped_attend(q, qkv, rows, seq, s, sink, plan):
+def grouped_attend(q, qkv, rows, seq, s, sink, plan, into=None):
     B, T = q.shape[:2]
     out = torch.zeros(B, T, s.heads, s.vdp)
     for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
@@ -245,9 +281,13 @@ def grouped_attend(q, qkv, rows, seq, s, sink, plan):
             continue
         key = torch.arange(start + n)
         if plan.ring:  # positions that are seen no more have lost their rows
-            key = key[(key < plan.head) | (key > start - s.span)]
-        kv = rows[slot, _places(plan, key)].float().repeat_interleave(s.heads // s.kv_heads, dim=1)
-        hidden = ~_seen(s, start + torch.arange(n), key)
+            key = key[((key < plan.head) & (s.pool == 0)) | (key > start - s.span)]
+        places, hidden = _places(s, plan, key), ~_seen(s, start + torch.arange(n), key)
+        if s.pool:
+            block = torch.arange((start + n) // s.pool)
+            places = torch.cat((block, places))
+            hidden = torch.cat(((block[None] + 1) * s.pool - 1 > start + torch.arange(n)[:, None] - s.window, hidden), 1)
+        kv = rows[slot, places].float().repeat_interleave(s.heads // s.kv_heads, dim=1)
         maps = []
         for u in range(s.maps):
             score = torch.einsum("thd,jhd->htj", q[b, :n, u :: s.maps].float(), kv[..., u * s.dimp : (u + 1) * s.dimp]) * s.scale
@@ -257,15 +297,16 @@ def grouped_attend(q, qkv, rows, seq, s, sink, plan):
             if s.sink:
                 add = torch.zeros(s.heads) if sink is None else sink
                 score = torch.cat((score, add.view(-1, 1, 1).expand(-1, n, 1)), dim=-1)
-            maps.append(torch.einsum("htj,jhv->thv", score.softmax(-1)[..., : len(key)], kv[..., s.maps * s.dimp :]))
+            maps.append(torch.einsum("htj,jhv->thv", score.softmax(-1)[..., : len(places)], kv[..., s.maps * s.dimp :]))
         if s.maps == 2:
             d = maps[0] - s.lam * maps[1]
-            maps[0] = d / torch.sqrt(d.square().sum(-1, keepdim=True) / s.vdim + s.eps) * s.post
-        out[b, :n] = maps[0]
+            maps[0] = d / torch.sqrt(d.square().sum(-1, keepdim=True) / s.vdim + s.eps)
+        out[b, :n] = maps[0] * s.post
     if s.gate:
         gate = torch.sigmoid(qkv[..., s.gate_col : s.gate_col + s.heads * s.gate_cols].float())
         out = out * gate.view(B, T, s.heads, s.gate_cols)
-    return out.view(B, T, -1).to(q.dtype)
+    out = out.view(B, T, -1).to(q.dtype)
+    return out if into is None else into.copy_(out)
 
 
 # ---- retention
@@ -293,9 +334,11 @@ def retention_scan(qk, v, decay, log2_decay, state, seq, s):
     return y.view(B, T, -1).to(qk.dtype)
 
 
-def head_norm_gate(y, gate, s, eps):
+def head_norm_gate(y, gate, s, eps, weight=None):
     x = y.float().view(*y.shape[:-1], s.heads, s.vdp)
     x = x / torch.sqrt(x.square().sum(-1, keepdim=True) / s.vdim + eps)
+    if weight is not None:
+        x = x * weight
     return (x.view(y.shape) * F.silu(gate[..., : s.inner].float())).to(y.dtype)
 
 
@@ -305,17 +348,67 @@ def retention_step(u, freq, decay, state, seq, s, eps, dtype):
     return head_norm_gate(y, u[..., s.qk + s.inner :], s, eps).to(dtype)
 
 
-# ---- state-space recurrence
-def short_conv(u, w, bias, ring, seq, s):
-    B, T, _ = u.shape
-    x = u[..., s.inner : s.dt_col].float()
-    out = torch.empty(B, T, s.channels, dtype=u.dtype)
+# ---- gated linear attention
+def _log_decay(a, decay, s):
+    """Logarithms of the decays ``(B, T, heads, np)``."""
+    z = a.float()[..., : s.rank] @ decay.weight + decay.bias
+    return (F.logsigmoid(z) / s.tau).view(*a.shape[:-1], s.heads, s.np)
+
+
+def gated_linear_scan(qka, v, decay, state, seq, s):
+    B, T = qka.shape[:2]
+    q, k = qka[..., : s.qk].view(B, T, 2, s.heads, s.np).unbind(2)
+    alpha = torch.exp(_log_decay(qka[..., s.qk :], decay, s))
+    dtype, v = v.dtype, v[..., : s.inner].float().reshape(B, T, s.heads, s.vdp)
+    y = torch.zeros(B, T, s.heads, s.vdp)
     for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
-        before = [ring[slot, p % s.taps].float() if p >= 0 else torch.zeros(s.channels) for p in range(start - s.taps + 1, start)]
+        S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+        for t in range(n):
+            S = alpha[b, t, :, :, None] * S + k[b, t, :, :, None] * v[b, t, :, None]
+            y[b, t] = torch.einsum("hnp,hn->hp", S, q[b, t] * s.query_scale)
+        if n > 0:
+            state[slot] = S
+    return y.view(B, T, -1).to(dtype)
+
+
+def gated_linear_step(u, decay, weight, state, seq, s, eps, dtype):
+    y = gated_linear_scan(u[..., : s.qk + s.rp], u[..., s.qk + s.rp :], decay, state, seq, s)
+    return head_norm_gate(y, u[..., s.qk + s.rp + s.inner :], s, eps, weight).to(dtype)
+
+
+# ---- gated recurrence per channel
+def gated_recurrence(u, w, ring, state, seq, s, scale, out):
+    B, T, _ = u.shape
+    x = short_conv(u, s.channels, w.conv, w.conv_bias, ring, seq, False)
+    z = torch.einsum("btpk,pkn->btpn", x.float().view(B, T, s.blocks, s.pp), w.gates.float())
+    r, i = (torch.sigmoid(g.reshape(B, T, -1) + b) for g, b in zip(z.split(s.pp, dim=-1), (w.bias_r, w.bias_i)))
+    log_a = r * w.rate * math.log(2.0)
+    a, add = torch.exp(log_a), torch.sqrt(-torch.expm1(2 * log_a)) * i * x.float()
+    y = F.gelu(u[..., : s.channels].float(), approximate="tanh") * scale
+    out.zero_()
+    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
+        S = state[slot].clone() if start > 0 else torch.zeros_like(state[slot])
+        for t in range(n):
+            S = a[b, t] * S + add[b, t]
+            out[b, t] = (S * y[b, t]).to(out.dtype)
+        if n > 0:
+            state[slot] = S
+    return out
+
+
+# ---- state-space recurrence
+def short_conv(u, col, w, bias, ring, seq, silu=True):
+    B, T, _ = u.shape
+    taps, channels = w.shape
+    x = u[..., col : col + channels].float()
+    out = torch.empty(B, T, channels, dtype=u.dtype)
+    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
+        before = [ring[slot, p % taps].float() if p >= 0 else torch.zeros(channels) for p in range(start - taps + 1, start)]
         rows = torch.cat((torch.stack(before), x[b])) if before else x[b]
-        out[b] = F.silu(sum(w[k] * rows[k : k + T] for k in range(s.taps)) + bias)
-        for t in range(max(0, n - s.taps), n):
-            ring[slot, (start + t) % s.taps] = u[b, t, s.inner : s.dt_col]
+        y = sum(w[k] * rows[k : k + T] for k in range(taps)) + bias
+        out[b] = F.silu(y) if silu else y
+        for t in range(max(0, n - taps), n):
+            ring[slot, (start + t) % taps] = u[b, t, col : col + channels]
     return out
 
 
@@ -337,7 +430,7 @@ def state_scan(u, xbc, dt_bias, a_log, skip, state, seq, s):
 
 
 def state_step(u, w, bias, dt_bias, a_log, skip, ring, state, seq, s):
-    return state_scan(u, short_conv(u, w, bias, ring, seq, s), dt_bias, a_log, skip, state, seq, s)
+    return state_scan(u, short_conv(u, s.inner, w, bias, ring, seq), dt_bias, a_log, skip, state, seq, s)
 
 
 def gated_group_norm(y, u, weight, s, eps):

@@ -400,7 +400,7 @@ def sequential_kernel_table(config: Config, batch: int, tokens: int = 8192) -> L
         cw, cb, db, al, sk = f32(m.taps, m.channels), f32(m.channels), f32(m.heads) - 4, f32(m.heads), f32(m.heads)
         state_bytes = B * m.heads * m.np * m.vdp * 8
         if T > 1:
-            tab.add(f"{tag}: convolution, {m.channels} channels", lambda: LC.short_conv(u, cw, cb, ring, seq, m), gbytes=4 * n * m.channels / 1e9)
+            tab.add(f"{tag}: convolution, {m.channels} channels", lambda: LC.short_conv(u, m.inner, cw, cb, ring, seq, True), gbytes=4 * n * m.channels / 1e9)
             xbc = rand(B, T, m.channels)
             flop = n * (m.heads * (4 * m.np * m.vdp + 128 * m.vdp) + m.groups * 128 * m.np) / 1e12
             by = (2 * n * (m.channels + m.inner + m.heads) + state_bytes) / 1e9

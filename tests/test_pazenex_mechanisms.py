@@ -335,7 +335,7 @@ def test_short_conv(env, name):
         counts = [min(k, T - a) for k, a in zip(counts, at)]
         seq = tab.begin(2, n, counts)
         seq.start = seq.start.clone()
-        out = L.short_conv(part_of(u, at, n, counts), wp, bp, ring, seq, s)
+        out = L.short_conv(part_of(u, at, n, counts), s.inner, wp, bp, ring, seq)
         for i in range(2):
             if counts[i]:
                 close(out[i, : counts[i]], want[i][at[i] : at[i] + counts[i]], dtype)
@@ -435,7 +435,7 @@ def test_state_step(env, name):
             seq = tab.begin(2, prompt, [prompt, prompt - 2])
             seq.start = seq.start.clone()
             part = part_of(u, at, prompt, seq.count_host)
-            xbc = L.short_conv(part, wp, bp, ring, seq, s)
+            xbc = L.short_conv(part, s.inner, wp, bp, ring, seq)
             L.state_scan(part, xbc, *vec, state, seq, s)
             at = list(seq.count_host)
             move(tab, seq)
