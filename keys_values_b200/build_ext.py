@@ -1,7 +1,7 @@
 """Builds the CUDA/C++ sources under ``csrc/`` for sm_100a, in-tree, into two libraries:
 ``libkvb200.so`` (caches, attention, GEMM, collectives of the LitGPT-shaped models) and
 ``libkvb200_layers.so`` (kernels of models described layer by layer: latent and grouped attention,
-state-space recurrence, retention, routed experts, token shift, depth averages, norms). Each loads on its own, so a command that needs one
+state-space recurrence, retention, gated linear attention, gated recurrence, routed experts, token shift, depth averages, norms). Each loads on its own, so a command that needs one
 of them compiles no more than that.
 
 Usage: ``python -m keys_values_b200.build_ext [--force] [--verbose]``. nvcc
@@ -23,7 +23,7 @@ CSRC = ROOT / "csrc"
 BUILD = CSRC / "build"
 LIB = ROOT / "libkvb200.so"
 LAYERS_LIB = ROOT / "libkvb200_layers.so"
-LAYERS_SOURCES = ("grouped_attn", "latent_attn", "latent_sm100", "layer_edge", "moe", "moe_sm100", "norm_edge", "retention", "ssm", "ssm_sm100")
+LAYERS_SOURCES = ("gated_linear", "gated_recurrence", "grouped_attn", "latent_attn", "latent_sm100", "layer_edge", "moe", "moe_sm100", "norm_edge", "retention", "ssm", "ssm_sm100")
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

@@ -13,9 +13,18 @@ __host__ __device__ __forceinline__ int seen_from(const kvb_attention& a, int hi
   return a.window > 0 && hi >= a.window ? hi - a.window + 1 : 0;
 }
 
+// Blocks that position hi sees (at most as many as there are rows for: padding may lie beyond the cache).
+__host__ __device__ __forceinline__ int blocks_seen(const kvb_attention& a, int hi) {
+  const int before = hi - a.window + 1;  // positions ahead of the window
+  if (a.pool == 0 || before <= 0) return 0;
+  const int n = before / a.pool;
+  return n < a.head ? n : a.head;
+}
+
 // Row of a position: without a ring the position itself; with one the first `head` positions have rows of their own and the others
-// share `ring` rows.
+// share `ring` rows; with pooled blocks the first `head` rows are theirs.
 __host__ __device__ __forceinline__ int row_of(const kvb_attention& a, int pos) {
+  if (a.pool > 0) return a.head + pos % a.ring;
   return a.ring == 0 || pos < a.head ? pos : a.head + (pos - a.head) % a.ring;
 }
 

@@ -2,6 +2,7 @@
 //
 //   prep    root mean squares of the whole query and key projections or of every head, rotation (angles in fp32, once per token),
 //           padded queries out, keys and values to their positions in the cache;
+//   pool    means of keys and values of the blocks that a pass completes (one token: the end of prep);
 //   attend  CUDA cores: fp32, and shapes that the tcgen05 kernel (latent_sm100.cu) does not take;
 //   decode  one new token per sequence, bf16: the positions are split over CTAs, K and V tiles come by TMA and meet the heads
 //           of a group as mma.sync tiles; a second kernel puts the parts together.
@@ -36,6 +37,38 @@ struct GpParams {
   unsigned rot_magic, rest_magic;
 };
 
+// Columns [c, c + V) of the mean of the rows of block `block` of a sequence; slot: its first row.
+template <typename T, int V>
+__device__ __forceinline__ void pool_columns(T* slot, const kvb_attention& a, long long step, int block, int c) {
+  using Vec = GpVec<T, V>;
+  float s[V];
+#pragma unroll
+  for (int e = 0; e < V; ++e) s[e] = 0.f;
+#pragma unroll 8
+  for (int j = 0; j < a.pool; ++j) {
+    const Vec v = *reinterpret_cast<const Vec*>(slot + row_of(a, block * a.pool + j) * step + c);
+#pragma unroll
+    for (int e = 0; e < V; ++e) s[e] += to_f32(v.v[e]);
+  }
+  const float inv = 1.f / (float)a.pool;
+  Vec r;
+#pragma unroll
+  for (int e = 0; e < V; ++e) r.v[e] = from_f32<T>(s[e] * inv);
+  *reinterpret_cast<Vec*>(slot + block * step + c) = r;
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(GP_THREADS)
+grouped_pool_kernel(T* __restrict__ rows, const GpParams p) {
+  const int b = blockIdx.y, block = p.start[b] / p.a.pool + blockIdx.x;
+  // complete with this pass, and with a row of its own
+  if ((block + 1) * p.a.pool > p.start[b] + p.count[b] || block >= p.a.head) return;
+  const int row = p.a.maps * p.a.dimp + p.a.vdp;
+  const long long step = (long long)p.a.kv_heads * row;
+  T* slot = rows + (long long)p.slots[b] * p.len * step;
+  for (int c = threadIdx.x * V; c < step; c += GP_THREADS * V) pool_columns<T, V>(slot, p.a, step, block, c);
+}
+
 template <typename T, int V>
 __global__ void __launch_bounds__(GP_THREADS)
 grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict__ rows, const GpParams p) {
@@ -50,8 +83,17 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
   for (int k = threadIdx.x; k < half; k += GP_THREADS) sincosf((float)pos * p.freq[k], &cs_sm[half + k], &cs_sm[k]);
   const int maps = p.a.maps, row = maps * p.dimp + p.vdp, place = row_of(p.a, pos);
   // where the token's keys and values go; padding goes nowhere
-  T* const dst = (t < p.count[b] && place < p.len) ? rows + ((long long)p.slots[b] * p.len + place) * p.a.kv_heads * row : nullptr;
+  T* const dst = (!p.a.borrowed && t < p.count[b] && place < p.len) ? rows + ((long long)p.slots[b] * p.len + place) * p.a.kv_heads * row : nullptr;
   const bool shared = p.value_col == nq;
+  // a single token may complete a block; the rows before it are those of earlier passes
+  auto pool = [&]() {
+    const int size = p.a.pool;
+    if (size == 0 || p.T > 1 || !dst || (pos + 1) % size || pos / size >= p.a.head) return;  // the same for all threads
+    __syncthreads();
+    const long long step = (long long)p.a.kv_heads * row;
+    T* slot = rows + (long long)p.slots[b] * p.len * step;
+    for (int c = threadIdx.x * V; c < step; c += GP_THREADS * V) pool_columns<T, V>(slot, p.a, step, pos / size, c);
+  };
   // one piece of a head: the key part of the cache or the query
   auto put = [&](int h, int col, const Vec& v) {
     if (h < p.heads) *reinterpret_cast<Vec*>(q + (n * p.heads + h) * p.dimp + col) = v;
@@ -86,10 +128,12 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
       const float r = 1.f / sqrtf(s / (float)p.dim + p.a.eps);
       const int h = i / per_head, col = (i - h * per_head) * V;
       const float* w = (h < p.heads ? p.norm_q : p.norm_k) + col;
+      const float f = p.a.q_scale && h < p.heads ? r * p.a.q_scale[h / maps] : r;
 #pragma unroll
-      for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(to_f32(a.v[e]) * r * w[e]);
+      for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(to_f32(a.v[e]) * f * w[e]);
       put(h, col, a);
     }
+    pool();
     return;
   }
   float rq = 1.f, rk = 1.f;
@@ -135,10 +179,11 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
     rk = 1.f / sqrtf(s1 / (float)(p.kv_heads * p.dim) + p.a.eps);
   }
   auto normed = [&](int h, int col, const Vec& a, float (&x)[V]) {
-    const float r = p.norm_q && !whole ? head_r[h] : (h < p.heads ? rq : rk);
+    float r = p.norm_q && !whole ? head_r[h] : (h < p.heads ? rq : rk);
+    if (p.a.q_scale && h < p.heads) r *= p.a.q_scale[h / maps];
     const float* w = p.norm_q ? (h < p.heads ? p.norm_q + (whole ? h * p.dimp : 0) : p.norm_k + (whole ? (h - p.heads) * p.dimp : 0)) + col : nullptr;
 #pragma unroll
-    for (int e = 0; e < V; ++e) x[e] = p.norm_q ? to_f32(a.v[e]) * r * w[e] : to_f32(a.v[e]);
+    for (int e = 0; e < V; ++e) x[e] = p.norm_q ? to_f32(a.v[e]) * r * w[e] : to_f32(a.v[e]) * r;
   };
   const int all = p.heads + p.kv_heads;
   const int ru = half / V;
@@ -175,6 +220,7 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
     put(h, k, a);
   }
   if (!shared && dst) put_values();
+  pool();
 }
 
 template <typename T, int V>
@@ -187,6 +233,7 @@ static int gp_launch_vec(const void* qkv, void* q, void* rows, GpParams& p, int 
   const size_t smem = (size_t)(p.rot_dims + (p.a.head_norm ? p.heads + p.kv_heads : 0)) * sizeof(float) + 8;
   if (smem > 48 * 1024) return KVB_ERR_TOO_LARGE;
   grouped_prep_kernel<T, V><<<dim3(p.T, B), GP_THREADS, smem, s>>>((const T*)qkv, (T*)q, (T*)rows, p);
+  if (p.a.pool > 0 && p.T > 1) grouped_pool_kernel<T, 16 / sizeof(T)><<<dim3(p.T / p.a.pool + 1, B), GP_THREADS, 0, s>>>((T*)rows, p);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
@@ -225,7 +272,7 @@ grouped_attend_simple_kernel(const T* __restrict__ q, const T* __restrict__ rows
   float* qs = gq_all + warp * a.dimp;
   const T* base = rows + (long long)p.slots[b] * p.len * step + (long long)g * row;
   const int hi = a.ring ? p.start[b] + t : min(p.start[b] + t, p.len - 1);  // rows of padding may lie beyond the cache
-  const int lo = seen_from(a, hi), kept = min(a.keep, lo), seen = kept + hi - lo + 1;
+  const int lo = seen_from(a, hi), kept = a.pool ? blocks_seen(a, hi) : min(a.keep, lo), seen = kept + hi - lo + 1;
   const float sink = a.sink ? (a.sink_w ? a.sink_w[h] : 0.f) : -INFINITY;
   float acc[MAPS][GA_MAX_V];
 #pragma unroll
@@ -241,7 +288,7 @@ grouped_attend_simple_kernel(const T* __restrict__ q, const T* __restrict__ rows
       int place = 0;
       float s = -INFINITY;
       if (j < seen) {
-        place = row_of(a, j < kept ? j : lo + j - kept);
+        place = a.pool && j < kept ? j : row_of(a, j < kept ? j : lo + j - kept);
         const T* k = base + place * step + u * a.dimp;
         float a0 = 0.f, a1 = 0.f;
         for (int i = 0; i < a.dimp; i += 2) {
@@ -273,7 +320,7 @@ grouped_attend_simple_kernel(const T* __restrict__ q, const T* __restrict__ rows
 #pragma unroll
     for (int i = 0; i < GA_MAX_V; ++i) acc[u][i] *= inv;
   }
-  float post = 1.f;
+  float post = a.post;
   if (MAPS == 2) {
     float ss = 0.f;
 #pragma unroll
@@ -289,7 +336,7 @@ grouped_attend_simple_kernel(const T* __restrict__ q, const T* __restrict__ rows
     if (c >= a.vdp) continue;
     float y = acc[0][i] * post;
     if (gate) y *= gate_of(to_f32(gate[n * p.gate_ld + (a.gate_cols == 1 ? h : h * a.vdp + c)]));
-    out[(n * a.heads + h) * a.vdp + c] = from_f32<T>(y);
+    out[n * a.out_ld + h * a.vdp + c] = from_f32<T>(y);
   }
 }
 
@@ -317,7 +364,7 @@ constexpr int GD_CHUNK = GD_KEYS * 128;  // bytes of [64 rows x 64 columns]
 
 struct GdParams {
   const __nv_bfloat16 *q, *gate;
-  __nv_bfloat16* out;  // (B, heads, vdp)
+  __nv_bfloat16* out;  // (B, out_ld)
   float* part_o;       // (n_split, B, heads · maps, vdp)
   float* part_ml;      // (n_split, B, heads · maps, 2)
   const int *slots, *start;
@@ -370,8 +417,9 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   const int h0 = g * group + blockIdx.y % tiles_h * HEADS, h_end = min(h0 + HEADS, (g + 1) * group);
   const int hi = p.a.ring ? p.start[b] : min(p.start[b], p.len - 1);
   const int lo = seen_from(p.a, hi), first = lo / GD_KEYS, keep = p.a.keep;
-  // tiles of kept positions, then those of [lo, hi]
-  const int kept = min((keep + GD_KEYS - 1) / GD_KEYS, first);
+  // tiles of kept positions or of blocks, then those of [lo, hi]
+  const int blocks = blocks_seen(p.a, hi);
+  const int kept = p.a.pool ? (blocks + GD_KEYS - 1) / GD_KEYS : min((keep + GD_KEYS - 1) / GD_KEYS, first);
   const int nT = kept + hi / GD_KEYS - first + 1;
   auto tile_at = [&](int t) { return t < kept ? t : t - kept + first; };
   const int per = (nT + p.n_split - 1) / p.n_split;
@@ -403,7 +451,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         if (!(ok = mbar_wait_bounded(&empty[st], ph ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
         mbar_expect_tx(&full[st], (uint32_t)STAGE);
         uint8_t* d = gd_smem + st * STAGE;
-        const int row = row_of(p.a, tile_at(t) * GD_KEYS);
+        const int row = p.a.pool && t < kept ? t * GD_KEYS : row_of(p.a, tile_at(t) * GD_KEYS);
         for (int c = 0; c < KC; ++c) tma_load_4d(d + c * GD_CHUNK, &tmK, &full[st], 64 * c, g, row, slot);
         if (MAPS == 2)
           for (int c = 0; c < KC; ++c) tma_load_4d(d + (KC + c) * GD_CHUNK, &tmK2, &full[st], 64 * c, g, row, slot);
@@ -459,8 +507,10 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     // after a wait that ran out the tiles are worked on unseen: the status word tells, and the loop ends
     if (ok) ok = mbar_wait_bounded(&full[st], ph, abort_flag, p.status, STATUS_TIMEOUT_FULL);
     const uint32_t tile = smem_u32(gd_smem) + (uint32_t)(st * STAGE);
-    const int jw = tile_at(t) * GD_KEYS + warp * 16;  // this warp's 16 positions
-    if (jw <= hi && (jw + 15 >= lo || jw < keep)) {
+    const int jw = tile_at(t) * GD_KEYS + warp * 16;  // this warp's 16 positions, or blocks
+    const bool of_blocks = p.a.pool && t < kept;
+    const int first_j = of_blocks ? 0 : lo, last_j = of_blocks ? blocks - 1 : hi;
+    if (jw <= last_j && (jw + 15 >= first_j || jw < keep)) {
       float s[2][2][4];  // even and odd steps apart: two short chains instead of a long one
 #pragma unroll
       for (int n = 0; n < 2; ++n)
@@ -492,14 +542,14 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[0][n][e] = p.cap_out * cap_tanh(s[0][n][e]);
       }
-      if (jw + 15 > hi || (jw < lo && jw + 15 >= keep)) {
+      if (jw + 15 > last_j || (jw < first_j && jw + 15 >= keep)) {
         const int j0 = jw + (lane & 3) * 2;
 #pragma unroll
         for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int j = j0 + 8 * n + (e & 1);
-            if (j > hi || (j < lo && j >= keep)) s[0][n][e] = -INFINITY;
+            if (j > last_j || (j < first_j && j >= keep)) s[0][n][e] = -INFINITY;
           }
       }
       float f[2];
@@ -605,7 +655,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       }
       continue;
     }
-    __nv_bfloat16* dst = p.out + ((long long)b * p.heads + h) * p.vdp;
+    __nv_bfloat16* dst = p.out + b * p.a.out_ld + h * p.vdp;
     if (MAPS == 2) {
       const float f0 = 1.f / l[0], f1 = p.a.lambda / l[MAPS - 1];
       float ss = 0.f;
@@ -627,7 +677,7 @@ grouped_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     // the sink may lie far above all scores: everything relative to the larger of both
     const float sink = p.a.sink ? gd_sink(p, h) : -INFINITY;
     const float top = fmaxf(m[0], sink);
-    const float f = attn_exp2(m[0] - top), inv = f / (l[0] * f + (p.a.sink ? attn_exp2(sink - top) : 0.f));
+    const float f = attn_exp2(m[0] - top), inv = p.a.post * f / (l[0] * f + (p.a.sink ? attn_exp2(sink - top) : 0.f));
     for (int c = lane * 2; c < p.vdp; c += 64) {
       float2 v = *reinterpret_cast<const float2*>(so + e * p.vdp + c);
       v.x *= inv;
@@ -664,8 +714,9 @@ grouped_merge_kernel(const GdParams p) {
 #pragma unroll
     for (int i = 0; i < 2; ++i) f[i] = m[i] == -INFINITY ? 0.f : attn_exp2(m[i] - top);
     const float inv = 1.f / (warp_sum(f[0] * l[0] + f[1] * l[1]) + (p.a.sink ? attn_exp2(sink - top) : 0.f));
-    wt[warp][lane] = f[0] * inv;
-    wt[warp][lane + 32] = f[1] * inv;
+    const float scale = MAPS == 2 ? inv : inv * p.a.post;
+    wt[warp][lane] = f[0] * scale;
+    wt[warp][lane + 32] = f[1] * scale;
   }
   __syncthreads();
   const int c = threadIdx.x * 2;  // value sizes up to 256
@@ -698,7 +749,7 @@ grouped_merge_kernel(const GdParams p) {
     o[0].x *= gt.x;
     o[0].y *= gt.y;
   }
-  *reinterpret_cast<uint32_t*>(p.out + ((long long)b * p.heads + h) * p.vdp + c) = pack_bf16x2(o[0].x, o[0].y);
+  *reinterpret_cast<uint32_t*>(p.out + b * p.a.out_ld + h * p.vdp + c) = pack_bf16x2(o[0].x, o[0].y);
 }
 
 // chunks of 64 key columns and of 64 value columns that a kernel is compiled for
@@ -723,7 +774,7 @@ static int gd_split(int B, int len, const kvb_attention& a) {
   long long tiles = (len + GD_KEYS - 1) / GD_KEYS;
   const int span = a.chunk > 0 ? a.chunk : a.window;
   if (span > 0) {
-    const long long most = (a.keep + GD_KEYS - 1) / GD_KEYS + (span + GD_KEYS - 1) / GD_KEYS + 1;
+    const long long most = ((a.pool > 0 ? a.head : a.keep) + GD_KEYS - 1) / GD_KEYS + (span + GD_KEYS - 1) / GD_KEYS + 1;
     if (tiles > most) tiles = most;
   }
   const long long slots = 148 * (gd_stage_bytes(a) * 3 > 110 * 1024 ? 1 : 2);
@@ -759,6 +810,7 @@ static bool attention_valid(const kvb_attention* a) {
   return a && a->heads > 0 && a->kv_heads > 0 && a->heads % a->kv_heads == 0 && (a->maps == 1 || a->maps == 2) && a->dim > 0 && a->vdim > 0 &&
          a->dimp >= a->dim && a->vdp >= a->vdim && a->window >= 0 && a->keep >= 0 && a->chunk >= 0 && !(a->window && a->chunk) &&
          (a->window || !a->keep) && a->head >= 0 && a->ring >= 0 && a->head % 128 == 0 && a->ring % 128 == 0 && (!a->ring || a->head >= a->keep) &&
+         a->pool >= 0 && (!a->pool || (a->window > 0 && a->keep == 0 && a->ring > 0)) && a->out_ld >= (long long)a->heads * a->vdp &&
          a->softcap >= 0.f && !(a->maps == 2 && (a->sink || a->gate_cols)) && (a->gate_cols == 0 || a->gate_cols == 1 || a->gate_cols == a->vdp);
 }
 
@@ -778,10 +830,10 @@ extern "C" int kvb_grouped_prep(const void* qkv, long long ld, const float* norm
       (norm_q == nullptr) != (norm_k == nullptr) || (a->ring && a->head + a->ring > len))
     return KVB_ERR_ARG;
   if ((a->dimp | a->vdp | a->value_col) % 8) return KVB_ERR_ALIGN;
-  if (a->value_col == a->heads * a->maps * a->dimp && (a->vdp != a->dimp || a->maps != 1)) return KVB_ERR_ARG;
+  if (!a->borrowed && a->value_col == a->heads * a->maps * a->dimp && (a->vdp != a->dimp || a->maps != 1)) return KVB_ERR_ARG;
   kvb::GpParams p;
   p.ld = ld; p.norm_q = norm_q; p.norm_k = norm_k; p.freq = freq; p.slots = slots; p.start = start; p.count = count; p.a = *a;
-  p.T = T_; p.len = len; p.heads = a->heads * a->maps; p.kv_heads = a->kv_heads * a->maps; p.dim = a->dim; p.dimp = a->dimp; p.vdp = a->vdp;
+  p.T = T_; p.len = len; p.heads = a->heads * a->maps; p.kv_heads = a->borrowed ? 0 : a->kv_heads * a->maps; p.dim = a->dim; p.dimp = a->dimp; p.vdp = a->vdp;
   p.rot_dims = a->rot_dims; p.value_col = a->value_col;
   KVB_GROUPED_TYPES(dtype, return kvb::gp_launch<T>(qkv, q, rows, p, B, (cudaStream_t)stream));
 }
@@ -814,6 +866,7 @@ extern "C" int kvb_grouped_decode(const void* q, const void* rows, const void* g
     return KVB_ERR_ARG;
   if (!kvb_grouped_decode_supported(a)) return KVB_ERR_UNSUPPORTED;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(rows) | reinterpret_cast<uintptr_t>(out)) & 15) return KVB_ERR_ALIGN;
+  if (a->out_ld % 2) return KVB_ERR_ALIGN;
   if (a->gate_cols > 1 && (gate_ld & 1 || reinterpret_cast<uintptr_t>(gate) & 3)) return KVB_ERR_ALIGN;
   const uint64_t row = a->maps * a->dimp + a->vdp, G = a->kv_heads, sk[3] = {row, G * row, (uint64_t)len * G * row};
   const uint64_t dk[4] = {(uint64_t)a->dimp, G, (uint64_t)len, (uint64_t)n_slots}, dv[4] = {(uint64_t)a->vdp, G, (uint64_t)len, (uint64_t)n_slots};

@@ -18,8 +18,8 @@
 //
 // Masks are arithmetic: key row j of sequence b has position start[b] − P + j (P = start[b] in a grouped-query cache), query t sees
 // max(P + t − window + 1, P − start[b], 0) <= j <= P + t. Tiles outside the range of a query tile are skipped, tiles inside
-// the range of all its rows need no mask. A grouped query may also see the first `keep` keys: their tiles come ahead of the others. In
-// a chunked layer its range starts where its chunk does.
+// the range of all its rows need no mask. A grouped query may also see the first `keep` keys, or the means of blocks before its window: their
+// tiles come ahead of the others. In a chunked layer its range starts where its chunk does.
 #include <cuda.h>
 #include <limits.h>
 
@@ -47,6 +47,7 @@ struct LfParams {
   int ksu_last, ksr;     // 16-feature steps of the last unrotated chunk and of the rotated chunk(s) in total
   int kst, vst;          // stages of K and V
   int vdp, window;
+  long long out_ld;
   float scale_log2;
   int* status;
   const int* slots;          // grouped-query cache: slot of every row; NULL: keys and values of the pass
@@ -120,10 +121,11 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     first = min(first, ra[u]);
     last = max(last, rb[u]);
   }
-  // Tiles are counted as they are visited: `kept` ones from the start of the sequence, which every query tile visits, then those from
-  // `first` on; ra, rb, last are of that count from here on.
+  // Tiles are counted as they are visited: `kept` ones from the start of the sequence (or of blocks: as many as the last query of the CTA
+  // sees), which every query tile visits, then those from `first` on; ra, rb, last are of that count from here on.
   const int keep_tiles = (p.a.keep + LF_T - 1) / LF_T;
-  const int kept = last < 0 ? 0 : min(keep_tiles, first), skipped = first - kept;
+  const int last_query = min((DIFF ? pair + 1 : (pair + 1) * NQT) * LF_T, p.T) - 1;
+  const int kept = last < 0 ? 0 : p.a.pool ? (blocks_seen(p.a, P + last_query) + LF_T - 1) / LF_T : min(keep_tiles, first), skipped = first - kept;
 #pragma unroll
   for (int u = 0; u < NQT; ++u) {
     if (rb[u] < 0) continue;
@@ -179,7 +181,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       int ks = 0, vs = 0;
       uint32_t kph = 0, vph = 0;
       for (int t = 0; t <= last; ++t) {
-        const int krow = p.slots ? row_of(p.a, tile_at(t) * LF_T) : tile_at(t) * LF_T;
+        const int krow = p.a.pool && t < kept ? t * LF_T : p.slots ? row_of(p.a, tile_at(t) * LF_T) : tile_at(t) * LF_T;
         if (!(ok = mbar_wait_bounded(&k_empty[ks], kph ^ 1, abort_flag, p.status, STATUS_TIMEOUT_EMPTY))) break;
         mbar_expect_tx(&k_full[ks], (uint32_t)(MAPS * nk * LF_CHUNK));
         uint8_t* kd = sK + ks * MAPS * nk * LF_CHUNK;
@@ -291,6 +293,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
     // rows of the tile: all see keys in [lo of the last row, hi of the first row] and the kept ones up to the first row
     const int lo_max = seen(P + t0 + LF_T - 1), hi_min = P + t0;
     const int keep = min(p.a.keep, hi + 1);
+    const int blocks = blocks_seen(p.a, hi), blocks_min = blocks_seen(p.a, hi_min);  // the fewest of the tile: its first row's
     const uint32_t lane_base = (uint32_t)(quarter * 32) << 16;
     const uint32_t tmem_S = tmem_base + (uint32_t)(u * LF_T) + lane_base;
     const uint32_t tmem_O = tmem_base + (uint32_t)(NQT * LF_T + u * o_cols) + lane_base;
@@ -322,7 +325,14 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
         }
       }
       const int j0 = tile_at(t) * LF_T;
-      if (j0 + LF_T - 1 > hi_min || (j0 < lo_max && j0 + LF_T > p.a.keep)) {
+      if (p.a.pool && t < kept) {
+        if (j0 + LF_T > blocks_min) {
+          const int here = blocks - j0;
+#pragma unroll
+          for (int e = 0; e < LF_T; ++e)
+            if (e >= here) x[e] = 0xff800000u;
+        }
+      } else if (j0 + LF_T - 1 > hi_min || (j0 < lo_max && j0 + LF_T > p.a.keep)) {
         const uint32_t span = (uint32_t)(hi - lo);
         const uint32_t off = (uint32_t)(j0 - lo);
         const int keep_here = keep - j0;
@@ -420,7 +430,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       s_ss[u][row] = ss;
       named_barrier(1, 256);
       const float r = p.a.post / sqrtf((s_ss[0][row] + s_ss[1][row]) / (float)p.a.vdim + p.a.eps);
-      __nv_bfloat16* dst = p.out + (((long long)b * p.T + (tq < p.T ? tq : 0)) * p.heads + h) * p.vdp;
+      __nv_bfloat16* dst = p.out + ((long long)b * p.T + (tq < p.T ? tq : 0)) * p.out_ld + h * p.vdp;
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         const int c = c_begin + 8 * k;
@@ -434,10 +444,10 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQu, const __grid_const
       }
     } else if (ok && my_rb >= my_ra) {
       tc_fence_after();
-      float inv_l = l > 0.f ? 1.f / l : 0.f;
+      float inv_l = l > 0.f ? p.a.post / l : 0.f;
       if (p.gate && p.a.gate_cols == 1 && tq < p.T)  // one number per head
         inv_l *= lf_sigmoid(__bfloat162float(p.gate[((long long)b * p.T + tq) * p.gate_ld + h]));
-      __nv_bfloat16* dst = p.out + (((long long)b * p.T + (tq < p.T ? tq : 0)) * p.heads + h) * p.vdp;
+      __nv_bfloat16* dst = p.out + ((long long)b * p.T + (tq < p.T ? tq : 0)) * p.out_ld + h * p.vdp;
 #pragma unroll 1
       for (int c0 = 0; c0 < p.vdp; c0 += 16) {
         uint32_t o[16];
@@ -557,6 +567,7 @@ extern "C" int kvb_latent_attend_tc(const void* q, const void* kv, const void* l
   p.ksr = (rp + 15) / 16;
   p.vdp = vdp; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.slots = nullptr; p.group = 1; p.gate = nullptr; p.gate_ld = 0; p.cap_in = p.cap_out = 0.f; p.a = kvb_attention{};
+  p.a.post = 1.f; p.out_ld = (long long)heads * vdp;
   return pl.nqt == 2 ? lf_launch<2, false, false>(tm, p, pl.smem, (cudaStream_t)stream) : lf_launch<1, false, false>(tm, p, pl.smem, (cudaStream_t)stream);
 }
 
@@ -568,6 +579,7 @@ extern "C" int kvb_grouped_attend_tc(const void* q, const void* rows, const void
                                      const int* start, int B, int T, int n_slots, int len, const kvb_attention* a, int* status, void* stream) {
   using namespace kvb;
   if (!a || B <= 0 || T <= 0 || n_slots <= 0 || len <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || !(a->scale > 0.f) ||
+      (a->pool && (a->window <= 0 || a->keep || a->ring <= 0)) || a->out_ld < (long long)a->heads * a->vdp || a->out_ld % 8 ||
       (a->maps != 1 && a->maps != 2) || (a->maps == 2 && (a->sink || gate)) || (a->window && a->chunk) || (a->keep && !a->window) ||
       a->head % LF_T || a->ring % LF_T || (a->ring && (a->head < a->keep || a->head + a->ring > len)))
     return KVB_ERR_ARG;
@@ -601,6 +613,7 @@ extern "C" int kvb_grouped_attend_tc(const void* q, const void* rows, const void
   p.cap_out = a->softcap * ATTN_LOG2E;
   p.scale_log2 = a->softcap > 0.f ? 1.f : a->scale * ATTN_LOG2E;
   p.slots = slots; p.group = a->heads / a->kv_heads; p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate_ld; p.a = *a;
+  p.out_ld = a->out_ld;
   cudaStream_t s = (cudaStream_t)stream;
   auto launch = [&](auto capped) {
     constexpr bool CAP = decltype(capped)::value;

@@ -250,9 +250,24 @@ moe_gemm_simple_kernel(const T* __restrict__ in, const T* __restrict__ w, T* __r
 }
 
 // out[n, c] = silu(x[n, c]) · x[n, up + c], zero in the columns from ff to ldo. A CTA has one row.
-template <typename T, int V>
+// what a gated feed-forward does with gate and up projection
+struct SiluUnit {
+  template <typename T> __device__ __forceinline__ float of(float g, float u) const { return moe_glu<T>(g, u); }
+};
+// g · sigmoid(1.702 g) · (u + 1) with g at most the limit and u within it on both sides
+struct ClampedUnit {
+  float limit;
+  template <typename T> __device__ __forceinline__ float of(float g, float u) const {
+    g = fminf(g, limit);
+    const float e = -1.702f * g;
+    const float s = sizeof(T) == 2 ? __fdividef(g, 1.f + __expf(e)) : g / (1.f + expf(e));
+    return s * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+};
+
+template <typename T, int V, typename Unit>
 __global__ void __launch_bounds__(256)
-glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long ldx, int up, int ff, int ldo) {
+glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long ldx, int up, int ff, int ldo, const Unit unit) {
   struct alignas(sizeof(T) * V) Vec { T v[V]; };
   x += blockIdx.x * ldx;
   out += (long long)blockIdx.x * ldo;
@@ -262,7 +277,7 @@ glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long ldx, int up, 
     if (c < ff) {
       const Vec g = *reinterpret_cast<const Vec*>(x + c), u = *reinterpret_cast<const Vec*>(x + up + c);
 #pragma unroll
-      for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(moe_glu<T>(to_f32(g.v[e]), to_f32(u.v[e])));
+      for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(unit.template of<T>(to_f32(g.v[e]), to_f32(u.v[e])));
     } else {
 #pragma unroll
       for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(0.f);
@@ -271,15 +286,20 @@ glu_kernel(const T* __restrict__ x, T* __restrict__ out, long long ldx, int up, 
   }
 }
 
-template <typename T>
-static int glu_launch(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, cudaStream_t s) {
+template <typename T, typename Unit>
+static int glu_launch(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, const Unit& unit, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
   const bool vec = ff % V == 0 && up % V == 0 && ldx % V == 0 && ldo % V == 0;
   int threads = ((vec ? ldo / V : ldo) + 31) / 32 * 32;
   if (threads > 256) threads = 256;
-  if (vec) glu_kernel<T, V><<<(unsigned)n, threads, 0, s>>>((const T*)x, (T*)out, ldx, up, ff, ldo);
-  else glu_kernel<T, 1><<<(unsigned)n, threads, 0, s>>>((const T*)x, (T*)out, ldx, up, ff, ldo);
+  if (vec) glu_kernel<T, V><<<(unsigned)n, threads, 0, s>>>((const T*)x, (T*)out, ldx, up, ff, ldo, unit);
+  else glu_kernel<T, 1><<<(unsigned)n, threads, 0, s>>>((const T*)x, (T*)out, ldx, up, ff, ldo, unit);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+template <typename T>
+static int glu_type(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, float limit, cudaStream_t s) {
+  return limit > 0.f ? glu_launch<T>(x, out, n, ldx, up, ff, ldo, ClampedUnit{limit}, s) : glu_launch<T>(x, out, n, ldx, up, ff, ldo, SiluUnit{}, s);
 }
 
 int moe_gemm_tc(const void* in, const void* w, void* out, const int* plan, const int* tile_expert, const int* tile_row, int tile,
@@ -351,9 +371,9 @@ extern "C" int kvb_moe_gemm(const void* in, const void* w, void* out, const int*
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
-extern "C" int kvb_glu(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, int dtype, void* stream) {
+extern "C" int kvb_glu(const void* x, void* out, long long n, long long ldx, int up, int ff, int ldo, float limit, int dtype, void* stream) {
   if (n <= 0 || ff <= 0 || up < ff || ldx < up + ff || ldo < ff || n > 0x7fffffffLL) return KVB_ERR_ARG;
-  if (dtype == 0) return kvb::glu_launch<float>(x, out, n, ldx, up, ff, ldo, (cudaStream_t)stream);
-  if (dtype == 1) return kvb::glu_launch<__nv_bfloat16>(x, out, n, ldx, up, ff, ldo, (cudaStream_t)stream);
+  if (dtype == 0) return kvb::glu_type<float>(x, out, n, ldx, up, ff, ldo, limit, (cudaStream_t)stream);
+  if (dtype == 1) return kvb::glu_type<__nv_bfloat16>(x, out, n, ldx, up, ff, ldo, limit, (cudaStream_t)stream);
   return KVB_ERR_ARG;
 }

@@ -2,7 +2,7 @@
 // o normed per head and gated. The recurrence over several tokens is the one of state-space mixers (ssm.cu, ssm_sm100.cu); here are
 //
 //   prep   rotation of the fp32 projections of queries and keys, rounded once to the type of the scan's operands;
-//   norm   y / rms(y) · silu(gate), a few lanes per head of a token;
+//   norm   y / rms(y) · silu(gate), possibly with a weight (gated linear attention), a few lanes per head of a token;
 //   step   one new token per sequence: rotation, decay, state, output, norm and gate of a head in one kernel, all in fp32, bound by
 //          reading and writing the state once.
 #include "common.cuh"
@@ -71,6 +71,7 @@ constexpr int HN_ROWS = 4;  // rows (heads of tokens) that a group of lanes work
 constexpr int HN_MAX = 16;  // accesses per lane and row
 
 struct HeadNormParams {
+  const float* weight;  // (vdp), NULL: ones
   long long ld, rows;
   int heads, vdim, vdp;
   float eps;
@@ -126,7 +127,10 @@ head_norm_gate_kernel(const T* __restrict__ y, const T* __restrict__ gate, T* __
       if (c >= p.vdp) break;
       Vec o;
 #pragma unroll
-      for (int e = 0; e < V; ++e) o.v[e] = from_f32<T>(to_f32(v[i][k].v[e]) * f * ss_silu_for<T>(to_f32(z[i][k].v[e])));
+      for (int e = 0; e < V; ++e) {
+        const float w = p.weight ? f * p.weight[c + e] : f;
+        o.v[e] = from_f32<T>(to_f32(v[i][k].v[e]) * w * ss_silu_for<T>(to_f32(z[i][k].v[e])));
+      }
       *reinterpret_cast<Vec*>(out + (long long)r * p.vdp + c) = o;
     }
   }
@@ -281,13 +285,13 @@ extern "C" int kvb_retention_prep(const float* in, long long ld, const float* fr
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
-extern "C" int kvb_head_norm_gate(const void* y, const void* gate, long long ld, void* out, long long n, int heads, int vdim, int vdp,
+extern "C" int kvb_head_norm_gate(const void* y, const void* gate, long long ld, const float* weight, void* out, long long n, int heads, int vdim, int vdp,
                                   float eps, int dtype, void* stream) {
   if (n <= 0 || heads <= 0 || vdim <= 0 || vdp < vdim || n * heads > 0x7f000000LL) return KVB_ERR_ARG;
   if (vdp % 8 || ld % 8 || (reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15)
     return KVB_ERR_ALIGN;
   kvb::HeadNormParams p;
-  p.ld = ld; p.rows = n * heads; p.heads = heads; p.vdim = vdim; p.vdp = vdp; p.eps = eps;
+  p.weight = weight; p.ld = ld; p.rows = n * heads; p.heads = heads; p.vdim = vdim; p.vdp = vdp; p.eps = eps;
   KVB_RETENTION_TYPES(dtype, return kvb::hn_type<T>(y, gate, out, p, (cudaStream_t)stream));
 }
 

@@ -29,7 +29,7 @@ struct ConvParams {
   const float *w, *bias;  // (taps, channels), (channels)
   const int *slots, *start, *count;
   long long ld;
-  int T, col, channels, taps, run;
+  int T, col, channels, taps, run, silu;
 };
 
 // TAPS 0: any number, inputs are read once per tap
@@ -89,7 +89,7 @@ short_conv_kernel(const T* __restrict__ u, T* __restrict__ out, T* __restrict__ 
           float acc = bias[e];
 #pragma unroll
           for (int k = 0; k < TAPS; ++k) acc = fmaf(w[k][e], x[k][e], acc);
-          y.v[e] = from_f32<T>(ss_silu_for<T>(acc));
+          y.v[e] = from_f32<T>(p.silu ? ss_silu_for<T>(acc) : acc);
         }
         *reinterpret_cast<Vec*>(dst + (long long)(t + i) * p.channels) = y;
       }
@@ -106,7 +106,7 @@ short_conv_kernel(const T* __restrict__ u, T* __restrict__ out, T* __restrict__ 
       }
       Vec y;
 #pragma unroll
-      for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(ss_silu_for<T>(acc[e]));
+      for (int e = 0; e < V; ++e) y.v[e] = from_f32<T>(p.silu ? ss_silu_for<T>(acc[e]) : acc[e]);
       *reinterpret_cast<Vec*>(dst + (long long)t * p.channels) = y;
     }
   }
@@ -136,12 +136,22 @@ constexpr int SN_COLS = 32;   // value columns of a CTA
 constexpr int SN_ROWS = 8;    // rows of the state that are worked on side by side
 constexpr int SN_CHUNK = 8;   // tokens staged at a time
 
-// NR: rows of the state per thread; thread (p, r) has column p of rows r, r + SN_ROWS, ...
-template <typename T, int NR>
+// Decays of their own for every row of the state (gated linear attention), from the same input as B and C.
+struct RowDecay {
+  kvb_gated_linear g;
+  const int* only;  // heads of rows of the pass to work on, NULL: all
+};
+
+// NR: rows of the state per thread; thread (p, r) has column p of rows r, r + SN_ROWS, ... TB: type of B and C; BY_ROW: decays by row, and C is
+// scaled
+template <typename T, typename TB, int NR, bool BY_ROW>
 __global__ void __launch_bounds__(SN_COLS * SN_ROWS)
-state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long long ldx, const T* __restrict__ bm, const T* __restrict__ cm,
-                         long long ldb, T* __restrict__ y, const ScanParams p) {
+state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long long ldx, const TB* __restrict__ bm, const TB* __restrict__ cm,
+                         long long ldb, T* __restrict__ y, const ScanParams p, const RowDecay rd) {
   constexpr int NP = NR * SN_ROWS;
+  constexpr int SN_CHUNK = BY_ROW ? 4 : kvb::SN_CHUNK;
+  __shared__ float srow[BY_ROW ? SN_CHUNK : 1][BY_ROW ? NP : 1];
+  if (BY_ROW && rd.only && !rd.only[blockIdx.z * p.heads + blockIdx.y]) return;
   __shared__ float sb[SN_CHUNK][NP], sc[SN_CHUNK][NP], sx[SN_CHUNK][SN_COLS], sdt[SN_CHUNK], sa[SN_CHUNK];
   __shared__ float part[SN_CHUNK][SN_ROWS][SN_COLS];
   const int p0 = blockIdx.x * SN_COLS, h = blockIdx.y, b = blockIdx.z;
@@ -155,7 +165,8 @@ state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long 
     const int row = r + i * SN_ROWS;
     s[i] = p.start[b] > 0 && mine && row < p.np ? st[(long long)row * p.vdp] : 0.f;
   }
-  const float rate = p.decay ? 0.f : -expf(p.a_log[h]), skip = p.decay ? 0.f : p.skip[h], bias = p.decay ? 0.f : p.dt_bias[h];
+  const bool fixed = BY_ROW || p.decay;
+  const float rate = fixed ? 0.f : -expf(p.a_log[h]), skip = fixed ? 0.f : p.skip[h], bias = fixed ? 0.f : p.dt_bias[h];
   x += (long long)b * p.T * ldx;
   bm += (long long)b * p.T * ldb;
   cm += (long long)b * p.T * ldb;
@@ -165,15 +176,20 @@ state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long 
       const int t = i / NP, k = i - t * NP;
       const long long at = (long long)(t0 + t) * ldb + g * p.np + k;
       sb[t][k] = k < p.np ? to_f32(bm[at]) : 0.f;
-      sc[t][k] = k < p.np ? to_f32(cm[at]) : 0.f;
+      sc[t][k] = k < p.np ? to_f32(cm[at]) * (BY_ROW ? rd.g.q_scale : 1.f) : 0.f;
+      if constexpr (BY_ROW) {
+        float d = 0.f;
+        if (k < p.np) d = ss_decay(gl_log_decay(rd.g, rd.g.in + ((long long)b * p.T + t0 + t) * rd.g.ld + 2 * rd.g.heads * p.np, h * p.np + k));
+        srow[t][k] = d;
+      }
     }
     for (int i = tid; i < nt * SN_COLS; i += SN_COLS * SN_ROWS) {
       const int t = i / SN_COLS, k = i - t * SN_COLS;
       sx[t][k] = p0 + k < p.vdp ? to_f32(x[(long long)(t0 + t) * ldx + h * p.vdp + p0 + k]) : 0.f;
     }
-    if (tid < nt && p.decay) {
+    if (tid < nt && fixed) {
       sdt[tid] = 1.f;
-      sa[tid] = p.decay[h];
+      sa[tid] = BY_ROW ? 0.f : p.decay[h];
     } else if (tid < nt) {
       const float dt = ss_softplus(to_f32(u[((long long)b * p.T + t0 + tid) * p.ld + p.dt_col + h]) + bias);
       sdt[tid] = dt;
@@ -186,7 +202,7 @@ state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long 
         const float a = sa[t], dx = sdt[t] * sx[t][col];
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-          s[i] = fmaf(a, s[i], dx * sb[t][r + i * SN_ROWS]);
+          s[i] = fmaf(BY_ROW ? srow[t][r + i * SN_ROWS] : a, s[i], dx * sb[t][r + i * SN_ROWS]);
           acc = fmaf(s[i], sc[t][r + i * SN_ROWS], acc);
         }
       }
@@ -211,12 +227,12 @@ state_scan_simple_kernel(const T* __restrict__ u, const T* __restrict__ x, long 
   }
 }
 
-template <typename T>
+template <typename T, typename TB = T, bool BY_ROW = false>
 static int scan_simple_launch(const void* u, const void* x, long long ldx, const void* bm, const void* cm, long long ldb, void* y,
-                              const ScanParams& p, int B, cudaStream_t s) {
+                              const ScanParams& p, int B, cudaStream_t s, const RowDecay& rd = RowDecay{}) {
   const dim3 grid((p.vdp + SN_COLS - 1) / SN_COLS, p.heads, B);
-#define KVB_SCAN(NR) state_scan_simple_kernel<T, NR><<<grid, SN_COLS * SN_ROWS, 0, s>>>( \
-    (const T*)u, (const T*)x, ldx, (const T*)bm, (const T*)cm, ldb, (T*)y, p)
+#define KVB_SCAN(NR) state_scan_simple_kernel<T, TB, NR, BY_ROW><<<grid, SN_COLS * SN_ROWS, 0, s>>>( \
+    (const T*)u, (const T*)x, ldx, (const TB*)bm, (const TB*)cm, ldb, (T*)y, p, rd)
   if (p.np <= 4 * SN_ROWS) KVB_SCAN(4);
   else if (p.np <= 16 * SN_ROWS) KVB_SCAN(16);
   else if (p.np <= 32 * SN_ROWS) KVB_SCAN(32);
@@ -448,13 +464,13 @@ relu_squared_kernel(T* __restrict__ x, long long n) {
   }
 
 extern "C" int kvb_short_conv(const void* u, long long ld, int col, const float* w, const float* bias, void* out, void* ring,
-                              const int* slots, const int* start, const int* count, int B, int T_, int channels, int taps, int dtype,
-                              void* stream) {
+                              const int* slots, const int* start, const int* count, int B, int T_, int channels, int taps, int silu,
+                              int dtype, void* stream) {
   if (B <= 0 || B > 65535 || T_ <= 0 || channels <= 0 || taps <= 0) return KVB_ERR_ARG;
   if (channels % 8 || col % 8 || ld % 8) return KVB_ERR_ALIGN;
   kvb::ConvParams p;
   p.w = w; p.bias = bias; p.slots = slots; p.start = start; p.count = count; p.ld = ld; p.T = T_; p.col = col; p.channels = channels;
-  p.taps = taps;
+  p.taps = taps; p.silu = silu;
   KVB_SSM_TYPES(dtype, return kvb::conv_launch<T>(u, out, ring, p, B, (cudaStream_t)stream));
 }
 
@@ -479,6 +495,19 @@ extern "C" int kvb_retention_scan(const void* v, long long ldv, const void* qk, 
   p.T = T_; p.dt_col = 0; p.heads = heads; p.groups = heads; p.vdp = vdp; p.np = np; p.inner = heads * vdp; p.channels = 0;
   KVB_SSM_TYPES(dtype, const T* q = (const T*)qk;
                 return kvb::scan_simple_launch<T>(nullptr, v, ldv, q + heads * np, q, ldqk, y, p, B, (cudaStream_t)stream));
+}
+
+extern "C" int kvb_gated_linear_scan(const kvb_gated_linear* g, const void* v, long long ldv, float* state, void* y, const int* only,
+                                     const int* slots, const int* start, const int* count, int B, int T_, int vdp, int dtype, void* stream) {
+  if (!g || B <= 0 || B > 65535 || T_ <= 0 || g->heads <= 0 || g->heads > 65535 || vdp <= 0 || g->np <= 0 || g->rank <= 0 ||
+      g->ld < 2LL * g->heads * g->np + g->rank)
+    return KVB_ERR_ARG;
+  kvb::ScanParams p;
+  p.dt_bias = p.a_log = p.skip = p.decay = nullptr; p.slots = slots; p.start = start; p.count = count; p.state = state; p.ld = 0;
+  p.T = T_; p.dt_col = 0; p.heads = g->heads; p.groups = g->heads; p.vdp = vdp; p.np = g->np; p.inner = g->heads * vdp; p.channels = 0;
+  const kvb::RowDecay rd{*g, only};
+  KVB_SSM_TYPES(dtype, return (kvb::scan_simple_launch<T, float, true>(nullptr, v, ldv, g->in + g->heads * g->np, g->in, g->ld, y, p, B,
+                                                                       (cudaStream_t)stream, rd)));
 }
 
 extern "C" int kvb_state_step(const void* u, long long ld, int col, int dt_col, const float* w, const float* bias, const float* dt_bias,

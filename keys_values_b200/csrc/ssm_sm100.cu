@@ -18,6 +18,11 @@
 // With a fixed decay per head (retention: B the keys, C the queries, x the values) the step size is 1, the running sums are multiples
 // of its logarithm and there is no D.
 //
+// With a decay per token and key channel (gated linear attention, ROWS) queries and keys come with the decays since, and up to, the middle of
+// their chunk in them (gated_linear.cu). The state is kept in units of the decay up to that middle: a chunk starts with multiplying its rows
+// by (second half of the chunk before) · (first half of this one), which a row of the state is a lane of TMEM for. Nothing else is weighted:
+// P is the masked G, and x itself enters the state.
+//
 // Long passes of few heads are cut into segments: a first launch (STATES) finds what each segment adds to the state and its total
 // decay, a small kernel chains them, and the segments then run side by side from their own starting states.
 #include <cuda.h>
@@ -41,7 +46,10 @@ struct SdParams {
   const __nv_bfloat16* u;
   __nv_bfloat16* y;
   float* seg_state;  // (n_seg, B, heads, np, vdp): states at the segments' starts; before the chaining, entry k + 1 holds what k adds
-  float* seg_decay;  // (n_seg, B, heads): log2 of the segments' decays
+  float* seg_decay;  // (n_seg, B, heads; ROWS: · np): log2 of the segments' decays
+  const float* factor;  // ROWS: (B, chunks, heads, np, 2), log2 of the decays of a chunk's halves
+  const int* far;       // ROWS: (B, heads), 1: the head is not worked on here
+  int chunks;
   int* status;
   int B, n_seg, seg_chunks, n_unit;  // n_unit: CTAs per sequence and segment
 };
@@ -50,18 +58,6 @@ __device__ __forceinline__ float sd_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
-}
-// log(1 + exp(x)) = max(x, 0) + log(1 + e) with e = exp(−|x|) <= 1, and log(1 + e) = 2 artanh(s), s = e / (2 + e) <= 1/3: seven terms of
-// the series leave a relative error of 2e-8
-__device__ __forceinline__ float sd_softplus(float x) {
-  const float e = __expf(-fabsf(x)), s = __fdividef(e, 2.f + e), q = s * s;
-  float r = fmaf(q, 1.f / 13.f, 1.f / 11.f);
-  r = fmaf(q, r, 1.f / 9.f);
-  r = fmaf(q, r, 1.f / 7.f);
-  r = fmaf(q, r, 1.f / 5.f);
-  r = fmaf(q, r, 1.f / 3.f);
-  r = fmaf(q, r, 1.f);
-  return fmaf(2.f * s, r, fmaxf(x, 0.f));
 }
 __device__ __forceinline__ void sd_store_4d(const void* tmap, const void* smem, int x, int y, int z, int w) {
   asm volatile("cp.async.bulk.tensor.4d.global.shared::cta.bulk_group [%0, {%2, %3, %4, %5}], [%1];" ::"l"(tmap), "r"(smem_u32(smem)),
@@ -87,8 +83,8 @@ struct SdShared {
 };
 
 // NH heads per CTA, NV tiles of 64 value columns, KC tiles of 64 columns of C and B (columns beyond the sizes are zero); STATES: only
-// what the segment adds to the state
-template <int NH, int NV, int KC, bool STATES>
+// what the segment adds to the state; ROWS: decays by row of the state
+template <int NH, int NV, int KC, bool STATES, bool ROWS>
 __global__ void __launch_bounds__(SD_FRONT + 256 * NH, 1)
 state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmB, const __grid_constant__ CUtensorMap tmC,
                   const __grid_constant__ CUtensorMap tmY, const SdParams q) {
@@ -109,12 +105,13 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
   const int unit = blockIdx.x % q.n_unit, seg = blockIdx.x / q.n_unit % q.n_seg, b = blockIdx.x / (q.n_unit * q.n_seg);
   const int h0 = unit * NH, g = h0 / (p.heads / p.groups);
   const int n = p.count[b];
+  if (ROWS && q.far[b * p.heads + h0]) return;  // the same for all threads, before anything is set up
   const int ca = seg * q.seg_chunks;
   const int cb = min(ca + q.seg_chunks, (n + SD_T - 1) / SD_T);  // chunks beyond the last real token change nothing
   const int n_chunks = max(0, cb - ca);
   // chunk of turn i. What a segment adds is summed from its end: a chunk's weights then hold the decay up to there, and the sum in
-  // TMEM needs no scaling between chunks
-  auto chunk_of = [&](int i) { return STATES ? ca + n_chunks - 1 - i : ca + i; };
+  // TMEM needs no scaling between chunks (ROWS: weights are no number per token, the order is that of time)
+  auto chunk_of = [&](int i) { return STATES && !ROWS ? ca + n_chunks - 1 - i : ca + i; };
   constexpr int VC = 64 * NV;
   if (threadIdx.x == 0) {
     mbar_init(&sh.c_full, 1);
@@ -127,7 +124,7 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
     }
     for (int u = 0; u < NH; ++u) {
       mbar_init(&sh.x_full[u], 1);
-      mbar_init(&sh.x_empty[u], 8);
+      mbar_init(&sh.x_empty[u], ROWS ? 1 : 8);
       mbar_init(&sh.y_staged[u], 8);
       mbar_init(&sh.s_ready[u], 8);
       mbar_init(&sh.g_full[u], 1);
@@ -235,19 +232,28 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
 #pragma unroll
             for (int k = 0; k < 4 * KC; ++k)
               umma_f16_ss(tY, dC + (k >> 2) * TILE + (k & 3) * STEP_K, dW + part * NV * TILE + k * STEP_MN, id_y, part != 0 || k != 0 ? 1u : 0u);
-          umma_commit(&sh.cs_full[u]);
+          if (!ROWS) umma_commit(&sh.cs_full[u]);
           umma_commit(&sh.c_empty);
         }
-        if (!(ok = mbar_wait_bounded(&sh.w_ready[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
-        tc_fence_after();
+        if (ROWS) {  // the state has been scaled (s_ready; STATES: w_ready), and x enters as it is
+          if (STATES && !(ok = mbar_wait_bounded(&sh.w_ready[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
+          if (!(ok = mbar_wait_bounded(&sh.x_full[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
+          tc_fence_after();
 #pragma unroll
-        for (int part = 0; part < 2; ++part)
+          for (int k = 0; k < SD_T / 16; ++k) umma_f16_ss(tS, dBt + stage + k * STEP_MN, dX + k * STEP_MN, id_s, 1u);
+          if (STATES) umma_commit(&sh.x_empty[u]);
+        } else {
+          if (!(ok = mbar_wait_bounded(&sh.w_ready[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
+          tc_fence_after();
 #pragma unroll
-          for (int k = 0; k < SD_T / 16; ++k) umma_f16_ss(tS, dBt + stage + k * STEP_MN, dW + part * NV * TILE + k * STEP_MN, id_s, 1u);
+          for (int part = 0; part < 2; ++part)
+#pragma unroll
+            for (int k = 0; k < SD_T / 16; ++k) umma_f16_ss(tS, dBt + stage + k * STEP_MN, dW + part * NV * TILE + k * STEP_MN, id_s, 1u);
+        }
         umma_commit(&sh.s_done[u]);
         umma_commit(&sh.b_empty[st]);
         if (!STATES) {
-          if (!(ok = mbar_wait_bounded(&sh.x_full[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
+          if (!ROWS && !(ok = mbar_wait_bounded(&sh.x_full[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
           if (!(ok = mbar_wait_bounded(&sh.p_ready[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL))) break;
           tc_fence_after();
 #pragma unroll
@@ -260,10 +266,10 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
     }
   } else if (warp == 3) {
     // ------------------- step sizes and running sums (base 2) of the decays, up to two chunks ahead; lane = four tokens.
-    // Padding has step 0 and changes nothing
+    // Padding has step 0 and changes nothing. ROWS: nothing to do
     float rate[NH], bias[NH];
 #pragma unroll
-    for (int u = 0; u < NH; ++u) {
+    for (int u = 0; u < NH && !ROWS; ++u) {
       rate[u] = p.decay ? p.decay[h0 + u] : -expf(p.a_log[h0 + u]) * SD_LOG2E;
       bias[u] = p.decay ? 0.f : p.dt_bias[h0 + u];
     }
@@ -277,15 +283,15 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
         for (int u = 0; u < NH; ++u) raw[u][j] = raw_dt && t < n ? __bfloat162float(raw_dt[(long long)t * p.ld + u]) : 0.f;
       }
     };
-    if (n_chunks > 0) fetch(0);
+    if (n_chunks > 0 && !ROWS) fetch(0);
     bool ok = true;
-    for (int i = 0; i < n_chunks; ++i) {
+    for (int i = 0; i < n_chunks && !ROWS; ++i) {
       const int t0 = chunk_of(i) * SD_T + 4 * lane;
       float dt[NH][4], c[NH][4];
 #pragma unroll
       for (int u = 0; u < NH; ++u)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) dt[u][j] = t0 + j >= n ? 0.f : p.decay ? 1.f : sd_softplus(raw[u][j] + bias[u]);
+        for (int j = 0; j < 4; ++j) dt[u][j] = t0 + j >= n ? 0.f : p.decay ? 1.f : ss_softplus_fast(raw[u][j] + bias[u]);
       if (i + 1 < n_chunks) fetch(i + 1);
       if (ok) ok = mbar_wait_bounded(&sh.d_empty[i & 1], (uint32_t)((i >> 1) & 1) ^ 1, abort_flag, q.status, STATUS_TIMEOUT_EMPTY);
 #pragma unroll
@@ -324,7 +330,7 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
     float* const seg_base = q.seg_state ? q.seg_state + ((long long)b * p.heads + h) * p.np * p.vdp : nullptr;
     // starting state of this CTA, NULL: zero
     const float* from = STATES ? nullptr : (q.n_seg > 1 ? seg_base + seg * seg_step : (p.start[b] > 0 ? own : nullptr));
-    const float skip = p.decay ? 0.f : p.skip[h];
+    const float skip = ROWS || p.decay ? 0.f : p.skip[h];
     bool ok = true;  // after a wait that ran out the work goes on unseen: the status word tells, and the loop ends
     float decay_log2 = 0.f;
     auto state_at = [&](const float* base, int c) {  // four columns of this row, zero beyond the sizes
@@ -372,17 +378,26 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
       __syncwarp();
       if (lane == 0) mbar_arrive(&sh.y_staged[u]);
     };
+    // ROWS: log2 of the halves of a chunk's decay of this row
+    auto halves = [&](int i) {
+      return row < p.np ? *reinterpret_cast<const float2*>(q.factor + ((((long long)b * q.chunks + ca + i) * p.heads + h) * p.np + row) * 2)
+                        : make_float2(0.f, 0.f);
+    };
+    float2 ahead = ROWS && n_chunks > 0 ? halves(0) : make_float2(0.f, 0.f);
+    float rest_log2 = 0.f;  // ROWS: second half of the chunk before
 #pragma unroll 1
     for (int i = 0; i < n_chunks; ++i) {
       const uint32_t ph = (uint32_t)(i & 1), xph = (uint32_t)((i >> 1) & 1);
       const float* const s_cum = sh.cum[i & 1][u];
       const float* const s_dt = sh.dt[i & 1][u];
-      if (ok) ok = mbar_wait_bounded(&sh.d_full[i & 1], xph, abort_flag, q.status, STATUS_TIMEOUT_FULL);
-      const float total = sh.total[i & 1][u];
-      const float cum = s_cum[row], dt = s_dt[row];
+      if (!ROWS && ok) ok = mbar_wait_bounded(&sh.d_full[i & 1], xph, abort_flag, q.status, STATUS_TIMEOUT_FULL);
+      const float total = ROWS ? ahead.x + ahead.y : sh.total[i & 1][u];
+      const float cum = ROWS ? 0.f : s_cum[row], dt = ROWS ? 0.f : s_dt[row];
       const float later = decay_log2;  // STATES: of the chunks behind this one
       decay_log2 += total;
-      const float decay = sd_exp2(total);
+      const float decay = sd_exp2(ROWS ? rest_log2 + ahead.x : total);
+      rest_log2 = ahead.y;
+      if (ROWS && i + 1 < n_chunks) ahead = halves(i + 1);
       // ---- the state: operand of Y (value and rest), then scaled in place
       if (!STATES && i > 0 && ok) ok = mbar_wait_bounded(&sh.s_done[u], ph ^ 1, abort_flag, q.status, STATUS_TIMEOUT_TMEM_FULL);
       tc_fence_after();
@@ -393,6 +408,15 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
           tmem_ld_32x32b_x32(tS + (uint32_t)c0, r);
           tmem_ld_wait();
           const uint32_t tile = (uint32_t)((col0 + c0) / 64 * SD_TILE);
+          auto scale = [&]() {
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              const float2 v = fmul2(sd_pair(r[e], r[e + 1]), make_float2(decay, decay));
+              r[e] = __float_as_uint(v.x);
+              r[e + 1] = __float_as_uint(v.y);
+            }
+          };
+          if (ROWS) scale();  // queries meet the state in the same units
 #pragma unroll
           for (int k = 0; k < 4; ++k) {
             uint32_t hi[4], lo[4];
@@ -402,12 +426,7 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
             *reinterpret_cast<uint4*>(w_hi + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
             *reinterpret_cast<uint4*>(w_lo + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
           }
-#pragma unroll
-          for (int e = 0; e < 32; e += 2) {
-            const float2 v = fmul2(sd_pair(r[e], r[e + 1]), make_float2(decay, decay));
-            r[e] = __float_as_uint(v.x);
-            r[e + 1] = __float_as_uint(v.y);
-          }
+          if (!ROWS) scale();
           tmem_st_32x32b_x16(tS + (uint32_t)c0, r);
           tmem_st_32x32b_x16(tS + (uint32_t)(c0 + 16), r + 16);
         }
@@ -421,14 +440,14 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
         // factor is one of the row times one of the column, both at most 1
         if (ok) ok = mbar_wait_bounded(&sh.g_full[u], ph, abort_flag, q.status, STATUS_TIMEOUT_TMEM_FULL);
         tc_fence_after();
-        const float ref = quarter > 0 ? s_cum[32 * quarter - 1] : 0.f;
+        const float ref = !ROWS && quarter > 0 ? s_cum[32 * quarter - 1] : 0.f;
         const float rf = sd_exp2(cum - ref);
         const float2 rf2 = make_float2(rf, rf);
         float* const fac = sh.fac[u][wi];
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           const int k = j == 0 ? half : 3 - half;
-          if (k < quarter) fac[32 * j + lane] = sd_exp2(ref - s_cum[32 * k + lane]) * s_dt[32 * k + lane];
+          if (!ROWS && k < quarter) fac[32 * j + lane] = sd_exp2(ref - s_cum[32 * k + lane]) * s_dt[32 * k + lane];
         }
         __syncwarp();
 #pragma unroll 1
@@ -440,7 +459,15 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
             tmem_ld_wait();
           }
           uint32_t hi[16], lo[16];
-          if (k < quarter) {
+          if (ROWS && k <= quarter) {
+            // behind the diagonal keys are not weighted down: what they give there may be anything
+#pragma unroll
+            for (int e = 0; e < 32; e += 2) {
+              if (k == quarter && e > lane) x[e] = 0u;
+              if (k == quarter && e + 1 > lane) x[e + 1] = 0u;
+              sd_split(sd_pair(x[e], x[e + 1]), hi[e / 2], lo[e / 2]);
+            }
+          } else if (k < quarter) {
 #pragma unroll
             for (int e = 0; e < 32; e += 4) {
               const float4 f = *reinterpret_cast<const float4*>(fac + 32 * j + e);
@@ -471,6 +498,33 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
           tmem_st_32x32b_x16(tG + (uint32_t)(32 * k), hi);
           tmem_st_32x32b_x16(tG + (uint32_t)(32 * k + 16), lo);
         }
+      }
+      if constexpr (ROWS) {
+        if (STATES) {
+          if (i > 0) {  // at first the state is zero
+            if (ok) ok = mbar_wait_bounded(&sh.s_done[u], ph ^ 1, abort_flag, q.status, STATUS_TIMEOUT_TMEM_FULL);
+            tc_fence_after();
+#pragma unroll
+            for (int c0 = 0; c0 < HC; c0 += 32) {
+              uint32_t r[32];
+              tmem_ld_32x32b_x32(tS + (uint32_t)c0, r);
+              tmem_ld_wait();
+#pragma unroll
+              for (int e = 0; e < 32; e += 2) {
+                const float2 v = fmul2(sd_pair(r[e], r[e + 1]), make_float2(decay, decay));
+                r[e] = __float_as_uint(v.x);
+                r[e + 1] = __float_as_uint(v.y);
+              }
+              tmem_st_32x32b_x16(tS + (uint32_t)c0, r);
+              tmem_st_32x32b_x16(tS + (uint32_t)(c0 + 16), r + 16);
+            }
+          }
+        }
+        tmem_st_wait();  // the scaled state, or P
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(STATES ? &sh.w_ready[u] : &sh.p_ready[u]);
+        continue;
       }
       // ---- W, in the place of the state's copy once that has been used
       if (ok) ok = mbar_wait_bounded(&sh.x_full[u], ph, abort_flag, q.status, STATUS_TIMEOUT_FULL);
@@ -537,6 +591,7 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
     // ---- the state goes on: to the chaining kernel, or (last segment) to its sequence
     if (n_chunks > 0 && ok) ok = mbar_wait_bounded(&sh.s_done[u], (uint32_t)((n_chunks - 1) & 1), abort_flag, q.status, STATUS_TIMEOUT_TMEM_FULL);
     tc_fence_after();
+    const float last = ROWS ? sd_exp2(rest_log2) : 1.f;  // to the end of the last chunk
     float* const to = STATES ? seg_base + (seg + 1) * seg_step : (seg == q.n_seg - 1 && n > 0 ? own : nullptr);
     if (to && ok) {
 #pragma unroll 1
@@ -550,14 +605,16 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
         for (int e = 0; e < 16; e += 4) {
           float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
           if (n_chunks > 0)
-            v = make_float4(__uint_as_float(r[e]), __uint_as_float(r[e + 1]), __uint_as_float(r[e + 2]), __uint_as_float(r[e + 3]));
+            v = make_float4(__uint_as_float(r[e]) * last, __uint_as_float(r[e + 1]) * last, __uint_as_float(r[e + 2]) * last, __uint_as_float(r[e + 3]) * last);
           else if (from)
             v = state_at(from, c0 + e);
           if (row < p.np && col0 + c0 + e < p.vdp) *reinterpret_cast<float4*>(to + (long long)row * p.vdp + col0 + c0 + e) = v;
         }
       }
     }
-    if (STATES && row == 0 && half == 0) q.seg_decay[((long long)(seg + 1) * q.B + b) * p.heads + h] = decay_log2;
+    if (ROWS) {
+      if (STATES && half == 0 && row < p.np) q.seg_decay[(((long long)(seg + 1) * q.B + b) * p.heads + h) * p.np + row] = decay_log2;
+    } else if (STATES && row == 0 && half == 0) q.seg_decay[((long long)(seg + 1) * q.B + b) * p.heads + h] = decay_log2;
   }
   tc_fence_before();
   __syncthreads();
@@ -570,19 +627,21 @@ state_scan_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant
 // Starting states of the segments: entry 0 is the sequence's state, entry k + 1 what segment k makes of entry k.
 constexpr int SD_CHAIN = 256;
 
+template <bool ROWS>
 __global__ void __launch_bounds__(SD_CHAIN)
 state_chain_kernel(const SdParams q) {
   const ScanParams& p = q.s;
   const int h = blockIdx.y, b = blockIdx.z, i = blockIdx.x * SD_CHAIN + threadIdx.x;
   const long long size = (long long)p.np * p.vdp, step = (long long)q.B * p.heads * size / 4;
-  if (i >= size / 4) return;
+  if (i >= size / 4 || (ROWS && q.far[b * p.heads + h])) return;
+  const int row = ROWS ? 4 * i / p.vdp : 0, rows = ROWS ? p.np : 1;  // of the decays
   const float4* own = reinterpret_cast<const float4*>(p.state + ((long long)p.slots[b] * p.heads + h) * size);
   float4* seg = reinterpret_cast<float4*>(q.seg_state + ((long long)b * p.heads + h) * size) + i;
   float4 s = p.start[b] > 0 ? own[i] : make_float4(0.f, 0.f, 0.f, 0.f);
   seg[0] = s;
 #pragma unroll 4
   for (int k = 1; k < q.n_seg; ++k) {
-    const float f = sd_exp2(q.seg_decay[((long long)k * q.B + b) * p.heads + h]);
+    const float f = sd_exp2(q.seg_decay[(((long long)k * q.B + b) * p.heads + h) * rows + row]);
     const float4 add = seg[k * step];
     s = make_float4(fmaf(f, s.x, add.x), fmaf(f, s.y, add.y), fmaf(f, s.z, add.z), fmaf(f, s.w, add.w));
     seg[k * step] = s;
@@ -612,22 +671,22 @@ static SdPlan sd_plan(int B, int T, int heads, int groups, int vdp, int np) {
   return pl;
 }
 
-template <int NH, int NV, int KC>
+template <int NH, int NV, int KC, bool ROWS>
 static int sd_launch(const CUtensorMap* tm, SdParams& q, int smem, cudaStream_t s) {
   static PerDeviceOnce once;
   if (once.first()) {
-    cudaFuncSetAttribute(state_scan_kernel<NH, NV, KC, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SD_SMEM_LIMIT);
-    cudaFuncSetAttribute(state_scan_kernel<NH, NV, KC, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SD_SMEM_LIMIT);
+    cudaFuncSetAttribute(state_scan_kernel<NH, NV, KC, false, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SD_SMEM_LIMIT);
+    cudaFuncSetAttribute(state_scan_kernel<NH, NV, KC, true, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, SD_SMEM_LIMIT);
   }
   q.n_unit = q.s.heads / NH;
   const int per_seg = q.n_unit * q.B, n_seg = q.n_seg;
   if (n_seg > 1) {
     q.n_seg = n_seg - 1;  // what the last segment adds is nobody's start
-    state_scan_kernel<NH, NV, KC, true><<<per_seg * (n_seg - 1), SD_FRONT + 256 * NH, smem, s>>>(tm[0], tm[1], tm[2], tm[3], q);
+    state_scan_kernel<NH, NV, KC, true, ROWS><<<per_seg * (n_seg - 1), SD_FRONT + 256 * NH, smem, s>>>(tm[0], tm[1], tm[2], tm[3], q);
     q.n_seg = n_seg;
-    state_chain_kernel<<<dim3((q.s.np * q.s.vdp / 4 + SD_CHAIN - 1) / SD_CHAIN, q.s.heads, q.B), SD_CHAIN, 0, s>>>(q);
+    state_chain_kernel<ROWS><<<dim3((q.s.np * q.s.vdp / 4 + SD_CHAIN - 1) / SD_CHAIN, q.s.heads, q.B), SD_CHAIN, 0, s>>>(q);
   }
-  state_scan_kernel<NH, NV, KC, false><<<per_seg * n_seg, SD_FRONT + 256 * NH, smem, s>>>(tm[0], tm[1], tm[2], tm[3], q);
+  state_scan_kernel<NH, NV, KC, false, ROWS><<<per_seg * n_seg, SD_FRONT + 256 * NH, smem, s>>>(tm[0], tm[1], tm[2], tm[3], q);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
@@ -672,9 +731,13 @@ static int sd_run(SdParams& q, const __nv_bfloat16* x, long long ldx, const __nv
   if ((rc = tmap_bf16(&tm[2], cm, 4, db, sb, box))) return rc;
   const uint64_t sy[3] = {(uint64_t)p.vdp, (uint64_t)p.inner, (uint64_t)T * p.inner};
   if ((rc = tmap_bf16(&tm[3], q.y, 4, dx, sy, box))) return rc;
-  if (pl.nh == 2) return pl.kc == 1 ? sd_launch<2, 1, 1>(tm, q, pl.smem, s) : sd_launch<2, 1, 2>(tm, q, pl.smem, s);
-  if (pl.nv == 1) return pl.kc == 1 ? sd_launch<1, 1, 1>(tm, q, pl.smem, s) : sd_launch<1, 1, 2>(tm, q, pl.smem, s);
-  return pl.kc == 1 ? sd_launch<1, 2, 1>(tm, q, pl.smem, s) : sd_launch<1, 2, 2>(tm, q, pl.smem, s);
+  if (q.factor) {  // heads do not share keys
+    if (pl.nv == 1) return pl.kc == 1 ? sd_launch<1, 1, 1, true>(tm, q, pl.smem, s) : sd_launch<1, 1, 2, true>(tm, q, pl.smem, s);
+    return pl.kc == 1 ? sd_launch<1, 2, 1, true>(tm, q, pl.smem, s) : sd_launch<1, 2, 2, true>(tm, q, pl.smem, s);
+  }
+  if (pl.nh == 2) return pl.kc == 1 ? sd_launch<2, 1, 1, false>(tm, q, pl.smem, s) : sd_launch<2, 1, 2, false>(tm, q, pl.smem, s);
+  if (pl.nv == 1) return pl.kc == 1 ? sd_launch<1, 1, 1, false>(tm, q, pl.smem, s) : sd_launch<1, 1, 2, false>(tm, q, pl.smem, s);
+  return pl.kc == 1 ? sd_launch<1, 2, 1, false>(tm, q, pl.smem, s) : sd_launch<1, 2, 2, false>(tm, q, pl.smem, s);
 }
 
 }  // namespace kvb
@@ -689,6 +752,7 @@ extern "C" int kvb_state_scan_tc(const void* u, long long ld, int dt_col, const 
   p.state = state; p.ld = ld; p.T = T; p.dt_col = dt_col; p.heads = heads; p.groups = groups; p.vdp = vdp; p.np = np; p.inner = heads * vdp;
   p.channels = heads * vdp + 2 * groups * np;
   q.u = (const __nv_bfloat16*)u; q.y = (__nv_bfloat16*)y; q.status = status; q.B = B;
+  q.factor = nullptr; q.far = nullptr; q.chunks = 0;
   const __nv_bfloat16* x = (const __nv_bfloat16*)xbc;
   return sd_run(q, x, p.channels, x + p.inner, x + p.inner + groups * np, p.channels, (float*)scratch, (cudaStream_t)stream);
 }
@@ -703,6 +767,27 @@ extern "C" int kvb_retention_scan_tc(const void* v, long long ldv, const void* q
   p.dt_bias = p.a_log = p.skip = nullptr; p.decay = log2_decay; p.slots = slots; p.start = start; p.count = count; p.state = state;
   p.ld = 0; p.T = T; p.dt_col = 0; p.heads = heads; p.groups = heads; p.vdp = vdp; p.np = np; p.inner = heads * vdp; p.channels = 0;
   q.u = nullptr; q.y = (__nv_bfloat16*)y; q.status = status; q.B = B;
+  q.factor = nullptr; q.far = nullptr; q.chunks = 0;
   const __nv_bfloat16* c = (const __nv_bfloat16*)qk;
   return sd_run(q, (const __nv_bfloat16*)v, ldv, c + heads * np, c, ldqk, (float*)scratch, (cudaStream_t)stream);
+}
+
+extern "C" long long kvb_gated_linear_scan_tc_scratch_bytes(int B, int T, int heads, int vdp, int np) {
+  const kvb::SdPlan pl = kvb::sd_plan(B, T, heads, heads, vdp, np);
+  return pl.n_seg > 1 ? (long long)pl.n_seg * B * heads * np * ((long long)vdp + 1) * 4 : 0;
+}
+
+extern "C" int kvb_gated_linear_scan_tc(const void* v, long long ldv, const void* qk, const float* factor, const int* far, float* state, void* y,
+                                        void* scratch, const int* slots, const int* start, const int* count, int B, int T, int heads, int vdp,
+                                        int np, int* status, void* stream) {
+  using namespace kvb;
+  if (!factor || !far) return KVB_ERR_ARG;
+  SdParams q;
+  ScanParams& p = q.s;
+  p.dt_bias = p.a_log = p.skip = p.decay = nullptr; p.slots = slots; p.start = start; p.count = count; p.state = state;
+  p.ld = 0; p.T = T; p.dt_col = 0; p.heads = heads; p.groups = heads; p.vdp = vdp; p.np = np; p.inner = heads * vdp; p.channels = 0;
+  q.u = nullptr; q.y = (__nv_bfloat16*)y; q.status = status; q.B = B;
+  q.factor = factor; q.far = far; q.chunks = (T + SD_T - 1) / SD_T;
+  const __nv_bfloat16* c = (const __nv_bfloat16*)qk;
+  return sd_run(q, (const __nv_bfloat16*)v, ldv, c + heads * np, c, 2 * heads * np, (float*)scratch, (cudaStream_t)stream);
 }

@@ -27,7 +27,8 @@ class _Attention(ctypes.Structure):
 
     _fields_ = [(n, ctypes.c_int) for n in ("heads", "kv_heads", "maps", "dim", "dimp", "vdim", "vdp", "rot_dims", "value_col", "head_norm",
                                             "window", "keep", "chunk", "head", "ring", "sink", "gate_cols")]
-    _fields_ += [(n, ctypes.c_float) for n in ("scale", "softcap", "lam", "post", "eps")] + [("sink_w", ctypes.c_void_p)]
+    _fields_ += [(n, ctypes.c_float) for n in ("scale", "softcap", "lam", "post", "eps")]
+    _fields_ += [("pool", ctypes.c_int), ("borrowed", ctypes.c_int), ("out_ld", ctypes.c_longlong), ("sink_w", ctypes.c_void_p), ("q_scale", ctypes.c_void_p)]
 
 
 class _Router(ctypes.Structure):
@@ -36,10 +37,36 @@ class _Router(ctypes.Structure):
     _fields_ = [(n, ctypes.c_int) for n in ("score", "groups", "keep", "renormalize")] + [("eps", ctypes.c_float), ("correction", ctypes.c_void_p)]
 
 
+class _EdgeTokens(ctypes.Structure):
+    """``kvb_edge_tokens`` of ``kvb200_layers.h``."""
+
+    _fields_ = [(n, ctypes.c_void_p) for n in ("slots", "start", "count")] + [("T", ctypes.c_int), ("taps", ctypes.c_int), ("table", ctypes.c_void_p),
+                ("table_rows", ctypes.c_longlong), ("conv_w", ctypes.c_void_p), ("conv_ring", ctypes.c_void_p)]
+
+
+class _GatedLinear(ctypes.Structure):
+    """``kvb_gated_linear`` of ``kvb200_layers.h``."""
+
+    _fields_ = [(n, ctypes.c_void_p) for n in ("input", "w", "bias")] + [("ld", ctypes.c_longlong)]
+    _fields_ += [(n, ctypes.c_int) for n in ("heads", "np", "rank")] + [("inv_tau", ctypes.c_float), ("q_scale", ctypes.c_float)]
+
+
+class _GatedRecurrence(ctypes.Structure):
+    """``kvb_gated_recurrence`` of ``kvb200_layers.h``."""
+
+    _fields_ = [(n, ctypes.c_void_p) for n in ("conv", "conv_bias", "bias_r", "bias_i", "rate", "gates")]
+    _fields_ += [(n, ctypes.c_int) for n in ("blocks", "pp", "taps")] + [("scale", ctypes.c_float)]
+
+
+def _ptr(t: Optional[torch.Tensor]) -> Optional[int]:
+    return None if t is None else t.data_ptr()
+
+
 @functools.lru_cache(maxsize=512)
-def _attention(s, plan, eps: float, sink: Optional[int]) -> _Attention:
+def _attention(s, plan, eps: float, sink: Optional[int] = None, q_scale: Optional[int] = None, out_ld: int = 0) -> _Attention:
     return _Attention(s.heads, s.kv_heads, s.maps, s.dim, s.dimp, s.vdim, s.vdp, s.rot_dims, s.value_col, int(s.head_norm), s.window, s.keep,
-                      s.chunk, plan.head, plan.ring, int(s.sink), s.gate_cols, s.scale, s.softcap, s.lam, s.post, eps, sink)
+                      s.chunk, plan.head, plan.ring, int(s.sink), s.gate_cols, s.scale, s.softcap, s.lam, s.post, eps,
+                      s.pool, int(s.borrowed), out_ld or s.inner, sink, q_scale)
 
 
 def lib():
@@ -51,6 +78,7 @@ def lib():
         _LIB.kvb_grouped_decode_scratch_bytes.restype = ctypes.c_longlong
         _LIB.kvb_state_scan_tc_scratch_bytes.restype = ctypes.c_longlong
         _LIB.kvb_latent_decode_scratch_bytes.restype = ctypes.c_longlong
+        _LIB.kvb_gated_linear_scan_tc_scratch_bytes.restype = ctypes.c_longlong
     return _LIB
 
 
@@ -162,7 +190,18 @@ def latent_decode(q_abs, q, ring, seq, shape, scale) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------------------------ sequential layers
-def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None) -> None:
+def _edge_tokens(tokens):
+    if tokens is None:
+        return None
+    seq, table, conv, ring = tokens
+    _contiguous(table, conv, ring)
+    if conv is not None and ring.dtype != torch.float32:
+        raise NativeError("the inputs of a convolution are kept in fp32")
+    return ctypes.byref(_EdgeTokens(seq.slots.data_ptr(), seq.start.data_ptr(), seq.count.data_ptr(), seq.length, 0 if conv is None else conv.shape[0],
+                                    _ptr(table), 0 if table is None else table.shape[0], _ptr(conv), _ptr(ring)))
+
+
+def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None, tokens=None) -> None:
     width = x_out.shape[-1]
     out, row, weight = experts if experts is not None else (None, None, None)
     _contiguous(x_in, sub, after, x_out, before, h, idx, embed, step, out, row, weight)
@@ -170,7 +209,7 @@ def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center,
     _check(lib().kvb_norm_edge(_p(x_in), _p(sub), _p(out), _p(row), _p(weight), 0 if weight is None else weight.shape[1],
                                _ll(0 if out is None else out.shape[1]), _p(after), _p(x_out), _p(before), _p(h), _p(idx), _p(embed),
                                _ll(0 if embed is None else embed.shape[0]), _p(step), _ll(x_out.numel() // width), width, _f(eps), int(center),
-                               code(dtype), _p(status_word(x_out.device)), _stream(x_out)), "norm_edge")
+                               code(dtype), _edge_tokens(tokens), _p(status_word(x_out.device)), _stream(x_out)), "norm_edge")
     _count()
 
 
@@ -179,7 +218,7 @@ def row_norm(x, weight, eps, center, dtype) -> torch.Tensor:
     y = torch.empty((n, width), dtype=dtype, device=x.device)
     _contiguous(x, weight)
     _check(lib().kvb_norm_edge(_p(x), None, None, None, None, 0, _ll(0), None, None, _p(weight), _p(y), None, None, _ll(0), None, _ll(n), width, _f(eps), int(center),
-                               code(dtype), _p(status_word(x.device)), _stream(x)), "row_norm")
+                               code(dtype), None, _p(status_word(x.device)), _stream(x)), "row_norm")
     _count()
     return y
 
@@ -192,26 +231,28 @@ def activate(x, act: int) -> torch.Tensor:
 
 
 # ------------------------------------------------------------------------------------------ grouped attention
-def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan) -> torch.Tensor:
-    B, T, ld = qkv.shape
+def grouped_prep(qkv, norm_q, norm_k, freq, rows, seq, s, eps, plan, q_scale=None) -> torch.Tensor:
+    B, T, _ = qkv.shape
+    ld = _rows_of(qkv)
     q = torch.empty((B, T, s.heads * s.maps, s.dimp), dtype=qkv.dtype, device=qkv.device)
-    _contiguous(qkv, norm_q, norm_k, freq, rows)
-    a = _attention(s, plan, eps, None)
+    _contiguous(norm_q, norm_k, freq, rows, q_scale)
+    a = _attention(s, plan, eps, None, _ptr(q_scale))
     _check(lib().kvb_grouped_prep(_p(qkv), _ll(ld), _p(norm_q), _p(norm_k), _p(freq), _p(q), _p(rows), _p(seq.slots), _p(seq.start),
                                   _p(seq.count), B, T, rows.shape[1], ctypes.byref(a), code(qkv.dtype), _stream(qkv)), "grouped_prep")
-    _count()
+    _count(2 if s.pool and T > 1 else 1)
     return q
 
 
-def grouped_attend(q, qkv, rows, seq, s, sink, plan) -> torch.Tensor:
+def grouped_attend(q, qkv, rows, seq, s, sink, plan, out=None) -> torch.Tensor:
     B, T = q.shape[:2]
-    out = torch.empty((B, T, s.heads * s.vdp), dtype=q.dtype, device=q.device)
-    _contiguous(q, qkv, rows, sink)
+    if out is None:
+        out = torch.empty((B, T, s.inner), dtype=q.dtype, device=q.device)
+    _contiguous(q, rows, sink)
     gate = qkv.data_ptr() + s.gate_col * qkv.element_size() if s.gate else None
-    gate_args = (ctypes.c_void_p(gate), _ll(qkv.shape[-1]))
+    gate_args = (ctypes.c_void_p(gate), _ll(_rows_of(qkv) if s.gate else 0))
     where = (_p(seq.slots), _p(seq.start))
     length = rows.shape[1]
-    a = ctypes.byref(_attention(s, plan, s.eps, None if sink is None else sink.data_ptr()))
+    a = ctypes.byref(_attention(s, plan, s.eps, _ptr(sink), None, _rows_of(out)))
     fast = q.dtype == torch.bfloat16 and not FORCE_SIMPLE
     if fast and T == 1 and lib().kvb_grouped_decode_supported(a):
         nbytes = int(lib().kvb_grouped_decode_scratch_bytes(B, length, a))
@@ -265,10 +306,10 @@ def retention_scan(qk, v, decay, log2_decay, state, seq, s) -> torch.Tensor:
     return y
 
 
-def head_norm_gate(y, gate, s, eps) -> torch.Tensor:
+def head_norm_gate(y, gate, s, eps, weight=None) -> torch.Tensor:
     out = torch.empty_like(y)
-    _contiguous(y)
-    _check(lib().kvb_head_norm_gate(_p(y), _p(gate), _ll(_rows_of(gate)), _p(out), _ll(y.numel() // s.inner), s.heads, s.vdim, s.vdp, _f(eps),
+    _contiguous(y, weight)
+    _check(lib().kvb_head_norm_gate(_p(y), _p(gate), _ll(_rows_of(gate)), _p(weight), _p(out), _ll(y.numel() // s.inner), s.heads, s.vdim, s.vdp, _f(eps),
                                     code(y.dtype), _stream(y)), "head_norm_gate")
     _count()
     return out
@@ -284,13 +325,83 @@ def retention_step(u, freq, decay, state, seq, s, eps, dtype) -> torch.Tensor:
     return out
 
 
+# --------------------------------------------------------------------------------------- gated linear attention
+# rank of the decays' projection that the kernel in front of the chunked scan has room for
+GATED_LINEAR_MAX_RANK = 256
+
+
+def _gated_linear(u, decay, s) -> _GatedLinear:
+    _contiguous(u, *decay)
+    return _GatedLinear(u.data_ptr(), decay.weight.data_ptr(), decay.bias.data_ptr(), u.shape[-1], s.heads, s.np, s.rank, 1.0 / s.tau, s.query_scale)
+
+
+def gated_linear_scan(qka, v, decay, state, seq, s) -> torch.Tensor:
+    B, T, _ = qka.shape
+    y = torch.empty((B, T, s.inner), dtype=v.dtype, device=v.device)
+    _contiguous(state)
+    g = _gated_linear(qka, decay, s)
+    where, stream = (_p(seq.slots), _p(seq.start), _p(seq.count), B, T), _stream(qka)
+    far = None
+    if v.dtype == torch.bfloat16 and not FORCE_SIMPLE and s.rank <= GATED_LINEAR_MAX_RANK and lib().kvb_state_scan_tc_supported(s.heads, s.heads, s.vdp, s.np):
+        chunks = (T + 127) // 128
+        qk = torch.empty((B, T, s.qk), dtype=v.dtype, device=v.device)
+        factor = torch.empty((B, chunks, s.keys, 2), dtype=torch.float32, device=v.device)
+        far = torch.empty((B, s.heads), dtype=torch.int32, device=v.device)
+        _check(lib().kvb_gated_linear_prep(ctypes.byref(g), _p(qk), _p(factor), _p(far), _p(seq.count), B, T, stream), "gated_linear_prep")
+        nbytes = int(lib().kvb_gated_linear_scan_tc_scratch_bytes(B, T, s.heads, s.vdp, s.np))
+        scratch = torch.empty(nbytes, dtype=torch.uint8, device=v.device) if nbytes else None
+        _check(lib().kvb_gated_linear_scan_tc(_p(v), _ll(_rows_of(v)), _p(qk), _p(factor), _p(far), _p(state), _p(y), _p(scratch), *where, s.heads,
+                                              s.vdp, s.np, _p(status_word(v.device)), stream), "gated_linear_scan_tc")
+        _count(4 if nbytes else 2)
+    # after the chunked kernel: the heads whose decays are beyond its range, usually none
+    _check(lib().kvb_gated_linear_scan(ctypes.byref(g), _p(v), _ll(_rows_of(v)), _p(state), _p(y), _p(far), *where, s.vdp, code(v.dtype), stream),
+           "gated_linear_scan")
+    _count()
+    return y
+
+
+def gated_linear_step(u, decay, weight, state, seq, s, eps, dtype) -> torch.Tensor:
+    B = u.shape[0]
+    out = torch.empty((B, 1, s.inner), dtype=dtype, device=u.device)
+    _contiguous(weight, state)
+    g = _gated_linear(u, decay, s)
+    _check(lib().kvb_gated_linear_step(ctypes.byref(g), s.qk + s.rp, _p(weight), _p(state), _p(out), _p(seq.slots), _p(seq.start), _p(seq.count), B,
+                                       s.vdim, s.vdp, _f(eps), code(dtype), _stream(u)), "gated_linear_step")
+    _count()
+    return out
+
+
+# ------------------------------------------------------------------------------------ gated recurrence per channel
+def gated_recurrence(u, w, ring, state, seq, s, scale, out) -> torch.Tensor:
+    B, T, _ = u.shape
+    _contiguous(*w, ring, state)
+    g = ctypes.byref(_GatedRecurrence(*(t.data_ptr() for t in (w.conv, w.conv_bias, w.bias_r, w.bias_i, w.rate, w.gates)), s.blocks, s.pp, s.taps, scale))
+    where = (_p(seq.slots), _p(seq.start), _p(seq.count), B)
+    ld, ldo = _ll(_rows_of(u)), _ll(_rows_of(out))
+    if T == 1:
+        _check(lib().kvb_gated_recurrence_step(g, _p(u), ld, _p(ring), _p(state), _p(out), ldo, *where, code(u.dtype), _stream(u)), "gated_recurrence_step")
+        _count()
+        return out
+    x = short_conv(u, s.channels, w.conv, w.conv_bias, ring, seq, False)
+    z = bmm_fp32(x.view(B * T, s.blocks, s.pp).transpose(0, 1), w.gates)
+    _check(lib().kvb_gated_recurrence_scan(g, _p(x), _p(z), _p(u), ld, _p(state), _p(out), ldo, *where, T, code(u.dtype), _stream(u)), "gated_recurrence_scan")
+    _count()
+    return out
+
+
+def bmm_fp32(a, b) -> torch.Tensor:
+    """Batched library product with an fp32 result."""
+    return torch.bmm(a, b) if a.dtype == torch.float32 else torch.bmm(a, b, out_dtype=torch.float32)
+
+
 # --------------------------------------------------------------------------------------- state-space recurrence
-def short_conv(u, w, bias, ring, seq, s) -> torch.Tensor:
-    B, T, ld = u.shape
-    out = torch.empty((B, T, s.channels), dtype=u.dtype, device=u.device)
-    _contiguous(u, w, bias, ring)
-    _check(lib().kvb_short_conv(_p(u), _ll(ld), s.inner, _p(w), _p(bias), _p(out), _p(ring), _p(seq.slots), _p(seq.start), _p(seq.count), B, T,
-                                s.channels, s.taps, code(u.dtype), _stream(u)), "short_conv")
+def short_conv(u, col, w, bias, ring, seq, silu=True) -> torch.Tensor:
+    B, T, _ = u.shape
+    taps, channels = w.shape
+    out = torch.empty((B, T, channels), dtype=u.dtype, device=u.device)
+    _contiguous(w, bias, ring)
+    _check(lib().kvb_short_conv(_p(u), _ll(_rows_of(u)), col, _p(w), _p(bias), _p(out), _p(ring), _p(seq.slots), _p(seq.start), _p(seq.count), B, T,
+                                channels, taps, int(silu), code(u.dtype), _stream(u)), "short_conv")
     _count()
     return out
 
@@ -333,11 +444,11 @@ def gated_group_norm(y, u, weight, s, eps) -> torch.Tensor:
     return out
 
 
-def glu(x, ff) -> torch.Tensor:
+def glu(x, ff, limit=None) -> torch.Tensor:
     half = x.shape[-1] // 2
     out = torch.empty((*x.shape[:-1], half), dtype=x.dtype, device=x.device)
     _contiguous(x)
-    _check(lib().kvb_glu(_p(x), _p(out), _ll(x.numel() // (2 * half)), _ll(2 * half), half, ff, half, code(x.dtype), _stream(x)), "glu")
+    _check(lib().kvb_glu(_p(x), _p(out), _ll(x.numel() // (2 * half)), _ll(2 * half), half, ff, half, _f(limit or 0.0), code(x.dtype), _stream(x)), "glu")
     _count()
     return out
 
