@@ -266,7 +266,7 @@ def run_layered(args) -> dict:
     prompt = 8192 if args.seq_len == 131072 else args.seq_len
     decode = 64 if args.decode == 512 else args.decode
     chunk = 2048 if args.chunk_size == 1024 else args.chunk_size
-    names = ["Mezilix-2k", "Mezilix-4k", "Pazenex-2k", "Pazenex-4k", "Ladadra-2k", "Ladadra-4k"] if args.model == "Qwen3-4B" else [args.model]
+    names = ["Mezilix-2k", "Mezilix-4k", "Pazenex-2k", "Pazenex-4k", "Ladadra-2k", "Ladadra-4k", "Dotorax-2k", "Dotorax-4k"] if args.model == "Qwen3-4B" else [args.model]
     sampler = ClockSampler(0)
     sampler.start()
     models, kernels = [], {}

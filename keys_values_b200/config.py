@@ -302,6 +302,38 @@ def _grouped_experts(n_expert: int, top: int, ff: int, groups: int, keep: int, s
                 renormalize_eps=1e-20, groups=dict(count=groups, keep=keep), shared=shared)
 
 
+def _dotorax(width: int, layers: List[dict], **kwargs: Any) -> dict:
+    """Fields of a model of sequential layers whose inputs pass a short convolution; ``layers`` as in ``Config.layers``."""
+    first = next(x["mixer"] for x in layers if x["mixer"]["kind"] == "grouped_attention")
+    return dict(
+        n_embd=width, n_layer=len(layers), layers=layers, n_head=first["n_head"], n_query_groups=first["n_kv_head"], head_size=first["dim"],
+        norm_class_name="StreamOffsetRMSNorm", parallel_residual=False, post_attention_norm=True, post_mlp_norm=True, bias=False,
+        position_table=True, architecture="Dotorax", **kwargs,
+    )
+
+
+def _shared_runs(times: int, heads: int, kv_heads: int, dim: int, rope_dims: int, linear: dict, parallel: dict, ff: int, limit: float = 7.0) -> List[dict]:
+    """``times`` runs of: attention, gated linear attention, attention over the first one's keys and values, two mixers side by side."""
+    out = []
+    for i in range(times):
+        a = dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=dim, scale=dim**-0.5, rope_base=250000.0, rope_dims=rope_dims,
+                 gate="head")
+        out += [a, linear, dict(a, kv_from=4 * i), parallel]
+    return [dict(mixer=m, mlp=dict(kind="gated", ff=ff, limit=limit)) for m in out]
+
+
+def _gated_linear(heads: int, dim: int, vdim: int, rank: int = 16, tau: float = 16.0) -> dict:
+    return dict(kind="gated_linear_attention", n_head=heads, dim=dim, v_dim=vdim, rank=rank, tau=tau)
+
+
+def _pooled_beside_recurrence(heads: int, kv_heads: int, dim: int, rope_dims: int, window: int, pool: int, width: int, blocks: int,
+                              scales: Tuple[float, float] = (0.7, 1.0)) -> dict:
+    left = dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=dim, scale=dim**-0.5, rope_base=50000.0, rope_dims=rope_dims,
+                rope_interleaved=True, qk_norm="unit", temperature=True, window=window, pool=pool)
+    return dict(kind="side_by_side", left=left, left_scale=scales[0], right=dict(kind="gated_recurrence", width=width, blocks=blocks, conv=4),
+                right_scale=scales[1])
+
+
 _llama_like = dict(
     rotary_percentage=1.0,
     parallel_residual=False,
@@ -411,6 +443,23 @@ configs: List[dict] = [
             dict(mixer=_chunked(32, 8, 128, 128, chunk=16384, rope_dims=64), mlp=_gated(11008)),
             dict(mixer=_chunked(32, 8, 128, 128, chunk=16384, rope_dims=64), mlp=_grouped_experts(32, 4, 2048, 4, 2, 2816)),
         ] * 3),
+    ),
+    # Dotorax: attention (half of it over another layer's keys and values), gated linear attention, a window with pooled blocks side by side
+    # with a gated recurrence; short convolutions in front of the sublayers, a position table
+    dict(
+        name="tiny-dotorax", block_size=1024, vocab_size=288, padded_vocab_size=288, norm_eps=1e-5, input_conv=3, residual_mult=0.8,
+        **_dotorax(112, _shared_runs(1, 6, 3, 24, 16, _gated_linear(3, 40, 24, rank=8),
+                                     _pooled_beside_recurrence(4, 2, 24, 8, 48, 6, 120, 5), 152, limit=2.0)),
+    ),
+    dict(
+        name="Dotorax-2k", block_size=1 << 15, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5, input_conv=4, residual_mult=0.7,
+        **_dotorax(2048, _shared_runs(4, 16, 4, 128, 64, _gated_linear(16, 128, 128),
+                                      _pooled_beside_recurrence(16, 4, 128, 64, 2048, 64, 2048, 16), 5632)),
+    ),
+    dict(
+        name="Dotorax-4k", block_size=1 << 15, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5, input_conv=4, residual_mult=0.7,
+        **_dotorax(4096, _shared_runs(3, 32, 8, 128, 64, _gated_linear(32, 128, 128),
+                                      _pooled_beside_recurrence(32, 8, 128, 64, 2048, 64, 4096, 16), 11008)),
     ),
     # Qwen 2.5
     dict(

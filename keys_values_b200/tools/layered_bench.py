@@ -5,7 +5,7 @@ time of every kernel of the design beside the like kernel of that model, each ag
 
 Random-init weights, synthetic tokens. For Mezilix the closest model has the same width, depth, heads, window and experts
 (count, chosen per token, expert weights per token): grouped-query attention over a sliding window, SwiGLU experts
-(``LLaMAMoE``), or a dense SwiGLU of the width that a token's chosen experts add up to. For Pazenex and Ladadra it has the same width,
+(``LLaMAMoE``), or a dense SwiGLU of the width that a token's chosen experts add up to. For Pazenex, Ladadra and Dotorax it has the same width,
 depth, heads and key/value heads, attention in every layer and a dense SwiGLU that makes the number of weights that a token meets
 equal. Kernel times are
 CUDA-event medians with an L2 flush (256 MB written, another 256 MB read) before every launch.
@@ -39,9 +39,14 @@ def closest_config(config: Config, dense: bool = False) -> Config:
     return Config(mlp_class_name="LLaMAMoE", intermediate_size=ff, moe_intermediate_size=ff, n_expert=f["n_expert"], n_expert_per_token=f["top"], **kw)
 
 
-def layer_weights(layer: Dict, width: int) -> int:
-    """Weights of the products that a token meets in one sequential layer."""
-    x, f = layer["mixer"], layer["mlp"]
+def mixer_weights(x: Dict, width: int) -> int:
+    """Weights of the products that a token meets in a mixer."""
+    if x["kind"] == "side_by_side":
+        return mixer_weights(x["left"], width) + mixer_weights(x["right"], width)
+    if x["kind"] == "gated_recurrence":
+        return 3 * width * x["width"] + 2 * x["width"] ** 2 // x["blocks"]
+    if x["kind"] == "gated_linear_attention":
+        return width * (x["n_head"] * (2 * x["dim"] + 3 * x["v_dim"]) + x["rank"]) + x["rank"] * x["n_head"] * x["dim"]
     if x["kind"] == "mamba2":
         inner, bc = x["n_head"] * x["v_dim"], x["groups"] * x["state"]
         n = width * (3 * inner + 2 * bc + x["n_head"])
@@ -52,6 +57,14 @@ def layer_weights(layer: Dict, width: int) -> int:
         H, G = x["n_head"], x["n_kv_head"]
         n = width * ((H + G) * maps * x["dim"] + H * x["v_dim"])
         n += width * ((0 if x.get("shared_value") else G * x["v_dim"]) + {True: H * x["v_dim"], "head": H}.get(x.get("gate"), 0))
+        if x.get("kv_from") is not None:
+            n -= width * G * (x["dim"] + x["v_dim"])
+    return n
+
+
+def layer_weights(layer: Dict, width: int) -> int:
+    """Weights of the products that a token meets in one sequential layer."""
+    n, f = mixer_weights(layer["mixer"], width), layer["mlp"]
     if f is None:
         return n
     if f["kind"] == "routed":
@@ -196,6 +209,8 @@ def _window_pairs(T: int, P: int, window: int) -> int:
 def kernel_table(config: Config, batch: int, tokens: int = 8192, dense_like: bool = True) -> List[Dict]:
     """Kernels of one middle layer of ``config`` (Pazenex: of one layer of each kind): a pass of ``tokens`` new tokens of one sequence with a full window before them,
     and a single-token pass of ``batch`` sequences with full rings; like kernels of the closest model after each."""
+    if any(x["mixer"]["kind"] == "side_by_side" for x in config.layers):
+        return side_by_side_kernel_table(config, batch, tokens)
     if any(x["mixer"]["kind"] == "retention" for x in config.layers):
         return output_norm_kernel_table(config, batch, tokens)
     if any(x["mixer"]["kind"] != "latent_attention" for x in config.layers):
@@ -567,6 +582,152 @@ def output_norm_kernel_table(config: Config, batch: int, tokens: int = 8192) -> 
                 gbytes=(2 * n * W + 2 * r.qk * W + 4 * n * r.qk) / 1e9, tflop=2 * n * r.qk * W / 1e12)
         tab.add(f"{tag}:   like: with bf16 result", lambda: torch.mm(hn, w3.t()), gbytes=2 * (n * W + r.qk * W + n * r.qk) / 1e9, tflop=2 * n * r.qk * W / 1e12)
         del hn, w3, x, sub, h, a, rr
+        torch.cuda.empty_cache()
+    ops.check_status(dev)
+    return tab.rows
+
+
+@torch.inference_mode()
+def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) -> List[Dict]:
+    """Kernels of one layer of each kind of a model with gated linear attention and a pooled window side by side with a gated recurrence: prompts
+    of ``tokens`` tokens, and a single-token pass of ``batch`` sequences at that position; like kernels of the closest model after each."""
+    from keys_values_b200 import ops
+    from keys_values_b200.kvcache.sequences import SequenceTable
+    from keys_values_b200.models.gated_linear import gated_linear_shape
+    from keys_values_b200.models.gated_recurrence import recurrence_shape
+    from keys_values_b200.models.grouped_attention import grouped_shape
+    from keys_values_b200.ops import cuda as cu
+    from keys_values_b200.ops import layers as L
+    from keys_values_b200.ops import layers_cuda as LC
+
+    dev, bf = torch.device("cuda"), torch.bfloat16
+    tab = KernelTable()
+    mixers = [x["mixer"] for x in config.layers]
+    both = next(x for x in mixers if x["kind"] == "side_by_side")
+    plain = grouped_shape(next(x for x in mixers if x["kind"] == "grouped_attention" and x.get("kv_from") is None))
+    borrowed = grouped_shape(next(x for x in mixers if x.get("kv_from") is not None))
+    pooled, r = grouped_shape(both["left"]), recurrence_shape(both["right"])
+    m = gated_linear_shape(next(x for x in mixers if x["kind"] == "gated_linear_attention"))
+    ff, limit = config.layers[0]["mlp"]["ff"], config.layers[0]["mlp"]["limit"]
+    W, eps, taps = config.n_embd, config.norm_eps, config.input_conv
+    rand = lambda *shape: torch.randn(*shape, device=dev, dtype=bf)  # noqa: E731
+    f32 = lambda *shape: torch.rand(*shape, device=dev)  # noqa: E731
+    tiles = lambda n: -(-n // 128) * 128  # noqa: E731
+    for B, T, start in ((1, tokens, 0), (4, tokens, 0), (batch, 1, tokens - 1)):
+        n = B * T
+        tag = f"prefill {B} x {T} tokens" if T > 1 else f"decode {B} rows"
+        table = SequenceTable(B, dev)
+        table.set_batch([table.acquire() for _ in range(B)])
+        table.pos.fill_(start)
+        table.pos_host = [start] * B
+        seq = table.begin(B, T)
+        seq.start = seq.start.clone()
+        # ---- between sublayers
+        x, sub, h, w1, w2 = torch.randn(B, T, W, device=dev), rand(B, T, W), rand(B, T, W), f32(W), f32(W)
+        out = torch.empty_like(x) if T > 1 else x
+        edge = L.EdgeTokens(seq, None, f32(taps, W), f32(B, taps, W))
+        tab.add(f"{tag}: norm, residual sum, norm, convolution", lambda: LC.norm_edge(x, sub, w1, out, w2, h, None, None, None, eps, False, None, edge),
+                gbytes=(n * W * 12 + (0 if T > 1 else B * taps * W * 4)) / 1e9)
+        a, rr, w = rand(n, W), rand(n, W), rand(W)
+        fused = cu.add_rmsnorm_supported(a)
+        like_norm = lambda: cu.add_rmsnorm_fwd(a, rr, w, eps, False) if fused else cu.rmsnorm_fwd(a, w, eps, False)  # noqa: E731
+        norm_bytes = n * W * (8 if fused else 4) / 1e9
+        tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+        up = rand(n, 2 * ff)
+        tab.add(f"{tag}: clamped unit", lambda: LC.glu(up, ff, limit), gbytes=n * ff * 6 / 1e9)
+        u1 = up.view(2, n, ff)
+        tab.add(f"{tag}:   like: SwiGLU", lambda: cu.swiglu_fwd(u1[0], u1[1]), gbytes=n * ff * 6 / 1e9)
+        del up, u1, out
+        # ---- attentions
+        for what, s in (("attention", plain), ("attention over another layer's keys", borrowed), ("pooled window", pooled)):
+            H, G, D, V = s.heads, s.kv_heads, s.dim, s.vdim
+            plan = L.RowPlan(tiles(tokens // s.pool), tiles(tokens + 64)) if s.pool else L.RowPlan()
+            length = sum(plan) if s.pool else tokens + 64
+            qkv, freq, rows = rand(B, T, s.ld), f32(s.rot_dims // 2), rand(B, length, G, s.row)
+            unit, temp = (torch.ones(s.dimp, device=dev), f32(H)) if s.pool else (None, None)
+            own = 0 if s.borrowed else G * (D + V)
+            tab.add(f"{tag}: {what}: " + ("norm, " if s.pool else "") + "rotation" + ("" if s.borrowed else ", into the cache") + (", means of blocks" if s.pool else ""),
+                    lambda: LC.grouped_prep(qkv, unit, unit, freq, rows, seq, s, eps, plan, temp), gbytes=2 * n * 2 * (H * D + own) / 1e9)
+            qkv2, cs, wq = rand(B, T, (H + 2 * G) * 128), f32(T, 128), rand(128)
+            tab.add(f"{tag}:   like: QK norm, split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, H, G, 128, eps, 128, False),
+                    gbytes=2 * 2 * n * (H + 2 * G) * 128 / 1e9)
+            q = rand(B, T, H, s.dimp)
+            q2, k2 = rand(B, H, T, 128), rand(B, G, tokens, 128)
+            seen = s.window or 1 << 40
+            win = s.window if s.window and s.window < tokens else 0
+            blocks = lambda t: max(0, (start + t - s.window + 1) // s.pool) if s.pool else 0  # noqa: E731
+            if T > 1:
+                pairs = B * H * (_window_pairs(T, 0, seen) + sum(blocks(t) for t in range(T)))
+                tab.add(f"{tag}: {what}, {H} heads on {G}" + (f", {s.window} tokens and blocks of {s.pool}" if s.pool else ", gate"),
+                        lambda: LC.grouped_attend(q, qkv, rows, seq, s, None, plan), tflop=2 * pairs * (D + V) / 1e12)
+                like = B * H * _window_pairs(T, 0, seen)
+                tab.add(f"{tag}:   like: attention 128 / 128" + (f", window {win}" if win else ""),
+                        lambda: cu.sdpa_fwd(q2, k2, k2, 0.09, 0, None, False, win, None) if win else cu.sdpa_fwd(q2, k2, k2, 0.09, 0), tflop=2 * like * 256 / 1e12)
+            else:
+                k = min(tokens, seen) + blocks(0)
+                tab.add(f"{tag}: {what} over {k} rows, {H} heads on {G}", lambda: LC.grouped_attend(q, qkv, rows, seq, s, None, plan),
+                        gbytes=2 * B * G * k * (D + V) / 1e9)
+                k3, v3 = rand(B, G, min(tokens, seen), 128), rand(B, G, min(tokens, seen), 128)
+                tab.add(f"{tag}:   like: attention over {k3.shape[2]} slots", lambda: cu.decode_attention(q2, k3, v3, 0.09, k3.shape[2]),
+                        gbytes=2 * B * G * k3.shape[2] * 256 / 1e9)
+                del k3, v3
+            del rows, k2, q2, q, qkv2, qkv
+        # ---- gated linear attention
+        state = 0.01 * torch.randn(B, m.heads, m.np, m.vdp, device=dev)
+        decay, wn = L.DecayWeights(0.3 * torch.randn(m.rank, m.keys, device=dev), 2 + f32(m.keys)), f32(m.vdp)
+        state_bytes = B * m.heads * m.np * m.vdp * 8
+        if T > 1:
+            qka, vg = torch.randn(B, T, m.qk + m.rp, device=dev), rand(B, T, 2 * m.inner)
+            g, chunks = LC._gated_linear(qka, decay, m), -(-T // 128)
+            qk, factor = torch.empty(B, T, m.qk, device=dev, dtype=bf), torch.empty(B, chunks, m.keys, 2, device=dev)
+            far = torch.zeros(B, m.heads, dtype=torch.int32, device=dev)
+            prep = lambda: cu._check(LC.lib().kvb_gated_linear_prep(LC.ctypes.byref(g), cu._p(qk), cu._p(factor), cu._p(far), cu._p(seq.count), B, T,  # noqa: E731
+                                                                    cu._stream(qka)), "prep")
+            tab.add(f"{tag}: gated linear: decays, queries and keys", prep, gbytes=n * (6 * m.qk + 4 * m.rp) / 1e9)
+            qkv2, cs, wq = rand(B, T, 2 * m.qk), f32(T, 128), rand(128)
+            tab.add(f"{tag}:   like: QK norm, split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, 2 * m.qk // 128 - 16, 8, 128, eps, 128, False),
+                    gbytes=8 * n * m.qk / 1e9)
+            flop = n * m.heads * (4 * m.np * m.vdp + 128 * (m.np + m.vdp)) / 1e12
+            tab.add(f"{tag}: gated linear scan (all kernels), {m.heads} heads of {m.np} x {m.vdp}", lambda: LC.gated_linear_scan(qka, vg, decay, state, seq, m),
+                    gbytes=(n * (4 * (m.qk + m.rp) + 4 * m.inner) + state_bytes) / 1e9, tflop=flop)
+            q2 = rand(B, m.heads, T, 128)
+            tab.add(f"{tag}:   like: attention 128 / 128, {m.heads} heads", lambda: cu.sdpa_fwd(q2, q2, q2, 0.09, 0),
+                    tflop=2 * B * m.heads * (T * (T + 1) // 2) * 256 / 1e12)
+            y = rand(B, T, m.inner)
+            tab.add(f"{tag}: gated linear: norm per head, gate", lambda: LC.head_norm_gate(y, vg[..., m.inner :], m, eps, wn), gbytes=6 * n * m.inner / 1e9)
+            tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+            del qka, vg, qk, q2, qkv2, y, factor
+        else:
+            u = torch.randn(B, 1, m.qk + m.rp + 2 * m.inner, device=dev)
+            tab.add(f"{tag}: gated linear step, {m.heads} heads of {m.np} x {m.vdp}", lambda: LC.gated_linear_step(u, decay, wn, state, seq, m, eps, bf),
+                    gbytes=(state_bytes + 4 * n * u.shape[-1]) / 1e9)
+        del state
+        # ---- gated recurrence
+        C = r.channels
+        u, ring, state, y = rand(B, T, 2 * C), rand(B, r.taps, C), f32(B, C), rand(B, T, C)
+        gw = L.RecurrenceWeights(f32(r.taps, C), f32(C), 0.1 * rand(r.blocks, r.pp, 2 * r.pp), f32(C), f32(C), -f32(C))
+        if T > 1:
+            tab.add(f"{tag}: convolution, {C} channels", lambda: LC.short_conv(u, C, gw.conv, gw.conv_bias, ring, seq, False), gbytes=4 * n * C / 1e9)
+            tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+            xc = rand(n, r.blocks, r.pp).transpose(0, 1)
+            tab.add(f"{tag}: library products of the gates, fp32 results", lambda: LC.bmm_fp32(xc, gw.gates), gbytes=n * C * 10 / 1e9, tflop=4 * n * C * r.pp / 1e12)
+            z, xs = LC.bmm_fp32(xc, gw.gates), rand(B, T, C)
+            g = LC._GatedRecurrence(*(t.data_ptr() for t in (gw.conv, gw.conv_bias, gw.bias_r, gw.bias_i, gw.rate, gw.gates)), r.blocks, r.pp, r.taps, 1.0)
+            scan = lambda: cu._check(LC.lib().kvb_gated_recurrence_scan(LC.ctypes.byref(g), cu._p(xs), cu._p(z), cu._p(u), cu._ll(2 * C), cu._p(state), cu._p(y),  # noqa: E731
+                                                                        cu._ll(C), cu._p(seq.slots), cu._p(seq.start), cu._p(seq.count), B, T, 1, cu._stream(u)), "scan")
+            tab.add(f"{tag}: gated recurrence scan, {C} channels", scan, gbytes=n * C * 14 / 1e9)
+            tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+            del z, xs, xc
+        else:
+            tab.add(f"{tag}: convolution, gates and recurrence step, {C} channels", lambda: LC.gated_recurrence(u, gw, ring, state, seq, r, 1.0, y),
+                    gbytes=(n * C * (2 * (2 + r.taps) + 8 + 2) + 4 * C * r.pp) / 1e9)
+            tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+        # ---- products (library, in both models)
+        hn, w3 = rand(n, W), rand(m.qk + m.rp, W)
+        tab.add(f"{tag}: library product with fp32 result {n} x {m.qk + m.rp} x {W}", lambda: L.linear_fp32(hn, w3),
+                gbytes=(2 * n * W + 2 * m.qk * W + 4 * n * m.qk) / 1e9, tflop=2 * n * m.qk * W / 1e12)
+        tab.add(f"{tag}:   like: with bf16 result", lambda: torch.mm(hn, w3.t()), gbytes=2 * (n * W + m.qk * W + n * m.qk) / 1e9, tflop=2 * n * m.qk * W / 1e12)
+        del hn, w3, x, sub, h, a, rr, u, ring, state, y
         torch.cuda.empty_cache()
     ops.check_status(dev)
     return tab.rows

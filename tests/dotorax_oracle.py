@@ -68,17 +68,19 @@ def blocks_seen(i, size, pool):
     return n
 
 
+def pooled_row(i, q, k, v, scale, size, pool):
+    """Result of one query at position ``i`` over a window of tokens and the means of the blocks that lie before it, in one softmax."""
+    n, first = blocks_seen(i, size, pool), max(0, i - size + 1)
+    keys, values = list(k[first : i + 1]), list(v[first : i + 1])
+    for b in range(n):
+        keys.append(k[b * pool : (b + 1) * pool].mean(0))
+        values.append(v[b * pool : (b + 1) * pool].mean(0))
+    return softmax_sum(torch.stack(keys) @ q * scale, torch.stack(values))
+
+
 def attend_pooled(q, k, v, scale, size, pool):
-    """One head over a window of tokens and the means of the blocks that lie before it, in one softmax."""
-    kb = [k[b * pool : (b + 1) * pool].mean(0) for b in range(len(k) // pool)]
-    vb = [v[b * pool : (b + 1) * pool].mean(0) for b in range(len(k) // pool)]
-    out = []
-    for i in range(len(q)):
-        n, first = blocks_seen(i, size, pool), max(0, i - size + 1)
-        keys = torch.cat([k[first : i + 1]] + [x[None] for x in kb[:n]])
-        values = torch.cat([v[first : i + 1]] + [x[None] for x in vb[:n]])
-        out.append(softmax_sum(keys @ q[i] * scale, values))
-    return torch.stack(out)
+    """One head."""
+    return torch.stack([pooled_row(i, q[i], k, v, scale, size, pool) for i in range(len(q))])
 
 
 def keys_values(h, w, m):
@@ -231,7 +233,7 @@ def gla_layer(heads=3, dim=16, vdim=24, tau=8.0, mlp=None):
     return {"type": "gla", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}}
 
 
-def content(layers, width=40, vocab=61, eps=1e-4, taps=3, mult=0.8, positions=400):
+def content(layers, width=40, vocab=61, eps=2e-2, taps=3, mult=0.5, positions=400):
     return {"architecture": "Dotorax", "vocab": vocab, "width": width, "norm": {"eps": eps}, "canon": {"taps": taps}, "residual_mult": mult,
             "max_positions": positions, "layers": layers}
 
