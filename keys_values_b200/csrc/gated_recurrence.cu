@@ -1,14 +1,17 @@
 // Gated recurrence per channel: S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t x_t with log2 a_t = rate · r_t, gates r and i sigmoids; the result is
 // S · gelu(y).
 //
-//   scan   several new tokens, behind the convolution (ssm.cu) and the gates' products: a CTA has 32 channels of one sequence and takes 128 tokens
-//          at a time. A warp has 16 of them and a lane one channel: decays and additions stay in registers, the warps exchange what their
-//          tokens make of a state, and then every warp runs through its tokens from the right start. Everything is read once;
+//   scan   several new tokens, behind the convolution (ssm.cu) and the gates' products: a cluster of up to eight CTAs has 64 channels of one
+//          sequence and takes 64 tokens per CTA at a time. A warp has 8 of them and a lane two channels: decays and additions stay in registers;
+//          the warps of a CTA, then the CTAs (over distributed shared memory) exchange what their tokens make of a state, and every warp runs
+//          through its tokens from the right start. Everything is read once;
 //   step   one new token per sequence: convolution, gates (a part's products on CUDA cores, weights read once for eight sequences), recurrence
 //          and output in one kernel. The inputs of the convolution lie in a ring with one row more than it looks back, so CTAs that share
 //          a part do not disturb each other.
 //
 // Everything from the gates' products on is fp32.
+#include <cooperative_groups.h>
+
 #include "common.cuh"
 #include "kvb200_layers.h"
 #include "ssm.cuh"
@@ -57,8 +60,10 @@ __device__ __forceinline__ void gr_token(float zr, float zi, float x, float rate
 
 // ------------------------------------------------------------------------------------------------ scan
 constexpr int GR_WARPS = 8;
-constexpr int GR_RUN = 16;  // tokens of a warp
+constexpr int GR_RUN = 8;    // tokens of a warp
+constexpr int GR_COLS = 64;  // channels of a CTA
 constexpr int GR_STEP = GR_WARPS * GR_RUN;
+constexpr int GR_CLUSTER = 8;
 
 struct GrScanParams {
   kvb_gated_recurrence g;
@@ -70,12 +75,26 @@ struct GrScanParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(GR_WARPS * 32)
+struct alignas(2 * sizeof(T)) GrPair {
+  T v[2];
+};
+
+// what tokens make of the states of two channels: s -> decay · s + sum
+struct GrMade {
+  float2 decay, sum;
+};
+__device__ __forceinline__ float2 gr_apply(const GrMade& m, float2 s) { return ffma2(m.decay, s, m.sum); }
+__device__ __forceinline__ GrMade gr_then(const GrMade& a, const GrMade& b) { return {fmul2(a.decay, b.decay), ffma2(b.decay, a.sum, b.sum)}; }
+
+template <typename T>
+__global__ void __launch_bounds__(GR_WARPS * 32, 2)
 gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T* __restrict__ out, const GrScanParams p) {
-  __shared__ float2 made[2][GR_WARPS][32];  // decay and addition of a warp's tokens
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.y;
-  const int channels = p.g.blocks * p.g.pp, c = blockIdx.x * 32 + lane;
-  const bool mine = c < channels;
+  __shared__ GrMade by_warp[2][GR_WARPS][32], by_cta[2][GR_CLUSTER][32];
+  cooperative_groups::cluster_group cluster = cooperative_groups::this_cluster();
+  const int rank = (int)cluster.block_rank(), ranks = (int)cluster.num_blocks();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.z;
+  const int channels = p.g.blocks * p.g.pp, c = blockIdx.y * GR_COLS + 2 * lane;
+  const bool mine = c < channels;  // parts are multiples of 8: both channels are of one
   const int cc = mine ? c : 0, part = cc / p.g.pp, j = cc - part * p.g.pp;
   const int n = p.count[b];
   const long long row0 = (long long)b * p.T;
@@ -83,63 +102,103 @@ gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T
   x += row0 * channels + cc;
   y += row0 * p.ldy + cc;
   out += row0 * p.ldo + cc;
-  const float rate = p.g.rate[cc], br = p.g.bias_r[cc], bi = p.g.bias_i[cc];
-  float* own = p.state + (long long)p.slots[b] * channels + cc;
-  float carry = mine && p.start[b] > 0 ? *own : 0.f;
+  const float2 rate = *reinterpret_cast<const float2*>(p.g.rate + cc), br = *reinterpret_cast<const float2*>(p.g.bias_r + cc),
+               bi = *reinterpret_cast<const float2*>(p.g.bias_i + cc);
+  float2* own = reinterpret_cast<float2*>(p.state + (long long)p.slots[b] * channels + cc);
+  float2 carry = mine && p.start[b] > 0 ? *own : make_float2(0.f, 0.f);
+  const GrMade nothing = {make_float2(1.f, 1.f), make_float2(0.f, 0.f)};
   int turn = 0;
-  for (int t0 = 0; t0 < n; t0 += GR_STEP, turn ^= 1) {
-    const int t1 = t0 + warp * GR_RUN;
-    float a[GR_RUN], add[GR_RUN];
-    T xv[GR_RUN], yv[GR_RUN];
+  for (int t0 = 0; t0 < n; t0 += ranks * GR_STEP, turn ^= 1) {
+    const int t1 = t0 + rank * GR_STEP + warp * GR_RUN;
+    float2 a[GR_RUN], add[GR_RUN];
+    GrPair<T> xv[GR_RUN], yv[GR_RUN];
 #pragma unroll
     for (int i = 0; i < GR_RUN; ++i) {
       const int t = t1 + i;
-      a[i] = add[i] = 0.f;
-      xv[i] = yv[i] = from_f32<T>(0.f);
+      a[i] = add[i] = make_float2(0.f, 0.f);
+      xv[i].v[0] = xv[i].v[1] = yv[i].v[0] = yv[i].v[1] = from_f32<T>(0.f);
       if (mine && t < n) {
-        a[i] = __ldcs(z + (long long)t * 2 * p.g.pp);
-        add[i] = __ldcs(z + (long long)t * 2 * p.g.pp + p.g.pp);
-        xv[i] = x[(long long)t * channels];
-        yv[i] = y[(long long)t * p.ldy];
+        a[i] = __ldcs(reinterpret_cast<const float2*>(z + (long long)t * 2 * p.g.pp));
+        add[i] = __ldcs(reinterpret_cast<const float2*>(z + (long long)t * 2 * p.g.pp + p.g.pp));
+        xv[i] = *reinterpret_cast<const GrPair<T>*>(x + (long long)t * channels);
+        yv[i] = *reinterpret_cast<const GrPair<T>*>(y + (long long)t * p.ldy);
       }
     }
-    float decay = 1.f, sum = 0.f;
+    GrMade own_tokens = nothing;
 #pragma unroll
     for (int i = 0; i < GR_RUN; ++i) {
       if (t1 + i < n) {
-        gr_token<T>(a[i] + br, add[i] + bi, to_f32(xv[i]), rate, a[i], add[i]);
+        gr_token<T>(a[i].x + br.x, add[i].x + bi.x, to_f32(xv[i].v[0]), rate.x, a[i].x, add[i].x);
+        gr_token<T>(a[i].y + br.y, add[i].y + bi.y, to_f32(xv[i].v[1]), rate.y, a[i].y, add[i].y);
       } else {  // changes nothing
-        a[i] = 1.f;
-        add[i] = 0.f;
+        a[i] = make_float2(1.f, 1.f);
+        add[i] = make_float2(0.f, 0.f);
       }
-      decay *= a[i];
-      sum = fmaf(a[i], sum, add[i]);
+      own_tokens = gr_then(own_tokens, {a[i], add[i]});
     }
-    made[turn][warp][lane] = make_float2(decay, sum);
+    by_warp[turn][warp][lane] = own_tokens;
     __syncthreads();
-    float s = carry;
+    GrMade before = nothing, all = nothing;
 #pragma unroll
     for (int w = 0; w < GR_WARPS; ++w) {
-      const float2 m = made[turn][w][lane];
-      if (w == warp) s = carry;
-      carry = fmaf(m.x, carry, m.y);
+      if (w == warp) before = all;
+      all = gr_then(all, by_warp[turn][w][lane]);
     }
+    if (ranks > 1) {  // every CTA of the cluster gets what the others' tokens make of a state
+      if (warp < ranks) cluster.map_shared_rank(&by_cta[turn][rank][lane], warp)[0] = all;
+      cluster.sync();
+      float2 s = carry;
+      for (int r = 0; r < ranks; ++r) {
+        if (r == rank) s = carry;
+        carry = gr_apply(by_cta[turn][r][lane], carry);
+      }
+      before = {before.decay, gr_apply(before, s)};
+    } else {
+      before.sum = gr_apply(before, carry);
+      carry = gr_apply(all, carry);
+    }
+    float2 s = before.sum;
 #pragma unroll
     for (int i = 0; i < GR_RUN; ++i) {
-      s = fmaf(a[i], s, add[i]);
-      if (mine && t1 + i < n) out[(long long)(t1 + i) * p.ldo] = from_f32<T>(s * gr_gelu<T>(to_f32(yv[i])) * p.g.scale);
+      s = ffma2(a[i], s, add[i]);
+      GrPair<T> o;
+      o.v[0] = from_f32<T>(s.x * gr_gelu<T>(to_f32(yv[i].v[0])) * p.g.scale);
+      o.v[1] = from_f32<T>(s.y * gr_gelu<T>(to_f32(yv[i].v[1])) * p.g.scale);
+      if (mine && t1 + i < n) *reinterpret_cast<GrPair<T>*>(out + (long long)(t1 + i) * p.ldo) = o;
     }
   }
+  if (ranks > 1) cluster.sync();  // nobody writes into the memory of a CTA that has gone
   if (!mine) return;
-  for (int t = n + warp; t < p.T; t += GR_WARPS) out[(long long)t * p.ldo] = from_f32<T>(0.f);
-  if (warp == 0 && n > 0) *own = carry;
+  GrPair<T> zero;
+  zero.v[0] = zero.v[1] = from_f32<T>(0.f);
+  for (int t = n + rank * GR_WARPS + warp; t < p.T; t += ranks * GR_WARPS) *reinterpret_cast<GrPair<T>*>(out + (long long)t * p.ldo) = zero;
+  if (rank == 0 && warp == 0 && n > 0) *own = carry;
+}
+
+template <typename T>
+static int gr_scan_launch(const void* x, const void* y, void* out, const GrScanParams& p, cudaStream_t s) {
+  const int tiles = (p.g.blocks * p.g.pp + GR_COLS - 1) / GR_COLS, steps = (p.T + GR_STEP - 1) / GR_STEP;
+  int ranks = 1;
+  while (ranks < GR_CLUSTER && ranks < steps) ranks *= 2;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(ranks, tiles, p.B);
+  cfg.blockDim = dim3(GR_WARPS * 32);
+  cfg.stream = s;
+  cudaLaunchAttribute attr;
+  attr.id = cudaLaunchAttributeClusterDimension;
+  attr.val.clusterDim.x = ranks;
+  attr.val.clusterDim.y = attr.val.clusterDim.z = 1;
+  cfg.attrs = &attr;
+  cfg.numAttrs = 1;
+  return cudaLaunchKernelEx(&cfg, gated_recurrence_scan_kernel<T>, (const T*)x, (const T*)y, (T*)out, p) == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 
 // ------------------------------------------------------------------------------------------------ step
-constexpr int GQ_ROWS = 8;    // sequences of a CTA
+constexpr int GQ_ROWS = 8;    // sequences of a CTA, one per warp for the convolution
 constexpr int GQ_COLS = 32;   // channels of a CTA, all of one part
-constexpr int GQ_SPLIT = 4;   // threads that share a product
-constexpr int GQ_THREADS = 2 * GQ_COLS * GQ_SPLIT;
+constexpr int GQ_SPLIT = 8;   // threads that share a product of two neighbouring channels
+constexpr int GQ_THREADS = GQ_COLS * GQ_SPLIT;
+constexpr int GQ_AHEAD = 16;  // weights of a thread that are on their way during the convolution
 
 struct GrStepParams {
   kvb_gated_recurrence g;
@@ -155,71 +214,85 @@ gated_recurrence_step_kernel(const T* __restrict__ u, T* __restrict__ ring, T* _
   extern __shared__ float gq_x[];  // (pp, GQ_ROWS): inputs behind the convolution
   __shared__ float zs[GQ_SPLIT][GQ_ROWS][2 * GQ_COLS];
   const int part = blockIdx.x / p.tiles, j0 = (blockIdx.x - part * p.tiles) * GQ_COLS, b0 = blockIdx.y * GQ_ROWS;
-  const int pp = p.g.pp, channels = p.g.blocks * pp, taps = p.g.taps, tid = threadIdx.x;
+  const int pp = p.g.pp, channels = p.g.blocks * pp, taps = p.g.taps, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rows = min(GQ_ROWS, p.B - b0);
-  for (int i = tid; i < pp * GQ_ROWS; i += GQ_THREADS) {
-    const int r = i / pp, k = i - r * pp, c = part * pp + k;
-    float v = 0.f;
-    if (r < rows) {
-      const int b = b0 + r, pos = p.start[b];
-      T* past = ring + (long long)p.slots[b] * taps * channels + c;
-      const T now = u[b * p.ld + channels + c];
-      v = fmaf(p.g.conv[(long long)(taps - 1) * channels + c], to_f32(now), p.g.conv_bias[c]);
-      for (int q = 1; q < taps; ++q)
-        if (pos - q >= 0) v = fmaf(p.g.conv[(long long)(taps - 1 - q) * channels + c], to_f32(past[(long long)((pos - q) % taps) * channels]), v);
-      v = to_f32(from_f32<T>(v));  // as the product of several tokens reads it
-      if (k >= j0 && k < j0 + GQ_COLS && p.count[b] > 0) past[(long long)(pos % taps) * channels] = now;
+  // thread (pair, split): two neighbouring columns of the decay gates (pairs below 16) or input gates, every GQ_SPLIT-th input
+  const int pair = tid % GQ_COLS, split = tid / GQ_COLS, col = 2 * (pair % (GQ_COLS / 2)), j = j0 + col;
+  const T* w = static_cast<const T*>(p.g.gates) + (long long)part * pp * 2 * pp + (pair < GQ_COLS / 2 ? 0 : pp) + j;
+  GrPair<T> ahead[GQ_AHEAD];
+  auto fetch = [&](int k0) {
+#pragma unroll
+    for (int i = 0; i < GQ_AHEAD; ++i) {
+      const int k = k0 + i * GQ_SPLIT;
+      if (j < pp && k < pp) ahead[i] = *reinterpret_cast<const GrPair<T>*>(w + (long long)k * 2 * pp);
+      else ahead[i].v[0] = ahead[i].v[1] = from_f32<T>(0.f);
     }
-    gq_x[k * GQ_ROWS + r] = v;
+  };
+  fetch(split);
+  {
+    const bool in = warp < rows;
+    const int b = b0 + (in ? warp : 0), pos = p.start[b];
+    const bool write = in && p.count[b] > 0;
+    T* past = ring + (long long)p.slots[b] * taps * channels + part * pp;
+    const T* now = u + b * p.ld + channels + part * pp;
+    const float* cw = p.g.conv + part * pp;
+#pragma unroll 4
+    for (int k = lane; k < pp; k += 32) {
+      float v = 0.f;
+      if (in) {
+        const T x = now[k];
+        v = fmaf(cw[(long long)(taps - 1) * channels + k], to_f32(x), p.g.conv_bias[part * pp + k]);
+#pragma unroll 4
+        for (int q = 1; q < taps; ++q)
+          if (pos - q >= 0) v = fmaf(cw[(long long)(taps - 1 - q) * channels + k], to_f32(past[(long long)((pos - q) % taps) * channels + k]), v);
+        v = to_f32(from_f32<T>(v));  // as the product of several tokens reads it
+        if (write && k >= j0 && k < j0 + GQ_COLS) past[(long long)(pos % taps) * channels + k] = x;
+      }
+      gq_x[k * GQ_ROWS + warp] = v;
+    }
   }
   __syncthreads();
   {
-    const int col = tid % (2 * GQ_COLS), split = tid / (2 * GQ_COLS);
-    const int j = j0 + col % GQ_COLS;
-    float acc[GQ_ROWS];
+    float2 acc[GQ_ROWS];
 #pragma unroll
-    for (int r = 0; r < GQ_ROWS; ++r) acc[r] = 0.f;
-    if (j < pp) {
-      const T* w = static_cast<const T*>(p.g.gates) + (long long)part * pp * 2 * pp + (col < GQ_COLS ? 0 : pp) + j;
-#pragma unroll 8
-      for (int k = split; k < pp; k += GQ_SPLIT) {
-        const float f = to_f32(w[(long long)k * 2 * pp]);
+    for (int r = 0; r < GQ_ROWS; ++r) acc[r] = make_float2(0.f, 0.f);
+    for (int k0 = split; k0 < pp;) {
+#pragma unroll
+      for (int i = 0; i < GQ_AHEAD; ++i) {
+        const int k = k0 + i * GQ_SPLIT;
+        if (k >= pp) break;
+        const float2 f = make_float2(to_f32(ahead[i].v[0]), to_f32(ahead[i].v[1]));
         const float4 lo = *reinterpret_cast<const float4*>(gq_x + k * GQ_ROWS), hi = *reinterpret_cast<const float4*>(gq_x + k * GQ_ROWS + 4);
-        acc[0] = fmaf(f, lo.x, acc[0]);
-        acc[1] = fmaf(f, lo.y, acc[1]);
-        acc[2] = fmaf(f, lo.z, acc[2]);
-        acc[3] = fmaf(f, lo.w, acc[3]);
-        acc[4] = fmaf(f, hi.x, acc[4]);
-        acc[5] = fmaf(f, hi.y, acc[5]);
-        acc[6] = fmaf(f, hi.z, acc[6]);
-        acc[7] = fmaf(f, hi.w, acc[7]);
+        const float v[GQ_ROWS] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+#pragma unroll
+        for (int r = 0; r < GQ_ROWS; ++r) acc[r] = ffma2(f, make_float2(v[r], v[r]), acc[r]);
       }
+      k0 += GQ_AHEAD * GQ_SPLIT;
+      if (k0 < pp) fetch(k0);
     }
 #pragma unroll
-    for (int r = 0; r < GQ_ROWS; ++r) zs[split][r][col] = acc[r];
+    for (int r = 0; r < GQ_ROWS; ++r) *reinterpret_cast<float2*>(&zs[split][r][(pair < GQ_COLS / 2 ? 0 : GQ_COLS) + col]) = acc[r];
   }
   __syncthreads();
-  for (int i = tid; i < GQ_ROWS * GQ_COLS; i += GQ_THREADS) {
-    const int r = i / GQ_COLS, j = j0 + i % GQ_COLS, c = part * pp + j;
-    if (r >= rows || j >= pp) continue;
-    const int b = b0 + r;
-    T* dst = out + b * p.ldo + c;
-    if (p.count[b] <= 0) {
-      *dst = from_f32<T>(0.f);
-      continue;
-    }
-    float zr = p.g.bias_r[c], zi = p.g.bias_i[c], a, add;
-#pragma unroll
-    for (int s = 0; s < GQ_SPLIT; ++s) {
-      zr += zs[s][r][i % GQ_COLS];
-      zi += zs[s][r][GQ_COLS + i % GQ_COLS];
-    }
-    gr_token<float>(zr, zi, gq_x[j * GQ_ROWS + r], p.g.rate[c], a, add);
-    float* own = p.state + (long long)p.slots[b] * channels + c;
-    const float s = fmaf(a, p.start[b] > 0 ? *own : 0.f, add);
-    *own = s;
-    *dst = from_f32<T>(s * gr_gelu<float>(to_f32(u[b * p.ld + c])) * p.g.scale);
+  const int jj = j0 + lane, c = part * pp + jj;  // a warp finishes a sequence
+  if (warp >= rows || jj >= pp) return;
+  const int b = b0 + warp;
+  T* dst = out + b * p.ldo + c;
+  if (p.count[b] <= 0) {
+    *dst = from_f32<T>(0.f);
+    return;
   }
+  float zr = p.g.bias_r[c], zi = p.g.bias_i[c], a, add;
+#pragma unroll
+  for (int s = 0; s < GQ_SPLIT; ++s) {
+    zr += zs[s][warp][lane];
+    zi += zs[s][warp][GQ_COLS + lane];
+  }
+  gr_token<float>(zr, zi, gq_x[jj * GQ_ROWS + warp], p.g.rate[c], a, add);
+  float* own = p.state + (long long)p.slots[b] * channels + c;
+  const float s = fmaf(a, p.start[b] > 0 ? *own : 0.f, add);
+  *own = s;
+  *dst = from_f32<T>(s * gr_gelu<float>(to_f32(u[b * p.ld + c])) * p.g.scale);
 }
 
 static bool gated_recurrence_valid(const kvb_gated_recurrence* g) {
@@ -242,10 +315,10 @@ extern "C" int kvb_gated_recurrence_scan(const kvb_gated_recurrence* g, const vo
     return KVB_ERR_ARG;
   kvb::GrScanParams p;
   p.g = *g; p.slots = slots; p.start = start; p.count = count; p.z = z; p.state = state; p.ldy = ldy; p.ldo = ldo; p.B = B; p.T = T_;
-  const dim3 grid((g->blocks * g->pp + 31) / 32, B);
-  KVB_RECURRENCE_TYPES(dtype, (kvb::gated_recurrence_scan_kernel<T><<<grid, kvb::GR_WARPS * 32, 0, (cudaStream_t)stream>>>(
-      (const T*)x, (const T*)y, (T*)out, p)));
-  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+  if (g->pp % 8 || ldy % 2 || ldo % 2 || (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(y) |
+                                          reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(state)) & 7)
+    return KVB_ERR_ALIGN;
+  KVB_RECURRENCE_TYPES(dtype, return kvb::gr_scan_launch<T>(x, y, out, p, (cudaStream_t)stream));
 }
 
 extern "C" int kvb_gated_recurrence_step(const kvb_gated_recurrence* g, const void* u, long long ld, void* ring, float* state, void* out,
@@ -254,6 +327,7 @@ extern "C" int kvb_gated_recurrence_step(const kvb_gated_recurrence* g, const vo
   if (!gated_recurrence_valid(g) || !g->gates || B <= 0 || ld < 2LL * g->blocks * g->pp || ldo < (long long)g->blocks * g->pp) return KVB_ERR_ARG;
   const size_t smem = (size_t)g->pp * GQ_ROWS * sizeof(float);
   if (smem > 200 * 1024 || B > 65535 * GQ_ROWS) return KVB_ERR_TOO_LARGE;
+  if (g->pp % 8 || (reinterpret_cast<uintptr_t>(g->gates) & 7)) return KVB_ERR_ALIGN;
   GrStepParams p;
   p.g = *g; p.slots = slots; p.start = start; p.count = count; p.state = state; p.ld = ld; p.ldo = ldo; p.B = B;
   p.tiles = (g->pp + GQ_COLS - 1) / GQ_COLS;

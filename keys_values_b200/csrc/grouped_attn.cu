@@ -37,36 +37,70 @@ struct GpParams {
   unsigned rot_magic, rest_magic;
 };
 
-// Columns [c, c + V) of the mean of the rows of block `block` of a sequence; slot: its first row.
+// Columns [c, c + V) of the sum of the rows first .. last - 1 of block `block` of a sequence; slot: its first row.
 template <typename T, int V>
-__device__ __forceinline__ void pool_columns(T* slot, const kvb_attention& a, long long step, int block, int c) {
+__device__ __forceinline__ void pool_columns(const T* slot, const kvb_attention& a, long long step, int block, int c, int first, int last, float (&s)[V]) {
   using Vec = GpVec<T, V>;
-  float s[V];
 #pragma unroll
   for (int e = 0; e < V; ++e) s[e] = 0.f;
-#pragma unroll 8
-  for (int j = 0; j < a.pool; ++j) {
-    const Vec v = *reinterpret_cast<const Vec*>(slot + row_of(a, block * a.pool + j) * step + c);
+  const int place = row_of(a, block * a.pool);  // a block's rows lie one behind the other up to the end of the ring
+  auto add = [&](const T* rows, int j0, int j1) {
+#pragma unroll 16
+    for (int j = j0; j < j1; ++j) {
+      const Vec v = *reinterpret_cast<const Vec*>(rows + (long long)j * step);
 #pragma unroll
-    for (int e = 0; e < V; ++e) s[e] += to_f32(v.v[e]);
+      for (int e = 0; e < V; ++e) s[e] += to_f32(v.v[e]);
+    }
+  };
+  for (int j0 = 0, at = place; j0 < a.pool; at = a.head) {
+    const int n = min(a.pool - j0, a.head + a.ring - at), mid = j0;
+    const int lo = max(first, mid), hi = min(last, mid + n);
+    if (lo < hi) add(slot + (at - mid) * step + c, lo, hi);
+    j0 += n;
   }
-  const float inv = 1.f / (float)a.pool;
-  Vec r;
-#pragma unroll
-  for (int e = 0; e < V; ++e) r.v[e] = from_f32<T>(s[e] * inv);
-  *reinterpret_cast<Vec*>(slot + block * step + c) = r;
 }
 
 template <typename T, int V>
-__global__ void __launch_bounds__(GP_THREADS)
+__device__ __forceinline__ void pool_store(T* slot, const kvb_attention& a, long long step, int block, int c, const float (&s)[V]) {
+  const float inv = 1.f / (float)a.pool;
+  GpVec<T, V> r;
+#pragma unroll
+  for (int e = 0; e < V; ++e) r.v[e] = from_f32<T>(s[e] * inv);
+  *reinterpret_cast<GpVec<T, V>*>(slot + block * step + c) = r;
+}
+
+// A CTA has a block, a thread V columns of some of its rows.
+constexpr int PL_SHARES = 4;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(GP_THREADS * PL_SHARES)
 grouped_pool_kernel(T* __restrict__ rows, const GpParams p) {
+  __shared__ float part[PL_SHARES - 1][GP_THREADS][V + 1];
   const int b = blockIdx.y, block = p.start[b] / p.a.pool + blockIdx.x;
   // complete with this pass, and with a row of its own
   if ((block + 1) * p.a.pool > p.start[b] + p.count[b] || block >= p.a.head) return;
   const int row = p.a.maps * p.a.dimp + p.a.vdp;
   const long long step = (long long)p.a.kv_heads * row;
   T* slot = rows + (long long)p.slots[b] * p.len * step;
-  for (int c = threadIdx.x * V; c < step; c += GP_THREADS * V) pool_columns<T, V>(slot, p.a, step, block, c);
+  const int lane = threadIdx.x % GP_THREADS, share = threadIdx.x / GP_THREADS, per = (p.a.pool + PL_SHARES - 1) / PL_SHARES;
+  for (int c0 = 0; c0 < step; c0 += GP_THREADS * V) {
+    const int c = c0 + lane * V;
+    float s[V];
+    if (c < step) pool_columns<T, V>(slot, p.a, step, block, c, share * per, min(p.a.pool, (share + 1) * per), s);
+    if (share > 0 && c < step) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) part[share - 1][lane][e] = s[e];
+    }
+    __syncthreads();
+    if (share == 0 && c < step) {
+#pragma unroll
+      for (int k = 0; k < PL_SHARES - 1; ++k)
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] += part[k][lane][e];
+      pool_store<T, V>(slot, p.a, step, block, c, s);
+    }
+    __syncthreads();
+  }
 }
 
 template <typename T, int V>
@@ -92,7 +126,11 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
     __syncthreads();
     const long long step = (long long)p.a.kv_heads * row;
     T* slot = rows + (long long)p.slots[b] * p.len * step;
-    for (int c = threadIdx.x * V; c < step; c += GP_THREADS * V) pool_columns<T, V>(slot, p.a, step, pos / size, c);
+    for (int c = threadIdx.x * V; c < step; c += GP_THREADS * V) {
+      float s[V];
+      pool_columns<T, V>(slot, p.a, step, pos / size, c, 0, size, s);
+      pool_store<T, V>(slot, p.a, step, pos / size, c, s);
+    }
   };
   // one piece of a head: the key part of the cache or the query
   auto put = [&](int h, int col, const Vec& v) {
@@ -233,7 +271,7 @@ static int gp_launch_vec(const void* qkv, void* q, void* rows, GpParams& p, int 
   const size_t smem = (size_t)(p.rot_dims + (p.a.head_norm ? p.heads + p.kv_heads : 0)) * sizeof(float) + 8;
   if (smem > 48 * 1024) return KVB_ERR_TOO_LARGE;
   grouped_prep_kernel<T, V><<<dim3(p.T, B), GP_THREADS, smem, s>>>((const T*)qkv, (T*)q, (T*)rows, p);
-  if (p.a.pool > 0 && p.T > 1) grouped_pool_kernel<T, 16 / sizeof(T)><<<dim3(p.T / p.a.pool + 1, B), GP_THREADS, 0, s>>>((T*)rows, p);
+  if (p.a.pool > 0 && p.T > 1) grouped_pool_kernel<T, 16 / sizeof(T)><<<dim3(p.T / p.a.pool + 1, B), GP_THREADS * PL_SHARES, 0, s>>>((T*)rows, p);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
 }
 

@@ -6,8 +6,9 @@
 // A CTA has one row, which stays in registers; means and squared deviations are separate sums (no cancellation).
 //
 // What a sublayer reads may pass a short causal convolution over time first. A single token finds the inputs before it in a ring of its
-// sequence. Of several tokens a CTA takes a run, some rows at a time, one per team of warps: the inputs of the rows stay in shared memory for
-// their successors, those of the tokens right before the run are worked out once more.
+// sequence. Of several tokens a CTA takes a run, one after the other, and keeps the inputs of the last ones in registers; those of the tokens
+// right before the run are worked out once more. (Convolutions of more than eight taps and wide rows keep them in shared memory, some rows at a
+// time, one per team of warps.)
 #include <type_traits>
 
 #include "common.cuh"
@@ -237,6 +238,172 @@ norm_edge_kernel(const NormEdgeParams p) {
 }
 
 // ------------------------------------------------------------------------- several tokens with a convolution
+// TAPS: taps that are kept in registers; a shorter convolution has zeros in front
+template <typename T, int V, int TH, int NC, int TAPS, bool CENTER>
+__global__ void __launch_bounds__(TH, TH == 128 ? 6 : TH == 256 ? 3 : 1)
+conv_run_kernel(const NormEdgeParams p) {
+  __shared__ float red[2][4][TH / 32];  // sums of a token, two tokens in turn
+  const int T_ = p.tok.T, taps = p.tok.taps, b = blockIdx.y, t0 = blockIdx.x * p.run, t1 = min(t0 + p.run, T_);
+  const int start = p.tok.start[b], count = p.tok.count[b], col = threadIdx.x * V;
+  constexpr int STRIDE = TH * V;
+  float* const ring = p.tok.conv_ring + (long long)p.tok.slots[b] * taps * p.width + col;
+  const long long row0 = (long long)b * T_;
+  float x[NC][V], y[NC][V], past[TAPS > 1 ? TAPS - 1 : 1][NC][V];  // past[k]: h of the token TAPS - 1 - k before
+  auto fetch = [&](int t) {  // what row t of the pass is made of, on its way
+    const long long o = (row0 + t) * p.width + col;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[i][e] = y[i][e] = 0.f;
+      if (col + i * STRIDE >= p.width) continue;
+      if (p.sub) RowVec<T, V>::load(static_cast<const T*>(p.sub) + o + i * STRIDE, y[i]);
+      if (p.x_in) RowVec<float, V>::load(p.x_in + o + i * STRIDE, x[i]);
+    }
+  };
+  // the row of the stream (stored if `out`) in x, then its h
+  auto work = [&](int t, bool out, float (&h)[NC][V], int next) {
+    float (*r2)[TH / 32] = red[t & 1];
+    const long long n = row0 + t, o = n * p.width + col;
+    long long tok = 0;
+    if (p.embed) {
+      tok = p.idx[n];
+      if (tok < 0 || tok >= p.vocab) {
+        if (p.status) atomicCAS(p.status, 0, STATUS_BAD_INDEX);
+        tok = 0;
+      }
+    }
+    const float r = p.after ? row_norm_factor<TH, NC, V, CENTER>(y, p, r2) : 1.f;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = col + i * STRIDE;
+      if (c >= p.width) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] = 0.f;
+        continue;
+      }
+      float w[V];
+      if (p.after) {
+        RowVec<float, V>::load(p.after + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] = fmaf(y[i][e] * r, w[e], x[i][e]);
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] = x[i][e] + y[i][e];
+      }
+      if (p.embed) {
+        RowVec<T, V>::load(static_cast<const T*>(p.embed) + tok * p.width + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] += w[e];
+      }
+      if (p.tok.table) {
+        RowVec<T, V>::load(static_cast<const T*>(p.tok.table) + table_row(p, n) * p.width + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] += w[e];
+      }
+      if (p.step) {
+        RowVec<float, V>::load(p.step + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] += w[e];
+      }
+      if (out && p.x_out) RowVec<float, V>::store(p.x_out + o + i * STRIDE, h[i]);
+    }
+    if (next >= 0) fetch(next);
+    if (!p.before) return;
+    const float f = row_norm_factor<TH, NC, V, CENTER>(h, p, r2 + 2);
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      if (col + i * STRIDE >= p.width) continue;
+      float w[V];
+      RowVec<float, V>::load(p.before + col + i * STRIDE, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) h[i][e] *= f * w[e];
+    }
+  };
+  const int first = t0 - taps + 1;
+  float h[NC][V];
+  fetch(max(first, 0));
+  for (int t = first; t < t1; ++t) {
+    if (t >= 0) {
+      work(t, t >= t0, h, t + 1 < t1 ? t + 1 : -1);
+    } else {  // before the pass, perhaps before the sequence
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+#pragma unroll
+        for (int e = 0; e < V; ++e) h[i][e] = 0.f;
+        if (start + t >= 0 && col + i * STRIDE < p.width) RowVec<float, V>::load(ring + (long long)((start + t) % taps) * p.width + i * STRIDE, h[i]);
+      }
+    }
+    if (t >= t0) {
+#pragma unroll
+      for (int i = 0; i < NC; ++i) {
+        const int c = col + i * STRIDE;
+        if (c >= p.width) continue;
+        float s[V], w[V];
+        RowVec<float, V>::load(p.tok.conv_w + (long long)(taps - 1) * p.width + c, w);
+#pragma unroll
+        for (int e = 0; e < V; ++e) s[e] = fmaf(w[e], h[i][e], h[i][e]);
+#pragma unroll
+        for (int k = TAPS - 2; k >= 0; --k) {
+          const int at = k - (TAPS - taps);
+          if (at < 0) break;
+          RowVec<float, V>::load(p.tok.conv_w + (long long)at * p.width + c, w);
+#pragma unroll
+          for (int e = 0; e < V; ++e) s[e] = fmaf(w[e], past[k][i][e], s[e]);
+        }
+        RowVec<T, V>::store(static_cast<T*>(p.h) + (row0 + t) * p.width + c, s);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NC; ++i)
+#pragma unroll
+      for (int e = 0; e < V; ++e) {
+#pragma unroll
+        for (int k = 0; k + 2 < TAPS; ++k) past[k][i][e] = past[k + 1][i][e];
+        if (TAPS > 1) past[TAPS - 2][i][e] = h[i][e];
+      }
+  }
+  // the ring takes the last ones of the sequence. Only the CTA of the first tokens has read it, so it alone may write there
+  if (t0 > 0) return;
+  for (int t = max(0, count - taps); t < count; ++t) {
+    fetch(t);
+    __syncthreads();  // sums of the tokens before have been read
+    work(t, false, h, -1);
+#pragma unroll
+    for (int i = 0; i < NC; ++i)
+      if (col + i * STRIDE < p.width) RowVec<float, V>::store(ring + (long long)((start + t) % taps) * p.width + i * STRIDE, h[i]);
+  }
+}
+
+template <typename T, int V, int TH, int NC, bool CENTER>
+static int conv_run_launch(NormEdgeParams& p, int B, cudaStream_t s) {
+  // a wave of CTAs, but no runs so short that most of the work is done twice
+  const int per_sm = TH == 128 ? 6 : TH == 256 ? 3 : 1;
+  long long runs = (148LL * per_sm) / B;
+  const long long most = (p.tok.T + 15) / 16;
+  if (runs > most) runs = most;
+  if (runs < 1) runs = 1;
+  p.run = (int)((p.tok.T + runs - 1) / runs);
+  if (p.run > 64) p.run = 64;  // many waves: even ends
+  if (p.run < p.tok.taps) p.run = p.tok.taps;
+  const dim3 grid((p.tok.T + p.run - 1) / p.run, B);
+  if (p.tok.taps <= 4) conv_run_kernel<T, V, TH, NC, 4, CENTER><<<grid, TH, 0, s>>>(p);
+  else conv_run_kernel<T, V, TH, NC, 8, CENTER><<<grid, TH, 0, s>>>(p);
+  return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+template <typename T, bool CENTER>
+static int conv_run_type(NormEdgeParams& p, int B, cudaStream_t s) {
+  if (p.width % 4) {
+    if (p.width <= 1024) return conv_run_launch<T, 1, 256, 4, CENTER>(p, B, s);
+    return KVB_ERR_TOO_LARGE;
+  }
+  if (p.width <= 512) return conv_run_launch<T, 4, 128, 1, CENTER>(p, B, s);
+  if (p.width <= 1024) return conv_run_launch<T, 4, 256, 1, CENTER>(p, B, s);
+  if (p.width <= 2048) return conv_run_launch<T, 4, 256, 2, CENTER>(p, B, s);
+  if (p.width <= 4096) return conv_run_launch<T, 4, 512, 2, CENTER>(p, B, s);
+  return KVB_ERR_TOO_LARGE;
+}
+
 constexpr int CE_WARPS = 8;
 
 // sums over the lanes of a team of `tw` warps (every warp of the CTA calls)
@@ -497,6 +664,13 @@ extern "C" int kvb_norm_edge(const float* x_in, const void* sub, const void* exp
   p.tok = tokens ? *tokens : kvb_edge_tokens{};
   p.run = 0;
   if (tokens && tokens->conv_w && tokens->T > 1) {
+    if (tokens->taps <= 8 && width <= (width % 4 ? 1024 : 4096)) {
+      const int B = (int)(n / tokens->T);
+      cudaStream_t s = (cudaStream_t)stream;
+      if (dtype == 0) return center ? kvb::conv_run_type<float, true>(p, B, s) : kvb::conv_run_type<float, false>(p, B, s);
+      if (dtype == 1) return center ? kvb::conv_run_type<__nv_bfloat16, true>(p, B, s) : kvb::conv_run_type<__nv_bfloat16, false>(p, B, s);
+      return KVB_ERR_ARG;
+    }
     if (dtype == 0) return kvb::conv_edge_type<float>(p, n, center, (cudaStream_t)stream);
     if (dtype == 1) return kvb::conv_edge_type<__nv_bfloat16>(p, n, center, (cudaStream_t)stream);
     return KVB_ERR_ARG;

@@ -23,7 +23,7 @@ struct alignas(sizeof(T) * V) SsVec {
 
 // ------------------------------------------------------------------------------------------------ conv
 constexpr int SC_THREADS = 128;
-constexpr int SC_RUN = 16;  // tokens of a thread
+constexpr int SC_RUN = 32;  // tokens of a thread
 
 struct ConvParams {
   const float *w, *bias;  // (taps, channels), (channels)
@@ -122,8 +122,8 @@ template <typename T>
 static int conv_launch(const void* u, void* out, void* ring, ConvParams& p, int B, cudaStream_t s) {
   constexpr int V = 16 / sizeof(T);
   const int blocks = (p.channels / V + SC_THREADS - 1) / SC_THREADS;
-  long long run = (long long)p.T * B * blocks / (148 * 8);  // enough CTAs first, then few inputs read twice
-  p.run = (int)(run < 4 ? 4 : (run > SC_RUN ? SC_RUN : run / 4 * 4));
+  long long run = ((long long)p.T * B * blocks + 148 * 4 - 1) / (148 * 4);  // a wave of CTAs first, then few inputs read twice
+  p.run = (int)(run < 4 ? 4 : (run > SC_RUN ? SC_RUN : (run + 3) / 4 * 4));
   if (p.run < p.taps) p.run = p.taps;  // only the first run of a channel may look back beyond the pass
   const dim3 grid(blocks, (p.T + p.run - 1) / p.run, B);
   if (p.taps == 4) short_conv_kernel<T, V, 4><<<grid, SC_THREADS, 0, s>>>((const T*)u, (T*)out, (T*)ring, p);

@@ -29,6 +29,7 @@ __device__ __forceinline__ float ss_decay(float x) { return 1.f + expm1f(x); }
 // logarithm of the decay of key channel c of a gated linear attention, from the token's low-rank input a
 __device__ __forceinline__ float gl_log_decay(const kvb_gated_linear& g, const float* a, int c) {
   float z = g.bias[c];
+#pragma unroll 8
   for (int r = 0; r < g.rank; ++r) z = fmaf(a[r], g.w[(long long)r * g.heads * g.np + c], z);
   return -ss_softplus(-z) * g.inv_tau;
 }

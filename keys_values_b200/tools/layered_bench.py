@@ -688,7 +688,7 @@ def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) ->
             tab.add(f"{tag}:   like: QK norm, split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, 2 * m.qk // 128 - 16, 8, 128, eps, 128, False),
                     gbytes=8 * n * m.qk / 1e9)
             flop = n * m.heads * (4 * m.np * m.vdp + 128 * (m.np + m.vdp)) / 1e12
-            tab.add(f"{tag}: gated linear scan (all kernels), {m.heads} heads of {m.np} x {m.vdp}", lambda: LC.gated_linear_scan(qka, vg, decay, state, seq, m),
+            tab.add(f"{tag}: gated linear scan with its preparation, {m.heads} heads of {m.np} x {m.vdp}", lambda: LC.gated_linear_scan(qka, vg, decay, state, seq, m),
                     gbytes=(n * (4 * (m.qk + m.rp) + 4 * m.inner) + state_bytes) / 1e9, tflop=flop)
             q2 = rand(B, m.heads, T, 128)
             tab.add(f"{tag}:   like: attention 128 / 128, {m.heads} heads", lambda: cu.sdpa_fwd(q2, q2, q2, 0.09, 0),

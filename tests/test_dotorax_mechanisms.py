@@ -20,7 +20,8 @@ EDGE_PASSES = [(9, [9, 6]), (1, [1, 1]), (2, [2, 2]), (1, [0, 1]), (40, [40, 33]
 
 
 @variant_param
-@pytest.mark.parametrize("width,taps", [(1, 3), (7, 1), (64, 2), (250, 4), (1028, 5), (2048, 4), (3000, 9), (5120, 4), (1030, 3)])
+@pytest.mark.parametrize("width,taps", [(1, 3), (7, 1), (64, 2), (250, 4), (1028, 5), (2048, 4), (3000, 9), (5120, 4), (1030, 3), (4096, 4), (3076, 3), (4096, 8),
+                                        (1024, 4), (512, 7), (1022, 6)])
 def test_edge_with_convolution(env, width, taps):
     """Residual sum of a normed result, norm, convolution, pass by pass: single tokens, runs that end anywhere, rows without tokens; a slot
     that is not part of the pass keeps what it holds."""
