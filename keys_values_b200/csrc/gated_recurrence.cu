@@ -58,6 +58,54 @@ __device__ __forceinline__ void gr_token(float zr, float zi, float x, float rate
   add = sqrtf(rest) * gr_sigmoid<T>(zi) * x;
 }
 
+// The same for results that are rounded to 16 bits, for two channels: few special-function results and paired multiply-adds. Gates in units of
+// log2: e = 2^-z, and both sigmoids 1 / (1 + e) come out of one reciprocal; rate2 = 2 ln 2 · rate.
+constexpr float GR_LOG2E = 1.4426950408889634f;
+__device__ __forceinline__ float gr_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float gr_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float gr_sqrt(float x) {
+  float y;
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float2 gr_both(float v) { return make_float2(v, v); }
+
+__device__ __forceinline__ void gr_token2(float2 zr, float2 zi, float2 x, float2 br, float2 bi, float2 rate, float2 rate2, float2& a, float2& add) {
+  const float2 ur = ffma2(zr, gr_both(-GR_LOG2E), br), ui = ffma2(zi, gr_both(-GR_LOG2E), bi);
+  // 2^60 and beyond: a closed gate either way, and the product stays a number
+  const float2 dr = fadd2(make_float2(gr_exp2(fminf(ur.x, 60.f)), gr_exp2(fminf(ur.y, 60.f))), gr_both(1.f));
+  const float2 di = fadd2(make_float2(gr_exp2(fminf(ui.x, 60.f)), gr_exp2(fminf(ui.y, 60.f))), gr_both(1.f));
+  const float2 d = fmul2(dr, di), inv = make_float2(gr_rcp(d.x), gr_rcp(d.y));
+  const float2 r = fmul2(di, inv), i = fmul2(dr, inv);
+  const float2 log2a = fmul2(rate, r), w = fmul2(rate2, r);  // w = 2 log a
+  a = make_float2(gr_exp2(log2a.x), gr_exp2(log2a.y));
+  // 1 - a^2 = 1 - e^w, near zero by the series
+  float2 s = ffma2(w, gr_both(1.f / 120.f), gr_both(1.f / 24.f));
+  s = ffma2(s, w, gr_both(1.f / 6.f));
+  s = ffma2(s, w, gr_both(0.5f));
+  s = ffma2(s, w, gr_both(1.f));
+  s = fmul2(s, make_float2(-w.x, -w.y));
+  const float2 na = make_float2(-a.x, -a.y), far = ffma2(na, a, gr_both(1.f));
+  const float2 rest = make_float2(w.x < -0.1f ? far.x : s.x, w.y < -0.1f ? far.y : s.y);
+  add = fmul2(fmul2(make_float2(gr_sqrt(rest.x), gr_sqrt(rest.y)), i), x);
+}
+
+// z · sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
+__device__ __forceinline__ float2 gr_gelu2(float2 z) {
+  constexpr float K = -1.5957691216057308f * GR_LOG2E;
+  const float2 u = fmul2(z, ffma2(fmul2(z, z), gr_both(0.044715f * K), gr_both(K)));
+  const float2 d = fadd2(make_float2(gr_exp2(u.x), gr_exp2(u.y)), gr_both(1.f));
+  return fmul2(z, make_float2(gr_rcp(d.x), gr_rcp(d.y)));
+}
+
 // ------------------------------------------------------------------------------------------------ scan
 constexpr int GR_WARPS = 8;
 constexpr int GR_RUN = 8;    // tokens of a warp
@@ -102,8 +150,14 @@ gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T
   x += row0 * channels + cc;
   y += row0 * p.ldy + cc;
   out += row0 * p.ldo + cc;
-  const float2 rate = *reinterpret_cast<const float2*>(p.g.rate + cc), br = *reinterpret_cast<const float2*>(p.g.bias_r + cc),
-               bi = *reinterpret_cast<const float2*>(p.g.bias_i + cc);
+  constexpr bool HALF = sizeof(T) == 2;
+  const float2 rate = *reinterpret_cast<const float2*>(p.g.rate + cc), rate2 = fmul2(rate, gr_both(2.f * GR_LN2));
+  float2 br = *reinterpret_cast<const float2*>(p.g.bias_r + cc), bi = *reinterpret_cast<const float2*>(p.g.bias_i + cc);
+  if (HALF) {
+    br = fmul2(br, gr_both(-GR_LOG2E));
+    bi = fmul2(bi, gr_both(-GR_LOG2E));
+  }
+  const float2 scale = gr_both(p.g.scale);
   float2* own = reinterpret_cast<float2*>(p.state + (long long)p.slots[b] * channels + cc);
   float2 carry = mine && p.start[b] > 0 ? *own : make_float2(0.f, 0.f);
   const GrMade nothing = {make_float2(1.f, 1.f), make_float2(0.f, 0.f)};
@@ -112,25 +166,37 @@ gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T
     const int t1 = t0 + rank * GR_STEP + warp * GR_RUN;
     float2 a[GR_RUN], add[GR_RUN];
     GrPair<T> xv[GR_RUN], yv[GR_RUN];
+    const float* zt = z + (long long)t1 * 2 * p.g.pp;
+    const T *xt = x + (long long)t1 * channels, *yt = y + (long long)t1 * p.ldy;
+    const int have = mine ? min(GR_RUN, n - t1) : 0;  // tokens of this warp
+    auto load = [&](int i) {
+      a[i] = __ldcs(reinterpret_cast<const float2*>(zt + i * 2 * p.g.pp));
+      add[i] = __ldcs(reinterpret_cast<const float2*>(zt + i * 2 * p.g.pp + p.g.pp));
+      xv[i] = *reinterpret_cast<const GrPair<T>*>(xt + i * channels);
+      yv[i] = *reinterpret_cast<const GrPair<T>*>(yt + i * p.ldy);
+    };
+    if (have == GR_RUN) {
 #pragma unroll
-    for (int i = 0; i < GR_RUN; ++i) {
-      const int t = t1 + i;
-      a[i] = add[i] = make_float2(0.f, 0.f);
-      xv[i].v[0] = xv[i].v[1] = yv[i].v[0] = yv[i].v[1] = from_f32<T>(0.f);
-      if (mine && t < n) {
-        a[i] = __ldcs(reinterpret_cast<const float2*>(z + (long long)t * 2 * p.g.pp));
-        add[i] = __ldcs(reinterpret_cast<const float2*>(z + (long long)t * 2 * p.g.pp + p.g.pp));
-        xv[i] = *reinterpret_cast<const GrPair<T>*>(x + (long long)t * channels);
-        yv[i] = *reinterpret_cast<const GrPair<T>*>(y + (long long)t * p.ldy);
+      for (int i = 0; i < GR_RUN; ++i) load(i);
+    } else {
+#pragma unroll
+      for (int i = 0; i < GR_RUN; ++i) {
+        a[i] = add[i] = make_float2(0.f, 0.f);
+        xv[i].v[0] = xv[i].v[1] = yv[i].v[0] = yv[i].v[1] = from_f32<T>(0.f);
+        if (i < have) load(i);
       }
     }
     GrMade own_tokens = nothing;
 #pragma unroll
     for (int i = 0; i < GR_RUN; ++i) {
-      if (t1 + i < n) {
-        gr_token<T>(a[i].x + br.x, add[i].x + bi.x, to_f32(xv[i].v[0]), rate.x, a[i].x, add[i].x);
-        gr_token<T>(a[i].y + br.y, add[i].y + bi.y, to_f32(xv[i].v[1]), rate.y, a[i].y, add[i].y);
-      } else {  // changes nothing
+      const float2 xi = make_float2(to_f32(xv[i].v[0]), to_f32(xv[i].v[1]));
+      if constexpr (HALF) {
+        gr_token2(a[i], add[i], xi, br, bi, rate, rate2, a[i], add[i]);
+      } else {
+        gr_token<T>(a[i].x + br.x, add[i].x + bi.x, xi.x, rate.x, a[i].x, add[i].x);
+        gr_token<T>(a[i].y + br.y, add[i].y + bi.y, xi.y, rate.y, a[i].y, add[i].y);
+      }
+      if (i >= have) {  // changes nothing
         a[i] = make_float2(1.f, 1.f);
         add[i] = make_float2(0.f, 0.f);
       }
@@ -158,13 +224,17 @@ gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T
       carry = gr_apply(all, carry);
     }
     float2 s = before.sum;
+    T* ot = out + (long long)t1 * p.ldo;
 #pragma unroll
     for (int i = 0; i < GR_RUN; ++i) {
       s = ffma2(a[i], s, add[i]);
+      const float2 yi = make_float2(to_f32(yv[i].v[0]), to_f32(yv[i].v[1]));
+      const float2 g = HALF ? gr_gelu2(yi) : make_float2(gr_gelu<T>(yi.x), gr_gelu<T>(yi.y));
+      const float2 v = fmul2(fmul2(s, g), scale);
       GrPair<T> o;
-      o.v[0] = from_f32<T>(s.x * gr_gelu<T>(to_f32(yv[i].v[0])) * p.g.scale);
-      o.v[1] = from_f32<T>(s.y * gr_gelu<T>(to_f32(yv[i].v[1])) * p.g.scale);
-      if (mine && t1 + i < n) *reinterpret_cast<GrPair<T>*>(out + (long long)(t1 + i) * p.ldo) = o;
+      o.v[0] = from_f32<T>(v.x);
+      o.v[1] = from_f32<T>(v.y);
+      if (i < have) *reinterpret_cast<GrPair<T>*>(ot + i * p.ldo) = o;
     }
   }
   if (ranks > 1) cluster.sync();  // nobody writes into the memory of a CTA that has gone

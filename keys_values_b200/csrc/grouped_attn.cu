@@ -147,9 +147,11 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
     }
   };
   const int per_head = p.dimp / V;
-  if (p.norm_q && p.a.head_norm && half == 0 && !shared && per_head <= 32 && (per_head & (per_head - 1)) == 0) {
-    // nothing is rotated and a head lies in neighbouring lanes: one pass without shared memory
+  const int partner = half / V;  // lanes from one half of a pair to the other
+  if (p.norm_q && p.a.head_norm && partner * V == half && (partner & (partner - 1)) == 0 && !shared && per_head <= 32 && (per_head & (per_head - 1)) == 0) {
+    // a head lies in neighbouring lanes: one pass, in which pairs of the rotation find each other by a shuffle
     if (dst) put_values();
+    if (half > 0) __syncthreads();
     const int total = (nq + nk) / V;
 #pragma unroll 4
     for (int i0 = 0; i0 < total; i0 += GP_THREADS) {
@@ -162,13 +164,28 @@ grouped_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q, T* __restrict_
         for (int e = 0; e < V; ++e) s = fmaf(to_f32(a.v[e]), to_f32(a.v[e]), s);
       }
       for (int o = per_head >> 1; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-      if (i >= total) continue;
+      const bool in = i < total;
       const float r = 1.f / sqrtf(s / (float)p.dim + p.a.eps);
-      const int h = i / per_head, col = (i - h * per_head) * V;
-      const float* w = (h < p.heads ? p.norm_q : p.norm_k) + col;
-      const float f = p.a.q_scale && h < p.heads ? r * p.a.q_scale[h / maps] : r;
+      const int h = in ? i / per_head : 0, col = (i - h * per_head) * V;
+      float x[V] = {};
+      if (in) {
+        const float* w = (h < p.heads ? p.norm_q : p.norm_k) + col;
+        const float f = p.a.q_scale && h < p.heads ? r * p.a.q_scale[h / maps] : r;
 #pragma unroll
-      for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(to_f32(a.v[e]) * f * w[e]);
+        for (int e = 0; e < V; ++e) x[e] = to_f32(a.v[e]) * f * w[e];
+      }
+      if (half > 0) {
+        const bool upper = col >= half, rotated = in && col < 2 * half;
+        const float* cs = cs_sm + (upper ? col - half : col);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const float y = __shfl_xor_sync(0xffffffffu, x[e], partner);
+          if (rotated) x[e] = x[e] * cs[e] + (upper ? y : -y) * cs[half + e];
+        }
+      }
+      if (!in) continue;
+#pragma unroll
+      for (int e = 0; e < V; ++e) a.v[e] = from_f32<T>(x[e]);
       put(h, col, a);
     }
     pool();

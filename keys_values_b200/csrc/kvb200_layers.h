@@ -44,16 +44,15 @@ int kvb_sequence_advance(const long long* idx, int* pos, int* prev_token, const 
 // weights and step fp32. center: layer norm, else RMS norm.
 //
 // tokens (NULL: the rows are no tokens of a pass): the n rows are T tokens of n / T rows of a pass. table (NULL: none): row start[b] + t is added
-// to x. conv_w (taps, width; NULL: none): h becomes h + sum_k conv_w[k] · (h of the token taps - 1 - k before), zero before a sequence's start;
-// conv_ring (slots, taps, width) fp32 holds the last h of every sequence, position p in row p mod taps. With T > 1 x_out must not be x_in, and
-// there are no experts.
+// to x. conv_w (taps, width; NULL: none; with T = 1): h becomes sum_k conv_w[k] · (h of the token taps - 1 - k before), zero before a sequence's
+// start; conv_ring (slots, taps, width) of `dtype` holds the last h of every sequence, position p in row p mod taps.
 typedef struct {
   const int *slots, *start, *count;
   int T, taps;
   const void* table;
   long long table_rows;
   const float* conv_w;
-  float* conv_ring;
+  void* conv_ring;
 } kvb_edge_tokens;
 int kvb_norm_edge(const float* x_in, const void* sub, const void* expert_out, const int* expert_row, const float* expert_w, int top,
                   long long expert_ld, const float* after, float* x_out, const float* before, void* h, const long long* idx,
@@ -111,7 +110,7 @@ int kvb_grouped_decode(const void* q, const void* rows, const void* gate, long l
 // ---- ssm.cu
 // Columns of u (ld): z (heads · vdp), from `col` on the channels x (heads · vdp) | B (groups · np) | C (groups · np), from
 // dt_col on the step sizes (heads). vdp, np multiples of 8. ring (slots, taps, channels), state (slots, heads, np, vdp) fp32.
-// The convolution has a silu behind it, or (silu 0) nothing.
+// The convolution has a bias (NULL: none) and a silu behind it, or (silu 0) nothing.
 int kvb_short_conv(const void* u, long long ld, int col, const float* w, const float* bias, void* out, void* ring, const int* slots,
                    const int* start, const int* count, int B, int T, int channels, int taps, int silu, int dtype, void* stream);
 int kvb_state_scan(const void* u, long long ld, int dt_col, const void* xbc, const float* dt_bias, const float* a_log,

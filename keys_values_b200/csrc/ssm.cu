@@ -60,7 +60,7 @@ short_conv_kernel(const T* __restrict__ u, T* __restrict__ out, T* __restrict__ 
   };
   float bias[V];
 #pragma unroll
-  for (int e = 0; e < V; ++e) bias[e] = p.bias[c + e];
+  for (int e = 0; e < V; ++e) bias[e] = p.bias ? p.bias[c + e] : 0.f;
   if constexpr (TAPS > 0) {
     float w[TAPS][V], x[TAPS][V];
 #pragma unroll
@@ -69,7 +69,7 @@ short_conv_kernel(const T* __restrict__ u, T* __restrict__ out, T* __restrict__ 
       for (int e = 0; e < V; ++e) w[k][e] = p.w[(long long)k * p.channels + c + e];
 #pragma unroll
     for (int k = 0; k < TAPS - 1; ++k) input(t0 - TAPS + 1 + k, x[k + 1]);
-    constexpr int AHEAD = 4;
+    constexpr int AHEAD = 8;
     for (int t = t0; t < t1; t += AHEAD) {
       Vec next[AHEAD];
 #pragma unroll
@@ -118,17 +118,22 @@ short_conv_kernel(const T* __restrict__ u, T* __restrict__ out, T* __restrict__ 
   }
 }
 
-template <typename T>
-static int conv_launch(const void* u, void* out, void* ring, ConvParams& p, int B, cudaStream_t s) {
-  constexpr int V = 16 / sizeof(T);
+template <typename T, int V>
+static int conv_launch_vec(const void* u, void* out, void* ring, ConvParams& p, int B, cudaStream_t s) {
   const int blocks = (p.channels / V + SC_THREADS - 1) / SC_THREADS;
-  long long run = ((long long)p.T * B * blocks + 148 * 4 - 1) / (148 * 4);  // a wave of CTAs first, then few inputs read twice
-  p.run = (int)(run < 4 ? 4 : (run > SC_RUN ? SC_RUN : (run + 3) / 4 * 4));
+  long long run = ((long long)p.T * B * blocks + 148 * 8 - 1) / (148 * 8);  // a wave of CTAs first, then few inputs read twice
+  p.run = (int)(run < 4 ? 4 : (run > SC_RUN ? SC_RUN : (run + 7) / 8 * 8));
   if (p.run < p.taps) p.run = p.taps;  // only the first run of a channel may look back beyond the pass
   const dim3 grid(blocks, (p.T + p.run - 1) / p.run, B);
   if (p.taps == 4) short_conv_kernel<T, V, 4><<<grid, SC_THREADS, 0, s>>>((const T*)u, (T*)out, (T*)ring, p);
   else short_conv_kernel<T, V, 0><<<grid, SC_THREADS, 0, s>>>((const T*)u, (T*)out, (T*)ring, p);
   return cudaGetLastError() == cudaSuccess ? KVB_OK : KVB_ERR_LAUNCH;
+}
+
+template <typename T>
+static int conv_launch(const void* u, void* out, void* ring, ConvParams& p, int B, cudaStream_t s) {
+  if (p.channels % 4 || p.col % 4 || p.ld % 4) return conv_launch_vec<T, 1>(u, out, ring, p, B, s);
+  return conv_launch_vec<T, 4>(u, out, ring, p, B, s);
 }
 
 // ------------------------------------------------------------------------------------------------ scan
@@ -467,7 +472,6 @@ extern "C" int kvb_short_conv(const void* u, long long ld, int col, const float*
                               const int* slots, const int* start, const int* count, int B, int T_, int channels, int taps, int silu,
                               int dtype, void* stream) {
   if (B <= 0 || B > 65535 || T_ <= 0 || channels <= 0 || taps <= 0) return KVB_ERR_ARG;
-  if (channels % 8 || col % 8 || ld % 8) return KVB_ERR_ALIGN;
   kvb::ConvParams p;
   p.w = w; p.bias = bias; p.slots = slots; p.start = start; p.count = count; p.ld = ld; p.T = T_; p.col = col; p.channels = channels;
   p.taps = taps; p.silu = silu;

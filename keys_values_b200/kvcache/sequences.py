@@ -1,8 +1,8 @@
 """State of the sequences a model is working on, one slot per sequence.
 
 A model whose rows may have different lengths keeps, per slot: the position of the next token, the previous
-token, and fp32 state of the edges between sublayers where there is one (the token shift's last normed input per layer; the last inputs of
-every sublayer, if these pass a convolution, in rings: position p in row p mod taps). Slots are handed
+token, and state of the edges between sublayers where there is one (fp32: the token shift's last normed input per layer; the last inputs
+of every sublayer, if these pass a convolution, in rings: position p in row p mod taps). Slots are handed
 out and taken back like cache blocks; a slot that starts at position 0 never reads what an earlier owner left.
 
 A pass (:class:`SequencePass`) names the slots of its rows, the position each row starts at and how many of its
@@ -37,7 +37,9 @@ class SequencePass:
 
 
 class SequenceTable:
-    def __init__(self, n_slots: int, device, shift_layers: int = 0, width: int = 0, conv_edges: int = 0, taps: int = 0):
+    def __init__(self, n_slots: int, device, shift_layers: int = 0, width: int = 0, conv_edges: int = 0, taps: int = 0,
+                 dtype: torch.dtype = torch.float32):
+        """``conv_edges``: sublayers whose input passes a convolution of ``taps``; these inputs are kept as ``dtype``."""
         if n_slots <= 0:
             raise ValueError("n_slots must be positive")
         self.n_slots = n_slots
@@ -46,7 +48,7 @@ class SequenceTable:
             self.pos = torch.zeros(n_slots, dtype=torch.int32, device=self.device)
             self.prev_token = torch.zeros(n_slots, dtype=torch.int32, device=self.device)
             self.shift = torch.zeros((shift_layers, n_slots, width), dtype=torch.float32, device=self.device) if shift_layers else None
-            self.conv = torch.zeros((conv_edges, n_slots, taps, width), dtype=torch.float32, device=self.device) if conv_edges else None
+            self.conv = torch.zeros((conv_edges, n_slots, taps, width), dtype=dtype, device=self.device) if conv_edges else None
         self._consts: Dict[Tuple[int, ...], torch.Tensor] = {}
         self.reset()
 
@@ -123,4 +125,4 @@ class SequenceTable:
 
     def size_estimate(self) -> int:
         """Bits held on the device."""
-        return 32 * (2 * self.n_slots + sum(t.numel() for t in (self.shift, self.conv) if t is not None))
+        return 64 * self.n_slots + sum(8 * t.numel() * t.element_size() for t in (self.shift, self.conv) if t is not None)

@@ -356,8 +356,6 @@ class SequentialBlock(Packed):
         if config.input_conv:  # (width, taps), the last column meets the token itself
             self.conv_1 = nn.Parameter(torch.zeros(config.n_embd, config.input_conv))
             self.conv_2 = None if self.mlp is None else nn.Parameter(torch.zeros(config.n_embd, config.input_conv))
-            if isinstance(self.mlp, RoutedMLP):
-                raise NotImplementedError("routed experts and an input convolution")
         if config.residual_mult != 1.0 and (self.post_attention_norm is None or self.mlp is not None and self.post_mlp_norm is None):
             raise NotImplementedError("a residual factor goes with norms after the sublayers, whose weights take it")
         self.center = STREAM_NORMS[config.norm_class_name]["center"]
@@ -369,19 +367,17 @@ class SequentialBlock(Packed):
         norms = dict(norm_1=(self.norm_1, 1.0), after_1=(self.post_attention_norm, mult), norm_2=(self.norm_2, 1.0), after_2=(self.post_mlp_norm, mult))
         pack = {k: None if n is None else n.packed()["weight"] * f for k, (n, f) in norms.items()}
         for k, w in dict(conv_1=self.conv_1, conv_2=self.conv_2).items():
-            pack[k] = None if w is None else w.float().t().contiguous()
+            pack[k] = None
+            if w is not None:  # h + convolution of h as one convolution
+                pack[k] = w.detach().float().t().clone(memory_format=torch.contiguous_format)
+                pack[k][-1] += 1
         return pack
 
     def _edge(self, model: "LayeredGPT", x: "LayerStream", y, after, before, conv, edge: int, want_h: bool = True, **kw: Any) -> None:
-        """From a sublayer's result to the next one's input, the ``edge``-th in the pass; ``conv``: what that input passes. A convolution over
-        several tokens reads a token's neighbours again, so the stream changes its place."""
-        ring = None if conv is None else model.sequences.conv[edge]
-        moves = conv is not None and x.x.shape[1] > 1
-        out = x.x if not moves else x.spare if x.spare is not None else torch.empty_like(x.x)
-        L.norm_edge(x.x, y, after, out, before, x.h if want_h else None, kw.get("idx"), kw.get("embed"), kw.get("step"), self.config.norm_eps, self.center,
-                    kw.get("experts"), None if conv is None else L.EdgeTokens(x.seq, None, conv, ring))
-        if moves:
-            x.x, x.spare = out, x.x
+        """From a sublayer's result to the next one's input, the ``edge``-th in the pass; ``conv``: what that input passes."""
+        tokens = None if conv is None else L.EdgeTokens(x.seq, None, conv, model.sequences.conv[edge])
+        L.norm_edge(x.x, y, after, x.x, before, x.h if want_h else None, kw.get("idx"), kw.get("embed"), kw.get("step"), self.config.norm_eps, self.center,
+                    kw.get("experts"), tokens)
 
     def enter(self, model: "LayeredGPT", idx: torch.Tensor, seq: SequencePass) -> "LayerStream":
         """The stream in front of this (the first) layer."""
@@ -530,7 +526,8 @@ class LayeredGPT(GPT):
             return
         c = self.config
         self.sequences = SequenceTable(min(x.max_batch_size for x in caches), self.lm_head.weight.device,
-                                       c.n_layer if c.token_shift else 0, c.n_embd, 2 * self.n_runs if c.input_conv else 0, c.input_conv)
+                                       c.n_layer if c.token_shift else 0, c.n_embd, 2 * self.n_runs if c.input_conv else 0, c.input_conv,
+                                       self.lm_head.weight.dtype)
         for x in caches:
             x.sequences = self.sequences
             if isinstance(x, BorrowedKVCache):

@@ -263,8 +263,8 @@ class RecurrenceWeights(NamedTuple):
 
 class EdgeTokens(NamedTuple):
     """What an edge between sublayers needs to know of its tokens: the pass; ``table`` (a vector per position is added to the stream); ``conv
-    (taps, width)`` fp32 and its ``ring (slots, taps, width)`` fp32 (what the sublayer reads, h, becomes h + a causal convolution of h; the ring
-    keeps the last h of every sequence, position p in row p mod taps)."""
+    (taps, width)`` fp32 and its ``ring (slots, taps, width)`` (what the sublayer reads, h, passes a causal convolution, whose last row meets the
+    token itself; the ring keeps the last h of every sequence, position p in row p mod taps)."""
 
     seq: object
     table: Optional[torch.Tensor] = None
@@ -359,9 +359,15 @@ def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps: float, 
     """``x = x_in + norm(s) · after`` with ``s = sub + Σ_k weight_k · expert output_k`` (``x_in``, ``sub`` or ``experts`` ``None``:
     without it; ``after`` ``None``: ``s`` as it is), then ``x += embed[idx] + step`` (each unless ``None``); ``x_out = x`` (fp32, may be
     ``x_in``) and, unless ``h`` is ``None``, ``h = norm(x) · before`` (``before`` ``None``: ``h = x``). The norm takes the mean off if
-    ``center``. ``experts``: ``(out, row, weight)`` of :func:`routed_experts`. ``tokens``: see :class:`EdgeTokens`; with a convolution over
-    several tokens ``x_out`` must not be ``x_in`` (a token's neighbours are read again)."""
-    _impl(x_out).norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts, tokens)
+    ``center``. ``experts``: ``(out, row, weight)`` of :func:`routed_experts`. ``tokens``: see :class:`EdgeTokens`; a single
+    token passes the convolution in the same kernel."""
+    impl = _impl(x_out)
+    if tokens is None or tokens.conv is None or tokens.seq.length == 1:
+        impl.norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts, tokens)
+        return
+    plain = torch.empty_like(h)
+    impl.norm_edge(x_in, sub, after, x_out, before, plain, idx, embed, step, eps, center, experts, tokens._replace(conv=None, ring=None))
+    impl.short_conv(plain, 0, tokens.conv, None, tokens.ring, tokens.seq, False, h)
 
 
 def row_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, center: bool, dtype: torch.dtype) -> torch.Tensor:
@@ -470,10 +476,10 @@ def gated_recurrence(u, w: RecurrenceWeights, ring, state, seq, shape: Recurrenc
 
 
 # ---- state-space recurrence
-def short_conv(u, col: int, w, bias, ring, seq, silu: bool = True) -> torch.Tensor:
-    """Causal convolution ``w (taps, channels)`` with bias (and silu) over the channels of ``u (B, T, ·)`` from ``col`` on; the inputs before the
+def short_conv(u, col: int, w, bias, ring, seq, silu: bool = True, out=None) -> torch.Tensor:
+    """Causal convolution ``w (taps, channels)`` with bias (unless ``None``) and silu (or without) over the channels of ``u (B, T, ·)`` from ``col`` on; the inputs before the
     pass come from ``ring (slots, taps, channels)``, which takes the last ones of the pass. Returns ``(B, T, channels)``."""
-    return _impl(u).short_conv(u, col, w, bias, ring, seq, silu)
+    return _impl(u).short_conv(u, col, w, bias, ring, seq, silu, out)
 
 
 def state_scan(u, xbc, dt_bias, a_log, skip, state, seq, shape: StateShape) -> torch.Tensor:

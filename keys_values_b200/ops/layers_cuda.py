@@ -195,8 +195,6 @@ def _edge_tokens(tokens):
         return None
     seq, table, conv, ring = tokens
     _contiguous(table, conv, ring)
-    if conv is not None and ring.dtype != torch.float32:
-        raise NativeError("the inputs of a convolution are kept in fp32")
     return ctypes.byref(_EdgeTokens(seq.slots.data_ptr(), seq.start.data_ptr(), seq.count.data_ptr(), seq.length, 0 if conv is None else conv.shape[0],
                                     _ptr(table), 0 if table is None else table.shape[0], _ptr(conv), _ptr(ring)))
 
@@ -395,11 +393,14 @@ def bmm_fp32(a, b) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------------------------- state-space recurrence
-def short_conv(u, col, w, bias, ring, seq, silu=True) -> torch.Tensor:
+def short_conv(u, col, w, bias, ring, seq, silu=True, out=None) -> torch.Tensor:
     B, T, _ = u.shape
     taps, channels = w.shape
-    out = torch.empty((B, T, channels), dtype=u.dtype, device=u.device)
-    _contiguous(w, bias, ring)
+    if out is None:
+        out = torch.empty((B, T, channels), dtype=u.dtype, device=u.device)
+    _contiguous(w, bias, ring, out)
+    if ring.dtype != u.dtype:
+        raise NativeError(f"inputs of type {u.dtype} are kept as {ring.dtype}")
     _check(lib().kvb_short_conv(_p(u), _ll(_rows_of(u)), col, _p(w), _p(bias), _p(out), _p(ring), _p(seq.slots), _p(seq.start), _p(seq.count), B, T,
                                 channels, taps, int(silu), code(u.dtype), _stream(u)), "short_conv")
     _count()

@@ -178,20 +178,6 @@ def _norm(x, weight, eps, center):
     return x / torch.sqrt(x.square().mean(-1, keepdim=True) + eps) * weight
 
 
-def _input_conv(h, w, ring, seq):
-    """h + causal convolution of h; the ring takes the last ones of every sequence."""
-    taps = w.shape[0]
-    B, T, _ = h.shape
-    out = h.clone()
-    for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
-        before = [ring[slot, p % taps] if p >= 0 else torch.zeros_like(h[b, 0]) for p in range(start - taps + 1, start)]
-        rows = torch.cat((torch.stack(before), h[b])) if before else h[b]
-        out[b] += sum(w[k] * rows[k : k + T] for k in range(taps))
-        for t in range(max(0, n - taps), n):
-            ring[slot, (start + t) % taps] = h[b, t]
-    return out
-
-
 def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center, experts=None, tokens=None) -> None:
     x = torch.zeros_like(x_out) if x_in is None else x_in
     s = None if sub is None else sub.float()
@@ -213,8 +199,9 @@ def norm_edge(x_in, sub, after, x_out, before, h, idx, embed, step, eps, center,
         x = x + step
     x_out.copy_(x)
     if h is not None:
-        y = x if before is None else _norm(x, before, eps, center)
-        h.copy_(y if tokens is None or tokens.conv is None else _input_conv(y, tokens.conv, tokens.ring, tokens.seq))
+        h.copy_(x if before is None else _norm(x, before, eps, center))
+        if tokens is not None and tokens.conv is not None:
+            short_conv(h.clone(), 0, tokens.conv, None, tokens.ring, tokens.seq, False, h)
 
 
 def row_norm(x, weight, eps, center, dtype):
@@ -397,15 +384,15 @@ def gated_recurrence(u, w, ring, state, seq, s, scale, out):
 
 
 # ---- state-space recurrence
-def short_conv(u, col, w, bias, ring, seq, silu=True):
+def short_conv(u, col, w, bias, ring, seq, silu=True, out=None):
     B, T, _ = u.shape
     taps, channels = w.shape
     x = u[..., col : col + channels].float()
-    out = torch.empty(B, T, channels, dtype=u.dtype)
+    out = torch.empty(B, T, channels, dtype=u.dtype) if out is None else out
     for b, (slot, start, n) in enumerate(zip(seq.slots.tolist(), seq.start.tolist(), seq.count.tolist())):
         before = [ring[slot, p % taps].float() if p >= 0 else torch.zeros(channels) for p in range(start - taps + 1, start)]
         rows = torch.cat((torch.stack(before), x[b])) if before else x[b]
-        y = sum(w[k] * rows[k : k + T] for k in range(taps)) + bias
+        y = sum(w[k] * rows[k : k + T] for k in range(taps)) + (0 if bias is None else bias)
         out[b] = F.silu(y) if silu else y
         for t in range(max(0, n - taps), n):
             ring[slot, (start + t) % taps] = u[b, t, col : col + channels]

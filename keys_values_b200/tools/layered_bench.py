@@ -624,20 +624,22 @@ def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) ->
         seq.start = seq.start.clone()
         # ---- between sublayers
         x, sub, h, w1, w2 = torch.randn(B, T, W, device=dev), rand(B, T, W), rand(B, T, W), f32(W), f32(W)
-        out = torch.empty_like(x) if T > 1 else x
-        edge = L.EdgeTokens(seq, None, f32(taps, W), f32(B, taps, W))
-        tab.add(f"{tag}: norm, residual sum, norm, convolution", lambda: LC.norm_edge(x, sub, w1, out, w2, h, None, None, None, eps, False, None, edge),
-                gbytes=(n * W * 12 + (0 if T > 1 else B * taps * W * 4)) / 1e9)
+        ring, cw = rand(B, taps, W), f32(taps, W)
+        edge = L.EdgeTokens(seq, None, cw, ring) if T == 1 else None
+        tab.add(f"{tag}: norm, residual sum, norm" + (", convolution" if T == 1 else ""),
+                lambda: LC.norm_edge(x, sub, w1, x, w2, h, None, None, None, eps, False, None, edge), gbytes=(n * W * 12 + (0 if T > 1 else B * taps * W * 2)) / 1e9)
         a, rr, w = rand(n, W), rand(n, W), rand(W)
         fused = cu.add_rmsnorm_supported(a)
         like_norm = lambda: cu.add_rmsnorm_fwd(a, rr, w, eps, False) if fused else cu.rmsnorm_fwd(a, w, eps, False)  # noqa: E731
         norm_bytes = n * W * (8 if fused else 4) / 1e9
         tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
+        if T > 1:
+            tab.add(f"{tag}: convolution of {W} inputs", lambda: LC.short_conv(sub, 0, cw, None, ring, seq, False, h), gbytes=4 * n * W / 1e9)
         up = rand(n, 2 * ff)
         tab.add(f"{tag}: clamped unit", lambda: LC.glu(up, ff, limit), gbytes=n * ff * 6 / 1e9)
         u1 = up.view(2, n, ff)
         tab.add(f"{tag}:   like: SwiGLU", lambda: cu.swiglu_fwd(u1[0], u1[1]), gbytes=n * ff * 6 / 1e9)
-        del up, u1, out
+        del up, u1
         # ---- attentions
         for what, s in (("attention", plain), ("attention over another layer's keys", borrowed), ("pooled window", pooled)):
             H, G, D, V = s.heads, s.kv_heads, s.dim, s.vdim

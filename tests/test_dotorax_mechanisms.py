@@ -16,6 +16,13 @@ from test_pazenex_mechanisms import check, close, env, move, padded, part_of, ta
 
 
 # ------------------------------------------------------------------------------------------------- between sublayers
+def plus_identity(w):
+    """h + conv(h) as one convolution ``(taps, width)``."""
+    w = w.t().clone(memory_format=torch.contiguous_format)
+    w[-1] += 1
+    return w
+
+
 EDGE_PASSES = [(9, [9, 6]), (1, [1, 1]), (2, [2, 2]), (1, [0, 1]), (40, [40, 33]), (1, [1, 1]), (3, [0, 3]), (5, [5, 1])]
 
 
@@ -34,7 +41,7 @@ def test_edge_with_convolution(env, width, taps):
     stream = torch.stack([x[b] + oracle.norm_rows(sub[b], after, eps) for b in range(2)])
     want = torch.stack([oracle.input_conv(oracle.norm_rows(s, before, eps), w) for s in stream])
     tab = table(dev, [0, 0], 3, [2, 0])
-    ring = torch.full((3, taps, width), 9.0, device=dev)  # what an earlier owner left
+    ring = torch.full((3, taps, width), 9.0, dtype=dtype, device=dev)  # what an earlier owner left
     f32 = lambda t: t.float().to(dev)  # noqa: E731
     at, got = [0, 0], [([], []), ([], [])]
     for n, counts in EDGE_PASSES:
@@ -42,7 +49,7 @@ def test_edge_with_convolution(env, width, taps):
         seq.start = seq.start.clone()
         xin, part = f32(part_of(x, at, n, counts)), part_of(sub, at, n, counts).to(dev, dtype)
         out, h = torch.empty_like(xin), torch.zeros(2, n, width, dtype=dtype, device=dev)
-        L.norm_edge(xin, part, f32(1 + after), out, f32(1 + before), h, None, None, None, eps, False, None, L.EdgeTokens(seq, None, f32(w.t().contiguous()), ring))
+        L.norm_edge(xin, part, f32(1 + after), out, f32(1 + before), h, None, None, None, eps, False, None, L.EdgeTokens(seq, None, f32(plus_identity(w)), ring))
         for b in range(2):
             got[b][0].append(out[b, : counts[b]])
             got[b][1].append(h[b, : counts[b]])
@@ -67,19 +74,19 @@ def test_entry_with_positions(env, T):
     start, counts = [0, 700 - T, 5], [T, T, max(1, T - 2)]
     tokens = torch.randint(0, vocab, (3, 700), generator=g)
     seq = table(dev, start).begin(3, T, counts)
-    ring = torch.zeros(3, taps, width, device=dev)
+    ring = torch.zeros(3, taps, width, dtype=dtype, device=dev)
     idx = torch.zeros(3, T, dtype=torch.int64)
     streams = []
     for b in range(3):
         x = embed[tokens[b]].double() + pos.double()
         h = oracle.norm_rows(x, before, eps)
         for p in range(max(0, start[b] - taps + 1), start[b]):
-            ring[b, p % taps] = h[p].float()
+            ring[b, p % taps] = h[p].to(dtype)
         idx[b, : counts[b]] = tokens[b, start[b] : start[b] + counts[b]]
         streams.append((x, oracle.input_conv(h, w)))
     x, h = torch.empty(3, T, width, device=dev), torch.zeros(3, T, width, dtype=dtype, device=dev)
     L.norm_edge(None, None, None, x, (1 + before).float().to(dev), h, idx.to(dev), embed.to(dev), None, eps, False, None,
-                L.EdgeTokens(seq, pos.to(dev), w.t().float().contiguous().to(dev), ring))
+                L.EdgeTokens(seq, pos.to(dev), plus_identity(w).float().to(dev), ring))
     for b, (xs, hs) in enumerate(streams):
         at = slice(start[b], start[b] + counts[b])
         close(x[b, : counts[b]], xs[at], torch.float32)
