@@ -3,8 +3,8 @@
 //
 //   scan   several new tokens, behind the convolution (ssm.cu) and the gates' products: a cluster of up to eight CTAs has 64 channels of one
 //          sequence and takes 64 tokens per CTA at a time. A warp has 8 of them and a lane two channels: decays and additions stay in registers;
-//          the warps of a CTA, then the CTAs (over distributed shared memory) exchange what their tokens make of a state, and every warp runs
-//          through its tokens from the right start. Everything is read once;
+//          the warps of a CTA, then the CTAs (asynchronous stores to distributed shared memory) exchange what their tokens make of a state, and
+//          every warp runs through its tokens from the right start. Everything is read once;
 //   step   one new token per sequence: convolution, gates (a part's products on CUDA cores, weights read once for eight sequences), recurrence
 //          and output in one kernel. The inputs of the convolution lie in a ring with one row more than it looks back, so CTAs that share
 //          a part do not disturb each other.
@@ -120,6 +120,7 @@ struct GrScanParams {
   float* state;
   long long ldy, ldo;
   int B, T;
+  int* status;
 };
 
 template <typename T>
@@ -128,9 +129,18 @@ struct alignas(2 * sizeof(T)) GrPair {
 };
 
 // what tokens make of the states of two channels: s -> decay · s + sum
-struct GrMade {
+struct alignas(16) GrMade {
   float2 decay, sum;
 };
+// to the same place of another CTA's shared memory, whose barrier counts the bytes
+__device__ __forceinline__ void gr_send(const GrMade* place, uint64_t* bar, int rank, const GrMade& m) {
+  uint32_t to, at;
+  asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(to) : "r"(smem_u32(place)), "r"(rank));
+  asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"(smem_u32(bar)), "r"(rank));
+  asm volatile("st.async.weak.shared::cluster.mbarrier::complete_tx::bytes.v4.b32 [%0], {%1, %2, %3, %4}, [%5];" ::"r"(to),
+               "r"(__float_as_uint(m.decay.x)), "r"(__float_as_uint(m.decay.y)), "r"(__float_as_uint(m.sum.x)), "r"(__float_as_uint(m.sum.y)), "r"(at)
+               : "memory");
+}
 __device__ __forceinline__ float2 gr_apply(const GrMade& m, float2 s) { return ffma2(m.decay, s, m.sum); }
 __device__ __forceinline__ GrMade gr_then(const GrMade& a, const GrMade& b) { return {fmul2(a.decay, b.decay), ffma2(b.decay, a.sum, b.sum)}; }
 
@@ -138,6 +148,9 @@ template <typename T>
 __global__ void __launch_bounds__(GR_WARPS * 32, 2)
 gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T* __restrict__ out, const GrScanParams p) {
   __shared__ GrMade by_warp[2][GR_WARPS][32], by_cta[2][GR_CLUSTER][32];
+  __shared__ uint64_t arrived[2];
+  __shared__ int abort_word;
+  volatile int* abort_flag = &abort_word;
   cooperative_groups::cluster_group cluster = cooperative_groups::this_cluster();
   const int rank = (int)cluster.block_rank(), ranks = (int)cluster.num_blocks();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.z;
@@ -161,8 +174,21 @@ gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T
   float2* own = reinterpret_cast<float2*>(p.state + (long long)p.slots[b] * channels + cc);
   float2 carry = mine && p.start[b] > 0 ? *own : make_float2(0.f, 0.f);
   const GrMade nothing = {make_float2(1.f, 1.f), make_float2(0.f, 0.f)};
-  int turn = 0;
-  for (int t0 = 0; t0 < n; t0 += ranks * GR_STEP, turn ^= 1) {
+  if (ranks > 1) {
+    if (threadIdx.x == 0) {
+      mbar_init(&arrived[0], 1);
+      mbar_init(&arrived[1], 1);
+      *abort_flag = 0;
+      mbar_fence_init();
+    }
+    cluster.sync();
+  }
+  bool ok = true;  // after a wait that ran out the work goes on with what there is: the status word tells
+  int turn = 0, phase = 0;
+  for (int t0 = 0; t0 < n; t0 += ranks * GR_STEP, turn ^= 1, phase += turn == 0) {
+    // Buffers in turn are enough: a CTA that sends for the turn after next has got everybody's results of the next one, which they send after
+    // they have read those of this one
+    if (ranks > 1 && threadIdx.x == 0) mbar_expect_tx(&arrived[turn], (uint32_t)(ranks * 32 * sizeof(GrMade)));
     const int t1 = t0 + rank * GR_STEP + warp * GR_RUN;
     float2 a[GR_RUN], add[GR_RUN];
     GrPair<T> xv[GR_RUN], yv[GR_RUN];
@@ -211,8 +237,8 @@ gated_recurrence_scan_kernel(const T* __restrict__ x, const T* __restrict__ y, T
       all = gr_then(all, by_warp[turn][w][lane]);
     }
     if (ranks > 1) {  // every CTA of the cluster gets what the others' tokens make of a state
-      if (warp < ranks) cluster.map_shared_rank(&by_cta[turn][rank][lane], warp)[0] = all;
-      cluster.sync();
+      if (warp < ranks) gr_send(&by_cta[turn][rank][lane], &arrived[turn], warp, all);
+      if (ok) ok = mbar_wait_bounded(&arrived[turn], (uint32_t)(phase & 1), abort_flag, p.status, STATUS_TIMEOUT_FULL);
       float2 s = carry;
       for (int r = 0; r < ranks; ++r) {
         if (r == rank) s = carry;
@@ -379,12 +405,12 @@ static bool gated_recurrence_valid(const kvb_gated_recurrence* g) {
   }
 
 extern "C" int kvb_gated_recurrence_scan(const kvb_gated_recurrence* g, const void* x, const float* z, const void* y, long long ldy, float* state,
-                                         void* out, long long ldo, const int* slots, const int* start, const int* count, int B, int T_, int dtype,
+                                         void* out, long long ldo, const int* slots, const int* start, const int* count, int B, int T_, int dtype, int* status,
                                          void* stream) {
   if (!kvb::gated_recurrence_valid(g) || !z || B <= 0 || B > 65535 || T_ <= 0 || ldy < (long long)g->blocks * g->pp || ldo < (long long)g->blocks * g->pp)
     return KVB_ERR_ARG;
   kvb::GrScanParams p;
-  p.g = *g; p.slots = slots; p.start = start; p.count = count; p.z = z; p.state = state; p.ldy = ldy; p.ldo = ldo; p.B = B; p.T = T_;
+  p.g = *g; p.slots = slots; p.start = start; p.count = count; p.z = z; p.state = state; p.ldy = ldy; p.ldo = ldo; p.B = B; p.T = T_; p.status = status;
   if (g->pp % 8 || ldy % 2 || ldo % 2 || (reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(y) |
                                           reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(state)) & 7)
     return KVB_ERR_ALIGN;

@@ -183,7 +183,7 @@ typedef struct {
 } kvb_gated_recurrence;
 // x (B, T, channels) behind its convolution, z (blocks, B · T, 2 pp) fp32, y (ldy) channels; out (ldo) = S · gelu(y) · scale, zero in padding
 int kvb_gated_recurrence_scan(const kvb_gated_recurrence* g, const void* x, const float* z, const void* y, long long ldy, float* state, void* out,
-                              long long ldo, const int* slots, const int* start, const int* count, int B, int T, int dtype, void* stream);
+                              long long ldo, const int* slots, const int* start, const int* count, int B, int T, int dtype, int* status, void* stream);
 // One token per sequence, convolution and gates included: u (ld) = [y: channels | x: channels]; ring (slots, taps, channels)
 int kvb_gated_recurrence_step(const kvb_gated_recurrence* g, const void* u, long long ld, void* ring, float* state, void* out, long long ldo,
                               const int* slots, const int* start, const int* count, int B, int dtype, void* stream);

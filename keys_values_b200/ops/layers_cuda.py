@@ -382,7 +382,8 @@ def gated_recurrence(u, w, ring, state, seq, s, scale, out) -> torch.Tensor:
         return out
     x = short_conv(u, s.channels, w.conv, w.conv_bias, ring, seq, False)
     z = bmm_fp32(x.view(B * T, s.blocks, s.pp).transpose(0, 1), w.gates)
-    _check(lib().kvb_gated_recurrence_scan(g, _p(x), _p(z), _p(u), ld, _p(state), _p(out), ldo, *where, T, code(u.dtype), _stream(u)), "gated_recurrence_scan")
+    _check(lib().kvb_gated_recurrence_scan(g, _p(x), _p(z), _p(u), ld, _p(state), _p(out), ldo, *where, T, code(u.dtype), _p(status_word(u.device)),
+                                           _stream(u)), "gated_recurrence_scan")
     _count()
     return out
 

@@ -716,7 +716,8 @@ def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) ->
             z, xs = LC.bmm_fp32(xc, gw.gates), rand(B, T, C)
             g = LC._GatedRecurrence(*(t.data_ptr() for t in (gw.conv, gw.conv_bias, gw.bias_r, gw.bias_i, gw.rate, gw.gates)), r.blocks, r.pp, r.taps, 1.0)
             scan = lambda: cu._check(LC.lib().kvb_gated_recurrence_scan(LC.ctypes.byref(g), cu._p(xs), cu._p(z), cu._p(u), cu._ll(2 * C), cu._p(state), cu._p(y),  # noqa: E731
-                                                                        cu._ll(C), cu._p(seq.slots), cu._p(seq.start), cu._p(seq.count), B, T, 1, cu._stream(u)), "scan")
+                                                                        cu._ll(C), cu._p(seq.slots), cu._p(seq.start), cu._p(seq.count), B, T, 1,
+                                                                        cu._p(cu.status_word(dev)), cu._stream(u)), "scan")
             tab.add(f"{tag}: gated recurrence scan, {C} channels", scan, gbytes=n * C * 14 / 1e9)
             tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
             del z, xs, xc

@@ -42,7 +42,7 @@ MODELS = {
                            R(heads=1, dim=11, vdim=13, tau=1.0, mlp=dense(ff=15)), A(heads=3, kv_heads=1, dim=7, vdim=5, dims=4),
                            A(heads=3, kv_heads=1, dim=7, vdim=5, dims=4, kv_from=2, mlp=dense(ff=7))], width=31, vocab=43, taps=2, mult=1.3),
     # one of everything
-    "one": oracle.content([R(heads=1, dim=1, vdim=8, tau=2.0, mlp=dense(ff=1)), A(heads=1, kv_heads=1, dim=8, vdim=8, dims=2),
+    "one": oracle.content([R(heads=1, dim=8, vdim=8, tau=2.0, mlp=dense(ff=1)), A(heads=1, kv_heads=1, dim=8, vdim=8, dims=2),
                            P(heads=1, kv_heads=1, dim=8, vdim=16, dims=2, size=1, pool=1, width=8, blocks=1, conv=1, mlp=dense(ff=8))], width=24, taps=1, mult=1.0),
     # sizes of the kernels' tiles
     "tiles": oracle.content([A(heads=24, kv_heads=1, dim=16, vdim=16, dims=16, mlp=dense(ff=64)), R(heads=2, dim=64, vdim=128, tau=16.0),

@@ -358,7 +358,7 @@ def run_gla(env, case, passes):
 
 GLA = {
     "plain": (3, 16, 24, 5, 8.0), "full": (2, 128, 128, 16, 16.0), "narrow": (4, 64, 40, 1, 16.0), "odd": (1, 7, 9, 3, 2.0), "large": (2, 200, 24, 20, 16.0),
-    "wide": (1, 24, 200, 33, 4.0),
+    "wide": (1, 24, 200, 33, 4.0), "one": (1, 1, 1, 1, 2.0),
 }
 
 
