@@ -207,30 +207,20 @@ norm_edge_kernel(const NormEdgeParams p) {
     }
     if (p.x_out) RowVec<float, V>::store(p.x_out + o + c, x[i]);
   }
-  // columns of h, the convolution of a single token included; then out
-  auto put_h = [&](int c, float (&w)[V]) {
-    if (p.tok.conv_w) conv_single<T, V>(p, (int)n, c, w);
-    RowVec<T, V>::store(static_cast<T*>(p.h) + o + c, w);
-  };
-  if (!p.before) {
-    if (!p.h) return;
-#pragma unroll
-    for (int i = 0; i < NC; ++i) {
-      const int c = (i * TH + threadIdx.x) * V;
-      if (c < p.width) put_h(c, x[i]);
-    }
-    return;
-  }
-  r = row_norm_factor<TH, NC, V, CENTER>(x, p, red + 2);
+  if (!p.h) return;
+  if (p.before) r = row_norm_factor<TH, NC, V, CENTER>(x, p, red + 2);
 #pragma unroll
   for (int i = 0; i < NC; ++i) {
     const int c = (i * TH + threadIdx.x) * V;
     if (c >= p.width) continue;
-    float w[V];
-    RowVec<float, V>::load(p.before + c, w);
+    if (p.before) {
+      float w[V];
+      RowVec<float, V>::load(p.before + c, w);
 #pragma unroll
-    for (int e = 0; e < V; ++e) w[e] *= x[i][e] * r;
-    put_h(c, w);
+      for (int e = 0; e < V; ++e) x[i][e] = w[e] * (x[i][e] * r);
+    }
+    if (p.tok.conv_w) conv_single<T, V>(p, (int)n, c, x[i]);
+    RowVec<T, V>::store(static_cast<T*>(p.h) + o + c, x[i]);
   }
 }
 
