@@ -294,6 +294,8 @@ constexpr int GQ_ROWS = 8;    // sequences of a CTA, one per warp for the convol
 constexpr int GQ_COLS = 32;   // channels of a CTA, all of one part
 constexpr int GQ_SPLIT = 8;   // threads that share a product of two neighbouring channels
 constexpr int GQ_THREADS = GQ_COLS * GQ_SPLIT;
+constexpr int GQ_TAPS = 4;    // taps of the convolution without a loop
+constexpr int GQ_CHANNELS = 4;
 constexpr int GQ_AHEAD = 16;  // weights of a thread that are on their way during the convolution
 
 struct GrStepParams {
@@ -332,19 +334,47 @@ gated_recurrence_step_kernel(const T* __restrict__ u, T* __restrict__ ring, T* _
     T* past = ring + (long long)p.slots[b] * taps * channels + part * pp;
     const T* now = u + b * p.ld + channels + part * pp;
     const float* cw = p.g.conv + part * pp;
-#pragma unroll 4
-    for (int k = lane; k < pp; k += 32) {
-      float v = 0.f;
-      if (in) {
-        const T x = now[k];
-        v = fmaf(cw[(long long)(taps - 1) * channels + k], to_f32(x), p.g.conv_bias[part * pp + k]);
-#pragma unroll 4
-        for (int q = 1; q < taps; ++q)
-          if (pos - q >= 0) v = fmaf(cw[(long long)(taps - 1 - q) * channels + k], to_f32(past[(long long)((pos - q) % taps) * channels + k]), v);
-        v = to_f32(from_f32<T>(v));  // as the product of several tokens reads it
-        if (write && k >= j0 && k < j0 + GQ_COLS) past[(long long)(pos % taps) * channels + k] = x;
+    // rows of the ring by how far back they are; up to GQ_TAPS of them, and a run of channels, are on their way together
+    int row[GQ_TAPS];
+#pragma unroll
+    for (int q = 1; q < GQ_TAPS; ++q) row[q] = q < taps && q <= pos ? (pos - q) % taps * channels : -1;
+    for (int k0 = lane; k0 < pp; k0 += 32 * GQ_CHANNELS) {
+      T x[GQ_CHANNELS], v[GQ_CHANNELS][GQ_TAPS];
+      float w[GQ_CHANNELS][GQ_TAPS], bias[GQ_CHANNELS];
+#pragma unroll
+      for (int i = 0; i < GQ_CHANNELS; ++i) {
+        const int k = k0 + 32 * i;
+        const bool there = in && k < pp;
+        x[i] = from_f32<T>(0.f);
+        bias[i] = w[i][0] = 0.f;
+        if (there) {
+          x[i] = now[k];
+          bias[i] = p.g.conv_bias[part * pp + k];
+          w[i][0] = cw[(long long)(taps - 1) * channels + k];
+        }
+#pragma unroll
+        for (int q = 1; q < GQ_TAPS; ++q) {
+          v[i][q] = from_f32<T>(0.f);
+          w[i][q] = 0.f;
+          if (there && row[q] >= 0) {
+            v[i][q] = past[row[q] + k];
+            w[i][q] = cw[(long long)(taps - 1 - q) * channels + k];
+          }
+        }
       }
-      gq_x[k * GQ_ROWS + warp] = v;
+#pragma unroll
+      for (int i = 0; i < GQ_CHANNELS; ++i) {
+        const int k = k0 + 32 * i;
+        if (k >= pp) break;
+        float s = fmaf(w[i][0], to_f32(x[i]), bias[i]);
+#pragma unroll
+        for (int q = 1; q < GQ_TAPS; ++q) s = fmaf(w[i][q], to_f32(v[i][q]), s);
+        for (int q = GQ_TAPS; in && q < taps && q <= pos; ++q)
+          s = fmaf(cw[(long long)(taps - 1 - q) * channels + k], to_f32(past[(long long)((pos - q) % taps) * channels + k]), s);
+        // rounded as the product of several tokens reads it
+        gq_x[k * GQ_ROWS + warp] = in ? to_f32(from_f32<T>(s)) : 0.f;
+        if (write && k >= j0 && k < j0 + GQ_COLS) past[(long long)(pos % taps) * channels + k] = x[i];
+      }
     }
   }
   __syncthreads();

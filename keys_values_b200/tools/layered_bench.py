@@ -613,7 +613,7 @@ def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) ->
     rand = lambda *shape: torch.randn(*shape, device=dev, dtype=bf)  # noqa: E731
     f32 = lambda *shape: torch.rand(*shape, device=dev)  # noqa: E731
     tiles = lambda n: -(-n // 128) * 128  # noqa: E731
-    for B, T, start in ((1, tokens, 0), (4, tokens, 0), (batch, 1, tokens - 1)):
+    for B, T, start in ((1, tokens, 0), (4, tokens, 0), (batch, 1, tokens - 2)):
         n = B * T
         tag = f"prefill {B} x {T} tokens" if T > 1 else f"decode {B} rows"
         table = SequenceTable(B, dev)
