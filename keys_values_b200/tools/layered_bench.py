@@ -690,6 +690,13 @@ def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) ->
             tab.add(f"{tag}:   like: QK norm, split + RoPE", lambda: cu.qknorm_rope_fwd(qkv2, cs, cs, wq, wq, 2 * m.qk // 128 - 16, 8, 128, eps, 128, False),
                     gbytes=8 * n * m.qk / 1e9)
             flop = n * m.heads * (4 * m.np * m.vdp + 128 * (m.np + m.vdp)) / 1e12
+            y = torch.empty(B, T, m.inner, device=dev, dtype=bf)
+            nbytes = int(LC.lib().kvb_gated_linear_scan_tc_scratch_bytes(B, T, m.heads, m.vdp, m.np))
+            scratch = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=dev)
+            alone = lambda: cu._check(LC.lib().kvb_gated_linear_scan_tc(  # noqa: E731
+                cu._p(vg), cu._ll(2 * m.inner), cu._p(qk), cu._p(factor), cu._p(far), cu._p(state), cu._p(y), cu._p(scratch), cu._p(seq.slots),
+                cu._p(seq.start), cu._p(seq.count), B, T, m.heads, m.vdp, m.np, cu._p(cu.status_word(dev)), cu._stream(vg)), "scan")
+            tab.add(f"{tag}: gated linear scan, {m.heads} heads of {m.np} x {m.vdp}", alone, gbytes=(n * (2 * m.qk + 4 * m.inner) + state_bytes) / 1e9, tflop=flop)
             tab.add(f"{tag}: gated linear scan with its preparation, {m.heads} heads of {m.np} x {m.vdp}", lambda: LC.gated_linear_scan(qka, vg, decay, state, seq, m),
                     gbytes=(n * (4 * (m.qk + m.rp) + 4 * m.inner) + state_bytes) / 1e9, tflop=flop)
             q2 = rand(B, m.heads, T, 128)
@@ -698,7 +705,7 @@ def side_by_side_kernel_table(config: Config, batch: int, tokens: int = 8192) ->
             y = rand(B, T, m.inner)
             tab.add(f"{tag}: gated linear: norm per head, gate", lambda: LC.head_norm_gate(y, vg[..., m.inner :], m, eps, wn), gbytes=6 * n * m.inner / 1e9)
             tab.add(f"{tag}:   like: (add +) RMSNorm", like_norm, gbytes=norm_bytes)
-            del qka, vg, qk, q2, qkv2, y, factor
+            del qka, vg, qk, q2, qkv2, y, factor, scratch
         else:
             u = torch.randn(B, 1, m.qk + m.rp + 2 * m.inner, device=dev)
             tab.add(f"{tag}: gated linear step, {m.heads} heads of {m.np} x {m.vdp}", lambda: LC.gated_linear_step(u, decay, wn, state, seq, m, eps, bf),
