@@ -316,7 +316,7 @@ def _shared_runs(times: int, heads: int, kv_heads: int, dim: int, rope_dims: int
     """``times`` runs of: attention, gated linear attention, attention over the first one's keys and values, two mixers side by side."""
     out = []
     for i in range(times):
-        a = dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=dim, scale=dim**-0.5, rope_base=250000.0, rope_dims=rope_dims,
+        a = dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=dim, scale=dim**-0.5, rope_base=500000.0, rope_dims=rope_dims,
                  gate="head")
         out += [a, linear, dict(a, kv_from=4 * i), parallel]
     return [dict(mixer=m, mlp=dict(kind="gated", ff=ff, limit=limit)) for m in out]
@@ -328,7 +328,7 @@ def _gated_linear(heads: int, dim: int, vdim: int, rank: int = 16, tau: float = 
 
 def _pooled_beside_recurrence(heads: int, kv_heads: int, dim: int, rope_dims: int, window: int, pool: int, width: int, blocks: int,
                               scales: Tuple[float, float] = (0.7, 1.0)) -> dict:
-    left = dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=dim, scale=dim**-0.5, rope_base=50000.0, rope_dims=rope_dims,
+    left = dict(kind="grouped_attention", n_head=heads, n_kv_head=kv_heads, dim=dim, v_dim=dim, scale=dim**-0.5, rope_base=10000.0, rope_dims=rope_dims,
                 rope_interleaved=True, qk_norm="unit", temperature=True, window=window, pool=pool)
     return dict(kind="side_by_side", left=left, left_scale=scales[0], right=dict(kind="gated_recurrence", width=width, blocks=blocks, conv=4),
                 right_scale=scales[1])
@@ -452,12 +452,12 @@ configs: List[dict] = [
                                      _pooled_beside_recurrence(4, 2, 24, 8, 48, 6, 120, 5), 152, limit=2.0)),
     ),
     dict(
-        name="Dotorax-2k", block_size=1 << 15, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5, input_conv=4, residual_mult=0.7,
+        name="Dotorax-2k", block_size=1 << 15, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5, input_conv=4, residual_mult=0.9,
         **_dotorax(2048, _shared_runs(4, 16, 4, 128, 64, _gated_linear(16, 128, 128),
                                       _pooled_beside_recurrence(16, 4, 128, 64, 2048, 64, 2048, 16), 5632)),
     ),
     dict(
-        name="Dotorax-4k", block_size=1 << 15, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5, input_conv=4, residual_mult=0.7,
+        name="Dotorax-4k", block_size=1 << 15, vocab_size=32000, padded_vocab_size=32000, norm_eps=1e-5, input_conv=4, residual_mult=0.9,
         **_dotorax(4096, _shared_runs(3, 32, 8, 128, 64, _gated_linear(32, 128, 128),
                                       _pooled_beside_recurrence(32, 8, 128, 64, 2048, 64, 4096, 16), 11008)),
     ),

@@ -164,7 +164,7 @@ MIXERS = {
     "shared": [A(heads=6, kv_heads=3, dim=16, vdim=24, dims=16), A(heads=6, kv_heads=3, dim=16, vdim=24, dims=16, scale=0.2, kv_from=0),
                A(heads=4, dim=24), A(heads=4, dim=24, scale=0.7, kv_from=2), A(heads=6, kv_heads=3, dim=16, vdim=24, dims=16, kv_from=0)],
     "parallel": [P()],
-    "parallel, wide": [P(heads=8, kv_heads=1, dim=64, vdim=32, dims=64, scale=0.4, size=40, pool=16, width=128, blocks=2, conv=4)],
+    "parallel, wide": [P(heads=8, kv_heads=1, dim=64, vdim=32, dims=64, scale=0.4, size=44, pool=16, width=128, blocks=2, conv=4)],
     "parallel, odd": [P(heads=3, kv_heads=1, dim=7, vdim=5, dims=4, size=3, pool=5, left_scale=-0.4, right_scale=2.5, width=33, blocks=11, conv=1)],
     "parallel, pool of one": [P(heads=2, kv_heads=2, dim=40, vdim=136, dims=8, scale=0.5, size=1, pool=1, width=8, blocks=1, conv=7)],
     "parallel, deep": [P(heads=2, kv_heads=1, dim=136, vdim=40, dims=136, scale=0.6, size=70, pool=3, width=300, blocks=3, conv=2)],
@@ -497,7 +497,7 @@ def recurrence_case(width, blocks, taps, T, dtype, seed=0, lam=(-3.0, 1.5)):
 
 
 @variant_param
-@pytest.mark.parametrize("width,blocks,taps", [(36, 3, 3), (64, 1, 4), (33, 11, 1), (256, 4, 4), (80, 2, 7), (1, 1, 2)])
+@pytest.mark.parametrize("width,blocks,taps", [(36, 3, 3), (64, 1, 4), (33, 11, 1), (320, 5, 4), (80, 2, 7), (1, 1, 2)])
 def test_gated_recurrence(env, width, blocks, taps):
     """Convolution, gates, recurrence and output over passes of several sizes and single tokens; columns of wider rows; a factor."""
     dev, dtype = env
